@@ -1,11 +1,12 @@
 """Typed configurations and the architecture registry."""
 from .hunyuan_dense import (ALIASES, ARCHITECTURE, ConfigError, HunyuanDenseConfig, RopeScaling,
                             build_spec, read_config_json)
-from . import mufevik, radorax, vodelix, zudarax
+from . import mufevik, pogarax, radorax, vodelix, zudarax
 from .radorax import RadoraxConfig
 from .vodelix import VodelixConfig
 from .mufevik import MufevikConfig
 from .zudarax import ZudaraxConfig
+from .pogarax import PogaraxConfig
 from .registry import (Architecture, UnknownArchitecture, register_architecture, registered,
                        resolve)
 from .spec import LayerSpec, ModelSpec, PartSpec, ScheduleStep
@@ -16,7 +17,8 @@ register_architecture(radorax.ARCHITECTURE, RadoraxConfig.from_dict, radorax.bui
 register_architecture(vodelix.ARCHITECTURE, VodelixConfig.from_dict, vodelix.build_spec, vodelix.ALIASES)
 register_architecture(mufevik.ARCHITECTURE, MufevikConfig.from_dict, mufevik.build_spec, mufevik.ALIASES)
 register_architecture(zudarax.ARCHITECTURE, ZudaraxConfig.from_dict, zudarax.build_spec, zudarax.ALIASES)
+register_architecture(pogarax.ARCHITECTURE, PogaraxConfig.from_dict, pogarax.build_spec, pogarax.ALIASES)
 
-__all__ = ["ConfigError", "HunyuanDenseConfig", "RadoraxConfig", "VodelixConfig", "MufevikConfig", "ZudaraxConfig", "RopeScaling", "read_config_json", "Architecture",
+__all__ = ["ConfigError", "HunyuanDenseConfig", "RadoraxConfig", "VodelixConfig", "MufevikConfig", "ZudaraxConfig", "PogaraxConfig", "RopeScaling", "read_config_json", "Architecture",
            "UnknownArchitecture", "register_architecture", "registered", "resolve", "LayerSpec",
            "ModelSpec", "PartSpec", "ScheduleStep", "EngineConfig", "parse_memory_limit"]

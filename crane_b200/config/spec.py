@@ -11,6 +11,11 @@ from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional
 
 
+# the workspace buffer that holds the residual stream in the model type, for models whose sublayers read the
+# stream itself (the embedding part's ``model_copy``; kept up to date by the block)
+STREAM_COPY = "stream_model"
+
+
 @dataclass
 class PartSpec:
     """One part: ``kind`` is its role (mixer, ffn, norm, position, embed, head),

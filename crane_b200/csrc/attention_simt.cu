@@ -7,7 +7,8 @@
 // request e attends the keys of positions max(0, p - window + 1) .. p of the
 // same request, found through the request's block table.  Scores, softmax
 // statistics and the weighted sum are float whatever the storage type.  `sink`: the
-// softmax has one more candidate of score 0 and no value (p_j = exp(s_j) / (1 + sum exp(s))).
+// softmax has one more candidate of score 0 and no value (p_j = exp(s_j) / (1 + sum exp(s))); `sinks`: of a
+// score of its own per query head.
 // `ScoreMod` says what happens to a score before it becomes a weight: squashed to cap * tanh(s / cap);
 // keys seen only within the query's own block of `chunk` positions (blocks counted from position 0);
 // weights sigmoid(s + bias of the head) that are not normalised over the keys instead of a softmax; a
@@ -34,6 +35,7 @@ struct ScoreMod {
     int d_row;                  // elements of a query / key row of a head (>= maps * d_map)
     int d_map;                  // elements from one map's start to the next
     float* out_f32;             // float [token][head][map][dv] instead of `out`, or null
+    const float* sinks;         // [nq]: one more candidate of this score and no value per head, or null
 };
 
 template <typename T>
@@ -122,7 +124,11 @@ paged_attention_simt_kernel(const T* __restrict__ q, T* __restrict__ out,
     if (__any_sync(0xffffffffu, bad) && lane == 0) atomicOr(err, CRANE_ERR_PAGE_RANGE);
     // a sink: one more candidate of score 0 that has no value, so it only adds exp(0 - m) to the sum
     if (sink) l += expf(-m);
-    const float inv = sm.sigmoid ? 1.f : l > 0.f ? 1.f / l : 0.f;
+    float inv = sm.sigmoid ? 1.f : l > 0.f ? 1.f / l : 0.f;
+    if (sm.sinks != nullptr) {
+        const float s = sm.sinks[h], top = fmaxf(m, s), mine = expf(m - top);
+        inv = mine / fmaf(l, mine, expf(s - top));
+    }
     if (sm.out_f32 != nullptr) {
         float* op = sm.out_f32 + ((long long)t * pairs + hv) * dv;
 #pragma unroll
@@ -180,9 +186,9 @@ CRANE_API int crane_paged_attention_simt(int dtype, const void* q, void* out, co
                                          const int* tok_entry, const int* block_table,
                                          int max_blocks, int num_pages, int page_size,
                                          int n_tokens, int nq, int nkv, int d, int dv,
-                                         int v_stride, int window, float scale, int sink, float* out_cross,
-                                         int* err, cudaStream_t st) {
-    const ScoreMod plain{0.f, 0, 0, nullptr, 1, d, d, nullptr};
+                                         int v_stride, int window, float scale, int sink, const float* sinks,
+                                         float* out_cross, int* err, cudaStream_t st) {
+    const ScoreMod plain{0.f, 0, 0, nullptr, 1, d, d, nullptr, sinks};
     return launch_simt(dtype, q, out, k_pool, v_pool, positions, tok_entry, block_table, max_blocks, num_pages,
                        page_size, n_tokens, nq, nkv, d, dv, v_stride, window, scale, sink, out_cross, plain, err, st);
 }
@@ -195,7 +201,7 @@ CRANE_API int crane_scored_attention_simt(int dtype, const void* q, void* out, c
                                           float scale, float softcap, int chunk, int sigmoid,
                                           const float* head_bias, int maps, int d_row, int d_map, float* out_f32,
                                           int* err, cudaStream_t st) {
-    const ScoreMod sm{softcap, chunk, sigmoid, head_bias, maps, d_row, d_map, out_f32};
+    const ScoreMod sm{softcap, chunk, sigmoid, head_bias, maps, d_row, d_map, out_f32, nullptr};
     return launch_simt(dtype, q, out, k_pool, v_pool, positions, tok_entry, block_table, max_blocks, num_pages,
                        page_size, n_tokens, nq, nkv, d, dv, v_stride, window, scale, 0, nullptr, sm, err, st);
 }

@@ -17,6 +17,11 @@
 // Launched with programmatic dependent launch: the first tiles of the weights
 // are requested before the kernel waits for its predecessor (see the producer).
 //
+// Grouped activations: with `group_features` > 0 the activations are several row blocks of one tensor,
+// `group_rows` apart, and output features f read block f / group_features (projections that each read an
+// input of their own, one launch).  group_features is a multiple of the tile's features, so a tile
+// reads one block; a tile's rows past the block's end belong to the next block and are not stored.
+//
 // Every wait on an mbarrier is bounded: when it runs out the kernel records
 // CRANE_ERR_WAIT_TIMEOUT, all roles leave their loops, tensor memory is freed
 // and the kernel returns.
@@ -121,7 +126,12 @@ struct GemmParams {
     int* err;
     const uint8_t* prefetch;        // what the NEXT product of the step will stream (its weights), or null:
     long long prefetch_bytes;       // asked into L2 by this kernel's idle warp as soon as it starts
+    int group_features, group_rows; // grouped activations (0: all features read the same rows)
 };
+// The first row of the activations that features from `feature` on read.
+__device__ __forceinline__ int group_row0(const GemmParams& p, int feature) {
+    return p.group_features > 0 ? feature / p.group_features * p.group_rows : 0;
+}
 
 // The kernels of a decode step run one after the other, each for a few microseconds, and each begins
 // by waiting for its operands to arrive from DRAM.  A product that is told what the next product
@@ -165,6 +175,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int a0 = blockIdx.x * BM, b0 = blockIdx.y * BN;
+    const int ag = TRANSPOSED ? a0 : a0 + group_row0(p, b0);          // where the operands' rows lie
+    const int bg = TRANSPOSED ? b0 + group_row0(p, a0) : b0;
     // the k-blocks are dealt out to the slices as evenly as they go
     const int num_kb_total = (p.k + BK - 1) / BK;
     const int kb_begin = (int)(((long long)blockIdx.z * num_kb_total) / gridDim.z);
@@ -204,15 +216,15 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             const uint32_t bar = smem_u32(&full[i]);
             mbar_expect_tx(bar, A_BYTES + B_BYTES);
             const int k0 = (kb_begin + i) * BK;
-            if (TRANSPOSED) tma_load_2d(smem_u32(smem_a + i * A_BYTES), &map_a, bar, k0, a0);
-            else tma_load_2d(smem_u32(smem_b + i * B_BYTES), &map_b, bar, k0, b0);
+            if (TRANSPOSED) tma_load_2d(smem_u32(smem_a + i * A_BYTES), &map_a, bar, k0, ag);
+            else tma_load_2d(smem_u32(smem_b + i * B_BYTES), &map_b, bar, k0, bg);
         }
         pdl_wait();
         for (int i = 0; i < pre; ++i) {
             const uint32_t bar = smem_u32(&full[i]);
             const int k0 = (kb_begin + i) * BK;
-            if (TRANSPOSED) tma_load_2d(smem_u32(smem_b + i * B_BYTES), &map_b, bar, k0, b0);
-            else tma_load_2d(smem_u32(smem_a + i * A_BYTES), &map_a, bar, k0, a0);
+            if (TRANSPOSED) tma_load_2d(smem_u32(smem_b + i * B_BYTES), &map_b, bar, k0, bg);
+            else tma_load_2d(smem_u32(smem_a + i * A_BYTES), &map_a, bar, k0, ag);
         }
         for (int i = pre; i < num_kb; ++i) {
             const int s = i % STAGES;
@@ -221,8 +233,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             const uint32_t bar = smem_u32(&full[s]);
             mbar_expect_tx(bar, A_BYTES + B_BYTES);
             const int k0 = (kb_begin + i) * BK;
-            tma_load_2d(smem_u32(smem_a + s * A_BYTES), &map_a, bar, k0, a0);
-            tma_load_2d(smem_u32(smem_b + s * B_BYTES), &map_b, bar, k0, b0);
+            tma_load_2d(smem_u32(smem_a + s * A_BYTES), &map_a, bar, k0, ag);
+            tma_load_2d(smem_u32(smem_b + s * B_BYTES), &map_b, bar, k0, bg);
         }
     } else if (warp == 1 && lane == 0) {
         // ---------------- MMA issuer ----------------
@@ -503,7 +515,8 @@ gemm_bf16_persistent_kernel(const __grid_constant__ CUtensorMap map_a,
         pdl_wait();                                          // the activations come from the kernel before
         int it = 0;                                          // k-blocks issued so far, over all tiles
         for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x) {
-            const int a0 = (tile % tiles_a) * (MT * BM), b0 = (tile / tiles_a) * BN;
+            const int b0 = (tile / tiles_a) * BN;
+            const int a0 = (tile % tiles_a) * (MT * BM) + group_row0(p, b0);
             for (int kb = 0; kb < num_kb; ++kb, ++it) {
                 const int s = it % STAGES;
                 if (!mbar_wait(smem_u32(&empty[s]), ((it / STAGES) & 1) ^ 1, abort_flag)) goto done;
@@ -720,7 +733,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
         pdl_wait();
         int it = 0;
         for (int tile = pair; tile < num_tiles; tile += num_pairs) {
-            const int a0 = (tile % tiles_a) * TILE_ROWS + (int)rank * BM;
+            const int a0 = (tile % tiles_a) * TILE_ROWS + (int)rank * BM + group_row0(p, (tile / tiles_a) * BN);
             const int b0 = (tile / tiles_a) * BN + (int)rank * BH;
             for (int kb = 0; kb < num_kb; ++kb, ++it) {
                 const int s = it % STAGES;
@@ -898,7 +911,7 @@ int launch_persistent(const CUtensorMap& ma, const CUtensorMap& mb, const GemmPa
 
 template <int BN, int STAGES, bool SILU, int MT = 1>
 int launch_pair(const void* A, const void* B, int rows_a, int rows_b, int k, long long lda, long long ldb,
-                const GemmParams& p, cudaStream_t st) {
+                const GemmParams& p, int map_rows_a, cudaStream_t st) {
     constexpr size_t smem = STAGES * (MT * BM * BK * 2 + (BN / 2) * BK * 2) + (2 * STAGES + 4) * 8 + 16 + 1024;
     static_assert(smem <= 232448, "more shared memory than a CTA can have");
     auto kern = gemm_bf16_pair_kernel<BN, STAGES, SILU, MT>;
@@ -913,7 +926,7 @@ int launch_pair(const void* A, const void* B, int rows_a, int rows_b, int k, lon
         configured = true;
     }
     CUtensorMap ma, mb;
-    if (!make_map(&ma, A, rows_a, k, lda, BM) || !make_map(&mb, B, rows_b, k, ldb, BN / 2))
+    if (!make_map(&ma, A, map_rows_a, k, lda, BM) || !make_map(&mb, B, rows_b, k, ldb, BN / 2))
         return (int)cudaErrorInvalidValue;
     const int tiles = ((rows_a + 2 * BM * MT - 1) / (2 * BM * MT)) * ((rows_b + BN - 1) / BN);
     const int pairs = tiles < sms / 2 ? tiles : sms / 2;
@@ -942,13 +955,15 @@ int dispatch_bn(int bn, const CUtensorMap& ma, const CUtensorMap& mb, const Gemm
 // epilogue: 0 none, 1 silu(gate) * up (see the persistent kernel).
 // out_f32 / transposed as in the kernel; split_k > 1 writes float partial sums
 // [split_k][...] into `out` (which must then be float) `split_stride` apart.
+// group_features > 0: grouped activations (see the top of the file): row blocks of `group_rows` rows each, and
+// rows of a block in use = the product's number of tokens.  No silu epilogue.
 // Requirements (checked, cudaErrorInvalidValue otherwise): k % 8 == 0, lda and
 // ldb multiples of 8 elements, A and B 16-byte aligned.
 CRANE_API int crane_gemm_bf16_tcgen05(const void* A, const void* B, const float* bias, void* out,
                                       int rows_a, int rows_b, int k, long long lda, long long ldb,
                                       long long ld_out, int bn, int tile_rows, int out_f32, int transposed,
-                                      int split_k, long long split_stride, int epilogue,
-                                      const void* prefetch, long long prefetch_bytes, int* err,
+                                      int split_k, long long split_stride, int epilogue, int group_features,
+                                      int group_rows, const void* prefetch, long long prefetch_bytes, int* err,
                                       cudaStream_t st) {
     if (rows_a <= 0 || rows_b <= 0) return 0;
     if (k <= 0 || (k & 7) || (lda & 7) || (ldb & 7) || ((uintptr_t)A & 15) || ((uintptr_t)B & 15))
@@ -956,13 +971,20 @@ CRANE_API int crane_gemm_bf16_tcgen05(const void* A, const void* B, const float*
     if (split_k < 1) split_k = 1;
     if (split_k > 1 && !out_f32) return (int)cudaErrorInvalidValue;
     CUtensorMap ma, mb;
-    if (!make_map(&ma, A, rows_a, k, lda, BM) || !make_map(&mb, B, rows_b, k, ldb, bn))
+    int map_rows_a = rows_a, map_rows_b = rows_b;
+    if (group_features > 0) {
+        const int features = transposed ? rows_a : rows_b, tokens = transposed ? rows_b : rows_a;
+        if (group_features % (transposed ? BM : bn) || group_rows < tokens || epilogue != 0) return (int)cudaErrorInvalidValue;
+        (transposed ? map_rows_b : map_rows_a) = (features + group_features - 1) / group_features * group_rows;
+    }
+    if (!make_map(&ma, A, map_rows_a, k, lda, BM) || !make_map(&mb, B, map_rows_b, k, ldb, bn))
         return (int)cudaErrorInvalidValue;
     const int num_kb = (k + BK - 1) / BK;
     if (split_k > num_kb) split_k = num_kb;
     GemmParams p;
     p.rows_a = rows_a; p.rows_b = rows_b; p.k = k;
     p.out = out; p.ld_out = ld_out; p.split_stride = split_stride; p.bias = bias; p.err = err;
+    p.group_features = group_features; p.group_rows = group_rows;
     p.prefetch = ((uintptr_t)prefetch & 15) ? nullptr : (const uint8_t*)prefetch;   // (only the narrow-tile kernel asks)
     p.prefetch_bytes = prefetch_bytes > 0 ? prefetch_bytes : 0;
     dim3 grid((rows_a + BM - 1) / BM, (rows_b + bn - 1) / bn, split_k);
@@ -1020,7 +1042,8 @@ CRANE_API int crane_gemm_bf16_tcgen05(const void* A, const void* B, const float*
 // tiles, bn in 192, 224, 256.  epilogue as there.
 CRANE_API int crane_gemm_bf16_pair(const void* A, const void* B, const float* bias, void* out, int rows_a,
                                    int rows_b, int k, long long lda, long long ldb, long long ld_out,
-                                   int bn, int tile_rows, int epilogue, int* err, cudaStream_t st) {
+                                   int bn, int tile_rows, int epilogue, int group_features, int group_rows,
+                                   int* err, cudaStream_t st) {
     if (rows_a <= 0 || rows_b <= 0) return 0;
     if (k <= 0 || (k & 7) || (lda & 7) || (ldb & 7) || ((uintptr_t)A & 15) || ((uintptr_t)B & 15))
         return (int)cudaErrorInvalidValue;
@@ -1030,34 +1053,40 @@ CRANE_API int crane_gemm_bf16_pair(const void* A, const void* B, const float* bi
     p.rows_a = rows_a; p.rows_b = rows_b; p.k = k;
     p.out = out; p.ld_out = ld_out; p.split_stride = 0; p.bias = bias; p.err = err;
     p.prefetch = nullptr; p.prefetch_bytes = 0;
+    p.group_features = group_features; p.group_rows = group_rows;
+    int map_rows = rows_a;
+    if (group_features > 0) {
+        if (group_features % bn || group_rows < rows_a || epilogue != 0) return (int)cudaErrorInvalidValue;
+        map_rows = (rows_b + group_features - 1) / group_features * group_rows;
+    }
     if (epilogue == 1) {
         if (bias != nullptr || (rows_b & 31) || (ld_out & 7) || ((uintptr_t)out & 15)) return (int)cudaErrorInvalidValue;
         if (tall) switch (bn) {
-            case 192: return launch_pair<192, 5, true, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-            case 224: return launch_pair<224, 4, true, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-            case 256: return launch_pair<256, 4, true, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
+            case 192: return launch_pair<192, 5, true, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+            case 224: return launch_pair<224, 4, true, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+            case 256: return launch_pair<256, 4, true, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
             default: return (int)cudaErrorInvalidValue;
         }
         switch (bn) {
-            case 128: return launch_pair<128, 8, true>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-            case 192: return launch_pair<192, 7, true>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-            case 224: return launch_pair<224, 6, true>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-            case 256: return launch_pair<256, 6, true>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
+            case 128: return launch_pair<128, 8, true>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+            case 192: return launch_pair<192, 7, true>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+            case 224: return launch_pair<224, 6, true>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+            case 256: return launch_pair<256, 6, true>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
         }
         return (int)cudaErrorInvalidValue;
     }
     if (epilogue != 0) return (int)cudaErrorInvalidValue;
     if (tall) switch (bn) {
-        case 192: return launch_pair<192, 5, false, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-        case 224: return launch_pair<224, 4, false, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-        case 256: return launch_pair<256, 4, false, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
+        case 192: return launch_pair<192, 5, false, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+        case 224: return launch_pair<224, 4, false, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+        case 256: return launch_pair<256, 4, false, 2>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
         default: return (int)cudaErrorInvalidValue;
     }
     switch (bn) {
-        case 128: return launch_pair<128, 8, false>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-        case 192: return launch_pair<192, 7, false>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-        case 224: return launch_pair<224, 6, false>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
-        case 256: return launch_pair<256, 6, false>(A, B, rows_a, rows_b, k, lda, ldb, p, st);
+        case 128: return launch_pair<128, 8, false>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+        case 192: return launch_pair<192, 7, false>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+        case 224: return launch_pair<224, 6, false>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
+        case 256: return launch_pair<256, 6, false>(A, B, rows_a, rows_b, k, lda, ldb, p, map_rows, st);
     }
     return (int)cudaErrorInvalidValue;
 }

@@ -7,11 +7,12 @@
 //    g.  Both happen in one kernel, a row in shared memory between its passes; either half may be
 //    absent (no pending result: the streams stay; `first`: all streams start as the embedding output).
 //    R = 1 with mix = out = in = 1 is the plain residual sum.
-// 2. `route_grouped`: softmax over all experts, a correction added for the choice only, experts in
+// 2. `route_grouped`: scores by softmax over all experts or by a sigmoid each, a correction added for the choice only, experts in
 //    equal groups of neighbours of which the best few groups stay eligible, the `top` largest choice
 //    scores chosen, weighted by their uncorrected scores; an optional further logit becomes the
 //    sigmoid gate of a shared expert.
-// 3. `gated_activation`: silu(gate) * up per feed-forward column, times the column's routing weight.
+// 3. `gated_activation`: silu(gate) * up per feed-forward column, times the column's routing weight, or with
+//    that weight on the expert's input: silu(w gate) * (w up).
 // All arithmetic in 32-bit; T is the storage type of activations (float or bf16).
 #include "common.cuh"
 
@@ -78,7 +79,7 @@ streams_norm_kernel(float* __restrict__ streams, long long stream_stride, int R,
 __global__ void __launch_bounds__(128)
 route_grouped_kernel(const float* __restrict__ z, int ld, const float* __restrict__ correction,
                      float* __restrict__ route, int n, int experts, int top, int groups, int keep,
-                     int shared_gate) {
+                     int shared_gate, int sigmoid_scores) {
     extern __shared__ float sm[];                     // per warp: score [E], choice [E], group score [groups]
     pdl_launch_dependents();
     pdl_wait();
@@ -90,22 +91,33 @@ route_grouped_kernel(const float* __restrict__ z, int ld, const float* __restric
     float* gscore = choice + experts;
     const float* zr = z + (long long)t * ld;
     float* r = route + (long long)t * (experts + shared_gate);
-    float zmax = -INFINITY;
-    for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, zr[e]);
-    zmax = warp_max(zmax);
-    float sum = 0.f;
-    for (int e = lane; e < experts; e += 32) {
-        const float p = expf(zr[e] - zmax);
-        score[e] = p;
-        sum += p;
-    }
-    sum = warp_sum(sum);
-    const float inv = 1.f / sum;
-    for (int e = lane; e < experts; e += 32) {
-        const float s = score[e] * inv;
-        score[e] = s;
-        choice[e] = s + (correction != nullptr ? correction[e] : 0.f);
-        r[e] = 0.f;
+    if (sigmoid_scores) {
+        // (without a correction the choice goes by the logits: the same order, and scores that round to the
+        // same number keep it)
+        for (int e = lane; e < experts; e += 32) {
+            const float s = 1.f / (1.f + expf(-zr[e]));
+            score[e] = s;
+            choice[e] = correction != nullptr ? s + correction[e] : zr[e];
+            r[e] = 0.f;
+        }
+    } else {
+        float zmax = -INFINITY;
+        for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, zr[e]);
+        zmax = warp_max(zmax);
+        float sum = 0.f;
+        for (int e = lane; e < experts; e += 32) {
+            const float p = expf(zr[e] - zmax);
+            score[e] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        const float inv = 1.f / sum;
+        for (int e = lane; e < experts; e += 32) {
+            const float s = score[e] * inv;
+            score[e] = s;
+            choice[e] = s + (correction != nullptr ? correction[e] : 0.f);
+            r[e] = 0.f;
+        }
     }
     __syncwarp();
     const int per = experts / groups;
@@ -162,12 +174,13 @@ route_grouped_kernel(const float* __restrict__ z, int ld, const float* __restric
 }
 
 // gu rows: [gate (cols) | up (cols)].  out[t][c] = silu(gate) * up * weight(c): route[t][c / per_expert]
-// for c < routed_cols, behind them route[t][experts] (`shared_gate`) or 1.
+// for c < routed_cols, behind them route[t][experts] (`shared_gate`) or 1.  `on_input`: the weight multiplies what
+// the expert reads, so both of its products: silu(w gate) * (w up).
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_activation_kernel(GemmOut<T> gu, T* __restrict__ out, long long n, int cols,
                         const float* __restrict__ route, int experts, int per_expert, int routed_cols,
-                        int shared_gate) {
+                        int shared_gate, int on_input) {
     pdl_launch_dependents();
     pdl_wait();
     const int rl = experts + shared_gate;
@@ -182,7 +195,8 @@ gated_activation_kernel(GemmOut<T> gu, T* __restrict__ out, long long n, int col
         }
         float v = 0.f;
         if (w != 0.f) {
-            const float a = gu.load(row * 2 * cols + c), b = gu.load(row * 2 * cols + cols + c);
+            const float z = gu.load(row * 2 * cols + c), b = gu.load(row * 2 * cols + cols + c);
+            const float a = on_input ? z * w : z;
             v = a / (1.f + expf(-a)) * b * w;
         }
         out[i] = from_f32<T>(v);
@@ -211,19 +225,20 @@ CRANE_API int crane_streams_norm(int dtype, float* streams, long long stream_str
 }
 
 CRANE_API int crane_route_grouped(const float* z, int ld, const float* correction, float* route, int n,
-                                  int experts, int top, int groups, int keep, int shared_gate, cudaStream_t st) {
+                                  int experts, int top, int groups, int keep, int shared_gate, int sigmoid_scores,
+                                  cudaStream_t st) {
     if (n <= 0) return 0;
     if (experts <= 0 || top <= 0 || groups <= 0 || experts % groups || keep <= 0 || keep > groups)
         return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)4 * (2 * experts + groups) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     return crane_launch(route_grouped_kernel, dim3((n + 3) / 4), dim3(128), smem, st, z, ld, correction, route, n,
-                        experts, top, groups, keep, shared_gate ? 1 : 0);
+                        experts, top, groups, keep, shared_gate ? 1 : 0, sigmoid_scores);
 }
 
 CRANE_API int crane_gated_activation(int dtype, const void* gu, const float* gu_parts, int n_parts,
                                      long long part_stride, void* out, int n_rows, int cols, const float* route,
-                                     int experts, int per_expert, int routed_cols, int shared_gate,
+                                     int experts, int per_expert, int routed_cols, int shared_gate, int on_input,
                                      cudaStream_t st) {
     if (n_rows <= 0 || cols <= 0) return 0;
     const long long n = (long long)n_rows * cols;
@@ -231,6 +246,6 @@ CRANE_API int crane_gated_activation(int dtype, const void* gu, const float* gu_
     DISPATCH_T(dtype, {
         GemmOut<T> u{(const T*)gu, gu_parts, n_parts, part_stride};
         return crane_launch(gated_activation_kernel<T>, dim3(blocks), dim3(256), 0, st, u, (T*)out, n, cols, route,
-                            experts, per_expert > 0 ? per_expert : 1, routed_cols, shared_gate ? 1 : 0);
+                            experts, per_expert > 0 ? per_expert : 1, routed_cols, shared_gate ? 1 : 0, on_input);
     });
 }

@@ -8,6 +8,8 @@
 // latent_prep   per token: c = RMSNorm(first rank columns of the down projection) * w and the rotated
 //               last rot columns go to the token's cache row [rank + rot]; the rotated part of every
 //               query head goes to columns rank.. of the absorbed query [token, head, rank + rot].
+//               Queries that come through a latent of their own take two launches: one with the cache row and
+//               the query latent's RMSNorm (which the queries' product then reads), one with the rotation.
 // head_linear   out[t, h, :] = W_h x[t, h, :] for every head (U_h^T on the unrotated query part; V_h on
 //               the attention's latent output, there times sigmoid(gate)): on the tensor cores in
 //               bfloat16 (widths that the MMA tiles take), else on the FP32 cores.
@@ -21,8 +23,8 @@ namespace {
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(GemmOut<T> proj, int cols, int q_off, int dkv_off, int heads, int dim, int rot,
-                   int rank, int rot_dims, const float* __restrict__ cos_tab,
+latent_prep_kernel(GemmOut<T> proj, int cols, int q_off, int dkv_off, int cq_off, int cq_rank,
+                   const float* __restrict__ cq_w, T* __restrict__ cq_out, int heads, int dim, int rot, int rank, int rot_dims, const float* __restrict__ cos_tab,
                    const float* __restrict__ sin_tab, int n_positions,
                    const int* __restrict__ positions, const int* __restrict__ tok_entry,
                    const int* __restrict__ block_table, int max_blocks, int num_pages, int page_size,
@@ -43,8 +45,19 @@ latent_prep_kernel(GemmOut<T> proj, int cols, int q_off, int dkv_off, int heads,
     const int half = rot_dims >> 1, pairs = rot >> 1, width = rank + rot;
     const float* cs = cos_tab + (long long)pos * half;
     const float* sn = sin_tab + (long long)pos * half;
-    // the rotated part of every query head
-    for (int i = threadIdx.x; i < heads * pairs; i += blockDim.x) {
+    // the query latent (cq_off >= 0): RMSNorm * w, a row of its own
+    if (cq_off >= 0) {
+        float sq = 0.f;
+        for (int c = threadIdx.x; c < cq_rank; c += blockDim.x) {
+            const float v = proj.load(prow + cq_off + c);
+            sq += v * v;
+        }
+        const float rq = 1.f / sqrtf(block_sum(sq, scratch) / (float)cq_rank + eps);
+        for (int c = threadIdx.x; c < cq_rank; c += blockDim.x)
+            cq_out[(long long)t * cq_rank + c] = from_f32<T>(proj.load(prow + cq_off + c) * rq * cq_w[c]);
+    }
+    // the rotated part of every query head (q_off < 0: the queries are not there yet)
+    for (int i = threadIdx.x; q_off >= 0 && i < heads * pairs; i += blockDim.x) {
         const int h = i / pairs, p = i % pairs;
         const long long src = prow + q_off + (long long)h * (dim + rot) + dim + 2 * p;
         float u = proj.load(src), v = proj.load(src + 1);
@@ -254,8 +267,8 @@ head_linear_mma_kernel(GemmOut<__nv_bfloat16> x, int x_cols, int x_off, int x_he
 }  // namespace
 
 CRANE_API int crane_latent_prep(int dtype, const void* proj, const float* proj_parts, int n_parts,
-                                long long part_stride, int cols, int q_off, int dkv_off, int heads,
-                                int dim, int rot, int rank, int rot_dims, const float* cos_tab,
+                                long long part_stride, int cols, int q_off, int dkv_off, int cq_off,
+                                int cq_rank, const float* cq_w, void* cq_out, int heads, int dim, int rot, int rank, int rot_dims, const float* cos_tab,
                                 const float* sin_tab, int n_positions, const int* positions,
                                 const int* tok_entry, const int* block_table, int max_blocks,
                                 int num_pages, int page_size, void* pool, const float* norm_w, float eps,
@@ -265,7 +278,7 @@ CRANE_API int crane_latent_prep(int dtype, const void* proj, const float* proj_p
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
         return crane_launch(latent_prep_kernel<T>, dim3(n_tokens), dim3(128), 0, st, p, cols, q_off, dkv_off,
-                            heads, dim, rot, rank, rot_dims, cos_tab, sin_tab, n_positions, positions,
+                            cq_off, cq_rank, cq_w, (T*)cq_out, heads, dim, rot, rank, rot_dims, cos_tab, sin_tab, n_positions, positions,
                             tok_entry, block_table, max_blocks, num_pages, page_size, (T*)pool, norm_w, eps,
                             (T*)q_abs, err);
     });

@@ -17,6 +17,10 @@
 // kernel merges them.  Key tiles of 64 rows come in by cp.async through the block table (a warp per
 // row, one page look-up per row), two buffers.  Scores, softmax statistics and sums are float.
 //
+// `window` > 0: a token sees its own position and the window - 1 before it; a tile starts at its first row's
+// first visible key.  `sinks`: a number per head that joins the softmax's sum without a key or a value,
+// where the sums are divided (at the end of the one slice, or in the merge).
+//
 // Widths are run-time numbers below compile-time bounds (two instantiations: up to 128 + 128 and
 // up to 256 key / 192 value columns); rank + rot a multiple of 16, rank a multiple of 8.
 #include "common.cuh"
@@ -75,6 +79,14 @@ __device__ __forceinline__ bool find_tile(int tile, const int* __restrict__ cu_q
     return false;
 }
 
+// What sums with maximum m (log2 units) and sum of weights l are multiplied by when the softmax's sum also holds
+// exp(sink).
+__device__ __forceinline__ float sink_share(float m, float l, float sink) {
+    const float s = sink * 1.4426950408889634f, top = fmaxf(m, s);
+    const float mine = exp2f(m - top);
+    return mine / fmaf(l, mine, exp2f(s - top));
+}
+
 template <bool SMALL, int MAXDK16, int MAXDV8>
 __global__ void __launch_bounds__(128)
 latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out,
@@ -82,7 +94,7 @@ latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __res
                        const __nv_bfloat16* __restrict__ pool, const int* __restrict__ cu_q,
                        const int* __restrict__ kv_len, const int* __restrict__ block_table, int max_blocks,
                        int num_pages, int page_shift, int n_entries, int heads, int dk, int dv, float scale,
-                       int* err) {
+                       int window, const float* __restrict__ sinks, int* err) {
     constexpr int WARPS = 4;
     constexpr int KT = KeyTile<SMALL>::value;
     constexpr int BM = SMALL ? 16 : 64;               // query rows of a tile
@@ -108,8 +120,11 @@ latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __res
     const int last_tok = (row0 + n_rows - 1) / heads;
     const int n_keys = pos0 + last_tok + 1;           // keys that the tile's last row sees
     const int key_tiles = (n_keys + KT - 1) / KT;
-    const int per = (key_tiles + splits - 1) / splits;
-    const int kt_lo = split * per, kt_hi = min(key_tiles, kt_lo + per);
+    // the first key that the tile's first row sees (what lies before it may have left the cache)
+    const int first_key = window > 0 ? max(0, pos0 + row0 / heads - window + 1) : 0;
+    const int kt_first = first_key / KT;
+    const int per = (key_tiles - kt_first + splits - 1) / splits;
+    const int kt_lo = kt_first + split * per, kt_hi = min(key_tiles, kt_lo + per);
     const int* table = block_table + (long long)entry * max_blocks;
     const int chunks = dk >> 3;                       // 16-byte pieces of a row
     pdl_wait();
@@ -125,7 +140,7 @@ latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __res
         __nv_bfloat16* dst = k_s + buf * KT * ld;
         for (int r = warp; r < KT; r += WARPS) {
             const int j = kt * KT + r;
-            bool ok = j < n_keys;
+            bool ok = j < n_keys && j >= first_key;
             long long src = 0;
             if (ok) {
                 const int page = table[j >> page_shift];
@@ -150,6 +165,7 @@ latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __res
     const int r_a = wrow + g, r_b = r_a + 8;
     const int see_a = pos0 + (row0 + min(r_a, n_rows - 1)) / heads;
     const int see_b = pos0 + (row0 + min(r_b, n_rows - 1)) / heads;
+    const int from_a = window > 0 ? see_a - window + 1 : 0, from_b = window > 0 ? see_b - window + 1 : 0;
     const float sl2 = scale * 1.4426950408889634f;   // scores in units of log2 e
 
     for (int kt = kt_lo; kt < kt_hi; ++kt) {
@@ -183,10 +199,10 @@ latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __res
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
             const int k0 = key0 + j * 8;
-            s[j][0] = k0 <= see_a ? s[j][0] * sl2 : -INFINITY;
-            s[j][1] = k0 + 1 <= see_a ? s[j][1] * sl2 : -INFINITY;
-            s[j][2] = k0 <= see_b ? s[j][2] * sl2 : -INFINITY;
-            s[j][3] = k0 + 1 <= see_b ? s[j][3] * sl2 : -INFINITY;
+            s[j][0] = k0 <= see_a && k0 >= from_a ? s[j][0] * sl2 : -INFINITY;
+            s[j][1] = k0 + 1 <= see_a && k0 + 1 >= from_a ? s[j][1] * sl2 : -INFINITY;
+            s[j][2] = k0 <= see_b && k0 >= from_b ? s[j][2] * sl2 : -INFINITY;
+            s[j][3] = k0 + 1 <= see_b && k0 + 1 >= from_b ? s[j][3] * sl2 : -INFINITY;
             mx_a = fmaxf(mx_a, fmaxf(s[j][0], s[j][1]));
             mx_b = fmaxf(mx_b, fmaxf(s[j][2], s[j][3]));
         }
@@ -296,14 +312,14 @@ latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __res
     }
 
     if (splits == 1) {
-        const float inv_a = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, inv_b = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const int r = half ? r_b : r_a;
             if (r >= n_rows) continue;
             const int row = row0 + r;
+            float inv = l_run[half] > 0.f ? 1.f / l_run[half] : 0.f;
+            if (sinks != nullptr) inv = sink_share(m_run[half], l_run[half], sinks[row % heads]);
             __nv_bfloat16* dst = out + ((long long)(q_first + row / heads) * heads + row % heads) * dv + 2 * t4;
-            const float inv = half ? inv_b : inv_a;
 #pragma unroll
             for (int i = 0; i < MAXDV8; ++i)
                 if (i < dv8)
@@ -336,7 +352,7 @@ template <bool SMALL>
 __global__ void __launch_bounds__(128)
 latent_attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                          __nv_bfloat16* __restrict__ out, const int* __restrict__ cu_q, int n_entries,
-                         int heads, int dv, int splits) {
+                         int heads, int dv, int splits, const float* __restrict__ sinks) {
     constexpr int BM = SMALL ? 16 : 64;
     __shared__ float wgt[MAX_SPLITS];
     __shared__ float inv_den;
@@ -360,7 +376,8 @@ latent_attn_merge_kernel(const float* __restrict__ part_o, const float* __restri
             den = fmaf(w, part_ml[(first + (long long)s * BM) * 2 + 1], den);
         }
         den = warp_sum(den);
-        if (threadIdx.x == 0) inv_den = den > 0.f ? 1.f / den : 0.f;
+        if (threadIdx.x == 0)
+            inv_den = sinks != nullptr ? sink_share(mx, den, sinks[(row0 + r) % heads]) : den > 0.f ? 1.f / den : 0.f;
     }
     __syncthreads();
     const int row = row0 + r;
@@ -379,7 +396,8 @@ latent_attn_merge_kernel(const float* __restrict__ part_o, const float* __restri
 template <bool SMALL, int MAXDK16, int MAXDV8>
 int launch(const __nv_bfloat16* q, __nv_bfloat16* out, float* part_o, float* part_ml, const __nv_bfloat16* pool,
            const int* cu_q, const int* kv_len, const int* block_table, int max_blocks, int num_pages, int page_size,
-           int n_entries, int tiles, int splits, int heads, int dk, int dv, float scale, int* err, cudaStream_t st) {
+           int n_entries, int tiles, int splits, int heads, int dk, int dv, float scale, int window,
+           const float* sinks, int* err, cudaStream_t st) {
     constexpr int BM = SMALL ? 16 : 64;
     constexpr int KT = KeyTile<SMALL>::value;
     int page_shift = 0;
@@ -393,10 +411,11 @@ int launch(const __nv_bfloat16* q, __nv_bfloat16* out, float* part_o, float* par
         attr_set = true;
     }
     int rc = crane_launch(kern, dim3(tiles, splits), dim3(128), smem, st, q, out, part_o, part_ml, pool, cu_q,
-                          kv_len, block_table, max_blocks, num_pages, page_shift, n_entries, heads, dk, dv, scale, err);
+                          kv_len, block_table, max_blocks, num_pages, page_shift, n_entries, heads, dk, dv, scale, window,
+                          sinks, err);
     if (rc != 0 || splits == 1) return rc;
     return crane_launch(latent_attn_merge_kernel<SMALL>, dim3(tiles, BM), dim3(128), 0, st, (const float*)part_o,
-                        (const float*)part_ml, out, cu_q, n_entries, heads, dv, splits);
+                        (const float*)part_ml, out, cu_q, n_entries, heads, dv, splits, sinks);
 }
 
 }  // namespace
@@ -412,8 +431,8 @@ CRANE_API int crane_latent_attention_mma_supports(int dk, int dv) {
 CRANE_API int crane_latent_attention_mma(const void* q, void* out, float* part_o, float* part_ml, const void* pool,
                                          const int* cu_q, const int* kv_len, const int* block_table,
                                          int max_blocks, int num_pages, int page_size, int n_entries, int tiles,
-                                         int splits, int small, int heads, int dk, int dv, float scale, int* err,
-                                         cudaStream_t st) {
+                                         int splits, int small, int heads, int dk, int dv, float scale, int window,
+                                         const float* sinks, int* err, cudaStream_t st) {
     if (tiles <= 0 || n_entries <= 0) return 0;
     if (!crane_latent_attention_mma_supports(dk, dv) || splits < 1 || splits > MAX_SPLITS ||
         (splits > 1 && (part_o == nullptr || part_ml == nullptr)))
@@ -423,7 +442,7 @@ CRANE_API int crane_latent_attention_mma(const void* q, void* out, float* part_o
     const auto* pb = (const __nv_bfloat16*)pool;
 #define CRANE_LATENT_LAUNCH(W, A, B)                                                                          \
     return launch<W, A, B>(qb, ob, part_o, part_ml, pb, cu_q, kv_len, block_table, max_blocks, num_pages,     \
-                           page_size, n_entries, tiles, splits, heads, dk, dv, scale, err, st)
+                           page_size, n_entries, tiles, splits, heads, dk, dv, scale, window, sinks, err, st)
     const bool narrow = dk <= 128 && dv <= 128;
     if (small) {
         if (narrow) CRANE_LATENT_LAUNCH(true, 8, 16);

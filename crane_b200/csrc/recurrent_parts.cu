@@ -4,17 +4,25 @@
 //     u  = beta_t (v_t - S^T k_t)            (`delta`: the delta rule's correction; else u = v_t)
 //     S <- S + k_t u^T
 //     o_t = S^T q_t                          (the read-out sees the token's own write)
+// or, `bonus`,
+//     o_t = S^T r_t + b_t v_t                (the read-out sees the state BEFORE the token's write, and of the
+//     S <- diag(w_t) S + k_t v_t^T            token itself only b_t = sum_i r_i u_i k_i, a number per head)
 //
 // `matrix_state_scan` walks each request's tokens in order.  Columns of S do not talk to one another:
 // a CTA holds a block of columns of one (request, head), a column's rows spread over LANES lanes of a
 // warp (ROWS rows each, in registers), dot products over the rows finished by shuffles.  The inputs of
 // every token (q, k, v, w, beta) are 32-bit rows of an `aux` buffer that a prep kernel writes:
 //   * `conv_delta_prep`: q, k, v through a short causal convolution over time and silu, q and k scaled
-//     to unit length per head, beta = sigmoid(.), w = exp(-exp(A) softplus(. + dt)) per head; the last
-//     taps - 1 inputs of the convolutions are part of the request's state (`conv_state_update`);
+//     to unit length per head, beta = sigmoid(.), w = exp(-exp(A) softplus(. + dt)) per head (unless a decay
+//     per key channel comes from elsewhere); the last taps - 1 inputs of the convolutions are part of the
+//     request's state (`conv_state_update`);
 //   * `decay_gate_prep`: q scaled, k, v, and w = sigmoid(z)^(1 / tau) per key channel with z a
-//     low-rank product plus bias.
-// `head_norm_gate` norms each head's read-out over dv, applies the weight and silu(gate).
+//     low-rank product plus bias;
+//   * `bonus_prep`: r, k, v and the number b per head.
+// `token_shift_mix` forms what the projections of the bonus recurrence read, h + (h' - h) mu with h' the
+// previous token's row, which is part of the request's state.  `low_rank_expand` is the second matrix of a
+// low-rank product with what follows it (a decay, or nothing).
+// `head_norm_gate` norms each head's read-out over dv, applies the weight and silu(gate) or sigmoid(gate).
 // `head_talk_mix` and `pair_norm_mean` belong to attention whose heads exchange their weights and to
 // two mixers side by side.
 // The state lives in 32-bit in the request's slot, in the order the scan's threads hold it:
@@ -29,8 +37,9 @@ __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); 
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 
 // ------------------------------------------------------ convolution + delta-rule inputs
-// proj row: [q (G d) | k (G d) | v (H dv) | gate (H dv) | b (H) | a (H)].  aux row: [q (G d) | k (G d) |
-// v (H dv) | w (H) | beta (H)].  conv_w [2 G d + H dv][taps] float.  conv_state: inside the slot's state
+// proj row: [q (G d) | k (G d) | v (H dv) | ...] with b (H) at column `b_off` and a (H) at `a_off` (-1: no
+// decay is formed here).  aux row: [q (G d) | k (G d) | v (H dv) | ...] with w (H) at `w_off` and beta (H) at
+// `beta_off`.  conv_w [2 G d + H dv][taps] float.  conv_state: inside the slot's state
 // at `conv_off`, [taps - 1][C].  Grid (tokens, blocks of heads); a warp per head of q, k or v (2 G + H of
 // them): a q or k head is written as the convolution left it, then scaled by the same lanes once its
 // sum of squares is known.
@@ -41,8 +50,8 @@ conv_delta_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
                        const int* __restrict__ slots, int n_slots, const float* __restrict__ state,
                        long long slot_stride, long long conv_off, const float* __restrict__ conv_w, int taps,
                        const float* __restrict__ a_log, const float* __restrict__ dt_bias,
-                       float* __restrict__ aux, int aux_cols, int H, int G, int d, int dv, float key_eps,
-                       float q_scale, int* err) {
+                       float* __restrict__ aux, int aux_cols, int H, int G, int d, int dv, int b_off, int a_off,
+                       int w_off, int beta_off, float key_eps, float q_scale, int* err) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -87,10 +96,10 @@ conv_delta_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
     }
     if (blockIdx.y == 0) {
         for (int h = threadIdx.x; h < H; h += blockDim.x) {
-            const long long row = (long long)t * cols + C + H * dv;
-            const float b = proj.load(row + h), a = proj.load(row + H + h);
-            out[C + h] = expf(-expf(a_log[h]) * softplus_f(a + dt_bias[h]));
-            out[C + H + h] = 1.f / (1.f + expf(-b));
+            const long long row = (long long)t * cols;
+            const float b = proj.load(row + b_off + h);
+            if (a_off >= 0) out[w_off + h] = expf(-expf(a_log[h]) * softplus_f(proj.load(row + a_off + h) + dt_bias[h]));
+            out[beta_off + h] = 1.f / (1.f + expf(-b));
         }
     }
 }
@@ -164,9 +173,221 @@ decay_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
         out[2 * hd + c] = proj.load(row + 2 * hd + c);
 }
 
+// ------------------------------------------------------ what the bonus recurrence's projections read
+// out[g][t][c] = h[t][c] + (h'[t][c] - h[t][c]) mu[g][c] for every mix g, h' the row of the request's token before
+// (zeros before its first one).  The row before a portion's first token lies in the slot, float [hidden] at
+// `row_off`; the thread that reads it there puts the portion's last row in its place.  Grid (tokens, column
+// blocks).
+template <typename T>
+__global__ void __launch_bounds__(256)
+token_shift_mix_kernel(const T* __restrict__ h, const float* __restrict__ mu, int mixes,
+                       const int* __restrict__ tok_entry, const int* __restrict__ cu_q,
+                       const int* __restrict__ kv_len, const int* __restrict__ slots, int n_slots,
+                       float* __restrict__ state, long long slot_stride, long long row_off, T* __restrict__ out,
+                       long long group_stride, int hidden, int* err) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int e = tok_entry[t];
+    if (e < 0) return;
+    const int first = cu_q[e], end = cu_q[e + 1];
+    const int slot = slots[e];
+    if (slot < 0 || slot >= n_slots) {
+        if (threadIdx.x == 0 && blockIdx.y == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
+        return;
+    }
+    const bool opens = t == first && kv_len[e] == end - first;       // the request's first token
+    float* kept = state + (long long)slot * slot_stride + row_off;
+    const long long row = (long long)t * hidden;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < hidden; c += gridDim.y * blockDim.x) {
+        const float x = to_f32(h[row + c]);
+        float before;
+        if (t == first) {
+            before = opens ? 0.f : kept[c];
+            kept[c] = to_f32(h[(long long)(end - 1) * hidden + c]);
+        } else {
+            before = to_f32(h[row - hidden + c]);
+        }
+        const float diff = before - x;
+        for (int g = 0; g < mixes; ++g)
+            out[(long long)g * group_stride + row + c] = from_f32<T>(fmaf(diff, mu[(long long)g * hidden + c], x));
+    }
+}
+
+// proj row: [r (H d) | k (H d) | v (H dv) | ...].  aux row: [r | k | v | ... ] with b (H) at column `b_off`:
+// b = sum_i r_i u_i k_i.  A warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(128)
+bonus_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, const float* __restrict__ u,
+                  float* __restrict__ aux, int aux_cols, int b_off, int n, int H, int d, int dv) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (wid >= (long long)n * H) return;
+    const int t = (int)(wid / H), h = (int)(wid % H);
+    if (tok_entry[t] < 0) return;
+    const long long row = (long long)t * cols;
+    float* out = aux + (long long)t * aux_cols;
+    const int hd = H * d;
+    float b = 0.f;
+    for (int c = lane; c < d; c += 32) {
+        const float r = proj.load(row + h * d + c), k = proj.load(row + hd + h * d + c);
+        out[h * d + c] = r;
+        out[hd + h * d + c] = k;
+        b = fmaf(r * u[h * d + c], k, b);
+    }
+    for (int c = lane; c < dv; c += 32) out[2 * hd + h * dv + c] = proj.load(row + 2 * hd + h * dv + c);
+    b = warp_sum(b);
+    if (lane == 0) out[b_off + h] = b;
+}
+
+// ------------------------------------------------------ the second matrix of a low-rank product
+// z[t][c] = sum_r in(low[t][low_off + r]) w[c][r], in the identity or tanh, then
+//   LR_PLAIN       out (T) = z
+//   LR_SOFT_DECAY  out (float) = exp(-exp(rate[c / per_rate]) softplus(z + bias[c]))
+//   LR_EXP_DECAY   out (float) = exp(-exp(z + bias[c]))
+// Up to two such products of one row of `low` (one mixer's decay and gate) are one launch.
+enum LowRankKind : int { LR_PLAIN = 0, LR_SOFT_DECAY = 1, LR_EXP_DECAY = 2 };
+struct LowRankPart {
+    const void* w;                // [n_out][ld_w] (MMA) or [rank][n_out] (FP32 cores), T
+    const float* bias;
+    const float* rate;
+    void* out;
+    long long out_ld;
+    int low_off, rank, ld_w, n_out, kind, tanh_in, per_rate;
+};
+struct LowRankArgs { LowRankPart part[2]; int col_blocks0; };       // column blocks of the first part
+
+template <typename T>
+__device__ __forceinline__ void low_rank_store(const LowRankPart& p, int t, int c, float z) {
+    const long long at = (long long)t * p.out_ld + c;
+    if (p.kind == LR_PLAIN) reinterpret_cast<T*>(p.out)[at] = from_f32<T>(z);
+    else {
+        z += p.bias[c];
+        const float r = p.kind == LR_SOFT_DECAY ? expf(p.rate[c / p.per_rate]) * softplus_f(z) : expf(z);
+        reinterpret_cast<float*>(p.out)[at] = expf(-r);
+    }
+}
+
+// FP32 cores: a CTA takes 16 tokens and 128 columns, a thread per column; r in order 0 .. rank - 1.
+constexpr int LR_TT = 16;
+template <typename T>
+__global__ void __launch_bounds__(128)
+low_rank_simt_kernel(GemmOut<T> low, int cols, const int* __restrict__ tok_entry, const LowRankArgs args, int n) {
+    extern __shared__ float xs[];                     // [LR_TT][rank]
+    pdl_launch_dependents();
+    pdl_wait();
+    const bool second = (int)blockIdx.y >= args.col_blocks0;
+    const LowRankPart& p = args.part[second ? 1 : 0];
+    const int t0 = blockIdx.x * LR_TT, nt = min(LR_TT, n - t0);
+    for (int i = threadIdx.x; i < LR_TT * p.rank; i += blockDim.x) {
+        const int tt = i / p.rank, r = i % p.rank;
+        float v = 0.f;
+        if (tt < nt && tok_entry[t0 + tt] >= 0) {
+            v = low.load((long long)(t0 + tt) * cols + p.low_off + r);
+            if (p.tanh_in) v = tanhf(v);
+        }
+        xs[i] = v;
+    }
+    __syncthreads();
+    const int c = ((int)blockIdx.y - (second ? args.col_blocks0 : 0)) * 128 + threadIdx.x;
+    if (c >= p.n_out) return;
+    const T* w = reinterpret_cast<const T*>(p.w);
+    float acc[LR_TT];
+#pragma unroll
+    for (int tt = 0; tt < LR_TT; ++tt) acc[tt] = 0.f;
+    for (int r = 0; r < p.rank; ++r) {
+        const float wv = to_f32(w[(long long)r * p.n_out + c]);
+#pragma unroll
+        for (int tt = 0; tt < LR_TT; ++tt) acc[tt] = fmaf(wv, xs[tt * p.rank + r], acc[tt]);
+    }
+#pragma unroll
+    for (int tt = 0; tt < LR_TT; ++tt)
+        if (tt < nt && tok_entry[t0 + tt] >= 0) low_rank_store<T>(p, t0 + tt, c, acc[tt]);
+}
+
+// Tensor cores (bf16, warp-level MMA), ranks up to 256: a CTA takes 64 tokens (16 per warp) and 64 columns, or
+// (FEW: a step of at most 16 tokens) 16 tokens and 64 columns, 16 per warp.  The weights' rows are stored
+// `ld_w` = rank rounded up to 16 long, zero-filled.
+__device__ __forceinline__ void lr_ldsm_x4(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3, const void* p) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(a));
+}
+constexpr int LR_COLS = 64;
+template <bool FEW>
+__global__ void __launch_bounds__(128)
+low_rank_mma_kernel(GemmOut<__nv_bfloat16> low, int cols, const int* __restrict__ tok_entry, const LowRankArgs args,
+                    int n) {
+    constexpr int BM = FEW ? 16 : 64;
+    extern __shared__ __align__(16) unsigned char lr_smem[];
+    const bool second = (int)blockIdx.y >= args.col_blocks0;
+    const LowRankPart& p = args.part[second ? 1 : 0];
+    const int ld = p.ld_w + 8;
+    __nv_bfloat16* a_s = reinterpret_cast<__nv_bfloat16*>(lr_smem);      // [BM][ld]
+    __nv_bfloat16* w_s = a_s + BM * ld;                                   // [64][ld]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+    const int t0 = blockIdx.x * BM;
+    const int c0 = ((int)blockIdx.y - (second ? args.col_blocks0 : 0)) * LR_COLS;
+    pdl_launch_dependents();
+    // the weights depend on no earlier kernel
+    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.w);
+    const int pieces = p.ld_w >> 3;
+    for (int i = threadIdx.x; i < LR_COLS * pieces; i += blockDim.x) {
+        const int r = i / pieces, q = i % pieces;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (c0 + r < p.n_out) v = *reinterpret_cast<const uint4*>(w + (long long)(c0 + r) * p.ld_w + q * 8);
+        *reinterpret_cast<uint4*>(w_s + r * ld + q * 8) = v;
+    }
+    pdl_wait();
+    for (int i = threadIdx.x; i < BM * p.ld_w; i += blockDim.x) {
+        const int tt = i / p.ld_w, r = i % p.ld_w;
+        float v = 0.f;
+        if (r < p.rank && t0 + tt < n && tok_entry[t0 + tt] >= 0) {
+            v = low.load((long long)(t0 + tt) * cols + p.low_off + r);
+            if (p.tanh_in) v = tanhf(v);
+        }
+        a_s[tt * ld + r] = __float2bfloat16_rn(v);
+    }
+    __syncthreads();
+    const int wrow = FEW ? 0 : warp * 16;
+    constexpr int NB = FEW ? 2 : 8;                   // blocks of 8 columns a warp takes
+    const int wcol = FEW ? warp * 16 : 0;
+    float acc[NB][4];
+#pragma unroll
+    for (int i = 0; i < NB; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int ks = 0; ks < (p.ld_w >> 4); ++ks) {
+        uint32_t a0, a1, a2, a3;
+        lr_ldsm_x4(a0, a1, a2, a3, a_s + (wrow + (lane & 15)) * ld + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int j = 0; j < NB / 2; ++j) {
+            uint32_t b0, b1, b2, b3;
+            lr_ldsm_x4(b0, b1, b2, b3, w_s + (wcol + j * 16 + (lane & 7) + (lane >> 4) * 8) * ld + ks * 16 + ((lane >> 3) & 1) * 8);
+            asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                         : "+f"(acc[2 * j][0]), "+f"(acc[2 * j][1]), "+f"(acc[2 * j][2]), "+f"(acc[2 * j][3])
+                         : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+            asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                         : "+f"(acc[2 * j + 1][0]), "+f"(acc[2 * j + 1][1]), "+f"(acc[2 * j + 1][2]), "+f"(acc[2 * j + 1][3])
+                         : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b2), "r"(b3));
+        }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int t = t0 + wrow + g + 8 * half;
+        if (t >= n || tok_entry[t] < 0) continue;
+#pragma unroll
+        for (int i = 0; i < NB; ++i) {
+            const int c = c0 + wcol + i * 8 + 2 * t4;
+            if (c < p.n_out) low_rank_store<__nv_bfloat16>(p, t, c, acc[i][2 * half]);
+            if (c + 1 < p.n_out) low_rank_store<__nv_bfloat16>(p, t, c + 1, acc[i][2 * half + 1]);
+        }
+    }
+}
+
 // ------------------------------------------------------ the recurrence
 // grid (entries, heads, column blocks); block = COLS columns x LANES lanes.  aux offsets: q_off, k_off,
-// v_off, w_off, beta_off (beta only with `delta`); q/k head of head h is h / qk_rep; w is [Hqk d]
+// v_off, w_off, beta_off (the delta rule's beta, or the bonus b); q/k head of head h is h / qk_rep; w is [H d]
 // (w_vec) or [H].  o_raw float [n][H dv].
 // Tokens come in tiles of `tile_tokens` whose vectors all threads copy into shared memory with 4-byte
 // asynchronous copies, the next tile while the current one is walked: a tile's fetch from DRAM is as
@@ -198,10 +419,11 @@ __device__ __forceinline__ float lanes_sum(float x, int lanes) {
 }
 // A lane holds ROWS neighbouring rows of its column.  FULL: the lanes' rows are exactly the dk rows; no row
 // is tested and a lane reads its part of a vector 16 bytes at a time.  WVEC: a decay per row (else one per
-// head).  DELTA: the delta rule's correction.  LANES: the lanes of a column when the kernel is compiled for
+// head).  MODE: what a token does (plain, the delta rule's correction, bonus).  LANES: the lanes of a column when the kernel is compiled for
 // them (0: any).  The first `walkers` threads walk the tokens; one more warp does nothing but copy the next
 // tile of tokens into shared memory meanwhile, since a walking warp's time is its instructions per token.
-template <int ROWS, bool FULL, bool DELTA, bool WVEC, int LANES>
+enum ScanMode : int { SCAN_PLAIN = 0, SCAN_DELTA = 1, SCAN_BONUS = 2 };
+template <int ROWS, bool FULL, int MODE, bool WVEC, int LANES>
 __global__ void __launch_bounds__(288)
 matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off, int k_off, int v_off, int w_off,
                          int beta_off, int qk_rep, const int* __restrict__ cu_q,
@@ -209,6 +431,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                          float* __restrict__ state, long long slot_stride, float* __restrict__ o_raw,
                          int H, int dk, int dv, int lanes_rt, int cols_per_block, int tile_tokens, int vec4,
                          int walkers, int* err) {
+    constexpr bool DELTA = MODE == SCAN_DELTA, BONUS = MODE == SCAN_BONUS;
     extern __shared__ __align__(16) float tile[];     // two tiles of [tile_tokens][3 dk + cols + 2, to a multiple of 4]
     pdl_launch_dependents();
     pdl_wait();
@@ -238,7 +461,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
     auto place = [&](int x, int& so, int& dofs) {                    // unit x of a token: where from, where to
         if (x < nq) so = q_off + hq * dk + x * unit, dofs = x * unit;
         else if (x < 2 * nq) so = k_off + hq * dk + (x - nq) * unit, dofs = dk + (x - nq) * unit;
-        else if (WVEC && x < 3 * nq) so = w_off + hq * dk + (x - 2 * nq) * unit, dofs = 2 * dk + (x - 2 * nq) * unit;
+        else if (WVEC && x < 3 * nq) so = w_off + h * dk + (x - 2 * nq) * unit, dofs = 2 * dk + (x - 2 * nq) * unit;
         else {
             const int y = x - (WVEC ? 3 : 2) * nq;
             so = v_off + h * dv + c0 + y * unit, dofs = 3 * dk + y * unit;
@@ -269,7 +492,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                 if (WVEC) b[3 * dk + cols_per_block] = 1.f;
                 else cp_async4(b + 3 * dk + cols_per_block, a + w_off + h);
             } else if (wl == 1) {
-                if (DELTA) cp_async4(b + 3 * dk + cols_per_block + 1, a + beta_off + h);
+                if (DELTA || BONUS) cp_async4(b + 3 * dk + cols_per_block + 1, a + beta_off + h);
                 else b[3 * dk + cols_per_block + 1] = 1.f;
             }
         }
@@ -326,6 +549,17 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                 }
                 const float vv = tp[3 * dk + vcol];    // a column that is not live reads a neighbour's and writes nothing
                 const float ws = WVEC ? 1.f : tp[3 * dk + cols_per_block];
+                if (BONUS) {
+                    float rd = 0.f;
+#pragma unroll
+                    for (int i = 0; i < ROWS; ++i) {
+                        rd = fmaf(s[i], qv[i], rd);
+                        s[i] = fmaf(s[i], WVEC ? wv[i] : ws, kv[i] * vv);
+                    }
+                    rd = lanes_sum<LANES>(rd, lanes);
+                    if (live && lane == 0) *op = fmaf(tp[3 * dk + cols_per_block + 1], vv, rd);
+                    continue;
+                }
                 float dot = 0.f;
 #pragma unroll
                 for (int i = 0; i < ROWS; ++i) {
@@ -356,13 +590,14 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
 }
 
 // ------------------------------------------------------ head norm and gate
-// out[t][h dv + c] = o_raw / rms_over_dv(o_raw) * norm_w[c] * silu(gate[t][gate_off + h dv + c]); a warp per
+// out[t][h dv + c] = o_raw / rms_over_dv(o_raw) * norm_w[h norm_step + c] * act(gate[t][gate_off + h dv + c]),
+// norm_step 0 (a weight that the heads share) or dv, act silu or, `sigmoid_gate`, sigmoid; a warp per
 // (token, head).
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols, int gate_off,
-                      const int* __restrict__ tok_entry, const float* __restrict__ norm_w, float eps,
-                      T* __restrict__ out, int n, int H, int dv) {
+                      const int* __restrict__ tok_entry, const float* __restrict__ norm_w, int norm_step,
+                      int sigmoid_gate, float eps, T* __restrict__ out, int n, int H, int dv) {
     pdl_launch_dependents();
     pdl_wait();
     const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -377,7 +612,8 @@ head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols
     const float rstd = rsqrtf(ss / (float)dv + eps);
     for (int c = lane; c < dv; c += 32) {
         const float g = proj.load((long long)t * cols + gate_off + h * dv + c);
-        out[((long long)t * H + h) * dv + c] = from_f32<T>(o[c] * rstd * norm_w[c] * silu_f(g));
+        const float a = sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g);
+        out[((long long)t * H + h) * dv + c] = from_f32<T>(o[c] * rstd * norm_w[h * norm_step + c] * a);
     }
 }
 
@@ -451,8 +687,9 @@ CRANE_API int crane_conv_delta_prep(int dtype, const void* proj, const float* pr
                                     const int* kv_len, const int* slots, int n_slots, float* state,
                                     long long slot_stride, long long conv_off, const float* conv_w, int taps,
                                     const float* a_log, const float* dt_bias, float* aux, int aux_cols,
-                                    int n_tokens, int n_entries, int H, int G, int d, int dv, float key_eps,
-                                    float q_scale, int* err, cudaStream_t st) {
+                                    int n_tokens, int n_entries, int H, int G, int d, int dv, int b_off, int a_off,
+                                    int w_off, int beta_off, float key_eps, float q_scale, int* err,
+                                    cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     const int C = 2 * G * d + H * dv;
     if (taps < 1 || taps > MAX_TAPS) return (int)cudaErrorInvalidValue;
@@ -464,7 +701,8 @@ CRANE_API int crane_conv_delta_prep(int dtype, const void* proj, const float* pr
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
         int rc = crane_launch(conv_delta_prep_kernel<T>, dim3(n_tokens, by), dim3(256), 0, st, p, cols, tok_entry,
                               cu_q, kv_len, slots, n_slots, (const float*)state, slot_stride, conv_off, conv_w,
-                              taps, a_log, dt_bias, aux, aux_cols, H, G, d, dv, key_eps, q_scale, err);
+                              taps, a_log, dt_bias, aux, aux_cols, H, G, d, dv, b_off, a_off, w_off, beta_off, key_eps,
+                              q_scale, err);
         if (rc != 0 || taps == 1) return rc;
         return crane_launch(conv_state_update_kernel<T>, dim3((C + 127) / 128, n_entries), dim3(128), 0, st, p,
                             cols, cu_q, kv_len, slots, n_slots, state, slot_stride, conv_off, taps, C);
@@ -486,6 +724,82 @@ CRANE_API int crane_decay_gate_prep(int dtype, const void* proj, const float* pr
     });
 }
 
+CRANE_API int crane_token_shift_mix(int dtype, const void* h, const float* mu, int mixes, const int* tok_entry,
+                                    const int* cu_q, const int* kv_len, const int* slots, int n_slots,
+                                    float* state, long long slot_stride, long long row_off, void* out,
+                                    long long group_stride, int n_tokens, int hidden, int* err, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    int by = (hidden + 255) / 256;
+    while (by > 1 && (long long)n_tokens * by > 4 * 148) by = (by + 1) / 2;
+    DISPATCH_T(dtype, return crane_launch(token_shift_mix_kernel<T>, dim3(n_tokens, by), dim3(256), 0, st, (const T*)h,
+                                          mu, mixes, tok_entry, cu_q, kv_len, slots, n_slots, state, slot_stride,
+                                          row_off, (T*)out, group_stride, hidden, err));
+}
+
+CRANE_API int crane_bonus_prep(int dtype, const void* proj, const float* proj_parts, int n_parts,
+                               long long part_stride, int cols, const int* tok_entry, const float* u, float* aux,
+                               int aux_cols, int b_off, int n_tokens, int H, int d, int dv, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    const long long warps = (long long)n_tokens * H;
+    DISPATCH_T(dtype, {
+        GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
+        return crane_launch(bonus_prep_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, st, p, cols,
+                            tok_entry, u, aux, aux_cols, b_off, n_tokens, H, d, dv);
+    });
+}
+
+// `mma` 1: bf16, weights [n_out][ld_w] with ld_w a multiple of 16 and at most 256, zero-filled behind the rank,
+// 16-byte aligned; 0: weights [rank][n_out] on the FP32 cores.  A second part with n_out2 = 0 is absent.
+CRANE_API int crane_low_rank_expand(int dtype, const void* low, const float* low_parts, int n_parts,
+                                    long long part_stride, int cols, const int* tok_entry, int mma,
+                                    const void* w1, const float* bias1, const float* rate1, int per_rate1,
+                                    void* out1, long long out_ld1, int low_off1, int rank1, int ld_w1, int n_out1,
+                                    int kind1, int tanh1, const void* w2, const float* bias2, const float* rate2,
+                                    int per_rate2, void* out2, long long out_ld2, int low_off2, int rank2, int ld_w2,
+                                    int n_out2, int kind2, int tanh2, int n_tokens, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    LowRankArgs a;
+    a.part[0] = LowRankPart{w1, bias1, rate1, out1, out_ld1, low_off1, rank1, ld_w1, n_out1, kind1, tanh1, per_rate1 > 0 ? per_rate1 : 1};
+    a.part[1] = LowRankPart{w2, bias2, rate2, out2, out_ld2, low_off2, rank2, ld_w2, n_out2, kind2, tanh2, per_rate2 > 0 ? per_rate2 : 1};
+    int widest = rank1;
+    if (n_out2 > 0 && rank2 > widest) widest = rank2;
+    if (mma) {
+        int ldm = ld_w1;
+        for (int i = 0; i < (n_out2 > 0 ? 2 : 1); ++i) {
+            const LowRankPart& p = a.part[i];
+            if (dtype != 1 || p.ld_w < p.rank || p.ld_w % 16 || p.ld_w <= 0 || p.ld_w > 256 || ((uintptr_t)p.w & 15))
+                return (int)cudaErrorInvalidValue;
+            if (p.ld_w > ldm) ldm = p.ld_w;
+        }
+        const int b0 = (n_out1 + LR_COLS - 1) / LR_COLS, b1 = n_out2 > 0 ? (n_out2 + LR_COLS - 1) / LR_COLS : 0;
+        a.col_blocks0 = b0;
+        const bool few = n_tokens <= 16;
+        const int bm = few ? 16 : 64;
+        const size_t smem = (size_t)(bm + LR_COLS) * (ldm + 8) * sizeof(__nv_bfloat16);
+        auto kern = few ? low_rank_mma_kernel<true> : low_rank_mma_kernel<false>;
+        static bool attr_set = false;
+        if (!attr_set) {
+            cudaFuncSetAttribute(low_rank_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 80 * 1024);
+            cudaFuncSetAttribute(low_rank_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 80 * 1024);
+            attr_set = true;
+        }
+        GemmOut<__nv_bfloat16> l{(const __nv_bfloat16*)low, low_parts, n_parts, part_stride};
+        return crane_launch(kern, dim3((n_tokens + bm - 1) / bm, b0 + b1), dim3(128), smem, st, l, cols, tok_entry, a,
+                            n_tokens);
+    }
+    const int b0 = (n_out1 + 127) / 128, b1 = n_out2 > 0 ? (n_out2 + 127) / 128 : 0;
+    a.col_blocks0 = b0;
+    const size_t smem = (size_t)LR_TT * (widest > 0 ? widest : 1) * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    DISPATCH_T(dtype, {
+        if (smem > 48 * 1024)
+            cudaFuncSetAttribute(low_rank_simt_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        GemmOut<T> l{(const T*)low, low_parts, n_parts, part_stride};
+        return crane_launch(low_rank_simt_kernel<T>, dim3((n_tokens + LR_TT - 1) / LR_TT, b0 + b1), dim3(128), smem, st, l,
+                            cols, tok_entry, a, n_tokens);
+    });
+}
+
 // The scan's geometry for a key size: (rows per lane, lanes per column); 0 rows: too wide.
 CRANE_API int crane_matrix_state_plan(int dk, int* rows, int* lanes) {
     int r = dk <= 256 ? 8 : 16, l = 1;
@@ -497,13 +811,15 @@ CRANE_API int crane_matrix_state_plan(int dk, int* rows, int* lanes) {
 }
 
 CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off, int k_off, int v_off, int w_off,
-                                      int beta_off, int w_vec, int delta, int qk_rep, const int* cu_q,
+                                      int beta_off, int w_vec, int mode, int qk_rep, const int* cu_q,
                                       const int* kv_len, const int* slots, int n_slots, float* state,
                                       long long slot_stride, float* o_raw, int n_entries, int H, int dk, int dv,
                                       int* err, cudaStream_t st) {
     if (n_entries <= 0) return 0;
     int rows, lanes;
-    if (crane_matrix_state_plan(dk, &rows, &lanes) || dv <= 0 || qk_rep <= 0) return (int)cudaErrorInvalidValue;
+    if (crane_matrix_state_plan(dk, &rows, &lanes) || dv <= 0 || qk_rep <= 0 || mode < 0 || mode > 2 ||
+        (mode == SCAN_BONUS && !w_vec))
+        return (int)cudaErrorInvalidValue;
     int cpb = 256 / lanes;
     if (cpb > dv) cpb = dv;
     // few entries and heads: narrower blocks of columns, so that more SMs walk (a column's result does not
@@ -519,13 +835,16 @@ CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off,
     if (tile_tokens < 1) return (int)cudaErrorInvalidValue;
     const size_t smem = 2 * (size_t)tile_tokens * per_token;
     const bool full = rows * lanes == dk;
-    using Kern = decltype(&matrix_state_scan_kernel<8, true, true, true, 0>);
+    using Kern = decltype(&matrix_state_scan_kernel<8, true, SCAN_DELTA, true, 0>);
+    const bool delta = mode == SCAN_DELTA;
     auto pick = [&](auto rows_c, auto lanes_c) -> Kern {
         constexpr int R = decltype(rows_c)::value, L = decltype(lanes_c)::value;
-        if (full) return delta ? (w_vec ? matrix_state_scan_kernel<R, true, true, true, L> : matrix_state_scan_kernel<R, true, true, false, L>)
-                               : (w_vec ? matrix_state_scan_kernel<R, true, false, true, L> : matrix_state_scan_kernel<R, true, false, false, L>);
-        return delta ? (w_vec ? matrix_state_scan_kernel<R, false, true, true, 0> : matrix_state_scan_kernel<R, false, true, false, 0>)
-                     : (w_vec ? matrix_state_scan_kernel<R, false, false, true, 0> : matrix_state_scan_kernel<R, false, false, false, 0>);
+        if (mode == SCAN_BONUS)
+            return full ? matrix_state_scan_kernel<R, true, SCAN_BONUS, true, L> : matrix_state_scan_kernel<R, false, SCAN_BONUS, true, 0>;
+        if (full) return delta ? (w_vec ? matrix_state_scan_kernel<R, true, SCAN_DELTA, true, L> : matrix_state_scan_kernel<R, true, SCAN_DELTA, false, L>)
+                               : (w_vec ? matrix_state_scan_kernel<R, true, SCAN_PLAIN, true, L> : matrix_state_scan_kernel<R, true, SCAN_PLAIN, false, L>);
+        return delta ? (w_vec ? matrix_state_scan_kernel<R, false, SCAN_DELTA, true, 0> : matrix_state_scan_kernel<R, false, SCAN_DELTA, false, 0>)
+                     : (w_vec ? matrix_state_scan_kernel<R, false, SCAN_PLAIN, true, 0> : matrix_state_scan_kernel<R, false, SCAN_PLAIN, false, 0>);
     };
     using std::integral_constant;
     Kern kern;
@@ -541,14 +860,14 @@ CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off,
 
 CRANE_API int crane_head_norm_gate(int dtype, const float* o_raw, const void* proj, const float* proj_parts,
                                    int n_parts, long long part_stride, int cols, int gate_off,
-                                   const int* tok_entry, const float* norm_w, float eps, void* out, int n_tokens,
-                                   int H, int dv, cudaStream_t st) {
+                                   const int* tok_entry, const float* norm_w, int norm_step, int sigmoid_gate,
+                                   float eps, void* out, int n_tokens, int H, int dv, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     const long long warps = (long long)n_tokens * H;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
         return crane_launch(head_norm_gate_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, st, o_raw, p,
-                            cols, gate_off, tok_entry, norm_w, eps, (T*)out, n_tokens, H, dv);
+                            cols, gate_off, tok_entry, norm_w, norm_step, sigmoid_gate, eps, (T*)out, n_tokens, H, dv);
     });
 }
 

@@ -19,7 +19,7 @@ from .csrc import build
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
 
 _SIGNATURES = {
-    "crane_embed_gather": [I, P, P, P, I, I, I, P, I, P, P],
+    "crane_embed_gather": [I, P, P, P, P, I, I, I, P, I, P, P],
     "crane_add_rmsnorm": [I, P, P, P, I, L, P, P, P, I, I, F, P],
     "crane_rope_norm_cache": [I, P, P, I, L, I, P, P, P, I, P, P, I, P, P, F, P, P, P, I, I, I, I,
                               I, I, I, I, I, I, I, F, P, P],
@@ -27,9 +27,9 @@ _SIGNATURES = {
     "crane_to_float": [I, P, P, L, P],
     "crane_sum_parts": [P, I, L, L, P, L, I, I, P],
     "crane_gemm_simt": [I, I, P, P, P, P, I, I, I, L, L, L, P],
-    "crane_gemm_bf16_tcgen05": [P, P, P, P, I, I, I, L, L, L, I, I, I, I, I, L, I, P, L, P, P],
-    "crane_gemm_bf16_pair": [P, P, P, P, I, I, I, L, L, L, I, I, I, P, P],
-    "crane_paged_attention_simt": [I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P],
+    "crane_gemm_bf16_tcgen05": [P, P, P, P, I, I, I, L, L, L, I, I, I, I, I, L, I, I, I, P, L, P, P],
+    "crane_gemm_bf16_pair": [P, P, P, P, I, I, I, L, L, L, I, I, I, I, I, P, P],
+    "crane_paged_attention_simt": [I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P, P],
     "crane_paged_decode_attention_supports": [I, I, I],
     "crane_paged_decode_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, P],
     "crane_paged_prefill_attention_supports": [I, I, I],
@@ -41,10 +41,10 @@ _SIGNATURES = {
     "crane_embed_bigram": [I, P, P, P, P, I, I, I, I, L, L, P, P, P, P, P, I, P, I, P, P],
     "crane_combine_layernorm": [I, P, P, L, I, P, P, I, L, P, P, I, L, P, P, P, P, P, P, P, P, I, I, F, P],
     "crane_xielu": [I, P, P, I, L, P, L, P, P],
-    "crane_latent_prep": [I, P, P, I, L, I, I, I, I, I, I, I, I, P, P, I, P, P, P, I, I, I, P, P, F, P, I, P, P],
+    "crane_latent_prep": [I, P, P, I, L, I, I, I, I, I, P, P, I, I, I, I, I, P, P, I, P, P, P, I, I, I, P, P, F, P, I, P, P],
     "crane_head_linear": [I, P, P, I, L, I, I, I, P, I, I, P, P, I, L, I, I, P, P, I, I, I, I, P],
     "crane_latent_attention_mma_supports": [I, I],
-    "crane_latent_attention_mma": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P],
+    "crane_latent_attention_mma": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P],
     "crane_embed_sinusoid": [I, P, P, P, P, P, P, I, I, I, P, I, P, P],
     "crane_stream_enter": [P, P, P, I, I, P],
     "crane_add_normed_norm": [I, P, P, P, I, L, P, P, P, P, I, I, F, F, P],
@@ -54,13 +54,17 @@ _SIGNATURES = {
     "crane_projection_norm_cache": [I, P, P, I, L, I, P, P, P, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I,
                                     P, P, I, I, P, P, P],
     "crane_streams_norm": [I, P, L, I, P, P, P, I, L, P, P, P, P, P, P, I, I, F, P],
-    "crane_route_grouped": [P, I, P, P, I, I, I, I, I, I, P],
-    "crane_gated_activation": [I, P, P, I, L, P, I, I, P, I, I, I, I, P],
-    "crane_conv_delta_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, I, P, P, P, I, I, I, I, I, I, I, F, F, P, P],
+    "crane_route_grouped": [P, I, P, P, I, I, I, I, I, I, I, P],
+    "crane_gated_activation": [I, P, P, I, L, P, I, I, P, I, I, I, I, I, P],
+    "crane_conv_delta_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P],
+    "crane_token_shift_mix": [I, P, P, I, P, P, P, P, I, P, L, L, P, L, I, I, P, P],
+    "crane_bonus_prep": [I, P, P, I, L, I, P, P, P, I, I, I, I, I, I, P],
+    "crane_low_rank_expand": [I, P, P, I, L, I, P, I, P, P, P, I, P, L, I, I, I, I, I, I, P, P, P, I, P, L, I, I, I, I, I, I,
+                              I, P],
     "crane_decay_gate_prep": [I, P, P, I, L, I, P, P, P, I, F, F, P, I, I, I, I, I, P],
     "crane_matrix_state_plan": [I, P, P],
     "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, I, I, I, I, P, P],
-    "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, F, P, I, I, I, P],
+    "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, I, I, F, P, I, I, I, P],
     "crane_head_talk_mix": [I, P, P, P, P, I, I, I, I, I, P],
     "crane_pair_norm_mean": [I, P, P, I, L, P, P, I, L, P, P, F, P, I, I, P],
     "crane_delta_rule_prep": [I, P, P, I, L, I, P, P, P, P, P, I, I, I, I, F, F, P],
@@ -168,11 +172,12 @@ class Kernels:
             raise KernelError(f"{what}: CUDA error {code}")
 
     # ---- elementwise ---------------------------------------------------
-    def embed_gather(self, tokens, table, x, err, deferred=None) -> None:
-        """``deferred`` int32 [R]: a token id <= -2 is read from its row -id - 2."""
+    def embed_gather(self, tokens, table, x, err, deferred=None, raw=None) -> None:
+        """``deferred`` int32 [R]: a token id <= -2 is read from its row -id - 2.  ``raw``: the rows once more,
+        in the table's type."""
         n, hidden = x.shape
         self._check(self.lib.crane_embed_gather(_dt(table.dtype), tokens.data_ptr(), table.data_ptr(),
-                                                x.data_ptr(), n, hidden, table.shape[0],
+                                                x.data_ptr(), _ptr(raw), n, hidden, table.shape[0],
                                                 deferred.data_ptr() if deferred is not None else None,
                                                 deferred.numel() if deferred is not None else 0,
                                                 err.data_ptr(), self._stream(x)), "embed_gather")
@@ -264,16 +269,19 @@ class Kernels:
                                          out.numel(), pq.data_ptr(), self._stream(out)), "xielu")
 
     def latent_prep(self, proj: Act, cols, q_off, dkv_off, heads, dim, rot, rank, rot_dims, cos, sin,
-                    positions, tok_entry, block_table, pool, page_size, norm_w, eps, q_abs, err) -> None:
+                    positions, tok_entry, block_table, pool, page_size, norm_w, eps, q_abs, err,
+                    cq_off: int = -1, cq_w=None, cq_out=None) -> None:
         """Latent attention's cache write and query rotation; ``dkv_off`` < 0: the
-        layer writes no cache.  ``pool`` [pages, 1, page_size, rank + rot]."""
+        layer writes no cache; ``q_off`` < 0: no query is rotated.  ``pool`` [pages, 1, page_size, rank + rot].
+        ``cq_off`` >= 0: the RMS norm of the query latent at that column, times ``cq_w``, goes to
+        ``cq_out`` [n, query rank]."""
         whole, parts, n_parts, stride = _split(proj)
         self._check(self.lib.crane_latent_prep(
-            _dt(q_abs.dtype), whole, parts, n_parts, stride, int(cols), int(q_off), int(dkv_off), heads, dim,
-            rot, rank, rot_dims, cos.data_ptr(), sin.data_ptr(), cos.shape[0], positions.data_ptr(),
+            _dt(pool.dtype), whole, parts, n_parts, stride, int(cols), int(q_off), int(dkv_off), int(cq_off),
+            cq_out.shape[1] if cq_out is not None else 0, _ptr(cq_w), _ptr(cq_out), heads, dim, rot, rank, rot_dims, cos.data_ptr(), sin.data_ptr(), cos.shape[0], positions.data_ptr(),
             tok_entry.data_ptr(), block_table.data_ptr(), block_table.shape[1], pool.shape[0], page_size,
-            pool.data_ptr(), _ptr(norm_w), float(eps), q_abs.data_ptr(), q_abs.shape[0], err.data_ptr(),
-            self._stream(q_abs)), "latent_prep")
+            pool.data_ptr(), _ptr(norm_w), float(eps), _ptr(q_abs), positions.shape[0], err.data_ptr(),
+            self._stream(pool)), "latent_prep")
 
     def head_linear(self, x: Act, x_cols, x_off, x_head, w, n_in, n_out, out, out_pitch, out_head,
                     heads, tok_entry=None, gate: Optional[Act] = None, g_cols=0, g_off=0) -> None:
@@ -291,17 +299,20 @@ class Kernels:
         return bool(self.lib.crane_latent_attention_mma_supports(int(dk), int(dv)))
 
     def latent_attention_mma(self, q, out, pool, cu_q, kv_len, block_table, page_size, tiles, splits,
-                             small: bool, heads, dk, dv, scale, part_o, part_ml, err) -> None:
+                             small: bool, heads, dk, dv, scale, part_o, part_ml, err, window: int = 0,
+                             sinks=None) -> None:
         """Attention over cache rows [dk] whose values are their leading ``dv`` columns,
         ``heads`` query heads per token (bfloat16).  One launch takes the entries of at
         most 16 rows (tokens x heads) in tiles of 16 (``small``) or the others in tiles
         of 64; ``tiles``: at least how many there are.  ``splits`` > 1 cuts every tile's
-        keys into slices that a second kernel merges (scratch: ``part_o``, ``part_ml``)."""
+        keys into slices that a second kernel merges (scratch: ``part_o``, ``part_ml``).  ``window``: a
+        token sees the last ``window`` positions, its own among them (0: all).  ``sinks`` float [heads]: a
+        candidate of that score without a value joins every softmax of its head."""
         self._check(self.lib.crane_latent_attention_mma(
             q.data_ptr(), out.data_ptr(), _ptr(part_o), _ptr(part_ml), pool.data_ptr(), cu_q.data_ptr(),
             kv_len.data_ptr(), block_table.data_ptr(), block_table.shape[1], pool.shape[0], page_size,
             kv_len.shape[0], int(tiles), int(splits), 1 if small else 0, heads, dk, dv, float(scale),
-            err.data_ptr(), self._stream(q)), "latent_attention_mma")
+            int(window), _ptr(sinks), err.data_ptr(), self._stream(q)), "latent_attention_mma")
 
     # ---- the stream of layers that norm what they add, routed feed-forwards ----
     def embed_sinusoid(self, tokens, positions, table, freq, x, keep, err, deferred=None) -> None:
@@ -420,26 +431,28 @@ class Kernels:
             out.shape[0], streams.shape[2], float(eps), self._stream(out)), "streams_norm")
 
     def route_grouped(self, z, correction, route, experts: int, top: int, groups: int, keep: int,
-                      shared_gate: bool) -> None:
-        """Per row of float ``z`` [n, >= experts (+ 1)]: scores = softmax over the experts; the ``top`` largest
+                      shared_gate: bool, sigmoid: bool = False) -> None:
+        """Per row of float ``z`` [n, >= experts (+ 1)]: scores = softmax over the experts (``sigmoid``: the
+        sigmoid of each); the ``top`` largest
         of score + correction among the experts of the ``keep`` best of ``groups`` groups are chosen;
         ``route`` [n, experts (+ 1)] gets their scores (zero elsewhere) and, ``shared_gate``, the
         sigmoid of column ``experts`` behind them."""
         assert z.dtype == torch.float32 and z.stride(1) == 1 and route.is_contiguous()
         self._check(self.lib.crane_route_grouped(
             z.data_ptr(), z.stride(0), _ptr(correction), route.data_ptr(), z.shape[0], int(experts), int(top),
-            int(groups), int(keep), 1 if shared_gate else 0, self._stream(z)), "route_grouped")
+            int(groups), int(keep), 1 if shared_gate else 0, 1 if sigmoid else 0, self._stream(z)), "route_grouped")
 
     def gated_activation(self, gu: Act, out, route=None, experts: int = 0, per_expert: int = 0,
-                         routed_cols: int = 0, shared_gate: bool = False) -> None:
+                         routed_cols: int = 0, shared_gate: bool = False, on_input: bool = False) -> None:
         """out[t, c] = silu(gu[t, c]) * gu[t, cols + c], times the column's routing weight:
         ``route[t, c // per_expert]`` for c < routed_cols, behind them ``route[t, experts]``
-        (``shared_gate``) or 1."""
+        (``shared_gate``) or 1.  ``on_input``: the weight multiplies what the expert reads instead, so both of
+        its products: silu(w gate) * (w up)."""
         whole, parts, n_parts, stride = _split(gu)
         self._check(self.lib.crane_gated_activation(
             _dt(out.dtype), whole, parts, n_parts, stride, out.data_ptr(), out.shape[0], out.shape[1], _ptr(route),
-            int(experts), int(per_expert), int(routed_cols), 1 if shared_gate else 0, self._stream(out)),
-            "gated_activation")
+            int(experts), int(per_expert), int(routed_cols), 1 if shared_gate else 0, 1 if on_input else 0,
+            self._stream(out)), "gated_activation")
 
     # ---- recurrences with a matrix state per head -----------------------
     def matrix_state_plan(self, dk: int):
@@ -451,18 +464,25 @@ class Kernels:
         return r.value, l.value
 
     def conv_delta_prep(self, proj: Act, cols, ctx, state, conv_off, conv_w, taps, a_log, dt_bias, aux, H, G, d, dv,
-                        key_eps, q_scale, err, dtype) -> None:
+                        key_eps, q_scale, err, dtype, b_off=None, a_off=None, w_off=None, beta_off=None) -> None:
         """Rows [q | k | v | gate | b | a] of a merged projection -> ``aux`` rows [q | k | v | w | beta] in
-        32-bit: q, k, v through their short convolutions (weights ``conv_w`` [channels, taps]) and silu,
+        32-bit (``b_off``, ``a_off`` and ``w_off``, ``beta_off``: other columns for them behind q, k, v;
+        ``a_off`` < 0: no decay is formed): q, k, v through their short convolutions (weights ``conv_w`` [channels, taps]) and silu,
         q and k to unit length per head (q times ``q_scale``), w = exp(-exp(a_log) softplus(a + dt_bias)),
         beta = sigmoid(b).  The convolutions' last taps - 1 inputs live in ``state`` [slots, floats] at
         ``conv_off`` and are replaced by a second kernel."""
         whole, parts, n_parts, stride = _split(proj)
+        C = 2 * G * d + H * dv
+        b_off = C + H * dv if b_off is None else b_off
+        a_off = b_off + H if a_off is None else a_off
+        w_off = C if w_off is None else w_off
+        beta_off = C + H if beta_off is None else beta_off
         self._check(self.lib.crane_conv_delta_prep(
             _dt(dtype), whole, parts, n_parts, stride, int(cols), ctx.tok_entry.data_ptr(), ctx.cu_q.data_ptr(),
             ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0),
-            int(conv_off), conv_w.data_ptr(), int(taps), a_log.data_ptr(), dt_bias.data_ptr(), aux.data_ptr(),
-            aux.shape[1], aux.shape[0], ctx.kv_len.shape[0], H, G, d, dv, float(key_eps), float(q_scale),
+            int(conv_off), conv_w.data_ptr(), int(taps), _ptr(a_log), _ptr(dt_bias), aux.data_ptr(),
+            aux.shape[1], aux.shape[0], ctx.kv_len.shape[0], H, G, d, dv, int(b_off), int(a_off), int(w_off),
+            int(beta_off), float(key_eps), float(q_scale),
             err.data_ptr(), self._stream(aux)), "conv_delta_prep")
 
     def decay_gate_prep(self, proj: Act, cols, tok_entry, a2t, bias, inv_tau, q_scale, aux, H, d, dv, dtype) -> None:
@@ -474,24 +494,98 @@ class Kernels:
             bias.data_ptr(), a2t.shape[0], float(inv_tau), float(q_scale), aux.data_ptr(), aux.shape[1],
             aux.shape[0], H, d, dv, self._stream(aux)), "decay_gate_prep")
 
-    def matrix_state_scan(self, aux, offs, w_vec: bool, delta: bool, qk_rep: int, ctx, state, o_raw, H, dk, dv,
+    def token_shift_mix(self, h, mu, ctx, state, row_off, out, err) -> None:
+        """out[g, t] = h[t] + (h' - h[t]) mu[g] for every mix g (``mu`` float [mixes, hidden], ``out`` [mixes, n,
+        hidden]), h' the request's row before: h[t - 1], or for a portion's first token the row kept in
+        ``state`` [slots, floats] at ``row_off`` (zeros before the request's first token), which the
+        portion's last row replaces."""
+        self._check(self.lib.crane_token_shift_mix(
+            _dt(h.dtype), h.data_ptr(), mu.data_ptr(), mu.shape[0], ctx.tok_entry.data_ptr(), ctx.cu_q.data_ptr(),
+            ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0),
+            int(row_off), out.data_ptr(), out.stride(0), h.shape[0], h.shape[1], err.data_ptr(), self._stream(h)),
+            "token_shift_mix")
+
+    def bonus_prep(self, proj: Act, cols, tok_entry, u, aux, b_off, H, d, dv, dtype) -> None:
+        """Rows [r | k | v | ...] of a projection -> ``aux`` rows [r | k | v | ...] in 32-bit with b = sum_i r_i u_i
+        k_i per head at column ``b_off`` (``u`` float [H, d])."""
+        whole, parts, n_parts, stride = _split(proj)
+        self._check(self.lib.crane_bonus_prep(
+            _dt(dtype), whole, parts, n_parts, stride, int(cols), tok_entry.data_ptr(), u.data_ptr(), aux.data_ptr(),
+            aux.stride(0), int(b_off), aux.shape[0], H, d, dv, self._stream(aux)), "bonus_prep")
+
+    @dataclass
+    class LowRank:
+        """The second matrix of a low-rank product (``w`` from ``pack_low_rank``), the columns of the first one's
+        result that it reads, and what becomes of z: ``kind`` "plain" (z in the model dtype), "soft_decay"
+        (exp(-exp(rate[c // per_rate]) softplus(z + bias)) in float) or "exp_decay" (exp(-exp(z + bias)) in float).
+        ``tanh``: of what it reads.  ``out`` [n, >= n_out], rows may be strided."""
+        w: torch.Tensor
+        rank: int
+        low_off: int
+        n_out: int
+        out: Optional[torch.Tensor] = None
+        kind: str = "plain"
+        bias: Optional[torch.Tensor] = None
+        rate: Optional[torch.Tensor] = None
+        per_rate: int = 1
+        tanh: bool = False
+        mma: bool = False
+
+    LOW_RANK_KINDS = {"plain": 0, "soft_decay": 1, "exp_decay": 2}
+    LOW_RANK_MMA_MOST = 256
+
+    @classmethod
+    def pack_low_rank(cls, w, exact: bool):
+        """(the second matrix [n_out, rank] as the kernel reads it, whether the tensor-core kernel takes it):
+        rows padded with zeros to a multiple of 16, or [rank, n_out] for the FP32 cores."""
+        n_out, rank = w.shape
+        padded = -(-rank // 16) * 16
+        if exact or w.dtype != torch.bfloat16 or padded > cls.LOW_RANK_MMA_MOST:
+            return w.t().contiguous(), False
+        out = torch.zeros((n_out, padded), dtype=w.dtype, device=w.device)
+        out[:, :rank] = w
+        return out, True
+
+    def low_rank_expand(self, low: Act, cols, tok_entry, n, dtype, a: "Kernels.LowRank", b=None) -> None:
+        """One or two second matrices of low-rank products over rows of ``low``, one launch."""
+        whole, parts, n_parts, stride = _split(low)
+        assert b is None or b.mma == a.mma
+
+        def args(p):
+            if p is None:
+                return [None, None, None, 1, None, 0, 0, 0, 0, 0, 0, 0]
+            return [p.w.data_ptr(), _ptr(p.bias), _ptr(p.rate), int(p.per_rate), p.out.data_ptr(), p.out.stride(0),
+                    int(p.low_off), int(p.rank), p.w.shape[1] if p.mma else 0, int(p.n_out),
+                    self.LOW_RANK_KINDS[p.kind], 1 if p.tanh else 0]
+        self._check(self.lib.crane_low_rank_expand(
+            _dt(dtype), whole, parts, n_parts, stride, int(cols), tok_entry.data_ptr(), 1 if a.mma else 0, *args(a),
+            *args(b), int(n), self._stream(a.out)), "low_rank_expand")
+
+    SCAN_MODES = {"plain": 0, "delta": 1, "bonus": 2}
+
+    def matrix_state_scan(self, aux, offs, w_vec: bool, mode, qk_rep: int, ctx, state, o_raw, H, dk, dv,
                           err) -> None:
-        """The recurrence S <- diag(w) S; u = beta (v - S^T k) (``delta``) or v; S <- S + k u^T; o = S^T q
+        """The recurrence S <- diag(w) S; u = beta (v - S^T k) (``mode`` "delta" or True) or v ("plain" or
+        False); S <- S + k u^T; o = S^T q; or (``mode`` "bonus") o = S^T q + beta v; S <- diag(w) S + k v^T,
         over every entry's tokens, from and to ``state`` [slots, floats] (its leading H * rows * lanes * dv
         floats).  ``offs``: columns of q, k, v, w, beta in ``aux``; ``o_raw`` float [n, H dv]."""
         self._check(self.lib.crane_matrix_state_scan(
-            aux.data_ptr(), aux.shape[1], *[int(o) for o in offs], 1 if w_vec else 0, 1 if delta else 0, int(qk_rep),
+            aux.data_ptr(), aux.shape[1], *[int(o) for o in offs], 1 if w_vec else 0,
+            self.SCAN_MODES[mode] if isinstance(mode, str) else int(bool(mode)), int(qk_rep),
             ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
             state.stride(0), o_raw.data_ptr(), ctx.kv_len.shape[0], H, dk, dv, err.data_ptr(),
             self._stream(o_raw)), "matrix_state_scan")
 
-    def head_norm_gate(self, o_raw, proj: Act, cols, gate_off, tok_entry, norm_w, eps, out, H, dv) -> None:
-        """out = o_raw / rms(o_raw per head) * norm_w * silu(gate columns of ``proj``)."""
+    def head_norm_gate(self, o_raw, proj: Act, cols, gate_off, tok_entry, norm_w, eps, out, H, dv,
+                       sigmoid: bool = False) -> None:
+        """out = o_raw / rms(o_raw per head) * norm_w * silu(gate columns of ``proj``), or ``sigmoid`` of them.
+        ``norm_w`` [dv] (shared by the heads) or [H dv]."""
+        norm_step = 0 if norm_w.numel() == dv else dv
         whole, parts, n_parts, stride = _split(proj)
         self._check(self.lib.crane_head_norm_gate(
             _dt(out.dtype), o_raw.data_ptr(), whole, parts, n_parts, stride, int(cols), int(gate_off),
-            tok_entry.data_ptr(), norm_w.data_ptr(), float(eps), out.data_ptr(), out.shape[0], H, dv,
-            self._stream(out)), "head_norm_gate")
+            tok_entry.data_ptr(), norm_w.data_ptr(), norm_step, 1 if sigmoid else 0, float(eps), out.data_ptr(),
+            out.shape[0], H, dv, self._stream(out)), "head_norm_gate")
 
     def head_talk_mix(self, cross, talk, tok_entry, out, H, G, dv, out_head) -> None:
         """out[t, h] = sum_g talk[h, g] cross[t, g, h // (H / G)]; heads ``out_head`` apart in ``out``."""
@@ -553,18 +647,20 @@ class Kernels:
     PAIR_TILES = (256, 224, 192, 128)
 
     def gemm_pair(self, x, w, bias, out, err, bn: int = 256, silu_mul: bool = False,
-                  tile_rows: int = 256) -> None:
+                  tile_rows: int = 256, group_features: int = 0, group_rows: int = 0) -> None:
         """out[M,N] (bf16) = x[M,K] @ w[N,K]^T (+ bias) for many tokens, every
         256 x ``bn`` tile computed by two SMs together (tcgen05 cta_group::2).
         ``silu_mul`` as in ``gemm_tcgen05``.  ``tile_rows`` 512: tiles of 512
-        tokens x ``bn`` (192, 224 or 256) features, two accumulators per SM."""
+        tokens x ``bn`` (192, 224 or 256) features, two accumulators per SM.
+        ``group_features`` as in ``gemm_tcgen05``."""
         M, K = x.shape
         N = w.shape[0]
         assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and bn in self.PAIR_TILES
         assert tuple(out.shape) == ((M, N // 2) if silu_mul else (M, N))
         self._check(self.lib.crane_gemm_bf16_pair(
             x.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), M, N, K, x.stride(0), w.stride(0),
-            out.stride(0), bn, tile_rows, 1 if silu_mul else 0, err.data_ptr(), self._stream(x)), "gemm_pair")
+            out.stride(0), bn, tile_rows, 1 if silu_mul else 0, int(group_features), int(group_rows),
+            err.data_ptr(), self._stream(x)), "gemm_pair")
 
     WIDE_TILES = (256, 224, 192, 160, 128)
 
@@ -658,7 +754,8 @@ class Kernels:
         return bn, rows
 
     def gemm_tcgen05(self, x, w, bias, out, err, split_k: int = 1, swap: bool = False,
-                     bn: int = 128, silu_mul: bool = False, prefetch=None, tile_rows: int = 128) -> None:
+                     bn: int = 128, silu_mul: bool = False, prefetch=None, tile_rows: int = 128,
+                     group_features: int = 0, group_rows: int = 0) -> None:
         """out[M,N] = x[M,K] @ w[N,K]^T (+ bias).  ``swap``: the weight fills the
         128-row side of the MMA and ``bn`` (16..64) covers the tokens.  With
         ``split_k`` > 1 ``out`` is float [slices, M, N] of partial sums.
@@ -667,7 +764,10 @@ class Kernels:
         bytes) of what the step's next product will stream, asked into L2 by the
         narrow-tile kernel while it runs (a hint; ignored by the other kernels).
         ``tile_rows`` 256: tiles of 256 tokens x ``bn`` (128, 192 or 256) features
-        (bf16 output, no slices, no swap, no silu)."""
+        (bf16 output, no slices, no swap, no silu).
+        ``group_features`` > 0: output feature f is of the rows ``group_rows * (f // group_features)`` onwards
+        of the tensor that ``x`` [M, K] is the first rows of (projections that each read an input of
+        their own, as one product); a multiple of a tile's features (128 with ``swap``, else ``bn``)."""
         M, K = x.shape
         N = w.shape[0]
         if silu_mul:
@@ -683,18 +783,19 @@ class Kernels:
         self._check(self.lib.crane_gemm_bf16_tcgen05(
             a.data_ptr(), b.data_ptr(), _ptr(bias), out.data_ptr(), a.shape[0], b.shape[0], K,
             a.stride(0), b.stride(0), ld, bn, tile_rows, 1 if out.dtype == torch.float32 else 0,
-            1 if swap else 0, split_k, stride, 1 if silu_mul else 0,
+            1 if swap else 0, split_k, stride, 1 if silu_mul else 0, int(group_features), int(group_rows),
             prefetch[0] if prefetch else None, prefetch[1] if prefetch else 0, err.data_ptr(),
             self._stream(x)), "gemm_tcgen05")
 
     # ---- attention ------------------------------------------------------
     def paged_attention_simt(self, q, out, k_pool, v_pool, positions, tok_entry, block_table,
                              page_size, nq, nkv, d, window, scale, err, dv=None, v_stride=None,
-                             sink: bool = False, out_cross=None) -> None:
+                             sink: bool = False, out_cross=None, sinks=None) -> None:
         """``dv``: width of a value row (default: the keys'), ``v_stride``: elements
         between value rows (default ``dv``).  With ``v_pool`` the key pool itself and
         ``v_stride == d`` the values are the leading ``dv`` columns of the key rows.
-        ``sink``: the softmax has one more candidate of score 0 that has no value.
+        ``sink``: the softmax has one more candidate of score 0 that has no value; ``sinks`` float [nq]: of
+        a score of its own per query head.
         ``out_cross`` float [n, nq, nkv, dv]: every query head's weights are applied to the values
         of EVERY key/value head (its scores still come from its own group's keys) and written there
         instead of ``out`` (which may be None), for attention whose heads exchange their weights."""
@@ -704,8 +805,8 @@ class Kernels:
             _dt(q.dtype), q.data_ptr(), _ptr(out), k_pool.data_ptr(), v_pool.data_ptr(),
             positions.data_ptr(), tok_entry.data_ptr(), block_table.data_ptr(),
             block_table.shape[1], k_pool.shape[0], page_size, q.shape[0], nq, nkv, d, dv, v_stride,
-            int(window), float(scale), 1 if sink else 0, _ptr(out_cross), err.data_ptr(), self._stream(q)),
-            "paged_attention_simt")
+            int(window), float(scale), 1 if sink else 0, _ptr(sinks), _ptr(out_cross), err.data_ptr(),
+            self._stream(q)), "paged_attention_simt")
 
     # ---- attention whose scores are worked on, and the block around it
     @dataclass

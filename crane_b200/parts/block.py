@@ -9,6 +9,9 @@ unadded ("pending") and receives the one of the block before it.
 x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))); then an optional per-layer
 token input joins the stream.
 
+``output_norm_residual``: the sublayers read x itself and only their results are normed,
+x += norm1(mixer(x)); x += norm2(ffn(x)).
+
 ``parallel_depth_average``: both branches read norms of the same x, their sum
 is added once, and what the next layer reads is a weighted sum of all layer
 results so far.
@@ -25,6 +28,7 @@ from __future__ import annotations
 
 import torch
 
+from ..config.spec import STREAM_COPY
 from ..weights.loader import TensorSpec
 from .base import Part, build_part, register_block, register_part
 from .norm import BranchSum, StreamUpdate, add_normed, combine_and_norm
@@ -215,6 +219,33 @@ class SandwichResidualBlock:
             _, raw = add_normed(x, f, self.norm2b, rt, raw_name=raw_name)
         if self.side is not None:
             self.side.forward(x, raw, ctx, rt)
+        return None
+
+
+@register_block("output_norm_residual")
+class OutputNormResidualBlock:
+    """x += norm1(mixer(x)), x += norm2(ffn(x)): the sublayers read the stream as it is, in the model type.
+    parts: ``norm1``, ``mixer`` and, unless the layer has no feed-forward, ``norm2``, ``ffn`` (a constant that
+    scales what is added is the norm's ``gain``).  Each addition is one kernel with the result's norm and the
+    copy of the new stream that the next reader takes; the copy lives in the workspace buffer
+    ``STREAM_COPY``, which the embedding part fills first (its ``model_copy``).  Nothing is left pending."""
+
+    def __init__(self, layer_spec):
+        p = layer_spec.parts
+        self.norm1, self.mixer = build_part(p["norm1"]), build_part(p["mixer"])
+        self.ffn = build_part(p["ffn"]) if "ffn" in p else None
+        self.norm2 = build_part(p["norm2"]) if self.ffn is not None else None
+
+    def parts(self):
+        return [q for q in (self.norm1, self.mixer, self.norm2, self.ffn) if q is not None]
+
+    def forward(self, x, pending, ctx, cache, rt):
+        h = rt.ws.get(STREAM_COPY, x.shape[0], x.shape[1], rt.dtype)
+        a = self.mixer.forward(h, ctx, cache, rt)
+        add_normed(x, a, self.norm1, rt, raw_name=STREAM_COPY)
+        if self.ffn is not None:
+            f = self.ffn.forward(h, ctx, rt)
+            add_normed(x, f, self.norm2, rt, raw_name=STREAM_COPY)
         return None
 
 

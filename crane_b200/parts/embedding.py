@@ -16,7 +16,8 @@ from .base import Part, register_part
 @register_part("embed", "token_embedding")
 class TokenEmbedding(Part):
     """params: ``vocab_size``, ``hidden_size``, ``table`` (tensor name behind the prefix; default
-    "weight").  Tensor [V,H]."""
+    "weight"), ``model_copy`` (a workspace buffer that also gets the rows, in the model type: for blocks whose
+    sublayers read the stream itself).  Tensor [V,H]."""
     kind = "embed"
 
     @classmethod
@@ -31,7 +32,9 @@ class TokenEmbedding(Part):
         """Writes the float residual rows ``x`` [N,H] for int32 ``tokens`` [N].
         A token id <= -2 names row ``-id - 2`` of ``deferred`` (int32, on the
         device): a token sampled by an earlier launch that the host has not read."""
-        rt.kernels.embed_gather(tokens, self.table, x, rt.err, deferred)
+        copy = self.params.get("model_copy")
+        raw = rt.ws.get(copy, x.shape[0], x.shape[1], rt.dtype) if copy else None
+        rt.kernels.embed_gather(tokens, self.table, x, rt.err, deferred, raw)
         rt.launches += 1
 
 

@@ -15,21 +15,24 @@ from .base import Part, register_part
 
 @register_part("ffn", "swiglu")
 class SwiGLU(Part):
-    """params: ``hidden_size``, ``intermediate_size``.  Tensors:
-    ``<prefix>gate_proj.weight`` [I,H], ``up_proj.weight`` [I,H], ``down_proj.weight`` [H,I]."""
+    """params: ``hidden_size``, ``intermediate_size``, ``names`` (gate, up, down; default
+    "gate_proj.weight", ...).  Tensors: gate [I,H], up [I,H], down [H,I]."""
     kind = "ffn"
+    NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
 
     @classmethod
     def manifest(cls, spec):
         h, i = spec.params["hidden_size"], spec.params["intermediate_size"]
         p = spec.prefix
-        return {p + "gate_proj.weight": TensorSpec((i, h)), p + "up_proj.weight": TensorSpec((i, h)),
-                p + "down_proj.weight": TensorSpec((h, i))}
+        nm = dict(cls.NAMES, **(spec.params.get("names") or {}))
+        return {p + nm["gate"]: TensorSpec((i, h)), p + nm["up"]: TensorSpec((i, h)),
+                p + nm["down"]: TensorSpec((h, i))}
 
     def load(self, weights, rt):
         p = self.prefix
+        nm = dict(self.NAMES, **(self.params.get("names") or {}))
         self.inter = int(self.params["intermediate_size"])
-        gate, up = weights.pop(p + "gate_proj.weight"), weights.pop(p + "up_proj.weight")
+        gate, up = weights.pop(p + nm["gate"]), weights.pop(p + nm["up"])
         # On the tensor-core path the merged matrix holds 16 gate rows, then the 16 up rows of
         # the same features, and so on: a tile of the product then has both halves of a
         # feature side by side and its epilogue can apply silu(gate) * up itself.
@@ -40,7 +43,7 @@ class SwiGLU(Part):
                 2 * self.inter, h).contiguous()
         else:
             self.gate_up = torch.cat([gate, up], dim=0).contiguous()
-        self.down = weights[p + "down_proj.weight"]
+        self.down = weights[p + nm["down"]]
 
     def forward(self, h, ctx, rt):
         act = rt.ws.get("ffn_act", h.shape[0], self.inter, rt.dtype)
@@ -209,14 +212,16 @@ class RoutedExperts(Part):
 @register_part("ffn", "grouped_experts")
 class GroupedExperts(Part):
     """A mixture of gated feed-forwards down_e(silu(gate_e(h)) * up_e(h)).  The router's logits
-    z = W_r h are formed in 32-bit; scores s = softmax(z) over ALL experts; an expert's choice score
+    z = W_r h are formed in 32-bit; scores s = softmax(z) over ALL experts, or sigmoid(z); an expert's choice score
     is s plus a learnt correction; experts come in ``groups`` equal groups of neighbours, a group
     counts as much as its best choice score, and only experts of the ``keep`` best groups can be
     chosen; the ``top`` largest choice scores among those are chosen (ties to the lower index) and
     weighted by their scores s, without the correction and without renormalising.  An optional shared
     expert of the same form runs for every token and is added, times sigmoid(w_sg . h) if it has a gate.
+    With ``weight_on`` "input" an expert's weight scales what it reads, expert_e(s_e h), not what it gives.
     params: ``hidden_size``, ``experts``, ``top``, ``groups``, ``keep``, ``expert_size``, ``shared_size``
-    (0: none), ``correction`` (tensor name or None), ``shared_gate`` (tensor name or None), ``names``.
+    (0: none), ``correction`` (tensor name or None), ``shared_gate`` (tensor name or None), ``scores``
+    ("softmax", the default, or "sigmoid"), ``weight_on`` ("output", the default, or "input"), ``names``.
     Tensors: router [E,H]; correction [E] (float); per expert gate, up [F,H], down [H,F]; shared gate,
     up [Fs,H], down [H,Fs]; shared_gate [1,H].
 
@@ -260,6 +265,10 @@ class GroupedExperts(Part):
         _, self.E, self.F, self.Fs = self._sizes(a)
         self.top, self.groups = int(a["top"]), int(a.get("groups") or 1)
         self.keep = int(a.get("keep") or self.groups)
+        scores, on = str(a.get("scores") or "softmax"), str(a.get("weight_on") or "output")
+        if scores not in ("softmax", "sigmoid") or on not in ("output", "input"):
+            raise ValueError(f"{p}: no scores '{scores}' or no weight on '{on}'")
+        self.sigmoid, self.on_input = scores == "sigmoid", on == "input"
         if not 0 < self.top <= self.E or self.E % self.groups or not 0 < self.keep <= self.groups:
             raise ValueError(f"{p}: {self.top} of {self.E} experts in {self.groups} groups ({self.keep} kept) cannot be chosen")
         self.correction = weights[p + a["correction"]] if a.get("correction") else None
@@ -280,9 +289,10 @@ class GroupedExperts(Part):
         n, k = h.shape[0], rt.kernels
         z = rt.linear(h, self.router, None, "router_logits", out_dtype=torch.float32)
         route = rt.ws.get("route_weights", n, self.E + (1 if self.shared_gate else 0), torch.float32)
-        k.route_grouped(z, self.correction, route, self.E, self.top, self.groups, self.keep, self.shared_gate)
+        k.route_grouped(z, self.correction, route, self.E, self.top, self.groups, self.keep, self.shared_gate,
+                        sigmoid=self.sigmoid)
         gu = rt.linear(h, self.gate_up, None, "experts_gate_up")
         act = rt.ws.get("experts_act", n, self.inter, rt.dtype)
-        k.gated_activation(gu, act, route, self.E, self.F, self.E * self.F, self.shared_gate)
+        k.gated_activation(gu, act, route, self.E, self.F, self.E * self.F, self.shared_gate, on_input=self.on_input)
         rt.launches += 2
         return rt.linear(act, self.down, None, "experts_down")

@@ -14,7 +14,8 @@ from .base import Part, register_part
 class RMSNorm(Part):
     """params: ``size``, ``eps``; ``weight`` (tensor name behind the prefix, default "weight");
     ``weight_offset`` (the norm multiplies by offset + w: 0, or 1 for weights stored around
-    zero; folded into the weight when it is loaded).  Tensor [size], kept float."""
+    zero; folded into the weight when it is loaded); ``gain`` (a constant that multiplies the normed row,
+    folded into the weight too: what a block scales a sublayer's result by).  Tensor [size], kept float."""
     kind = "norm"
 
     @classmethod
@@ -29,6 +30,9 @@ class RMSNorm(Part):
         offset = float(self.params.get("weight_offset") or 0.0)
         if offset:
             self.weight = (self.weight + offset).contiguous()
+        gain = self.params.get("gain")
+        if gain is not None and float(gain) != 1.0:
+            self.weight = (self.weight * float(gain)).contiguous()
         self.eps = float(self.params["eps"])
         self.size = int(self.params["size"])
 

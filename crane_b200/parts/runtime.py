@@ -150,17 +150,66 @@ class Runtime:
         self.launches += 1
         return True
 
-    def _linear_bf16(self, x, w, bias, out, hint_next: bool = True, own_parts: Optional[str] = None) -> Act:
+    def linear_grouped(self, xs: torch.Tensor, w: torch.Tensor, group_features: int, name: str) -> Act:
+        """Projections that each read an input of their own, as one product: column f of the result [M, N] is
+        xs[f // group_features] @ w[f]^T, for xs [groups, M, K] and w [N, K] (the last group may be
+        narrower)."""
+        _, M, K = xs.shape
+        N = w.shape[0]
+        k = self.kernels
+        out = self.ws.get(name, M, N, self.dtype)
+        groups = -(-N // group_features)
+        if not self.exact and self.use_tcgen05 and group_features % 128 == 0 and k.tcgen05_takes(xs[0], w):
+            serial = self.launches == self._after_product and k.pdl_default       # (as in ``linear``)
+            if serial:
+                k.lib.crane_set_pdl(0)
+            try:
+                return self._linear_bf16(xs[0], w, None, out, group=(int(group_features), M))
+            finally:
+                if serial:
+                    k.lib.crane_set_pdl(1)
+                self._after_product = self.launches
+        for g in range(groups):
+            lo, hi = g * group_features, min(N, (g + 1) * group_features)
+            x, wg, og = xs[g], w[lo:hi], out[:, lo:hi]
+            if self.exact or not (self.use_tcgen05 and k.tcgen05_takes(x, wg)):
+                k.gemm_simt(x, wg, None, og)
+                self.launches += 1
+                continue
+            # (behind a product: without programmatic dependent launch, as in ``linear``)
+            serial = (g > 0 or self.launches == self._after_product) and k.pdl_default
+            if serial:
+                k.lib.crane_set_pdl(0)
+            try:
+                if M <= self.split_rows:
+                    k.gemm_tcgen05(x, wg, None, og, self.err, swap=True, bn=self._few_rows_tile(M))
+                else:
+                    k.gemm_tcgen05(x, wg, None, og, self.err, bn=128)
+            finally:
+                if serial:
+                    k.lib.crane_set_pdl(1)
+            self.launches += 1
+            self._after_product = self.launches
+        return out
+
+    @staticmethod
+    def _few_rows_tile(M: int) -> int:
+        return 16 if M <= 16 else 32 if M <= 32 else 64 if M <= 64 else 128 if M <= 128 else 256
+
+    def _linear_bf16(self, x, w, bias, out, hint_next: bool = True, own_parts: Optional[str] = None,
+                     group=None) -> Act:
+        """``group``: (features, rows) of grouped activations (see ``Kernels.gemm_tcgen05``)."""
         k = self.kernels
         M, K = x.shape
         N = w.shape[0]
         tag = str(N) if own_parts is None else str(N) + ":" + own_parts
+        grp = {} if group is None else {"group_features": group[0], "group_rows": group[1]}
         if self.use_tcgen05 and k.tcgen05_takes(x, w):
             if M <= self.split_rows:
                 # few tokens: the weight rows fill the MMA's 128-wide side (the tokens its 16 to
                 # 256 wide side), and the inner dimension is cut into slices until every SM has a
                 # tile to stream
-                bn = 16 if M <= 16 else 32 if M <= 32 else 64 if M <= 64 else 128 if M <= 128 else 256
+                bn = self._few_rows_tile(M)
                 tiles = (N + 127) // 128
                 # at most 8: the consumers of partial sums fetch eight slices at a time
                 slices = min(k.slices_for(tiles, K, self.num_sms), 8)
@@ -175,14 +224,24 @@ class Runtime:
                     parts = self.ws.get("splitk:" + tag, slices * self.split_rows, N,
                                         torch.float32, cap=slices * self.split_rows)
                     parts = parts[:slices * M].view(slices, M, N)
-                    k.gemm_tcgen05(x, w, bias, parts, self.err, split_k=slices, swap=True, bn=bn, prefetch=nxt)
+                    k.gemm_tcgen05(x, w, bias, parts, self.err, split_k=slices, swap=True, bn=bn, prefetch=nxt, **grp)
                     self.launches += 1
                     if out.dtype == torch.float32:
                         k.sum_parts(Partials(parts), out)      # float logits: the slices added in order
                         self.launches += 1
                         return out
                     return Partials(parts)
-                k.gemm_tcgen05(x, w, bias, out, self.err, swap=True, bn=bn, prefetch=nxt)
+                k.gemm_tcgen05(x, w, bias, out, self.err, swap=True, bn=bn, prefetch=nxt, **grp)
+            elif group is not None:
+                # (a tile's features lie in one group)
+                pair, pair_rows = k.pair_plan(M, N, K, self.num_sms)
+                bn = 256 if group[0] % 256 == 0 else 128
+                if pair:
+                    k.gemm_pair(x, w, bias, out, self.err, bn=bn, tile_rows=pair_rows if bn == 256 else 256, **grp)
+                else:
+                    if k.tile_width_for(M, N, self.num_sms) < 192:
+                        bn = 128
+                    k.gemm_tcgen05(x, w, bias, out, self.err, bn=bn, **grp)
             else:
                 pair, pair_rows = k.pair_plan(M, N, K, self.num_sms) if out.dtype == torch.bfloat16 else (0, 0)
                 bn = k.tile_width_for(M, N, self.num_sms)

@@ -50,6 +50,8 @@ def random_tensors(manifest: Dict[str, TensorSpec], seed: int, dtype: torch.dtyp
             out[name] = torch.eye(shape[0], shape[1], device=dev) + std * t       # a mixing matrix near the identity
         elif spec.init == "unit":
             out[name] = 0.5 * t
+        elif spec.init == "slow":
+            out[name] = -3.0 + 0.5 * t
         elif spec.keep == "float32":
             out[name] = std * t
         else:

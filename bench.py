@@ -1218,6 +1218,248 @@ def zudarax_workload(args, pk):
     return out
 
 
+def pogarax_config(like, layers):
+    """A Pogarax model with the width, layer count and vocabulary of the Hunyuan configuration `like`: the layers
+    take turns between the delta rule with a decay per channel (heads of 64 across the width, half as many
+    query/key heads, a convolution of four taps, inner sizes of 64), time mixing (heads of 64 across the
+    width, inner size 64) and latent attention (the other's head count, heads of 128 + 32 rotated, values of
+    128, latents of 192 and 512, a window of 1,024 positions, every second one on the cache of the one
+    before); feed-forwards: dense of the other's inner size in the delta layers, eight experts of a quarter
+    of it of which two are chosen in the others."""
+    h, heads, ff = like["hidden_size"], like["num_attention_heads"], like["intermediate_size"]
+    delta = {"heads": h // 64, "kv_heads": max(1, h // 128), "dim": 64, "vdim": 64, "conv": 4, "decay_rank": 64, "gate_rank": 64}
+    wkv = {"heads": h // 64, "dim": 64, "decay_rank": 64}
+    latent = {"heads": heads, "dim": 128, "rot_dim": 32, "vdim": 128, "kv_rank": 192, "q_rank": 512, "scale": 160 ** -0.5,
+              "mask": {"size": 1024}, "rot": {"dims": 32, "base": 10000.0,
+                                              "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": ff // 4}}
+    ls, owner = [], None
+    for i in range(layers):
+        if i % 3 == 0:
+            ls.append({"type": "channel_delta", "mixer": delta, "mlp": dense})
+        elif i % 3 == 1:
+            ls.append({"type": "wkv", "mixer": wkv, "mlp": moe})
+        elif owner is None:
+            ls.append({"type": "latent_attention", "mixer": latent, "mlp": moe})
+            owner = i
+        else:
+            ls.append({"type": "latent_attention", "mixer": dict(latent, kv_from=owner), "mlp": moe})
+            owner = None
+    return {"architecture": "Pogarax", "vocab": like["vocab_size"], "width": h, "norm": {"eps": 1e-5},
+            "residual_mult": 0.5, "layers": ls}
+
+
+def pogarax_kernel_table(pcfg, pk, tokens, batch, context):
+    """Every kernel or option that only Pogarax runs beside the kernel of the engine's other models that does
+    the like job, each alone on synthetic operands of these layer sizes (L2 flushed between repetitions),
+    with the fraction of its roofline: algorithmic bytes over the measured copy rate, or FLOPs over the
+    measured bf16 rate, whichever takes longer."""
+    from types import SimpleNamespace
+    import numpy as np
+    import torch
+    from crane_b200.parts import Runtime
+    from crane_b200.parts.latent_attention import latent_attention_kernel
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    rt = Runtime(dev, bf, max(tokens, 256))
+    K = rt.kernels
+    flush = torch.zeros(128 << 20, dtype=f32, device=dev)
+    err = rt.err
+    W = pcfg["width"]
+    pick = lambda t: next(l["mixer"] for l in pcfg["layers"] if l["type"] == t)
+    dl, wk, la = pick("channel_delta"), pick("wkv"), pick("latent_attention")
+    moe = next(l["mlp"] for l in pcfg["layers"] if l["mlp"]["kind"] == "moe")
+    hbm, peak = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    rows = []
+
+    def add(name, like, ms, nbytes, flops, like_ms=0, like_bytes=0, like_flops=0):
+        def frac(ms_, b, f):
+            return round(max(b / hbm, f / peak) / (ms_ * 1e-3), 4)
+        rows.append({"kernel": name, "ms": round(ms, 4), "frac": frac(ms, nbytes, flops), "like": like,
+                     "like_ms": round(like_ms, 4) if like_ms else None,
+                     "like_frac": frac(like_ms, like_bytes, like_flops) if like_ms else None})
+
+    rnd = lambda *shape, dt=bf: torch.randn(*shape, device=dev, dtype=f32).to(dt)
+    ps = 64
+    E, top, F = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"]
+    for kind, n_req, q_len, kv in (("prefill", 1, tokens, tokens), ("decode", batch, 1, context)):
+        blocks = -(-kv // ps)
+        table = torch.arange(n_req * blocks, dtype=torch.int32, device=dev).view(n_req, blocks)
+        h_cu, h_kv = np.arange(n_req + 1, dtype=np.int32) * q_len, np.full(n_req, kv, dtype=np.int32)
+        cu_d, kv_d = torch.from_numpy(h_cu).to(dev), torch.from_numpy(h_kv).to(dev)
+        n = n_req * q_len
+        pos = torch.from_numpy(np.concatenate([np.arange(kv - q_len, kv, dtype=np.int32)] * n_req)).to(dev)
+        ent = torch.from_numpy(np.repeat(np.arange(n_req, dtype=np.int32), q_len)).to(dev)
+        slots = torch.arange(n_req, dtype=torch.int32, device=dev)
+        ctx = SimpleNamespace(tok_entry=ent, cu_q=cu_d, kv_len=kv_d, slots=slots)
+        # the addition of a normed result: with the copy of the stream / with the next norm
+        x, y, o1, w2 = rnd(n, W, dt=f32), rnd(n, W), torch.empty(n, W, device=dev, dtype=bf), [rnd(W, dt=f32) for _ in range(2)]
+        t_p = _median_ms(lambda: K.add_normed_norm(x, y, w2[0], 1e-5, raw=o1), flush=flush)
+        t_l = _median_ms(lambda: K.add_normed_norm(x, y, w2[0], 1e-5, w2[1], 1e-5, o1), flush=flush)
+        add(f"add_normed_norm with the stream's copy ({kind})", "add_normed_norm with the next norm (Vodelix)", t_p, n * W * 12, 0,
+            t_l, n * W * 12, 0)
+        # router and activation
+        z, route = rnd(n, E, dt=f32), torch.empty(n, E, device=dev)
+        t_p = _median_ms(lambda: K.route_grouped(z, None, route, E, top, 1, 1, False, sigmoid=True), flush=flush)
+        t_l = _median_ms(lambda: K.route_grouped(z, None, route, E, top, 1, 1, False), flush=flush)
+        add(f"route_grouped, sigmoid ({kind})", "route_grouped, softmax (Mufevik)", t_p, n * E * 8, 0, t_l, n * E * 8, 0)
+        gu, act = rnd(n, 2 * E * F), torch.empty(n, E * F, device=dev, dtype=bf)
+        t_p = _median_ms(lambda: K.gated_activation(gu, act, route, E, F, E * F, on_input=True), flush=flush)
+        t_l = _median_ms(lambda: K.gated_activation(gu, act, route, E, F, E * F), flush=flush)
+        add(f"gated_activation, weight on the input ({kind})", "gated_activation (Mufevik)", t_p, n * E * F * 6, 0, t_l, n * E * F * 6, 0)
+        del gu, act, x, y
+        # ---- the delta rule: preparation, the low-rank products, the recurrence, norm and gate
+        H, G, d, m, taps, ra, rg = (dl[k] for k in ("heads", "kv_heads", "dim", "vdim", "conv", "decay_rank", "gate_rank"))
+        C, gd, hv, hd = 2 * G * d + H * m, G * d, H * m, H * d
+        rws, lanes = K.matrix_state_plan(d)
+        conv_off = H * rws * lanes * m
+        state = torch.zeros(n_req, conv_off + (taps - 1) * C, device=dev)
+        conv_w, a_log, dtb, dtb_h = rnd(C, taps, dt=f32), rnd(H, dt=f32), rnd(hd, dt=f32), rnd(H, dt=f32)
+        cols = C + H + ra + rg
+        proj = rnd(n, cols)
+        w_at = -(-(C + H) // 4) * 4
+        aux = torch.rand(n, w_at + hd, device=dev)
+        like_cols = C + hv + 2 * H
+        like_proj, like_aux = rnd(n, like_cols), torch.rand(n, C + 2 * H, device=dev)
+        t_p = _median_ms(lambda: K.conv_delta_prep(proj, cols, ctx, state, conv_off, conv_w, taps, None, None, aux, H, G, d, m, 1e-6,
+                                                   d ** -0.5, err, bf, b_off=C, a_off=-1, w_off=0, beta_off=C), flush=flush)
+        t_l = _median_ms(lambda: K.conv_delta_prep(like_proj, like_cols, ctx, state, conv_off, conv_w, taps, a_log, dtb_h, like_aux, H,
+                                                   G, d, m, 1e-6, d ** -0.5, err, bf), flush=flush)
+        add(f"conv_delta_prep, no decay ({kind})", "conv_delta_prep (Mufevik)", t_p, n * C * 6, 0, t_l, n * C * 6, 0)
+        packs = [K.pack_low_rank(rnd(o, r), False) for o, r in ((hd, ra), (hv, rg))]
+        gate = torch.empty(n, hv, device=dev, dtype=bf)
+        A = K.LowRank(packs[0][0], ra, C + H, hd, out=aux[:, w_at:], kind="soft_decay", bias=dtb, rate=a_log, per_rate=d, mma=True)
+        B = K.LowRank(packs[1][0], rg, C + H + ra, hv, out=gate, mma=True)
+        t_p = _median_ms(lambda: K.low_rank_expand(proj, cols, ent, n, bf, A, B), flush=flush)
+        # the like kernel: one decay per channel from a low-rank product, with q, k, v brought to 32-bit
+        pc = 2 * hd + 2 * hv + ra
+        gp, ga, a2t = rnd(n, pc), torch.empty(n, 3 * hd + hv, device=dev), rnd(ra, hd, dt=f32)
+        t_g = _median_ms(lambda: K.decay_gate_prep(gp, pc, ent, a2t, dtb, 0.25, d ** -0.5, ga, H, d, m, bf), flush=flush)
+        b_g = n * (2 * hd + hv + ra) * 2 + n * (3 * hd + hv) * 4
+        add(f"low_rank_expand, decay and gate ({kind})", "decay_gate_prep (Mufevik)", t_p,
+            n * (ra + rg) * 2 + n * (hd * 4 + hv * 2) + (ra * hd + rg * hv) * 2, 0, t_g, b_g + ra * hd * 4, 0)
+        o_raw = torch.empty(n, hv, device=dev)
+        aux[:, w_at:].uniform_(0.9, 1.0)
+        sc = lambda a, offs, wv, mode, rep: K.matrix_state_scan(a, offs, wv, mode, rep, ctx, state, o_raw, H, d, m, err)
+        t_p = _median_ms(lambda: sc(aux, (0, gd, 2 * gd, w_at, C), True, "delta", H // G), flush=flush)
+        t_l = _median_ms(lambda: sc(like_aux, (0, gd, 2 * gd, C, C + H), False, "delta", H // G), flush=flush)
+        st = n_req * H * d * m * 8
+        add(f"matrix_state_scan, delta rule, decay per channel ({kind})", "matrix_state_scan, delta rule (Mufevik)", t_p,
+            n * (C + H + hd + hv) * 4 + (st if kind == "decode" else 0), 0, t_l, n * (C + 2 * H + hv) * 4 + (st if kind == "decode" else 0), 0)
+        nw, o = rnd(m, dt=f32), torch.empty(n, hv, device=dev, dtype=bf)
+        t_p = _median_ms(lambda: K.head_norm_gate(o_raw, gate, hv, 0, ent, nw, 1e-5, o, H, m, sigmoid=True), flush=flush)
+        t_l = _median_ms(lambda: K.head_norm_gate(o_raw, like_proj, like_cols, C, ent, nw, 1e-5, o, H, m), flush=flush)
+        add(f"head_norm_gate, sigmoid ({kind})", "head_norm_gate (Mufevik)", t_p, n * hv * 8, 0, t_l, n * hv * 8, 0)
+        del proj, aux, like_proj, like_aux, gate, state
+        # ---- time mixing: the mixes, the grouped product, preparation, decay, the recurrence
+        H, d, rk = wk["heads"], wk["dim"], wk["decay_rank"]
+        hd = H * d
+        rws, lanes = K.matrix_state_plan(d)
+        row_off = H * rws * lanes * d
+        state = torch.zeros(n_req, row_off + W, device=dev)
+        h, mu, xs = rnd(n, W), rnd(5, W, dt=f32), torch.empty(5, n, W, device=dev, dtype=bf)
+        t_p = _median_ms(lambda: K.token_shift_mix(h, mu, ctx, state, row_off, xs, err), flush=flush)
+        a2, b2 = rnd(n, W), rnd(n, W)
+        t_l = _median_ms(lambda: K.pair_norm_mean(a2, b2, w2[0], w2[1], 1e-5, o1), flush=flush)
+        add(f"token_shift_mix ({kind})", "pair_norm_mean (Mufevik)", t_p, n * W * 2 * 6, 0, t_l, n * W * 6, 0)
+        wts = rnd(4 * hd + rk, W)
+        t_p = _median_ms(lambda: rt.linear_grouped(xs, wts, hd, "bench_grouped"), flush=flush)
+        t_l = _median_ms(lambda: rt.linear(h, wts, None, "bench_plain"), flush=flush)
+        fl, by = 2 * n * W * (4 * hd + rk), (4 * hd + rk) * W * 2
+        add(f"grouped product, five inputs ({kind})", "the same product of one input", t_p, by + n * W * 10, fl, t_l, by + n * W * 2, fl)
+        proj, aux = rnd(n, 4 * hd + rk), torch.empty(n, 4 * hd + H, device=dev)
+        u = rnd(H, d, dt=f32)
+        t_p = _median_ms(lambda: K.bonus_prep(proj, 4 * hd + rk, ent, u, aux, 4 * hd, H, d, d, bf), flush=flush)
+        add(f"bonus_prep ({kind})", "decay_gate_prep (Mufevik)", t_p, n * 3 * hd * 6, 0, t_g, b_g, 0)
+        w2p, mma = K.pack_low_rank(rnd(hd, rk), False)
+        A = K.LowRank(w2p, rk, 4 * hd, hd, out=aux[:, 3 * hd:], kind="exp_decay", bias=rnd(hd, dt=f32), tanh=True, mma=mma)
+        t_p = _median_ms(lambda: K.low_rank_expand(proj, 4 * hd + rk, ent, n, bf, A), flush=flush)
+        add(f"low_rank_expand, tanh and decay ({kind})", "decay_gate_prep (Mufevik)", t_p, n * rk * 2 + n * hd * 4 + rk * hd * 2, 0,
+            t_g, b_g + ra * hd * 4, 0)
+        o_raw = torch.empty(n, hd, device=dev)
+        aux[:, 3 * hd:4 * hd].uniform_(0.9, 1.0)
+        t_p = _median_ms(lambda: K.matrix_state_scan(aux, (0, hd, 2 * hd, 3 * hd, 4 * hd), True, "bonus", 1, ctx, state, o_raw, H, d, d,
+                                                     err), flush=flush)
+        t_l = _median_ms(lambda: K.matrix_state_scan(aux, (0, hd, 2 * hd, 3 * hd, 0), True, "plain", 1, ctx, state, o_raw, H, d, d, err),
+                         flush=flush)
+        b_s = n * (5 * hd) * 4 + (n_req * H * d * d * 8 if kind == "decode" else 0)
+        add(f"matrix_state_scan, bonus ({kind})", "matrix_state_scan, decay per channel (Mufevik)", t_p, b_s, 0, t_l, b_s, 0)
+        del proj, aux, state, xs, wts
+        # ---- latent attention: preparation, attention with window and sinks
+        H, dim, rot, r, rq = (la[k] for k in ("heads", "dim", "rot_dim", "kv_rank", "q_rank"))
+        win = la["mask"]["size"]
+        width = r + rot
+        pool = rnd(n_req * blocks, 1, ps, width)
+        cos = torch.rand(kv, rot // 2, device=dev)
+        nw_r, nw_q = rnd(r, dt=f32), rnd(rq, dt=f32)
+        first, qp, q_abs = rnd(n, rq + width), rnd(n, H * (dim + rot)), rnd(n, H * width)
+        cq = torch.empty(n, rq, device=dev, dtype=bf)
+        meta = (cos, cos, pos, ent, table, pool, ps)
+        t_1 = _median_ms(lambda: K.latent_prep(first, rq + width, -1, rq, H, dim, rot, r, rot, *meta, nw_r, 1e-5, None, err, cq_off=0,
+                                               cq_w=nw_q, cq_out=cq), flush=flush)
+        t_2 = _median_ms(lambda: K.latent_prep(qp, H * (dim + rot), 0, -1, H, dim, rot, r, rot, *meta, None, 1e-5, q_abs, err), flush=flush)
+        merged = rnd(n, H * (dim + rot) + width)
+        t_l = _median_ms(lambda: K.latent_prep(merged, H * (dim + rot) + width, 0, H * (dim + rot), H, dim, rot, r, rot, *meta, nw_r, 1e-5,
+                                               q_abs, err), flush=flush)
+        b_l = n * (H * rot + width) * 4
+        add(f"latent_prep, cache row and query latent ({kind})", "latent_prep (Radorax)", t_1, n * (width + rq) * 4, 0, t_l, b_l, 0)
+        add(f"latent_prep, rotation of the queries ({kind})", "latent_prep (Radorax)", t_2, n * H * rot * 4, 0, t_l, b_l, 0)
+        o_lat, sinks = torch.empty(n, H * r, device=dev, dtype=bf), rnd(H, dt=f32)
+        scratch = lambda name, rows_, cols_, cap: rt.ws.get(name, rows_, cols_, f32, cap=cap)
+        at = lambda w_, s_: latent_attention_kernel(K, q_abs, o_lat, pool, pos, ent, cu_d, kv_d, h_cu, h_kv, table, ps, H, r, rot,
+                                                    la["scale"], err, False, num_sms=rt.num_sms, scratch=scratch, window=w_, sinks=s_)
+        t_p = _median_ms(lambda: at(win, sinks), flush=flush)
+        t_f = _median_ms(lambda: at(0, sinks), flush=flush)
+        t_l = _median_ms(lambda: at(0, None), flush=flush)
+        seen = lambda w_: sum(min(p + 1, w_ or p + 1) for p in range(kv - q_len, kv)) * n_req
+        read = lambda w_: n_req * min(kv, (w_ + q_len - 1) if w_ else kv) * width * 2
+        fl = lambda w_: 2 * seen(w_) * H * (width + r)
+        add(f"latent attention, window of {win} and sinks ({kind})", "latent attention (Radorax)", t_p, read(win), fl(win), t_l, read(0), fl(0))
+        add(f"latent attention, sinks, no window ({kind})", "latent attention (Radorax)", t_f, read(0), fl(0), t_l, read(0), fl(0))
+        del pool, merged, first, qp, q_abs
+    torch.cuda.synchronize()
+    assert int(err.item()) == 0
+    return rows
+
+
+def pogarax_workload(args, pk):
+    """Prefill and decode throughput of Pogarax at the layer sizes of --sizes beside Mufevik (the engine's
+    closest model: a delta rule behind convolutions, gated experts) at the same width, layers and
+    vocabulary, random weights, and its kernels beside their likes."""
+    import gc
+    import torch
+    hcfg = dict(MODEL)
+    hcfg.update(OTHER_SIZES.get(args.sizes, {}))
+    layers = args.layers or 12
+    hcfg["num_hidden_layers"] = layers
+    pcfg, mcfg = pogarax_config(hcfg, layers), mufevik_config(hcfg, layers)
+    page, pt = 64, args.prefill_tokens
+    out = {"workload": "pogarax", "sizes": args.sizes, "layers": layers, "batch": args.batch,
+           "context": args.context, "prefill_tokens": pt, "dtype": "bf16", "data": "synthetic", "models": {}}
+    for name, cfg in (("pogarax", pcfg), ("mufevik", mcfg)):
+        opts = dict(page_size=page, num_pages=(args.batch * (args.context + args.steps + args.warmup + 64) + pt) // page + 64,
+                    max_concurrent=max(64, args.batch), max_seq_len=max(args.context, pt) + 1024,
+                    max_batched_tokens=max(2048, pt), chunk_size=max(2048, pt))
+        model = build_model(cfg, opts)
+        pms = time_prefill(model, pt, cfg["vocab"], reps=3)
+        ids = fill_cache(model, args.batch, args.context)
+        with ClockSampler() as clk:
+            dms, launches = time_decode(model, ids, args.steps, args.warmup, cfg["vocab"])
+        weights = sum(t.numel() * t.element_size() for t in _model_tensors(model))
+        out["models"][name] = {"prefill_ms": round(pms, 3), "prefill_tokens_per_s": round(pt * 1000.0 / pms, 1),
+                               "decode_ms_per_step": round(dms, 4),
+                               "decode_tokens_per_s": round(args.batch * 1000.0 / dms, 1),
+                               "launches_per_decode_step": launches, "weight_bytes": weights,
+                               "layer_runs": len(model.runner.spec.schedule), "clocks": clk.summary()}
+        del model
+        gc.collect()
+        torch.cuda.empty_cache()
+    if not args.no_points:
+        out["kernels"] = pogarax_kernel_table(pcfg, pk, pt, args.batch, args.context)
+    out["peaks"] = pk
+    return out
+
+
 def _model_tensors(model):
     seen, out = set(), []
     parts = [model.runner.model.embed, model.runner.model.final_norm, model.runner.model.head]
@@ -1257,7 +1499,7 @@ def main():
                     help="layer sizes: Hunyuan 1.8B (the default, the headline configuration), 4B or 7B")
     ap.add_argument("--prefill-chunk", type=int, default=0,
                     help="with --only-prefill: also time the prompt in portions of this many tokens, a step each")
-    ap.add_argument("--workload", default="", choices=["", "serve", "mixed-step", "radorax", "vodelix", "mufevik", "zudarax"],
+    ap.add_argument("--workload", default="", choices=["", "serve", "mixed-step", "radorax", "vodelix", "mufevik", "zudarax", "pogarax"],
                     help="serve: a mix of requests through the scheduler; mixed-step: decoded tokens beside "
                          "one prompt portion in one step; radorax: prefill and decode of Radorax beside Hunyuan "
                          "Dense at equal layer sizes, and their kernels side by side; vodelix: the same for Vodelix; "
@@ -1281,6 +1523,9 @@ def main():
         return 2
     args.warmup = max(args.warmup, 3)
 
+    if args.workload == "pogarax":
+        print(json.dumps(pogarax_workload(args, peaks())))
+        return 0
     if args.workload == "zudarax":
         print(json.dumps(zudarax_workload(args, peaks())))
         return 0

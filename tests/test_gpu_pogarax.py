@@ -60,7 +60,7 @@ def _compare(got, tb, plain, dtype, label, tol_rms=3e-5):
         assert np.median(errs) <= 0.1, label
 
 
-@pytest.mark.parametrize("name, dtype", [(n, "float32") for n in SMALL] + [(n + a, "bfloat16") for n in SMALL for a in ("", "-all")])
+@pytest.mark.parametrize("name, dtype", [(n, "float32") for n in SMALL] + [(n + "-all", "bfloat16") for n in SMALL] + [("PA", "bfloat16")])
 def test_alone_whole_tail_portions(name, dtype, cases, tmp_path):
     folder, reqs, plain = cases(name, dtype)
     ps = tp.TINY[name]["page_size"]
@@ -74,7 +74,7 @@ def test_alone_whole_tail_portions(name, dtype, cases, tmp_path):
         tt.compare_cuts([(got, tb)], dtype, f"config {name}", tol=2e-5)
 
 
-@pytest.mark.parametrize("name, dtype", [(n, "float32") for n in SMALL] + [(n + a, "bfloat16") for n in SMALL for a in ("", "-all")])
+@pytest.mark.parametrize("name, dtype", [(n, "float32") for n in SMALL] + [(n + "-all", "bfloat16") for n in SMALL] + [("PA", "bfloat16")])
 def test_mixed_with_page_and_slot_reuse(name, dtype, cases, tmp_path):
     folder, reqs, plain = cases(name, dtype)
     ps = tp.TINY[name]["page_size"]

@@ -1306,7 +1306,8 @@ def pogarax_kernel_table(pcfg, pk, tokens, batch, context):
         gu, act = rnd(n, 2 * E * F), torch.empty(n, E * F, device=dev, dtype=bf)
         t_p = _median_ms(lambda: K.gated_activation(gu, act, route, E, F, E * F, on_input=True), flush=flush)
         t_l = _median_ms(lambda: K.gated_activation(gu, act, route, E, F, E * F), flush=flush)
-        add(f"gated_activation, weight on the input ({kind})", "gated_activation (Mufevik)", t_p, n * E * F * 6, 0, t_l, n * E * F * 6, 0)
+        by = n * F * (top * 4 + E * 2)             # (columns of experts that a token did not choose are not read)
+        add(f"gated_activation, weight on the input ({kind})", "gated_activation (Mufevik)", t_p, by, 0, t_l, by, 0)
         del gu, act, x, y
         # ---- the delta rule: preparation, the low-rank products, the recurrence, norm and gate
         H, G, d, m, taps, ra, rg = (dl[k] for k in ("heads", "kv_heads", "dim", "vdim", "conv", "decay_rank", "gate_rank"))
@@ -1369,13 +1370,12 @@ def pogarax_kernel_table(pcfg, pk, tokens, batch, context):
         add(f"grouped product, five inputs ({kind})", "the same product of one input", t_p, by + n * W * 10, fl, t_l, by + n * W * 2, fl)
         proj, aux = rnd(n, 4 * hd + rk), torch.empty(n, 4 * hd + H, device=dev)
         u = rnd(H, d, dt=f32)
-        t_p = _median_ms(lambda: K.bonus_prep(proj, 4 * hd + rk, ent, u, aux, 4 * hd, H, d, d, bf), flush=flush)
-        add(f"bonus_prep ({kind})", "decay_gate_prep (Mufevik)", t_p, n * 3 * hd * 6, 0, t_g, b_g, 0)
         w2p, mma = K.pack_low_rank(rnd(hd, rk), False)
         A = K.LowRank(w2p, rk, 4 * hd, hd, out=aux[:, 3 * hd:], kind="exp_decay", bias=rnd(hd, dt=f32), tanh=True, mma=mma)
-        t_p = _median_ms(lambda: K.low_rank_expand(proj, 4 * hd + rk, ent, n, bf, A), flush=flush)
-        add(f"low_rank_expand, tanh and decay ({kind})", "decay_gate_prep (Mufevik)", t_p, n * rk * 2 + n * hd * 4 + rk * hd * 2, 0,
-            t_g, b_g + ra * hd * 4, 0)
+        t_p = _median_ms(lambda: K.low_rank_expand(proj, 4 * hd + rk, ent, n, bf, A, bonus=K.Bonus(u, aux, 4 * hd, H, d, d)),
+                         flush=flush)
+        add(f"low_rank_expand, tanh and decay, with the bonus ({kind})", "decay_gate_prep (Mufevik)", t_p,
+            n * (3 * hd + rk) * 2 + n * 4 * hd * 4 + rk * hd * 2, 0, t_g, b_g + ra * hd * 4, 0)
         o_raw = torch.empty(n, hd, device=dev)
         aux[:, 3 * hd:4 * hd].uniform_(0.9, 1.0)
         t_p = _median_ms(lambda: K.matrix_state_scan(aux, (0, hd, 2 * hd, 3 * hd, 4 * hd), True, "bonus", 1, ctx, state, o_raw, H, d, d,

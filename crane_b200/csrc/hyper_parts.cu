@@ -77,7 +77,7 @@ streams_norm_kernel(float* __restrict__ streams, long long stream_stride, int R,
 // One warp per token.  z: float logits [n][ld], the first `experts` of a row the router's, column
 // `experts` (if `shared_gate`) the shared expert's gate.  route [n][experts + shared_gate].
 __global__ void __launch_bounds__(128)
-route_grouped_kernel(const float* __restrict__ z, int ld, const float* __restrict__ correction,
+route_grouped_kernel(GemmOut<float> z, int ld, const float* __restrict__ correction,
                      float* __restrict__ route, int n, int experts, int top, int groups, int keep,
                      int shared_gate, int sigmoid_scores) {
     extern __shared__ float sm[];                     // per warp: score [E], choice [E], group score [groups]
@@ -89,24 +89,25 @@ route_grouped_kernel(const float* __restrict__ z, int ld, const float* __restric
     float* score = sm + (size_t)wib * (2 * experts + groups);
     float* choice = score + experts;
     float* gscore = choice + experts;
-    const float* zr = z + (long long)t * ld;
+    const long long zr = (long long)t * ld;
+    for (int e = lane; e < experts; e += 32) score[e] = z.load(zr + e);       // (each lane reads its own again below)
     float* r = route + (long long)t * (experts + shared_gate);
     if (sigmoid_scores) {
         // (without a correction the choice goes by the logits: the same order, and scores that round to the
         // same number keep it)
         for (int e = lane; e < experts; e += 32) {
-            const float s = 1.f / (1.f + expf(-zr[e]));
+            const float logit = score[e], s = 1.f / (1.f + expf(-logit));
             score[e] = s;
-            choice[e] = correction != nullptr ? s + correction[e] : zr[e];
+            choice[e] = correction != nullptr ? s + correction[e] : logit;
             r[e] = 0.f;
         }
     } else {
         float zmax = -INFINITY;
-        for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, zr[e]);
+        for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, score[e]);
         zmax = warp_max(zmax);
         float sum = 0.f;
         for (int e = lane; e < experts; e += 32) {
-            const float p = expf(zr[e] - zmax);
+            const float p = expf(score[e] - zmax);
             score[e] = p;
             sum += p;
         }
@@ -170,7 +171,7 @@ route_grouped_kernel(const float* __restrict__ z, int ld, const float* __restric
         }
         __syncwarp();
     }
-    if (shared_gate && lane == 0) r[experts] = 1.f / (1.f + expf(-zr[experts]));
+    if (shared_gate && lane == 0) r[experts] = 1.f / (1.f + expf(-z.load(zr + experts)));
 }
 
 // gu rows: [gate (cols) | up (cols)].  out[t][c] = silu(gate) * up * weight(c): route[t][c / per_expert]
@@ -203,6 +204,40 @@ gated_activation_kernel(GemmOut<T> gu, T* __restrict__ out, long long n, int col
     }
 }
 
+// The same for bfloat16 products whose columns come in whole groups of 8: a thread takes 8 neighbouring columns of one
+// row (two 16-byte loads, one 16-byte store); grid (column groups, rows).
+__global__ void __launch_bounds__(256)
+gated_activation_vec_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int cols,
+                            const float* __restrict__ route, int experts, int per_expert, int routed_cols,
+                            int shared_gate, int on_input) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c0 = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (c0 >= cols) return;
+    const long long row = blockIdx.y;
+    float w = 1.f;
+    if (route != nullptr) {
+        const float* r = route + row * (experts + shared_gate);
+        if (c0 < routed_cols) w = r[c0 / per_expert];
+        else if (shared_gate) w = r[experts];
+    }
+    uint4 res = make_uint4(0u, 0u, 0u, 0u);
+    if (w != 0.f) {                                   // (an expert that was not chosen is not even read)
+        const uint4 graw = *(const uint4*)(gu + row * 2 * cols + c0);
+        const uint4 uraw = *(const uint4*)(gu + row * 2 * cols + cols + c0);
+        const __nv_bfloat162* g2 = (const __nv_bfloat162*)&graw;
+        const __nv_bfloat162* u2 = (const __nv_bfloat162*)&uraw;
+        __nv_bfloat162* o2 = (__nv_bfloat162*)&res;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 z = __bfloat1622float2(g2[i]), b = __bfloat1622float2(u2[i]);
+            const float ax = on_input ? z.x * w : z.x, ay = on_input ? z.y * w : z.y;
+            o2[i] = __floats2bfloat162_rn(ax / (1.f + expf(-ax)) * b.x * w, ay / (1.f + expf(-ay)) * b.y * w);
+        }
+    }
+    *(uint4*)(out + row * cols + c0) = res;
+}
+
 }  // namespace
 
 CRANE_API int crane_streams_norm(int dtype, float* streams, long long stream_stride, int n_streams,
@@ -224,7 +259,7 @@ CRANE_API int crane_streams_norm(int dtype, float* streams, long long stream_str
     });
 }
 
-CRANE_API int crane_route_grouped(const float* z, int ld, const float* correction, float* route, int n,
+CRANE_API int crane_route_grouped(const float* z, const float* z_parts, int n_parts, long long part_stride, int ld, const float* correction, float* route, int n,
                                   int experts, int top, int groups, int keep, int shared_gate, int sigmoid_scores,
                                   cudaStream_t st) {
     if (n <= 0) return 0;
@@ -232,7 +267,8 @@ CRANE_API int crane_route_grouped(const float* z, int ld, const float* correctio
         return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)4 * (2 * experts + groups) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-    return crane_launch(route_grouped_kernel, dim3((n + 3) / 4), dim3(128), smem, st, z, ld, correction, route, n,
+    return crane_launch(route_grouped_kernel, dim3((n + 3) / 4), dim3(128), smem, st,
+                        GemmOut<float>{z, z_parts, n_parts, part_stride}, ld, correction, route, n,
                         experts, top, groups, keep, shared_gate ? 1 : 0, sigmoid_scores);
 }
 
@@ -243,6 +279,11 @@ CRANE_API int crane_gated_activation(int dtype, const void* gu, const float* gu_
     if (n_rows <= 0 || cols <= 0) return 0;
     const long long n = (long long)n_rows * cols;
     const int blocks = (int)((n + 255) / 256 < 16384 ? (n + 255) / 256 : 16384);
+    if (dtype == 1 && gu != nullptr && cols % 8 == 0 && n_rows <= 65535 && ((uintptr_t)gu | (uintptr_t)out) % 16 == 0 &&
+        (route == nullptr || (per_expert > 0 && per_expert % 8 == 0 && routed_cols % 8 == 0)))
+        return crane_launch(gated_activation_vec_kernel, dim3((cols / 8 + 255) / 256, n_rows), dim3(256), 0, st,
+                            (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, cols, route, experts,
+                            per_expert > 0 ? per_expert : 1, routed_cols, shared_gate ? 1 : 0, on_input);
     DISPATCH_T(dtype, {
         GemmOut<T> u{(const T*)gu, gu_parts, n_parts, part_stride};
         return crane_launch(gated_activation_kernel<T>, dim3(blocks), dim3(256), 0, st, u, (T*)out, n, cols, route,

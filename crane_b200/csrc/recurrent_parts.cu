@@ -15,10 +15,11 @@
 //   * `conv_delta_prep`: q, k, v through a short causal convolution over time and silu, q and k scaled
 //     to unit length per head, beta = sigmoid(.), w = exp(-exp(A) softplus(. + dt)) per head (unless a decay
 //     per key channel comes from elsewhere); the last taps - 1 inputs of the convolutions are part of the
-//     request's state (`conv_state_update`);
+//     request's state, moved on by the lane that reads them in a step of single tokens, else by
+//     `conv_state_update`;
 //   * `decay_gate_prep`: q scaled, k, v, and w = sigmoid(z)^(1 / tau) per key channel with z a
 //     low-rank product plus bias;
-//   * `bonus_prep`: r, k, v and the number b per head.
+//   * `bonus_prep` (also as further blocks of `low_rank_expand`): r, k, v and the number b per head.
 // `token_shift_mix` forms what the projections of the bonus recurrence read, h + (h' - h) mu with h' the
 // previous token's row, which is part of the request's state.  `low_rank_expand` is the second matrix of a
 // low-rank product with what follows it (a decay, or nothing).
@@ -42,13 +43,15 @@ __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log
 // `beta_off`.  conv_w [2 G d + H dv][taps] float.  conv_state: inside the slot's state
 // at `conv_off`, [taps - 1][C].  Grid (tokens, blocks of heads); a warp per head of q, k or v (2 G + H of
 // them): a q or k head is written as the convolution left it, then scaled by the same lanes once its
-// sum of squares is known.
-template <typename T>
+// sum of squares is known.  SINGLE: every entry of the step has one token, so the lane that reads a channel's kept
+// inputs is the only one and moves them on.
+template <typename T, bool SINGLE>
 __global__ void __launch_bounds__(256)
 conv_delta_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry,
                        const int* __restrict__ cu_q, const int* __restrict__ kv_len,
                        const int* __restrict__ slots, int n_slots, const float* __restrict__ state,
-                       long long slot_stride, long long conv_off, const float* __restrict__ conv_w, int taps,
+                       float* state_out, long long slot_stride, long long conv_off,
+                       const float* __restrict__ conv_w, int taps,
                        const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                        float* __restrict__ aux, int aux_cols, int H, int G, int d, int dv, int b_off, int a_off,
                        int w_off, int beta_off, float key_eps, float q_scale, int* err) {
@@ -77,12 +80,23 @@ conv_delta_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
         for (int cc = lane; cc < width; cc += 32) {
             const int c = c_first + cc;
             float acc = 0.f;
-            for (int j = 0; j < taps; ++j) {
-                const int back = taps - 1 - j;
-                float x = 0.f;
-                if (i - back >= 0) x = proj.load((long long)(t - back) * cols + c);
-                else if (start + i - back >= 0) x = cs[(long long)(taps - 1 + i - back) * C + c];
-                acc = fmaf(conv_w[(long long)c * taps + j], x, acc);
+            if (SINGLE) {                              // (state_out: the same slots, through a pointer that may be written)
+                float* kept = state_out + (long long)slot * slot_stride + conv_off + c;
+                for (int j = 0; j < taps; ++j) {
+                    float x = 0.f;
+                    if (j == taps - 1) x = proj.load((long long)t * cols + c);
+                    else if (start - (taps - 1 - j) >= 0) x = kept[(long long)j * C];
+                    acc = fmaf(conv_w[(long long)c * taps + j], x, acc);
+                    if (j > 0) kept[(long long)(j - 1) * C] = x;
+                }
+            } else {
+                for (int j = 0; j < taps; ++j) {
+                    const int back = taps - 1 - j;
+                    float x = 0.f;
+                    if (i - back >= 0) x = proj.load((long long)(t - back) * cols + c);
+                    else if (start + i - back >= 0) x = cs[(long long)(taps - 1 + i - back) * C + c];
+                    acc = fmaf(conv_w[(long long)c * taps + j], x, acc);
+                }
             }
             const float v = silu_f(acc);
             out[c] = v;
@@ -104,7 +118,8 @@ conv_delta_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
     }
 }
 
-// One thread per (entry, channel): the last taps - 1 inputs of the channel after this step.
+// One thread per (entry, channel): the last taps - 1 inputs of the channel after this step (a step of
+// nothing but single tokens has moved them on already).
 constexpr int MAX_TAPS = 16;
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -216,21 +231,31 @@ token_shift_mix_kernel(const T* __restrict__ h, const float* __restrict__ mu, in
 
 // proj row: [r (H d) | k (H d) | v (H dv) | ...].  aux row: [r | k | v | ... ] with b (H) at column `b_off`:
 // b = sum_i r_i u_i k_i.  A warp per (token, head).
+struct BonusJob { const float* u; float* aux; int aux_cols, b_off, H, d, dv; };     // (u null: no such job)
 template <typename T>
-__global__ void __launch_bounds__(128)
-bonus_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, const float* __restrict__ u,
-                  float* __restrict__ aux, int aux_cols, int b_off, int n, int H, int d, int dv) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int lane = threadIdx.x & 31;
-    if (wid >= (long long)n * H) return;
-    const int t = (int)(wid / H), h = (int)(wid % H);
-    if (tok_entry[t] < 0) return;
+__device__ __forceinline__ void bonus_head(const GemmOut<T>& proj, int cols, const BonusJob& job, int t, int h, int lane) {
+    const float* u = job.u;
+    float* aux = job.aux;
+    const int aux_cols = job.aux_cols, b_off = job.b_off, H = job.H, d = job.d, dv = job.dv;
     const long long row = (long long)t * cols;
     float* out = aux + (long long)t * aux_cols;
     const int hd = H * d;
     float b = 0.f;
+    if (((cols | d | dv | aux_cols) & 1) == 0) {                              // two neighbours a lane
+        for (int c = 2 * lane; c < d; c += 64) {
+            const float2 r = proj.load2(row + h * d + c), k = proj.load2(row + hd + h * d + c), uv = ld2(u + h * d + c);
+            st2(out + h * d + c, r.x, r.y);
+            st2(out + hd + h * d + c, k.x, k.y);
+            b = fmaf(r.x * uv.x, k.x, fmaf(r.y * uv.y, k.y, b));
+        }
+        for (int c = 2 * lane; c < dv; c += 64) {
+            const float2 v = proj.load2(row + 2 * hd + h * dv + c);
+            st2(out + 2 * hd + h * dv + c, v.x, v.y);
+        }
+        b = warp_sum(b);
+        if (lane == 0) out[b_off + h] = b;
+        return;
+    }
     for (int c = lane; c < d; c += 32) {
         const float r = proj.load(row + h * d + c), k = proj.load(row + hd + h * d + c);
         out[h * d + c] = r;
@@ -240,6 +265,17 @@ bonus_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, 
     for (int c = lane; c < dv; c += 32) out[2 * hd + h * dv + c] = proj.load(row + 2 * hd + h * dv + c);
     b = warp_sum(b);
     if (lane == 0) out[b_off + h] = b;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+bonus_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, const BonusJob job, int n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (wid >= (long long)n * job.H) return;
+    const int t = (int)(wid / job.H);
+    if (tok_entry[t] >= 0) bonus_head<T>(proj, cols, job, t, (int)(wid % job.H), threadIdx.x & 31);
 }
 
 // ------------------------------------------------------ the second matrix of a low-rank product
@@ -257,17 +293,39 @@ struct LowRankPart {
     long long out_ld;
     int low_off, rank, ld_w, n_out, kind, tanh_in, per_rate;
 };
-struct LowRankArgs { LowRankPart part[2]; int col_blocks0; };       // column blocks of the first part
-
+// The grid's column blocks: the first part's, the second's up to `col_blocks`, then (if there is one) the bonus job's,
+// whose (token, head) pairs of the row tile are dealt out to the warps of those blocks.
+struct LowRankArgs { LowRankPart part[2]; int col_blocks0, col_blocks; BonusJob bonus; };
 template <typename T>
-__device__ __forceinline__ void low_rank_store(const LowRankPart& p, int t, int c, float z) {
+__device__ __forceinline__ void bonus_blocks(const GemmOut<T>& proj, int cols, const int* __restrict__ tok_entry,
+                                             const LowRankArgs& args, int t0, int nt) {
+    const int nw = blockDim.x >> 5, H = args.bonus.H;
+    const int first = ((int)blockIdx.y - args.col_blocks) * nw + (int)(threadIdx.x >> 5);
+    for (int x = first; x < nt * H; x += ((int)gridDim.y - args.col_blocks) * nw) {
+        const int t = t0 + x / H;
+        if (tok_entry[t] >= 0) bonus_head<T>(proj, cols, args.bonus, t, x % H, threadIdx.x & 31);
+    }
+}
+
+// What a column adds to z and multiplies the rate by.
+struct LowRankColumn { float bias, rate; };
+__device__ __forceinline__ LowRankColumn low_rank_column(const LowRankPart& p, int c) {
+    LowRankColumn k{0.f, 1.f};
+    if (p.kind != LR_PLAIN && c < p.n_out) {
+        k.bias = p.bias[c];
+        if (p.kind == LR_SOFT_DECAY) k.rate = expf(p.rate[c / p.per_rate]);
+    }
+    return k;
+}
+__device__ __forceinline__ float low_rank_decay(const LowRankPart& p, const LowRankColumn& k, float z) {
+    z += k.bias;
+    return expf(-(p.kind == LR_SOFT_DECAY ? k.rate * softplus_f(z) : expf(z)));
+}
+template <typename T>
+__device__ __forceinline__ void low_rank_store(const LowRankPart& p, const LowRankColumn& k, int t, int c, float z) {
     const long long at = (long long)t * p.out_ld + c;
     if (p.kind == LR_PLAIN) reinterpret_cast<T*>(p.out)[at] = from_f32<T>(z);
-    else {
-        z += p.bias[c];
-        const float r = p.kind == LR_SOFT_DECAY ? expf(p.rate[c / p.per_rate]) * softplus_f(z) : expf(z);
-        reinterpret_cast<float*>(p.out)[at] = expf(-r);
-    }
+    else reinterpret_cast<float*>(p.out)[at] = low_rank_decay(p, k, z);
 }
 
 // FP32 cores: a CTA takes 16 tokens and 128 columns, a thread per column; r in order 0 .. rank - 1.
@@ -278,9 +336,10 @@ low_rank_simt_kernel(GemmOut<T> low, int cols, const int* __restrict__ tok_entry
     extern __shared__ float xs[];                     // [LR_TT][rank]
     pdl_launch_dependents();
     pdl_wait();
+    const int t0 = blockIdx.x * LR_TT, nt = min(LR_TT, n - t0);
+    if ((int)blockIdx.y >= args.col_blocks) return bonus_blocks<T>(low, cols, tok_entry, args, t0, nt);
     const bool second = (int)blockIdx.y >= args.col_blocks0;
     const LowRankPart& p = args.part[second ? 1 : 0];
-    const int t0 = blockIdx.x * LR_TT, nt = min(LR_TT, n - t0);
     for (int i = threadIdx.x; i < LR_TT * p.rank; i += blockDim.x) {
         const int tt = i / p.rank, r = i % p.rank;
         float v = 0.f;
@@ -293,6 +352,7 @@ low_rank_simt_kernel(GemmOut<T> low, int cols, const int* __restrict__ tok_entry
     __syncthreads();
     const int c = ((int)blockIdx.y - (second ? args.col_blocks0 : 0)) * 128 + threadIdx.x;
     if (c >= p.n_out) return;
+    const LowRankColumn col = low_rank_column(p, c);
     const T* w = reinterpret_cast<const T*>(p.w);
     float acc[LR_TT];
 #pragma unroll
@@ -304,7 +364,7 @@ low_rank_simt_kernel(GemmOut<T> low, int cols, const int* __restrict__ tok_entry
     }
 #pragma unroll
     for (int tt = 0; tt < LR_TT; ++tt)
-        if (tt < nt && tok_entry[t0 + tt] >= 0) low_rank_store<T>(p, t0 + tt, c, acc[tt]);
+        if (tt < nt && tok_entry[t0 + tt] >= 0) low_rank_store<T>(p, col, t0 + tt, c, acc[tt]);
 }
 
 // Tensor cores (bf16, warp-level MMA), ranks up to 256: a CTA takes 64 tokens (16 per warp) and 64 columns, or
@@ -322,6 +382,11 @@ low_rank_mma_kernel(GemmOut<__nv_bfloat16> low, int cols, const int* __restrict_
                     int n) {
     constexpr int BM = FEW ? 16 : 64;
     extern __shared__ __align__(16) unsigned char lr_smem[];
+    if ((int)blockIdx.y >= args.col_blocks) {
+        pdl_launch_dependents();
+        pdl_wait();
+        return bonus_blocks<__nv_bfloat16>(low, cols, tok_entry, args, blockIdx.x * BM, min(BM, n - (int)blockIdx.x * BM));
+    }
     const bool second = (int)blockIdx.y >= args.col_blocks0;
     const LowRankPart& p = args.part[second ? 1 : 0];
     const int ld = p.ld_w + 8;
@@ -341,14 +406,18 @@ low_rank_mma_kernel(GemmOut<__nv_bfloat16> low, int cols, const int* __restrict_
         *reinterpret_cast<uint4*>(w_s + r * ld + q * 8) = v;
     }
     pdl_wait();
-    for (int i = threadIdx.x; i < BM * p.ld_w; i += blockDim.x) {
-        const int tt = i / p.ld_w, r = i % p.ld_w;
-        float v = 0.f;
-        if (r < p.rank && t0 + tt < n && tok_entry[t0 + tt] >= 0) {
-            v = low.load((long long)(t0 + tt) * cols + p.low_off + r);
-            if (p.tanh_in) v = tanhf(v);
+#pragma unroll 4
+    for (int tt = warp; tt < BM; tt += 4) {
+        const bool ok = t0 + tt < n && tok_entry[t0 + tt] >= 0;
+        const long long at = (long long)(t0 + tt) * cols + p.low_off;
+        for (int r = lane; r < p.ld_w; r += 32) {
+            float v = 0.f;
+            if (ok && r < p.rank) {
+                v = low.load(at + r);
+                if (p.tanh_in) v = tanhf(v);
+            }
+            a_s[tt * ld + r] = __float2bfloat16_rn(v);
         }
-        a_s[tt * ld + r] = __float2bfloat16_rn(v);
     }
     __syncthreads();
     const int wrow = FEW ? 0 : warp * 16;
@@ -372,15 +441,30 @@ low_rank_mma_kernel(GemmOut<__nv_bfloat16> low, int cols, const int* __restrict_
                          : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b2), "r"(b3));
         }
     }
+    const int ta = t0 + wrow + g;
+    bool live[2];
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-        const int t = t0 + wrow + g + 8 * half;
-        if (t >= n || tok_entry[t] < 0) continue;
+    for (int half = 0; half < 2; ++half) live[half] = ta + 8 * half < n && tok_entry[ta + 8 * half] >= 0;
+    // two neighbouring columns a store where rows are evenly long and the first element is aligned
+    const bool pairs = (p.out_ld & 1) == 0 && ((uintptr_t)p.out & 7) == 0;
 #pragma unroll
-        for (int i = 0; i < NB; ++i) {
-            const int c = c0 + wcol + i * 8 + 2 * t4;
-            if (c < p.n_out) low_rank_store<__nv_bfloat16>(p, t, c, acc[i][2 * half]);
-            if (c + 1 < p.n_out) low_rank_store<__nv_bfloat16>(p, t, c + 1, acc[i][2 * half + 1]);
+    for (int i = 0; i < NB; ++i) {
+        const int c = c0 + wcol + i * 8 + 2 * t4;
+        if (c >= p.n_out) continue;
+        const LowRankColumn ka = low_rank_column(p, c), kb = low_rank_column(p, c + 1);
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            if (!live[half]) continue;
+            const int t = ta + 8 * half;
+            const float za = acc[i][2 * half], zb = acc[i][2 * half + 1];
+            if (pairs && c + 1 < p.n_out) {
+                const long long at = (long long)t * p.out_ld + c;
+                if (p.kind == LR_PLAIN) st2(reinterpret_cast<__nv_bfloat16*>(p.out) + at, za, zb);
+                else st2(reinterpret_cast<float*>(p.out) + at, low_rank_decay(p, ka, za), low_rank_decay(p, kb, zb));
+            } else {
+                low_rank_store<__nv_bfloat16>(p, ka, t, c, za);
+                if (c + 1 < p.n_out) low_rank_store<__nv_bfloat16>(p, kb, t, c + 1, zb);
+            }
         }
     }
 }
@@ -606,6 +690,39 @@ head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols
     const int t = (int)(wid / H), h = (int)(wid % H);
     if (tok_entry[t] < 0) return;
     const float* o = o_raw + ((long long)t * H + h) * dv;
+    if (((dv | cols | gate_off) & 1) == 0 && (norm_step & 1) == 0) {          // heads of even size: two neighbours a lane
+        const long long gp = (long long)t * cols + gate_off + h * dv;
+        float2 v[4], gv[4];                                                   // (the first 256 elements stay in registers)
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = 2 * lane + 64 * i;
+            if (c < dv) {
+                v[i] = ld2(o + c);
+                gv[i] = proj.load2(gp + c);
+                ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
+            }
+        }
+        for (int c = 2 * lane + 256; c < dv; c += 64) {
+            const float2 a = ld2(o + c);
+            ss = fmaf(a.x, a.x, fmaf(a.y, a.y, ss));
+        }
+        ss = warp_sum(ss);
+        const float rstd = rsqrtf(ss / (float)dv + eps);
+        auto act = [&](float g) { return sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g); };
+        const float* w = norm_w + h * norm_step;
+        T* dst = out + ((long long)t * H + h) * dv;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int c = 2 * lane + 64 * i;
+            if (c < dv) st2(dst + c, v[i].x * rstd * w[c] * act(gv[i].x), v[i].y * rstd * w[c + 1] * act(gv[i].y));
+        }
+        for (int c = 2 * lane + 256; c < dv; c += 64) {
+            const float2 a = ld2(o + c), g = proj.load2(gp + c);
+            st2(dst + c, a.x * rstd * w[c] * act(g.x), a.y * rstd * w[c + 1] * act(g.y));
+        }
+        return;
+    }
     float ss = 0.f;
     for (int c = lane; c < dv; c += 32) { const float v = o[c]; ss = fmaf(v, v, ss); }
     ss = warp_sum(ss);
@@ -688,7 +805,7 @@ CRANE_API int crane_conv_delta_prep(int dtype, const void* proj, const float* pr
                                     long long slot_stride, long long conv_off, const float* conv_w, int taps,
                                     const float* a_log, const float* dt_bias, float* aux, int aux_cols,
                                     int n_tokens, int n_entries, int H, int G, int d, int dv, int b_off, int a_off,
-                                    int w_off, int beta_off, float key_eps, float q_scale, int* err,
+                                    int w_off, int beta_off, float key_eps, float q_scale, int all_single, int* err,
                                     cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     const int C = 2 * G * d + H * dv;
@@ -699,11 +816,12 @@ CRANE_API int crane_conv_delta_prep(int dtype, const void* proj, const float* pr
     while (by > 1 && (long long)n_tokens * by > 4 * 148) by = (by + 1) / 2;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
-        int rc = crane_launch(conv_delta_prep_kernel<T>, dim3(n_tokens, by), dim3(256), 0, st, p, cols, tok_entry,
-                              cu_q, kv_len, slots, n_slots, (const float*)state, slot_stride, conv_off, conv_w,
+        const auto kern = all_single ? conv_delta_prep_kernel<T, true> : conv_delta_prep_kernel<T, false>;
+        int rc = crane_launch(kern, dim3(n_tokens, by), dim3(256), 0, st, p, cols, tok_entry,
+                              cu_q, kv_len, slots, n_slots, (const float*)state, state, slot_stride, conv_off, conv_w,
                               taps, a_log, dt_bias, aux, aux_cols, H, G, d, dv, b_off, a_off, w_off, beta_off, key_eps,
                               q_scale, err);
-        if (rc != 0 || taps == 1) return rc;
+        if (rc != 0 || taps == 1 || all_single) return rc;
         return crane_launch(conv_state_update_kernel<T>, dim3((C + 127) / 128, n_entries), dim3(128), 0, st, p,
                             cols, cu_q, kv_len, slots, n_slots, state, slot_stride, conv_off, taps, C);
     });
@@ -743,8 +861,9 @@ CRANE_API int crane_bonus_prep(int dtype, const void* proj, const float* proj_pa
     const long long warps = (long long)n_tokens * H;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
+        const BonusJob job{u, aux, aux_cols, b_off, H, d, dv};
         return crane_launch(bonus_prep_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, st, p, cols,
-                            tok_entry, u, aux, aux_cols, b_off, n_tokens, H, d, dv);
+                            tok_entry, job, n_tokens);
     });
 }
 
@@ -756,9 +875,17 @@ CRANE_API int crane_low_rank_expand(int dtype, const void* low, const float* low
                                     void* out1, long long out_ld1, int low_off1, int rank1, int ld_w1, int n_out1,
                                     int kind1, int tanh1, const void* w2, const float* bias2, const float* rate2,
                                     int per_rate2, void* out2, long long out_ld2, int low_off2, int rank2, int ld_w2,
-                                    int n_out2, int kind2, int tanh2, int n_tokens, cudaStream_t st) {
+                                    int n_out2, int kind2, int tanh2, const float* bonus_u, float* bonus_aux,
+                                    int bonus_aux_cols, int bonus_off, int bonus_H, int bonus_d, int bonus_dv,
+                                    int n_tokens, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     LowRankArgs a;
+    a.bonus = BonusJob{bonus_u, bonus_aux, bonus_aux_cols, bonus_off, bonus_H, bonus_d, bonus_dv};
+    auto bonus_count = [&](int rows_per_tile) {              // blocks for the bonus job: about a pair a warp, 64 at most
+        if (bonus_u == nullptr) return 0;
+        const int blocks = ((n_tokens < rows_per_tile ? n_tokens : rows_per_tile) * bonus_H + 3) / 4;
+        return blocks < 64 ? blocks : 64;
+    };
     a.part[0] = LowRankPart{w1, bias1, rate1, out1, out_ld1, low_off1, rank1, ld_w1, n_out1, kind1, tanh1, per_rate1 > 0 ? per_rate1 : 1};
     a.part[1] = LowRankPart{w2, bias2, rate2, out2, out_ld2, low_off2, rank2, ld_w2, n_out2, kind2, tanh2, per_rate2 > 0 ? per_rate2 : 1};
     int widest = rank1;
@@ -773,6 +900,7 @@ CRANE_API int crane_low_rank_expand(int dtype, const void* low, const float* low
         }
         const int b0 = (n_out1 + LR_COLS - 1) / LR_COLS, b1 = n_out2 > 0 ? (n_out2 + LR_COLS - 1) / LR_COLS : 0;
         a.col_blocks0 = b0;
+        a.col_blocks = b0 + b1;
         const bool few = n_tokens <= 16;
         const int bm = few ? 16 : 64;
         const size_t smem = (size_t)(bm + LR_COLS) * (ldm + 8) * sizeof(__nv_bfloat16);
@@ -784,19 +912,20 @@ CRANE_API int crane_low_rank_expand(int dtype, const void* low, const float* low
             attr_set = true;
         }
         GemmOut<__nv_bfloat16> l{(const __nv_bfloat16*)low, low_parts, n_parts, part_stride};
-        return crane_launch(kern, dim3((n_tokens + bm - 1) / bm, b0 + b1), dim3(128), smem, st, l, cols, tok_entry, a,
-                            n_tokens);
+        return crane_launch(kern, dim3((n_tokens + bm - 1) / bm, b0 + b1 + bonus_count(bm)), dim3(128), smem, st, l, cols,
+                            tok_entry, a, n_tokens);
     }
     const int b0 = (n_out1 + 127) / 128, b1 = n_out2 > 0 ? (n_out2 + 127) / 128 : 0;
     a.col_blocks0 = b0;
+    a.col_blocks = b0 + b1;
     const size_t smem = (size_t)LR_TT * (widest > 0 ? widest : 1) * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     DISPATCH_T(dtype, {
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(low_rank_simt_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         GemmOut<T> l{(const T*)low, low_parts, n_parts, part_stride};
-        return crane_launch(low_rank_simt_kernel<T>, dim3((n_tokens + LR_TT - 1) / LR_TT, b0 + b1), dim3(128), smem, st, l,
-                            cols, tok_entry, a, n_tokens);
+        return crane_launch(low_rank_simt_kernel<T>, dim3((n_tokens + LR_TT - 1) / LR_TT, b0 + b1 + bonus_count(LR_TT)), dim3(128),
+                            smem, st, l, cols, tok_entry, a, n_tokens);
     });
 }
 

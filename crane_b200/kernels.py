@@ -54,13 +54,13 @@ _SIGNATURES = {
     "crane_projection_norm_cache": [I, P, P, I, L, I, P, P, P, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I,
                                     P, P, I, I, P, P, P],
     "crane_streams_norm": [I, P, L, I, P, P, P, I, L, P, P, P, P, P, P, I, I, F, P],
-    "crane_route_grouped": [P, I, P, P, I, I, I, I, I, I, I, P],
+    "crane_route_grouped": [P, P, I, L, I, P, P, I, I, I, I, I, I, I, P],
     "crane_gated_activation": [I, P, P, I, L, P, I, I, P, I, I, I, I, I, P],
-    "crane_conv_delta_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P],
+    "crane_conv_delta_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, I, P, P],
     "crane_token_shift_mix": [I, P, P, I, P, P, P, P, I, P, L, L, P, L, I, I, P, P],
     "crane_bonus_prep": [I, P, P, I, L, I, P, P, P, I, I, I, I, I, I, P],
     "crane_low_rank_expand": [I, P, P, I, L, I, P, I, P, P, P, I, P, L, I, I, I, I, I, I, P, P, P, I, P, L, I, I, I, I, I, I,
-                              I, P],
+                              P, P, I, I, I, I, I, I, P],
     "crane_decay_gate_prep": [I, P, P, I, L, I, P, P, P, I, F, F, P, I, I, I, I, I, P],
     "crane_matrix_state_plan": [I, P, P],
     "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, I, I, I, I, P, P],
@@ -118,6 +118,11 @@ def _dt(dtype: torch.dtype) -> int:
     if dtype == torch.bfloat16:
         return 1
     raise KernelError(f"kernels take float32 or bfloat16 storage, got {dtype}")
+
+
+def step_of_single_tokens(ctx) -> bool:
+    """Whether the step's shape says that every entry has one token (or none: a padding entry)."""
+    return bool(getattr(ctx, "all_single", False)) or getattr(ctx, "graph_bucket", 0) > 0
 
 
 def _split(a: Act):
@@ -432,15 +437,17 @@ class Kernels:
 
     def route_grouped(self, z, correction, route, experts: int, top: int, groups: int, keep: int,
                       shared_gate: bool, sigmoid: bool = False) -> None:
-        """Per row of float ``z`` [n, >= experts (+ 1)]: scores = softmax over the experts (``sigmoid``: the
+        """Per row of float ``z`` [n, >= experts (+ 1)] (whole or as partial sums): scores = softmax over the experts (``sigmoid``: the
         sigmoid of each); the ``top`` largest
         of score + correction among the experts of the ``keep`` best of ``groups`` groups are chosen;
         ``route`` [n, experts (+ 1)] gets their scores (zero elsewhere) and, ``shared_gate``, the
         sigmoid of column ``experts`` behind them."""
-        assert z.dtype == torch.float32 and z.stride(1) == 1 and route.is_contiguous()
+        whole, parts, n_parts, stride = _split(z)
+        rows = z.parts[0] if isinstance(z, Partials) else z
+        assert rows.dtype == torch.float32 and rows.stride(1) == 1 and route.is_contiguous()
         self._check(self.lib.crane_route_grouped(
-            z.data_ptr(), z.stride(0), _ptr(correction), route.data_ptr(), z.shape[0], int(experts), int(top),
-            int(groups), int(keep), 1 if shared_gate else 0, 1 if sigmoid else 0, self._stream(z)), "route_grouped")
+            whole, parts, n_parts, stride, rows.stride(0), _ptr(correction), route.data_ptr(), rows.shape[0], int(experts), int(top),
+            int(groups), int(keep), 1 if shared_gate else 0, 1 if sigmoid else 0, self._stream(route)), "route_grouped")
 
     def gated_activation(self, gu: Act, out, route=None, experts: int = 0, per_expert: int = 0,
                          routed_cols: int = 0, shared_gate: bool = False, on_input: bool = False) -> None:
@@ -470,7 +477,7 @@ class Kernels:
         ``a_off`` < 0: no decay is formed): q, k, v through their short convolutions (weights ``conv_w`` [channels, taps]) and silu,
         q and k to unit length per head (q times ``q_scale``), w = exp(-exp(a_log) softplus(a + dt_bias)),
         beta = sigmoid(b).  The convolutions' last taps - 1 inputs live in ``state`` [slots, floats] at
-        ``conv_off`` and are replaced by a second kernel."""
+        ``conv_off``; they are moved on in the same kernel in a step of single tokens (``ctx``), else by a second one."""
         whole, parts, n_parts, stride = _split(proj)
         C = 2 * G * d + H * dv
         b_off = C + H * dv if b_off is None else b_off
@@ -482,7 +489,7 @@ class Kernels:
             ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0),
             int(conv_off), conv_w.data_ptr(), int(taps), _ptr(a_log), _ptr(dt_bias), aux.data_ptr(),
             aux.shape[1], aux.shape[0], ctx.kv_len.shape[0], H, G, d, dv, int(b_off), int(a_off), int(w_off),
-            int(beta_off), float(key_eps), float(q_scale),
+            int(beta_off), float(key_eps), float(q_scale), 1 if step_of_single_tokens(ctx) else 0,
             err.data_ptr(), self._stream(aux)), "conv_delta_prep")
 
     def decay_gate_prep(self, proj: Act, cols, tok_entry, a2t, bias, inv_tau, q_scale, aux, H, d, dv, dtype) -> None:
@@ -546,8 +553,19 @@ class Kernels:
         out[:, :rank] = w
         return out, True
 
-    def low_rank_expand(self, low: Act, cols, tok_entry, n, dtype, a: "Kernels.LowRank", b=None) -> None:
-        """One or two second matrices of low-rank products over rows of ``low``, one launch."""
+    @dataclass
+    class Bonus:
+        """``bonus_prep``'s arguments, for its work to ride along in another kernel's launch."""
+        u: torch.Tensor
+        aux: torch.Tensor
+        b_off: int
+        H: int
+        d: int
+        dv: int
+
+    def low_rank_expand(self, low: Act, cols, tok_entry, n, dtype, a: "Kernels.LowRank", b=None, bonus=None) -> None:
+        """One or two second matrices of low-rank products over rows of ``low``, one launch; ``bonus`` (a
+        ``Kernels.Bonus``): ``bonus_prep`` over the same rows in the same launch."""
         whole, parts, n_parts, stride = _split(low)
         assert b is None or b.mma == a.mma
 
@@ -559,7 +577,10 @@ class Kernels:
                     self.LOW_RANK_KINDS[p.kind], 1 if p.tanh else 0]
         self._check(self.lib.crane_low_rank_expand(
             _dt(dtype), whole, parts, n_parts, stride, int(cols), tok_entry.data_ptr(), 1 if a.mma else 0, *args(a),
-            *args(b), int(n), self._stream(a.out)), "low_rank_expand")
+            *args(b), *([None, None, 0, 0, 0, 0, 0] if bonus is None else
+                        [bonus.u.data_ptr(), bonus.aux.data_ptr(), bonus.aux.stride(0), int(bonus.b_off), bonus.H, bonus.d,
+                         bonus.dv]),
+            int(n), self._stream(a.out)), "low_rank_expand")
 
     SCAN_MODES = {"plain": 0, "delta": 1, "bonus": 2}
 

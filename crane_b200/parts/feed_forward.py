@@ -287,7 +287,7 @@ class GroupedExperts(Part):
 
     def forward(self, h, ctx, rt):
         n, k = h.shape[0], rt.kernels
-        z = rt.linear(h, self.router, None, "router_logits", out_dtype=torch.float32)
+        z = rt.linear(h, self.router, None, "router_logits", out_dtype=torch.float32, keep_parts=True)
         route = rt.ws.get("route_weights", n, self.E + (1 if self.shared_gate else 0), torch.float32)
         k.route_grouped(z, self.correction, route, self.E, self.top, self.groups, self.keep, self.shared_gate,
                         sigmoid=self.sigmoid)

@@ -31,6 +31,7 @@ from dataclasses import replace
 
 import torch
 
+from ..kernels import step_of_single_tokens
 from ..weights.loader import TensorSpec
 from .base import CacheNeed, Part, register_part
 
@@ -224,7 +225,7 @@ class GatedDelta(Part):
         o = rt.ws.get("gated_delta_o", n, hv, rt.dtype)
         k.head_norm_gate(o_raw, gate, gate_cols, gate_off, ctx.tok_entry, self.norm_w, self.eps, o, H, self.m,
                          sigmoid=self.sigmoid_gate)
-        rt.launches += 4 if self.taps > 1 else 3
+        rt.launches += 4 if self.taps > 1 and not step_of_single_tokens(ctx) else 3
         return rt.linear(o, self.o_w, None, "delta_out")
 
 
@@ -276,11 +277,11 @@ class WkvTimeMix(Part):
         self.w, self.H, self.d = int(a["hidden_size"]), int(a["heads"]), int(a["dim"])
         nm = dict(self.NAMES, **(a.get("names") or {}))
         self.eps = float(a.get("norm_eps") or 0.0)
-        # the projections, each of a mix of its own, as one grouped product: [r | k | v | g | w1]
+        # the projections, each of a mix of its own, as one grouped product: [r | k | v | g | w1]; w1 is a product
+        # of its own where it is wider than the heads together (the last group can only be narrower)
         mats = [weights.pop(p + nm[n]) for n in ("r", "k", "v", "g", "w1")]
         self.rank, hd = mats[4].shape[0], self.H * self.d
-        if self.rank > hd:
-            raise ValueError(f"{p}: the decay's inner size {self.rank} is wider than the heads ({hd})")
+        self.w1 = mats.pop() if self.rank > hd else None
         self.w_in = torch.cat(mats, dim=0).contiguous()
         self.cols = self.w_in.shape[0]
         self.mu = torch.stack([weights[p + nm["mu_" + s]] for s in self.MIXES]).contiguous()
@@ -288,7 +289,7 @@ class WkvTimeMix(Part):
         if second.shape[1] != self.rank:
             raise ValueError(f"{p}: the decay's two matrices do not share their inner size")
         packed, mma = rt.kernels.pack_low_rank(second, rt.exact)
-        self.w2 = rt.kernels.LowRank(packed, self.rank, 4 * hd, hd, kind="exp_decay", bias=weights[p + nm["w0"]],
+        self.w2 = rt.kernels.LowRank(packed, self.rank, 4 * hd if self.w1 is None else 0, hd, kind="exp_decay", bias=weights[p + nm["w0"]],
                                      tanh=True, mma=mma)
         self.u, self.norm_w, self.o_w = weights[p + nm["u"]], weights[p + nm["norm"]], weights[p + nm["o"]]
         # rows of the recurrence's inputs: [r | k | v | w | b]
@@ -307,12 +308,18 @@ class WkvTimeMix(Part):
         k.token_shift_mix(h, self.mu, ctx, cache.state, self.row_off, xs, rt.err)
         proj = rt.linear_grouped(xs, self.w_in, hd, "time_mix_proj")
         aux = rt.ws.get("time_mix_aux", n, self.aux_cols, torch.float32)
-        k.bonus_prep(proj, self.cols, ctx.tok_entry, self.u, aux, 4 * hd, H, d, d, rt.dtype)
-        k.low_rank_expand(proj, self.cols, ctx.tok_entry, n, rt.dtype, replace(self.w2, out=aux[:, 3 * hd:]))
+        w2 = replace(self.w2, out=aux[:, 3 * hd:])
+        if self.w1 is None:
+            k.low_rank_expand(proj, self.cols, ctx.tok_entry, n, rt.dtype, w2, bonus=k.Bonus(self.u, aux, 4 * hd, H, d, d))
+        else:
+            k.bonus_prep(proj, self.cols, ctx.tok_entry, self.u, aux, 4 * hd, H, d, d, rt.dtype)
+            low = rt.linear(xs[4], self.w1, None, "time_mix_low", hold=True)
+            k.low_rank_expand(low, self.rank, ctx.tok_entry, n, rt.dtype, w2)
+            rt.launches += 1
         o_raw = rt.ws.get("time_mix_o_raw", n, hd, torch.float32)
         k.matrix_state_scan(aux, (0, hd, 2 * hd, 3 * hd, 4 * hd), True, "bonus", 1, ctx, cache.state, o_raw, H, d, d,
                             rt.err)
         o = rt.ws.get("time_mix_o", n, hd, rt.dtype)
         k.head_norm_gate(o_raw, proj, self.cols, 3 * hd, ctx.tok_entry, self.norm_w, self.eps, o, H, d)
-        rt.launches += 5
+        rt.launches += 4
         return rt.linear(o, self.o_w, None, "time_mix_out")

@@ -97,14 +97,15 @@ class Runtime:
     # ---- matrix product -------------------------------------------------
     def linear(self, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], name: str,
                out_dtype: Optional[torch.dtype] = None, cap: Optional[int] = None,
-               hint_next: bool = True, hold: bool = False) -> Act:
+               hint_next: bool = True, hold: bool = False, keep_parts: bool = False) -> Act:
         """x[M,K] @ w[N,K]^T (+ bias[N], float) -> [M,N] in ``out_dtype`` (the
         model dtype unless stated).  ``hint_next`` False: this product does not
         ask for the next product's weights (its caller streams so much between
         the two that they would not stay in L2).  ``hold``: the result is read
         only after other products have run (a branch of a parallel block): if it
         is left as partial sums, they get a buffer of this product's own name
-        instead of the one that all products of its width share."""
+        instead of the one that all products of its width share.  ``keep_parts``: a float
+        result may stay partial sums too (its reader adds them up)."""
         M, K = x.shape
         N = w.shape[0]
         out_dtype = out_dtype or self.dtype
@@ -126,7 +127,7 @@ class Runtime:
         if serial:
             self.kernels.lib.crane_set_pdl(0)
         try:
-            return self._linear_bf16(x, w, bias, out, hint_next, name if hold else None)
+            return self._linear_bf16(x, w, bias, out, hint_next, name if hold else None, keep_parts=keep_parts)
         finally:
             if serial:
                 self.kernels.lib.crane_set_pdl(1)
@@ -197,7 +198,7 @@ class Runtime:
         return 16 if M <= 16 else 32 if M <= 32 else 64 if M <= 64 else 128 if M <= 128 else 256
 
     def _linear_bf16(self, x, w, bias, out, hint_next: bool = True, own_parts: Optional[str] = None,
-                     group=None) -> Act:
+                     group=None, keep_parts: bool = False) -> Act:
         """``group``: (features, rows) of grouped activations (see ``Kernels.gemm_tcgen05``)."""
         k = self.kernels
         M, K = x.shape
@@ -226,7 +227,7 @@ class Runtime:
                     parts = parts[:slices * M].view(slices, M, N)
                     k.gemm_tcgen05(x, w, bias, parts, self.err, split_k=slices, swap=True, bn=bn, prefetch=nxt, **grp)
                     self.launches += 1
-                    if out.dtype == torch.float32:
+                    if out.dtype == torch.float32 and not keep_parts:
                         k.sum_parts(Partials(parts), out)      # float logits: the slices added in order
                         self.launches += 1
                         return out

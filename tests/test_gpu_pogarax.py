@@ -161,6 +161,9 @@ def _np(t):
 # step; slots in no order
 PLAN = [[(0, 20, 2), (1, 1, 0), (2, 4, 1)], [(2, 5, 1), (0, 1, 2)], [(0, 1, 2)], [(0, 15, 2), (3, 2, 0)], [(3, 9, 0)]]
 PLAN_LENS = [37, 1, 9, 11]
+PLAN_LONG = [[(0, 70, 2), (1, 2, 0), (2, 1, 1), (3, 6, 3)], [(2, 66, 1), (0, 1, 2), (3, 1, 3)], [(0, 3, 2), (3, 67, 3)], [(0, 1, 2), (3, 2, 3)],
+             [(2, 1, 1), (0, 1, 2)], [(0, 1, 2), (2, 1, 1), (3, 1, 3)], [(2, 3, 1), (0, 1, 2)]]
+PLAN_LONG_LENS = [78, 2, 72, 77]
 
 
 def _steps_of(lens, plan, pad=0):
@@ -217,20 +220,21 @@ def test_bonus_prep(K, dtype, H, d, dv):
     from crane_b200.kernels import Partials
     rng = np.random.default_rng(d)
     n, hd, hv = 9, H * d, H * dv
-    cols = 2 * hd + hv + 5
+    cols = 2 * hd + hv + (6 if d == 40 else 5)
     u = rng.standard_normal((H, d))
     ent = np.zeros(n, dtype=np.int32)
     ent[4] = -1
     for form in ("whole", "parts"):
         parts = _dev(rng.standard_normal((2, n, cols)))
         x = parts.sum(0).to(dtype)
-        aux = torch.full((n, 2 * hd + hv + H + 6), 5.0, device=DEV)
+        extra = (2 * hd + hv + H) % 2             # (rows of even length take two neighbours a lane)
+        aux = torch.full((n, 2 * hd + hv + H + 6 + extra), 5.0, device=DEV)
         K.bonus_prep(x if form == "whole" else Partials(parts), cols, _i32(ent), _dev(u), aux, 2 * hd + hv + 6, H, d, dv, dtype)
         xn, got = _np(x), _np(aux)
         b = (xn[:, :hd].reshape(n, H, d) * u * xn[:, hd:2 * hd].reshape(n, H, d)).sum(-1)
         keep = ent >= 0
         assert np.abs(got[keep, :2 * hd + hv] - xn[keep, :2 * hd + hv]).max() < 1e-6, form
-        assert np.abs(got[keep, 2 * hd + hv + 6:] - b[keep]).max() < 2e-5 * max(1.0, np.abs(b).max()), form
+        assert np.abs(got[keep, 2 * hd + hv + 6:2 * hd + hv + 6 + H] - b[keep]).max() < 2e-5 * max(1.0, np.abs(b).max()), form
         assert (got[4] == 5.0).all() and (got[:, 2 * hd + hv:2 * hd + hv + 6] == 5.0).all()
 
 
@@ -286,6 +290,30 @@ def test_low_rank_expand(K, dtype, n, ranks, outs):
         assert np.abs(g1[keep] - want1[keep]).max() < (2e-5 if exact else 8e-3) * max(1.0, np.abs(want1).max()), kind
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("n, H, d", [(1, 3, 16), (8, 5, 40), (70, 2, 64), (200, 33, 8)])
+def test_bonus_rides_along_with_the_low_rank_product(K, dtype, n, H, d):
+    """One launch for the decay and for r, k, v and the bonus gives what two launches give, row by row."""
+    rng = np.random.default_rng(n)
+    hd, rank = H * d, 10
+    cols = 3 * hd + rank
+    proj = _dev(rng.standard_normal((n, cols)), dtype)
+    u = _dev(rng.standard_normal((H, d)))
+    w, mma = K.pack_low_rank(_dev(rng.standard_normal((hd, rank)) * 0.3, dtype), dtype == torch.float32)
+    bias = _dev(rng.standard_normal(hd))
+    ent = np.zeros(n, dtype=np.int32)
+    if n > 4:
+        ent[3] = -1
+    one, two = (torch.full((n, 4 * hd + H), 5.0, device=DEV) for _ in range(2))
+    part = lambda aux: K.LowRank(w, rank, 3 * hd, hd, out=aux[:, 3 * hd:], kind="exp_decay", bias=bias, tanh=True, mma=mma)
+    K.low_rank_expand(proj, cols, _i32(ent), n, dtype, part(one), bonus=K.Bonus(u, one, 4 * hd, H, d, d))
+    K.bonus_prep(proj, cols, _i32(ent), u, two, 4 * hd, H, d, d, dtype)
+    K.low_rank_expand(proj, cols, _i32(ent), n, dtype, part(two))
+    assert torch.equal(one, two)
+    if n > 4:
+        assert (one[3] == 5.0).all()
+
+
 @pytest.mark.parametrize("mode", ["delta", "bonus"])
 @pytest.mark.parametrize("H, G, dk, dv", [(2, 2, 16, 8), (4, 2, 24, 40), (1, 1, 64, 32), (6, 3, 48, 16), (2, 1, 128, 128),
                                           (1, 1, 300, 20), (3, 1, 32, 12), (2, 2, 256, 4), (5, 5, 8, 8)])
@@ -337,9 +365,10 @@ def test_matrix_state_scan_with_a_decay_per_channel(K, mode, H, G, dk, dv):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("shared, sigmoid", [(True, True), (False, False), (False, True)])
-def test_head_norm_gate_options(K, dtype, shared, sigmoid):
+@pytest.mark.parametrize("dv, gate_off", [(40, 7), (40, 6), (300, 0), (128, 8)])
+def test_head_norm_gate_options(K, dtype, shared, sigmoid, dv, gate_off):
     rng = np.random.default_rng(3)
-    n, H, dv, eps, gate_off = 11, 3, 40, 1e-3, 7
+    n, H, eps = 11, 3, 1e-3
     cols = gate_off + H * dv + 2
     o_raw = rng.standard_normal((n, H, dv)) * 0.03                 # small, so that eps counts
     proj = _dev(rng.standard_normal((n, cols)), dtype)
@@ -352,22 +381,27 @@ def test_head_norm_gate_options(K, dtype, shared, sigmoid):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("H, G, d, dv, taps", [(4, 2, 16, 24, 3), (5, 1, 16, 8, 1), (3, 3, 24, 16, 5)])
-def test_conv_prep_without_a_decay(K, dtype, H, G, d, dv, taps):
-    """Other columns for beta, no decay formed, the columns where it would be left alone."""
-    import plain_mufevik as pm
+@pytest.mark.parametrize("H, G, d, dv, taps", [(4, 2, 16, 24, 3), (5, 1, 16, 8, 1), (3, 3, 24, 16, 5), (4, 4, 64, 128, 4),
+                                               (6, 3, 128, 70, 4), (2, 1, 8, 130, 4), (3, 1, 66, 64, 2), (2, 2, 9, 7, 4)])
+@pytest.mark.parametrize("plan, lens", [(PLAN, PLAN_LENS), (PLAN_LONG, PLAN_LONG_LENS)])
+def test_conv_prep_without_a_decay(K, dtype, H, G, d, dv, taps, plan, lens):
+    """Other columns for beta, no decay formed, the columns where it would be left alone; steps of many tokens,
+    whose tiles of tokens hold the ends and beginnings of entries, beside steps of few."""
     rng = np.random.default_rng(taps)
     C = 2 * G * d + H * dv
     b_off = C + 5
     cols = b_off + H + 3
+    cols += cols % 2
     conv_w = rng.standard_normal((C, taps))
-    proj = [_dev(rng.standard_normal((n, cols)), dtype) for n in PLAN_LENS]
+    proj = [_dev(rng.standard_normal((n, cols)), dtype) for n in lens]
     state = torch.full((4, 2 + (taps - 1) * C), 1e3, device=DEV)
     err = _err()
-    for ctx, ents in _steps_of(PLAN_LENS, PLAN):
+    for ctx, ents in _steps_of(lens, plan):
+        ctx.all_single = all(t == 1 for _, _, t, _ in ents)        # (the engine says so: the inputs then move on in one kernel)
         rows = torch.cat([proj[r][b:b + t] for r, b, t, _ in ents])
         n = rows.shape[0]
-        aux = torch.full((n, C + 4 + H), 5.0, device=DEV)
+        wide = C + 4 + H + (C + H) % 2
+        aux = torch.full((n, wide), 5.0, device=DEV)
         K.conv_delta_prep(rows, cols, ctx, state, 2, _dev(conv_w), taps, None, None, aux, H, G, d, dv, 1e-6, d ** -0.5, err, dtype,
                           b_off=b_off, a_off=-1, w_off=0, beta_off=C + 4)
         got = _np(aux)
@@ -379,7 +413,7 @@ def test_conv_prep_without_a_decay(K, dtype, H, G, d, dv, taps):
             k = pp.unit_vector(y[:, G * d:2 * G * d].reshape(-1, G, d))
             want = np.concatenate([q.reshape(len(x), -1), k.reshape(len(x), -1), y[:, 2 * G * d:]], axis=1)[b:b + t]
             assert np.abs(got[at:at + t, :C] - want).max() < 2e-5, (r, b)
-            assert np.abs(got[at:at + t, C + 4:] - pp.sigmoid(x[b:b + t, b_off:b_off + H])).max() < 1e-6
+            assert np.abs(got[at:at + t, C + 4:C + 4 + H] - pp.sigmoid(x[b:b + t, b_off:b_off + H])).max() < 1e-6
             at += t
         assert (got[:, C:C + 4] == 5.0).all()
     assert int(err.item()) == 0
@@ -393,8 +427,13 @@ def test_route_by_sigmoid_scores(K, experts, top):
     z[0] = 40.0 + np.arange(experts)                     # scores that all round to 1: the logits still order them
     z[1] = 0.25                                          # all equal: the lowest indices
     z[2] = -30.0 - np.arange(experts)                    # scores near zero
-    route = torch.full((n, experts), 5.0, device=DEV)
+    from crane_b200.kernels import Partials
+    route, route2 = torch.full((n, experts), 5.0, device=DEV), torch.full((n, experts), 5.0, device=DEV)
     K.route_grouped(_dev(z), None, route, experts, top, 1, 1, False, sigmoid=True)
+    # the logits left as partial sums
+    K.route_grouped(Partials(torch.stack([_dev(z), torch.zeros(n, experts, device=DEV)])), None, route2, experts, top, 1, 1, False,
+                    sigmoid=True)
+    assert torch.equal(route, route2)
     got = _np(route)
     for t in range(n):
         order = sorted(range(experts), key=lambda e: (-float(z[t, e]), e))[:top]
@@ -404,10 +443,11 @@ def test_route_by_sigmoid_scores(K, experts, top):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_weight_on_the_experts_input(K, dtype):
+@pytest.mark.parametrize("F", [6, 16, 264])
+def test_weight_on_the_experts_input(K, dtype, F):
     from crane_b200.kernels import Partials
     rng = np.random.default_rng(8)
-    n, E, F = 7, 4, 6
+    n, E = 7, 4
     cols = E * F
     route = rng.random((n, E)).astype(np.float32)
     route[:, 2] = 0.0
@@ -421,6 +461,9 @@ def test_weight_on_the_experts_input(K, dtype):
         want = pp.silu(w * gn[:, :cols]) * (w * gn[:, cols:])
         assert np.abs(_np(out) - want).max() < (1e-5 if dtype == torch.float32 else 2e-2) * np.abs(want).max(), form
         assert (out[:, 2 * F:3 * F] == 0).all()
+        K.gated_activation(gu if form == "whole" else Partials(parts), out, _dev(route), E, F, cols)
+        want = pp.silu(gn[:, :cols]) * gn[:, cols:] * w
+        assert np.abs(_np(out) - want).max() < (1e-5 if dtype == torch.float32 else 2e-2) * np.abs(want).max(), form
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -68,11 +68,12 @@ PB = {
     ],
 }
 
-# recurrences only (no layer asks for pages); heads of 8 and of 40 (rows past the lanes' own)
+# recurrences only (no layer asks for pages); heads of 8 and of 40 (rows past the lanes' own); a decay's inner size
+# above the heads' width
 PC = {
     "architecture": "Pogarax", "vocab": 89, "width": 56, "norm": {"eps": 1e-5}, "residual_mult": 1.7,
     "layers": [
-        _moe(_wkv(1, 40, 4), 6, 2, 16),
+        _moe(_wkv(1, 40, 44), 6, 2, 16),
         _none(_delta(2, 2, 40, 12, 2, 4, 4)),
         _dense(_wkv(5, 8, 3), 24),
         _moe(_delta(6, 3, 8, 8, 4, 2, 5), 4, 2, 8),

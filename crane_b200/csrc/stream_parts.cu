@@ -78,8 +78,55 @@ add_normed_norm_kernel(float* __restrict__ x, GemmOut<T> delta, const float* __r
     extern __shared__ __align__(16) float row[];
     __shared__ float scratch[32];
     pdl_launch_dependents();
-    pdl_wait();
     const long long base = (long long)blockIdx.x * hidden;
+    // Rows of four columns a thread (the few rows of a step of single tokens): everything a thread reads is in flight
+    // at once, the weights before the wait for the kernel before, and stays in its registers.
+    if (hidden % 4 == 0 && hidden <= 4 * (int)blockDim.x && delta.part_stride % 4 == 0 &&
+        ((uintptr_t)x | (uintptr_t)wd | (uintptr_t)wo | (uintptr_t)delta.parts) % 16 == 0 &&
+        ((uintptr_t)out | (uintptr_t)raw | (uintptr_t)delta.whole) % 8 == 0) {
+        const int c = threadIdx.x * 4;
+        const bool in = c < hidden;
+        float4 d = make_float4(0.f, 0.f, 0.f, 0.f), v = d, w1 = d, w2 = d;
+        if (in) {
+            w1 = *(const float4*)(wd + c);
+            if (out != nullptr) w2 = *(const float4*)(wo + c);
+        }
+        pdl_wait();
+        if (in) {
+            v = *(const float4*)(x + base + c);
+            if (delta.parts == nullptr) {
+                const float2 a = ld2(delta.whole + base + c), b = ld2(delta.whole + base + c + 2);
+                d = make_float4(a.x, a.y, b.x, b.y);
+            } else {                                   // slices added in order, rounded once, as GemmOut's readers do
+                for (int i = 0; i < delta.n_parts; i += 8) {
+                    float4 q[8];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j)
+                        q[j] = i + j < delta.n_parts ? *(const float4*)(delta.parts + (long long)(i + j) * delta.part_stride + base + c)
+                                                     : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) d.x += q[j].x, d.y += q[j].y, d.z += q[j].z, d.w += q[j].w;
+                }
+                d.x = to_f32(from_f32<T>(d.x)), d.y = to_f32(from_f32<T>(d.y));
+                d.z = to_f32(from_f32<T>(d.z)), d.w = to_f32(from_f32<T>(d.w));
+            }
+        }
+        const float rs = rsqrtf(block_sum((d.x * d.x + d.y * d.y) + (d.z * d.z + d.w * d.w), scratch) / (float)hidden + eps_d);
+        v = make_float4(v.x + d.x * rs * w1.x, v.y + d.y * rs * w1.y, v.z + d.z * rs * w1.z, v.w + d.w * rs * w1.w);
+        if (in) {
+            *(float4*)(x + base + c) = v;
+            if (raw != nullptr) { st2(raw + base + c, v.x, v.y); st2(raw + base + c + 2, v.z, v.w); }
+        }
+        if (out == nullptr) return;
+        if (!in) v = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float rn = rsqrtf(block_sum((v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w), scratch) / (float)hidden + eps_o);
+        if (in) {
+            st2(out + base + c, v.x * rn * w2.x, v.y * rn * w2.y);
+            st2(out + base + c + 2, v.z * rn * w2.z, v.w * rn * w2.w);
+        }
+        return;
+    }
+    pdl_wait();
     float ss = 0.f;
     // (rows of a multiple of 4 columns go four columns a thread and pass; `hidden` and the tensors'
     // alignment are the same for every row, so the branch is uniform)
@@ -300,9 +347,9 @@ CRANE_API int crane_add_normed_norm(int dtype, float* x, const void* delta, cons
         GemmOut<T> d{(const T*)delta, delta_parts, n_parts, part_stride};
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(add_normed_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        // few rows (a step of single tokens): more threads a row, so that a thread's loads, each of which
-        // waits for memory, are few
-        const int threads = n_rows <= 64 ? (hidden >= 4096 ? 1024 : hidden >= 1024 ? 512 : 256) : 256;
+        // few rows (a step of single tokens): four columns a thread where a block has that many
+        const int want = (hidden / 4 + 31) / 32 * 32;
+        const int threads = n_rows <= 64 ? (want < 256 ? 256 : want > 1024 ? 1024 : want) : 256;
         return crane_launch(add_normed_norm_kernel<T>, dim3(n_rows), dim3(threads), smem, st, x, d, wd, wo, (T*)out,
                             (T*)raw, hidden, eps_d, eps_o);
     });

@@ -155,7 +155,7 @@ def test_embed_sinusoid(K, hidden):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("hidden", [68, 96, 1000])
+@pytest.mark.parametrize("hidden", [67, 68, 96, 1000, 3072, 4104])
 def test_add_normed_norm(K, dtype, hidden):
     from crane_b200.kernels import Partials
     rng = np.random.default_rng(hidden)

@@ -56,6 +56,9 @@ struct FusedArgs {
     int general;                    // 0: the defaults (whole head, contiguous halves, norm after, plain w)
     int sink;                       // (the plain form too) the softmax has one more candidate of score 0 that
                                     // has no value: exp2(0 - max) joins the sum where the output is divided
+    const float* sinks;             // (the plain form too) the same with a score of its own per query head, float [nq]
+    int gate_off;                   // >= 0 (the plain form too, where qkv names the gate's product): the result is
+                                    // multiplied by the sigmoid of column gate_off + h D + c of the token's row
     int cross;                      // (the plain form only) a CTA per (slice, pair of key/value heads, request):
                                     // queries and keys of the first, values of the second; always through the
                                     // scratch memory, and the merge kernel writes float [row][nq][nkv][d]
@@ -65,8 +68,23 @@ struct FusedArgs {
 __device__ __forceinline__ float raw1(const FusedArgs& a, long long idx) {
     if (a.qkv_parts == nullptr) return __bfloat162float(a.qkv[idx]);
     float s = 0.f;
-    for (int i = 0; i < a.n_parts; ++i) s += a.qkv_parts[(long long)i * a.part_stride + idx];
+    for (int i = 0; i < a.n_parts; i += 8) {                 // eight loads in flight, added in slice order
+        float p[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) p[j] = (i + j < a.n_parts) ? a.qkv_parts[(long long)(i + j) * a.part_stride + idx] : 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s += p[j];
+    }
     return __bfloat162float(__float2bfloat16_rn(s));
+}
+
+// One output: acc over the softmax's sum L (scores relative to mb, in units of log2 e), sinks and gate applied.
+__device__ __forceinline__ float finish_out(const FusedArgs& a, int t, int h, int d, int c, float acc, float L, float mb) {
+    if (a.sink) L += exp2f(-mb);
+    if (a.sinks != nullptr) L += exp2f(a.sinks[h] * 1.4426950408889634f - mb);
+    const float r = L > 0.f ? acc / L : 0.f;
+    if (a.gate_off < 0) return r;
+    return r / (1.f + expf(-raw1(a, (long long)t * a.qkv_stride + a.gate_off + h * d + c)));
 }
 
 __device__ __forceinline__ float2 raw2(const FusedArgs& a, long long idx) {
@@ -501,8 +519,7 @@ paged_decode_attn_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
         }
         const int h = g * n_rep + r;
         if (n_splits == 1 && !fa.cross) {
-            if (fa.sink) L += exp2f(-mb);
-            out[((long long)t * nq + h) * D + c] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+            out[((long long)t * nq + h) * D + c] = __float2bfloat16_rn(finish_out(fa, t, h, D, c, O, L, mb));
         } else {
             const long long pi = (fa.cross ? ((long long)e * nq + h) * nkv + gv : (long long)e * nq + h) * n_splits + split;
             part_o[pi * D + c] = O;
@@ -967,8 +984,7 @@ paged_decode_attn_tma_kernel(const __grid_constant__ CUtensorMap k_map,
         }
         const int h = g * n_rep + r;
         if (n_splits == 1 && !fa.cross) {
-            if (fa.sink) L += exp2f(-mb);
-            out[((long long)t * nq + h) * D + c] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+            out[((long long)t * nq + h) * D + c] = __float2bfloat16_rn(finish_out(fa, t, h, D, c, O, L, mb));
         } else if (CLUSTER) {
             cl_o[r * D + c] = O;
             if (c == 0) { cl_ml[r * 2] = M; cl_ml[r * 2 + 1] = L; }
@@ -1013,8 +1029,8 @@ paged_decode_attn_tma_kernel(const __grid_constant__ CUtensorMap k_map,
                 L += f * ml[sp].y;
                 acc += f * ov[sp];
             }
-            if (fa.sink) L += exp2f(-mb);
-            out[((long long)t * nq + g * n_rep + r) * D + (idx % D)] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+            out[((long long)t * nq + g * n_rep + r) * D + (idx % D)] =
+                __float2bfloat16_rn(finish_out(fa, t, g * n_rep + r, D, idx % D, acc, L, mb));
         }
         // nobody leaves while a CTA of the cluster may still read its shared memory
         asm volatile("barrier.cluster.arrive.release.aligned;\n"
@@ -1027,7 +1043,7 @@ paged_decode_attn_tma_kernel(const __grid_constant__ CUtensorMap k_map,
 template <int MAXS>
 __device__ __forceinline__ void merge_column(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                              __nv_bfloat16* __restrict__ out, long long base, int t, int nq,
-                                             int h, int d, int n_splits, int sink, int out_float) {
+                                             int h, int d, int n_splits, const FusedArgs& fa, int out_float) {
     for (int c = threadIdx.x; c < d; c += blockDim.x) {
         float2 ml[MAXS];
         float o[MAXS];
@@ -1047,8 +1063,7 @@ __device__ __forceinline__ void merge_column(const float* __restrict__ part_o, c
             L += f * ml[s].y;
             acc += f * o[s];
         }
-        if (sink) L += exp2f(-mb);
-        const float r = L > 0.f ? acc / L : 0.f;
+        const float r = finish_out(fa, t, h, d, c, acc, L, mb);
         if (out_float) ((float*)out)[((long long)t * nq + h) * d + c] = r;
         else out[((long long)t * nq + h) * d + c] = __float2bfloat16_rn(r);
     }
@@ -1062,9 +1077,9 @@ __device__ __forceinline__ void merge_column(const float* __restrict__ part_o, c
 // four loads in flight per thread.  Always in slice order.
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     __nv_bfloat16* __restrict__ out, const int* __restrict__ cu_q,
-                                    int nq, int d, int n_splits, int sink, int out_float) {
+                                    int nq, int d, int n_splits, const FusedArgs fa, int out_float) {
     __shared__ float wgt[64];
-    __shared__ float m_s[64], l_s[64];
+    __shared__ float m_s[64], l_s[64], sum_s[2];
     pdl_launch_dependents();
     pdl_wait();
     const int e = blockIdx.x, h = blockIdx.y;
@@ -1073,9 +1088,9 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
     if (cu_q[e + 1] - t != 1) return;
     if (n_splits <= 64) {
         // all loads of a thread go out together; 16 slices' worth of registers when that is enough
-        if (n_splits <= 16) merge_column<16>(part_o, part_ml, out, base, t, nq, h, d, n_splits, sink, out_float);
-        else if (n_splits <= 32) merge_column<32>(part_o, part_ml, out, base, t, nq, h, d, n_splits, sink, out_float);
-        else merge_column<64>(part_o, part_ml, out, base, t, nq, h, d, n_splits, sink, out_float);
+        if (n_splits <= 16) merge_column<16>(part_o, part_ml, out, base, t, nq, h, d, n_splits, fa, out_float);
+        else if (n_splits <= 32) merge_column<32>(part_o, part_ml, out, base, t, nq, h, d, n_splits, fa, out_float);
+        else merge_column<64>(part_o, part_ml, out, base, t, nq, h, d, n_splits, fa, out_float);
         return;
     }
     for (int s = threadIdx.x; s < n_splits; s += blockDim.x) {
@@ -1093,9 +1108,8 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
             L += f * l_s[s];
             wgt[s] = f;
         }
-        if (sink) L += exp2f(-mb);
-        const float inv = L > 0.f ? 1.f / L : 0.f;
-        for (int s = 0; s < n_splits; ++s) wgt[s] *= inv;
+        sum_s[0] = L;
+        sum_s[1] = mb;
     }
     __syncthreads();
     for (int c = threadIdx.x; c < d; c += blockDim.x) {
@@ -1111,7 +1125,7 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
             a3 += wgt[s + 3] * v3;
         }
         for (; s < n_splits; ++s) a0 += wgt[s] * po[(long long)s * d];
-        const float r = (a0 + a1) + (a2 + a3);
+        const float r = finish_out(fa, t, h, d, c, (a0 + a1) + (a2 + a3), sum_s[0], sum_s[1]);
         if (out_float) ((float*)out)[((long long)t * nq + h) * d + c] = r;
         else out[((long long)t * nq + h) * d + c] = __float2bfloat16_rn(r);
     }
@@ -1238,7 +1252,7 @@ int launch_decode(const void* q, void* out, float* part_o, float* part_ml, const
         if ((n_splits > 1 && !cluster) || cross)
             return crane_launch(decode_merge_kernel, dim3(n_entries, nq_out), dim3(D >= 128 ? 128 : 64), 0, st,
                                 (const float*)part_o, (const float*)part_ml, (__nv_bfloat16*)out, cu_q, nq_out,
-                                D, n_splits, fa.sink, cross);
+                                D, n_splits, fa, cross);
         return 0;
     }
     int rc = crane_launch(kern, grid, dim3(WARPS * 32), smem, st, (const __nv_bfloat16*)q,
@@ -1248,7 +1262,7 @@ int launch_decode(const void* q, void* out, float* part_o, float* part_ml, const
     if (rc == 0 && (n_splits > 1 || cross))
         rc = crane_launch(decode_merge_kernel, dim3(n_entries, nq_out), dim3(D >= 128 ? 128 : 64), 0, st,
                           (const float*)part_o, (const float*)part_ml, (__nv_bfloat16*)out, cu_q, nq_out, D,
-                          n_splits, fa.sink, cross);
+                          n_splits, fa, cross);
     return rc;
 }
 }  // namespace
@@ -1314,19 +1328,25 @@ CRANE_API int crane_paged_decode_attention_supports(int d, int nq, int nkv) {
 // n_entries * nq * n_splits * d floats and part_ml n_entries * nq * n_splits * 2
 // when n_splits > 1.  cross != 0: `out` is float [rows][nq][nkv][d], every query head's weights
 // applied to the values of every key/value head; the scratch memory is always used and takes nkv
-// times as much.
+// times as much.  sinks and the gate as in crane_paged_prefill_attention (neither with cross).
 CRANE_API int crane_paged_decode_attention(const void* q, void* out, float* part_o, float* part_ml,
                                            const void* k_pool, const void* v_pool, const int* cu_q,
                                            const int* kv_len, const int* block_table, int max_blocks,
                                            int num_pages, int page_size, int n_entries, int nq, int nkv,
                                            int d, int window, float scale, int n_splits, int sink,
+                                           const float* sinks, const void* gate, const float* gate_parts,
+                                           int gate_n_parts, long long gate_stride, int gate_ld, int gate_off,
                                            int cross, int* err, cudaStream_t st) {
     if (n_entries <= 0) return 0;
     if (!crane_paged_decode_attention_supports(d, nq, nkv) || n_splits < 1 || n_splits > 64 ||
-        (cross && (part_o == nullptr || part_ml == nullptr)))
+        (cross && (part_o == nullptr || part_ml == nullptr || gate_ld > 0 || sinks != nullptr)))
         return (int)cudaErrorInvalidValue;
     FusedArgs none = {};
     none.sink = sink;
+    none.sinks = sinks;
+    none.qkv = (const __nv_bfloat16*)gate; none.qkv_parts = gate_parts; none.n_parts = gate_n_parts;
+    none.part_stride = gate_stride; none.qkv_stride = gate_ld;
+    none.gate_off = gate_ld > 0 ? gate_off : -1;
     none.cross = cross ? 1 : 0;
     return launch_for_head_size(d, 0, q, out, part_o, part_ml, k_pool, v_pool, cu_q, kv_len, block_table,
                                 max_blocks, num_pages, page_size, n_entries, nq, nkv, window, scale,
@@ -1337,7 +1357,8 @@ CRANE_API int crane_paged_decode_attention(const void* q, void* out, float* part
 // (`qkv` whole, or `qkv_parts` as n_parts float partial sums), one row of
 // [q | k | v] (q alone when has_kv == 0) per token.  The kernel encodes and
 // normalises them, writes the new key and value into their pages and attends; a
-// second kernel merges the slices.  Head sizes must be multiples of 4.
+// second kernel merges the slices.  Head sizes must be multiples of 4.  gate_off >= 0: the gate's
+// columns lie there in the same rows.
 CRANE_API int crane_paged_decode_attention_fused(
     const void* qkv, const float* qkv_parts, int n_parts, long long part_stride, int qkv_stride,
     int has_kv, int rotary, const float* cos_tab, const float* sin_tab, int table_len,
@@ -1345,7 +1366,7 @@ CRANE_API int crane_paged_decode_attention_fused(
     void* k_pool, void* v_pool, const int* cu_q, const int* kv_len,
     const int* block_table, int max_blocks, int num_pages, int page_size, int n_entries, int nq, int nkv,
     int d, int window, float scale, int n_splits, int rotary_dim, int interleaved, int norm_first,
-    float norm_offset, int* err, cudaStream_t st) {
+    float norm_offset, const float* sinks, int gate_off, int* err, cudaStream_t st) {
     if (n_entries <= 0) return 0;
     if (rotary_dim <= 0) rotary_dim = d;
     if (!crane_paged_decode_attention_supports(d, nq, nkv) || n_splits < 1 || n_splits > 64 || (d & 3) ||
@@ -1358,7 +1379,7 @@ CRANE_API int crane_paged_decode_attention_fused(
     fa.part_stride = part_stride; fa.qkv_stride = qkv_stride; fa.has_kv = has_kv; fa.rotary = rotary;
     fa.cos_tab = cos_tab; fa.sin_tab = sin_tab; fa.table_len = table_len; fa.q_norm_w = q_norm_w;
     fa.k_norm_w = k_norm_w; fa.eps = eps; fa.k_pool_w = (__nv_bfloat16*)k_pool;
-    fa.v_pool_w = (__nv_bfloat16*)v_pool;
+    fa.v_pool_w = (__nv_bfloat16*)v_pool; fa.sinks = sinks; fa.gate_off = gate_off;
     return launch_for_head_size(d, 1, nullptr, out, part_o, part_ml, k_pool, v_pool, cu_q, kv_len,
                                 block_table, max_blocks, num_pages, page_size, n_entries, nq, nkv, window,
                                 scale, n_splits, err, &fa, st);
@@ -1431,6 +1452,6 @@ CRANE_API int crane_paged_decode_attention_noalloc(const void* q, void* out, con
     }
     return crane_paged_decode_attention(q, out, part_o, part_ml, k_pool, v_pool, cu_q, kv_len,
                                         block_table, max_blocks, num_pages, page_size, n_entries, nq,
-                                        nkv, d, window, scale, n_splits, 0, 0, err, stream);
+                                        nkv, d, window, scale, n_splits, 0, nullptr, nullptr, nullptr, 0, 0, 0, -1, 0, err, stream);
 }
 #endif  // CRANE_HEAD_SIZE

@@ -28,8 +28,9 @@ paged_prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __
                           const __nv_bfloat16* __restrict__ v_pool, const int* __restrict__ cu_q,
                           const int* __restrict__ kv_len, const int* __restrict__ block_table,
                           int max_blocks, int num_pages, int page_size, int n_entries, int nq, int nkv,
-                          int window, float scale_log2, int skip_single, int sink,
-                          float* __restrict__ out_cross, int* err) {
+                          int window, float scale_log2, int skip_single, int sink, const float* __restrict__ sinks,
+                          const GemmOut<__nv_bfloat16> gate, int gate_ld, int gate_off, float* __restrict__ out_cross,
+                          int* err) {
     constexpr int RB = Tile<D>::ROW_BYTES;
     constexpr int TILE_BYTES = BKV * RB;
     constexpr int KS = D / 16, DN = D / 8;
@@ -194,6 +195,11 @@ paged_prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __
         l[0] += exp2f(-m[0]);
         l[1] += exp2f(-m[1]);
     }
+    if (sinks != nullptr) {                          // of a score of its own per query head
+        const float sh = sinks[h] * 1.4426950408889634f;
+        l[0] += exp2f(sh - m[0]);
+        l[1] += exp2f(sh - m[1]);
+    }
     const float inv_a = l[0] > 0.f ? 1.f / l[0] : 0.f, inv_b = l[1] > 0.f ? 1.f / l[1] : 0.f;
     const int c0 = (lane & 3) * 2;
     if (out_cross != nullptr) {
@@ -208,6 +214,20 @@ paged_prefill_attn_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __
                     make_float2(o[dn][2] * inv_b, o[dn][3] * inv_b);
         }
         return;
+    }
+    if (gate_ld > 0) {                               // times the sigmoid of the row's gate columns of this head
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh) {
+            const int r = hh ? rb : ra;
+            if (r >= r_end) continue;
+            const long long gp = (long long)(row0 + r) * gate_ld + gate_off + h * D + c0;
+#pragma unroll
+            for (int dn = 0; dn < DN; ++dn) {
+                const float2 z = gate.load2(gp + dn * 8);
+                o[dn][2 * hh] /= 1.f + expf(-z.x);
+                o[dn][2 * hh + 1] /= 1.f + expf(-z.y);
+            }
+        }
     }
 #pragma unroll
     for (int dn = 0; dn < DN; ++dn) {
@@ -224,7 +244,9 @@ template <int D>
 int launch_prefill(const void* q, void* out, const void* k_pool, const void* v_pool, const int* cu_q,
                    const int* kv_len, const int* block_table, int max_blocks, int num_pages,
                    int page_size, int n_entries, int total_q_tiles, int nq, int nkv, int window,
-                   float scale, int skip_single, int sink, float* out_cross, int* err, cudaStream_t st) {
+                   float scale, int skip_single, int sink, const float* sinks, const void* gate, const float* gate_parts,
+                   int gate_n_parts, long long gate_stride, int gate_ld, int gate_off, float* out_cross, int* err,
+                   cudaStream_t st) {
     constexpr int smem = 4 * BKV * Tile<D>::ROW_BYTES;
     auto kern = paged_prefill_attn_kernel<D>;
     static bool configured = false;
@@ -237,8 +259,10 @@ int launch_prefill(const void* q, void* out, const void* k_pool, const void* v_p
     kern<<<grid, THREADS, smem, st>>>((const __nv_bfloat16*)q, (__nv_bfloat16*)out,
                                       (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, cu_q,
                                       kv_len, block_table, max_blocks, num_pages, page_size, n_entries,
-                                      nq, nkv, window, scale * 1.4426950408889634f, skip_single, sink,
-                                      out_cross, err);
+                                      nq, nkv, window, scale * 1.4426950408889634f, skip_single, sink, sinks,
+                                      GemmOut<__nv_bfloat16>{(const __nv_bfloat16*)gate, gate_parts, gate_n_parts,
+                                                             gate_stride},
+                                      gate_ld, gate_off, out_cross, err);
     return crane_launch_status();
 }
 }  // namespace
@@ -251,12 +275,14 @@ int launch_prefill(const void* q, void* out, const void* k_pool, const void* v_p
     const void *q, void *out, const void *k_pool, const void *v_pool, const int *cu_q, const int *kv_len, \
         const int *block_table, int max_blocks, int num_pages, int page_size, int n_entries,            \
         int total_q_tiles, int nq, int nkv, int window, float scale, int skip_single, int sink,         \
-        float *out_cross, int *err, cudaStream_t st
+        const float *sinks, const void *gate, const float *gate_parts, int gate_n_parts, long long gate_stride, \
+        int gate_ld, int gate_off, float *out_cross, int *err, cudaStream_t st
 #ifdef CRANE_HEAD_SIZE
 extern "C" int CRANE_CAT(crane_prefill_launch_d, CRANE_HEAD_SIZE)(CRANE_PREFILL_LAUNCHER_ARGS) {
     return launch_prefill<CRANE_HEAD_SIZE>(q, out, k_pool, v_pool, cu_q, kv_len, block_table, max_blocks,
                                            num_pages, page_size, n_entries, total_q_tiles, nq, nkv, window,
-                                           scale, skip_single, sink, out_cross, err, st);
+                                           scale, skip_single, sink, sinks, gate, gate_parts, gate_n_parts, gate_stride,
+                                           gate_ld, gate_off, out_cross, err, st);
 }
 #else
 #ifdef CRANE_HEAD_SIZE_LIST          // the head sizes linked into this library (see attention_decode.cu)
@@ -280,20 +306,26 @@ CRANE_API int crane_paged_prefill_attention_supports(int d, int nq, int nkv) {
 // the real ones do nothing).  skip_single != 0: entries of exactly one token are left out (they
 // count no tile either); their rows of `out` are for the decode kernel to write.  out_cross
 // (float [rows][nq][nkv][d], or null): every query head's weights applied to the values of every
-// key/value head, written there instead of `out`.
+// key/value head, written there instead of `out`.  sinks (float [nq], or null): a candidate of that score without
+// a value joins every softmax of its head.  gate_ld > 0: the result is multiplied by the sigmoid of the row's columns
+// gate_off + h d .. of a product whose rows are gate_ld long (whole or as partial sums; all even).
 CRANE_API int crane_paged_prefill_attention(const void* q, void* out, const void* k_pool,
                                             const void* v_pool, const int* cu_q, const int* kv_len,
                                             const int* block_table, int max_blocks, int num_pages,
                                             int page_size, int n_entries, int total_q_tiles, int nq,
                                             int nkv, int d, int window, float scale, int skip_single,
-                                            int sink, float* out_cross, int* err, cudaStream_t st) {
+                                            int sink, const float* sinks, const void* gate, const float* gate_parts,
+                                            int gate_n_parts, long long gate_stride, int gate_ld, int gate_off,
+                                            float* out_cross, int* err, cudaStream_t st) {
     if (n_entries <= 0 || total_q_tiles <= 0) return 0;
+    if (gate_ld > 0 && (((gate_ld | gate_off) & 1) || (gate_stride & 1) || out_cross != nullptr)) return (int)cudaErrorInvalidValue;
     if (!crane_paged_prefill_attention_supports(d, nq, nkv)) return (int)cudaErrorInvalidValue;
 #define CASE(DD)                                                                                      \
     case DD:                                                                                          \
         return crane_prefill_launch_d##DD(q, out, k_pool, v_pool, cu_q, kv_len, block_table, max_blocks, \
                                           num_pages, page_size, n_entries, total_q_tiles, nq, nkv,      \
-                                          window, scale, skip_single, sink, out_cross, err, st);
+                                          window, scale, skip_single, sink, sinks, gate, gate_parts, gate_n_parts, gate_stride, \
+                                           gate_ld, gate_off, out_cross, err, st);
     switch (d) { CRANE_PREFILL_HEAD_SIZES(CASE) }
 #undef CASE
     return (int)cudaErrorInvalidValue;

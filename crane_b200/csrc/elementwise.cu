@@ -20,7 +20,8 @@ CRANE_API void crane_set_pdl(int on) { g_crane_pdl = on ? 1 : 0; }
 // earlier launch on this stream sampled and the host has not seen yet.
 template <typename T>
 __global__ void embed_gather_kernel(const int* __restrict__ tokens, const T* __restrict__ table,
-                                    float* __restrict__ x, T* __restrict__ raw, int hidden, int vocab,
+                                    float* __restrict__ x, T* __restrict__ raw, float scale, float* __restrict__ keep,
+                                    int hidden, int vocab,
                                     const int* __restrict__ deferred, int n_deferred, int* err) {
     pdl_launch_dependents();
     pdl_wait();
@@ -34,8 +35,10 @@ __global__ void embed_gather_kernel(const int* __restrict__ tokens, const T* __r
     const T* src = table + (long long)tok * hidden;
     float* dst = x + (long long)t * hidden;
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-        dst[c] = to_f32(src[c]);
-        if (raw != nullptr) raw[(long long)t * hidden + c] = src[c];       // the stream in the model type
+        const float v = to_f32(src[c]) * scale;
+        dst[c] = v;
+        if (raw != nullptr) raw[(long long)t * hidden + c] = from_f32<T>(v);   // the stream in the model type
+        if (keep != nullptr) keep[(long long)t * hidden + c] = v;
     }
 }
 
@@ -653,11 +656,12 @@ static bool norm_cluster_on() {
 // dtype: 0 = float, 1 = bf16.  Every function returns the CUDA launch status.
 
 CRANE_API int crane_embed_gather(int dtype, const int* tokens, const void* table, float* x, void* raw,
-                                 int n_tokens, int hidden, int vocab, const int* deferred,
+                                 float scale, float* keep, int n_tokens, int hidden, int vocab, const int* deferred,
                                  int n_deferred, int* err, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     DISPATCH_T(dtype, return crane_launch(embed_gather_kernel<T>, dim3(n_tokens), dim3(256), 0, st, tokens,
-                                          (const T*)table, x, (T*)raw, hidden, vocab, deferred, n_deferred, err));
+                                          (const T*)table, x, (T*)raw, scale, keep, hidden, vocab, deferred, n_deferred,
+                                          err));
 }
 
 CRANE_API int crane_add_rmsnorm(int dtype, float* x, const void* delta, const float* delta_parts,

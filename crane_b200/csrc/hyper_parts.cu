@@ -75,11 +75,12 @@ streams_norm_kernel(float* __restrict__ streams, long long stream_stride, int R,
 }
 
 // One warp per token.  z: float logits [n][ld], the first `experts` of a row the router's, column
-// `experts` (if `shared_gate`) the shared expert's gate.  route [n][experts + shared_gate].
+// `experts` (if `shared_gate`) the shared expert's gate.  route [n][experts + shared_gate]: the chosen experts' scores,
+// or, `renorm`, those over their sum (+ 1e-20), times `scale`; zero elsewhere.
 __global__ void __launch_bounds__(128)
 route_grouped_kernel(GemmOut<float> z, int ld, const float* __restrict__ correction,
                      float* __restrict__ route, int n, int experts, int top, int groups, int keep,
-                     int shared_gate, int sigmoid_scores) {
+                     int shared_gate, int sigmoid_scores, int renorm, float scale) {
     extern __shared__ float sm[];                     // per warp: score [E], choice [E], group score [groups]
     pdl_launch_dependents();
     pdl_wait();
@@ -171,6 +172,13 @@ route_grouped_kernel(GemmOut<float> z, int ld, const float* __restrict__ correct
         }
         __syncwarp();
     }
+    if (renorm || scale != 1.f) {                     // the chosen scores over their sum, times a constant
+        __syncwarp();
+        float sum = 0.f;
+        for (int e = lane; e < experts; e += 32) sum += r[e];
+        const float f = renorm ? scale / (warp_sum(sum) + 1e-20f) : scale;
+        for (int e = lane; e < experts; e += 32) r[e] *= f;
+    }
     if (shared_gate && lane == 0) r[experts] = 1.f / (1.f + expf(-z.load(zr + experts)));
 }
 
@@ -260,7 +268,7 @@ CRANE_API int crane_streams_norm(int dtype, float* streams, long long stream_str
 }
 
 CRANE_API int crane_route_grouped(const float* z, const float* z_parts, int n_parts, long long part_stride, int ld, const float* correction, float* route, int n,
-                                  int experts, int top, int groups, int keep, int shared_gate, int sigmoid_scores,
+                                  int experts, int top, int groups, int keep, int shared_gate, int sigmoid_scores, int renorm, float scale,
                                   cudaStream_t st) {
     if (n <= 0) return 0;
     if (experts <= 0 || top <= 0 || groups <= 0 || experts % groups || keep <= 0 || keep > groups)
@@ -269,7 +277,7 @@ CRANE_API int crane_route_grouped(const float* z, const float* z_parts, int n_pa
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     return crane_launch(route_grouped_kernel, dim3((n + 3) / 4), dim3(128), smem, st,
                         GemmOut<float>{z, z_parts, n_parts, part_stride}, ld, correction, route, n,
-                        experts, top, groups, keep, shared_gate ? 1 : 0, sigmoid_scores);
+                        experts, top, groups, keep, shared_gate ? 1 : 0, sigmoid_scores, renorm, scale);
 }
 
 CRANE_API int crane_gated_activation(int dtype, const void* gu, const float* gu_parts, int n_parts,

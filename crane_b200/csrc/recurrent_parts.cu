@@ -7,6 +7,9 @@
 // or, `bonus`,
 //     o_t = S^T r_t + b_t v_t                (the read-out sees the state BEFORE the token's write, and of the
 //     S <- diag(w_t) S + k_t v_t^T            token itself only b_t = sum_i r_i u_i k_i, a number per head)
+// or, `gated`,
+//     S <- w_t S + b_t k_t v_t^T,  N <- w_t N + b_t k_t     (N: one more column of S whose values are 1)
+//     o_t = S^T q_t,  den_t = N . q_t                       (divided where the head is normed)
 //
 // `matrix_state_scan` walks each request's tokens in order.  Columns of S do not talk to one another:
 // a CTA holds a block of columns of one (request, head), a column's rows spread over LANES lanes of a
@@ -19,11 +22,14 @@
 //     `conv_state_update`;
 //   * `decay_gate_prep`: q scaled, k, v, and w = sigmoid(z)^(1 / tau) per key channel with z a
 //     low-rank product plus bias;
+//   * `exp_gate_prep`: q scaled, k, v, and of exponential gates under a running maximum the kept share w, the new
+//     token's share b and the floor of the normaliser, per head; the maximum is part of the request's state;
 //   * `bonus_prep` (also as further blocks of `low_rank_expand`): r, k, v and the number b per head.
 // `token_shift_mix` forms what the projections of the bonus recurrence read, h + (h' - h) mu with h' the
 // previous token's row, which is part of the request's state.  `low_rank_expand` is the second matrix of a
 // low-rank product with what follows it (a decay, or nothing).
-// `head_norm_gate` norms each head's read-out over dv, applies the weight and silu(gate) or sigmoid(gate).
+// `head_norm_gate` norms each head's read-out over dv (of a `gated` scan after the division by its normaliser),
+// applies the weight and silu(gate) or sigmoid(gate).
 // `head_talk_mix` and `pair_norm_mean` belong to attention whose heads exchange their weights and to
 // two mixers side by side.
 // The state lives in 32-bit in the request's slot, in the order the scan's threads hold it:
@@ -186,6 +192,113 @@ decay_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
     }
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < hv; c += gridDim.y * blockDim.x)
         out[2 * hd + c] = proj.load(row + 2 * hd + c);
+}
+
+// ------------------------------------------------------ exponential gates under a running maximum
+// proj row: [q (H d) | k (H d) | v (H dv) | ...] with the input gate (H) at column `i_off` and the forget gate (H) at
+// `f_off`.  aux row: [q * q_scale | k | v | ...] with w, b and floor (H each) one behind the other at `w_off`:
+//     i = cap tanh((z_i + bias_i) / cap),  f = log sigmoid(cap tanh((z_f + bias_f) / cap))
+//     M' = max(f + M, i);  w = exp(f + M - M'),  b = exp(i - M'),  floor = exp(-M')
+// M (0 before a request's first token) lies in the slot, [H] at `m_off`.  The first `gate_blocks` CTAs work out the
+// gates, a warp per (entry, head); the others copy q, k and v, `by` CTAs a token.  M -> max(M + A, B) composes to
+// maps of the same form, so a warp takes 128 tokens at a time, four a lane, and finds the M before every lane's four by
+// a scan over the lanes; within a lane it goes token by token, and a token's w is taken from the very M that the token
+// before it left.
+template <typename T>
+__global__ void __launch_bounds__(256)
+exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, const int* __restrict__ cu_q,
+                     const int* __restrict__ kv_len, const int* __restrict__ slots, int n_slots,
+                     float* __restrict__ state, long long slot_stride, long long m_off,
+                     const float* __restrict__ bias_i, const float* __restrict__ bias_f, float cap, float q_scale,
+                     float* __restrict__ aux, int aux_cols, int n_entries, int H, int d, int dv, int i_off, int f_off,
+                     int w_off, int gate_blocks, int by, int* err) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int hd = H * d, hv = H * dv;
+    if ((int)blockIdx.x >= gate_blocks) {
+        const int t = ((int)blockIdx.x - gate_blocks) / by, part = ((int)blockIdx.x - gate_blocks) % by;
+        if (tok_entry[t] < 0) return;
+        const long long row = (long long)t * cols;
+        float* out = aux + (long long)t * aux_cols;
+        const int n = 2 * hd + hv;
+        if (((cols | aux_cols | hd | n) & 1) == 0) {
+            for (int c = 2 * (part * blockDim.x + threadIdx.x); c < n; c += 2 * by * blockDim.x) {
+                const float2 v = proj.load2(row + c);
+                const float f = c < hd ? q_scale : 1.f;
+                st2(out + c, v.x * f, v.y * f);
+            }
+        } else {
+            for (int c = part * blockDim.x + threadIdx.x; c < n; c += by * blockDim.x)
+                out[c] = proj.load(row + c) * (c < hd ? q_scale : 1.f);
+        }
+        return;
+    }
+    const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (wid >= n_entries * H) return;
+    const int e = wid / H, h = wid % H;
+    const int first = cu_q[e], q_len = cu_q[e + 1] - first;
+    if (q_len <= 0) return;
+    const int slot = slots[e];
+    if (slot < 0 || slot >= n_slots) {
+        if (lane == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
+        return;
+    }
+    float* kept = state + (long long)slot * slot_stride + m_off + h;
+    float m0 = kv_len[e] > q_len ? *kept : 0.f;
+    const float bi = bias_i[h], bf = bias_f[h];
+    constexpr int PER = 4;
+    float zi[PER], zf[PER];
+    auto fetch = [&](int t0) {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            const int t = t0 + lane * PER + j;
+            const long long row = (long long)(first + (t < q_len ? t : q_len - 1)) * cols + h;
+            zi[j] = proj.load(row + i_off);
+            zf[j] = proj.load(row + f_off);
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < q_len; t0 += 32 * PER) {
+        float li[PER], lf[PER], m[PER];
+        float A = 0.f, B = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            const bool in = t0 + lane * PER + j < q_len;
+            const float x = cap * tanhf((zf[j] + bf) / cap);
+            li[j] = in ? cap * tanhf((zi[j] + bi) / cap) : -INFINITY;          // (past the end: M stays)
+            lf[j] = in ? fminf(x, 0.f) - log1pf(expf(-fabsf(x))) : 0.f;
+            B = fmaxf(B + lf[j], li[j]);
+            A += lf[j];
+        }
+        if (t0 + 32 * PER < q_len) fetch(t0 + 32 * PER);
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float pa = __shfl_up_sync(0xffffffffu, A, o), pb = __shfl_up_sync(0xffffffffu, B, o);
+            if (lane >= o) {
+                B = fmaxf(pb + A, B);
+                A += pa;
+            }
+        }
+        const float pa = __shfl_up_sync(0xffffffffu, A, 1), pb = __shfl_up_sync(0xffffffffu, B, 1);
+        float run = lane == 0 ? m0 : fmaxf(m0 + pa, pb);
+#pragma unroll
+        for (int j = 0; j < PER; ++j) m[j] = run = fmaxf(lf[j] + run, li[j]);
+        const float left = __shfl_up_sync(0xffffffffu, m[PER - 1], 1);
+        float before = lane == 0 ? m0 : left;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            const int t = t0 + lane * PER + j;
+            if (t < q_len) {
+                float* out = aux + (long long)(first + t) * aux_cols + w_off + h;
+                out[0] = expf(lf[j] + before - m[j]);
+                out[H] = expf(li[j] - m[j]);
+                out[2 * H] = expf(-m[j]);
+            }
+            before = m[j];
+        }
+        m0 = __shfl_sync(0xffffffffu, m[PER - 1], 31);
+    }
+    if (lane == 0) *kept = m0;
 }
 
 // ------------------------------------------------------ what the bonus recurrence's projections read
@@ -503,10 +616,11 @@ __device__ __forceinline__ float lanes_sum(float x, int lanes) {
 }
 // A lane holds ROWS neighbouring rows of its column.  FULL: the lanes' rows are exactly the dk rows; no row
 // is tested and a lane reads its part of a vector 16 bytes at a time.  WVEC: a decay per row (else one per
-// head).  MODE: what a token does (plain, the delta rule's correction, bonus).  LANES: the lanes of a column when the kernel is compiled for
+// head).  MODE: what a token does (plain, the delta rule's correction, bonus, gated: there column dv is the normaliser, whose read-out goes
+// to `den`).  LANES: the lanes of a column when the kernel is compiled for
 // them (0: any).  The first `walkers` threads walk the tokens; one more warp does nothing but copy the next
 // tile of tokens into shared memory meanwhile, since a walking warp's time is its instructions per token.
-enum ScanMode : int { SCAN_PLAIN = 0, SCAN_DELTA = 1, SCAN_BONUS = 2 };
+enum ScanMode : int { SCAN_PLAIN = 0, SCAN_DELTA = 1, SCAN_BONUS = 2, SCAN_GATED = 3 };
 template <int ROWS, bool FULL, int MODE, bool WVEC, int LANES>
 __global__ void __launch_bounds__(288)
 matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off, int k_off, int v_off, int w_off,
@@ -514,8 +628,9 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                          const int* __restrict__ kv_len, const int* __restrict__ slots, int n_slots,
                          float* __restrict__ state, long long slot_stride, float* __restrict__ o_raw,
                          int H, int dk, int dv, int lanes_rt, int cols_per_block, int tile_tokens, int vec4,
-                         int walkers, int* err) {
-    constexpr bool DELTA = MODE == SCAN_DELTA, BONUS = MODE == SCAN_BONUS;
+                         int walkers, float* __restrict__ den, int* err) {
+    constexpr bool DELTA = MODE == SCAN_DELTA, BONUS = MODE == SCAN_BONUS, GATED = MODE == SCAN_GATED;
+    const int dvt = dv + (GATED ? 1 : 0);             // columns of the state
     extern __shared__ __align__(16) float tile[];     // two tiles of [tile_tokens][3 dk + cols + 2, to a multiple of 4]
     pdl_launch_dependents();
     pdl_wait();
@@ -540,7 +655,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
     // on 16 bytes and is a multiple of them) or of 4
     const int wl = threadIdx.x & 31;
     const int unit = vec4 ? 4 : 1;
-    const int nq = dk / unit, nvu = min(cols_per_block, dv - c0) / unit;
+    const int nq = dk / unit, nvu = max(0, min(cols_per_block, dv - c0)) / unit;
     const int n_units = (WVEC ? 3 : 2) * nq + nvu;
     auto place = [&](int x, int& so, int& dofs) {                    // unit x of a token: where from, where to
         if (x < nq) so = q_off + hq * dk + x * unit, dofs = x * unit;
@@ -576,7 +691,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                 if (WVEC) b[3 * dk + cols_per_block] = 1.f;
                 else cp_async4(b + 3 * dk + cols_per_block, a + w_off + h);
             } else if (wl == 1) {
-                if (DELTA || BONUS) cp_async4(b + 3 * dk + cols_per_block + 1, a + beta_off + h);
+                if (DELTA || BONUS || GATED) cp_async4(b + 3 * dk + cols_per_block + 1, a + beta_off + h);
                 else b[3 * dk + cols_per_block + 1] = 1.f;
             }
         }
@@ -589,24 +704,26 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
     const int lane = threadIdx.x % lanes, cl = threadIdx.x / lanes;
     const int r0 = lane * ROWS;                       // the lane's rows: r0 .. r0 + ROWS - 1
     const int col = c0 + cl;
-    const bool live = !producer && cl < cols_per_block && col < dv;
+    const bool live = !producer && cl < cols_per_block && col < dvt;
+    const bool idle = !__any_sync(0xffffffffu, live);   // (a warp without a column walks nothing)
     const int vcol = live ? cl : 0;
-    // state [H][ROWS][dv][lanes]
-    float* sp = state + (long long)slot * slot_stride + (long long)h * ROWS * dv * lanes;
+    // state [H][ROWS][columns][lanes]
+    float* sp = state + (long long)slot * slot_stride + (long long)h * ROWS * dvt * lanes;
     float s[ROWS];
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
-        s[i] = (live && start > 0 && (FULL || r0 + i < dk)) ? sp[((long long)i * dv + col) * lanes + lane] : 0.f;
+        s[i] = (live && start > 0 && (FULL || r0 + i < dk)) ? sp[((long long)i * dvt + col) * lanes + lane] : 0.f;
     __syncthreads();                                  // the first tile is there
-    const long long o_step = (long long)H * dv;
+    const bool norm_col = GATED && col == dv;
+    const long long o_step = norm_col ? H : (long long)H * dv;
     for (int it = 0; it < n_tiles; ++it) {
         const int t0 = it * tile_tokens;
         const int nt = min(tile_tokens, q_len - t0);
         if (producer) {
             if (it + 1 < n_tiles) fetch(t0 + tile_tokens, tile + ((it + 1) & 1) * tile_floats);
-        } else {
+        } else if (!idle) {
             const float* tp = tile + (it & 1) * tile_floats;
-            float* op = o_raw + (long long)(first + t0) * o_step + h * dv + (live ? col : 0);
+            float* op = (norm_col ? den + h : o_raw + h * dv + (live ? col : 0)) + (long long)(first + t0) * o_step;
 #pragma unroll(ROWS == 8 ? 2 : 1)
             for (int tt = 0; tt < nt; ++tt, tp += stride, op += o_step) {
                 float qv[ROWS], kv[ROWS], wv[ROWS];
@@ -651,6 +768,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                     if (DELTA) dot = fmaf(s[i], kv[i], dot);
                 }
                 float u = vv;
+                if (GATED) u = tp[3 * dk + cols_per_block + 1] * (norm_col ? 1.f : vv);
                 if (DELTA) {
                     dot = lanes_sum<LANES>(dot, lanes);
                     u = tp[3 * dk + cols_per_block + 1] * (vv - dot);
@@ -669,19 +787,21 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
     }
     if (live) {
 #pragma unroll
-        for (int i = 0; i < ROWS; ++i) sp[((long long)i * dv + col) * lanes + lane] = s[i];
+        for (int i = 0; i < ROWS; ++i) sp[((long long)i * dvt + col) * lanes + lane] = s[i];
     }
 }
 
 // ------------------------------------------------------ head norm and gate
 // out[t][h dv + c] = o_raw / rms_over_dv(o_raw) * norm_w[h norm_step + c] * act(gate[t][gate_off + h dv + c]),
 // norm_step 0 (a weight that the heads share) or dv, act silu or, `sigmoid_gate`, sigmoid; a warp per
-// (token, head).
+// (token, head).  `den` [n][H] (or null): o_raw is first divided by max(|den|, floor) + den_eps, floor of token t at
+// floor_at[t * floor_ld + h].
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols, int gate_off,
                       const int* __restrict__ tok_entry, const float* __restrict__ norm_w, int norm_step,
-                      int sigmoid_gate, float eps, T* __restrict__ out, int n, int H, int dv) {
+                      int sigmoid_gate, float eps, const float* __restrict__ den, const float* __restrict__ floor_at,
+                      int floor_ld, float den_eps, T* __restrict__ out, int n, int H, int dv) {
     pdl_launch_dependents();
     pdl_wait();
     const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -690,6 +810,9 @@ head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols
     const int t = (int)(wid / H), h = (int)(wid % H);
     if (tok_entry[t] < 0) return;
     const float* o = o_raw + ((long long)t * H + h) * dv;
+    // the read-out's own normaliser, if it has one, divides it first
+    const float inv = den == nullptr ? 1.f
+                                     : 1.f / (fmaxf(fabsf(den[(long long)t * H + h]), floor_at[(long long)t * floor_ld + h]) + den_eps);
     if (((dv | cols | gate_off) & 1) == 0 && (norm_step & 1) == 0) {          // heads of even size: two neighbours a lane
         const long long gp = (long long)t * cols + gate_off + h * dv;
         float2 v[4], gv[4];                                                   // (the first 256 elements stay in registers)
@@ -708,7 +831,7 @@ head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols
             ss = fmaf(a.x, a.x, fmaf(a.y, a.y, ss));
         }
         ss = warp_sum(ss);
-        const float rstd = rsqrtf(ss / (float)dv + eps);
+        const float rstd = inv * rsqrtf(ss * inv * inv / (float)dv + eps);
         auto act = [&](float g) { return sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g); };
         const float* w = norm_w + h * norm_step;
         T* dst = out + ((long long)t * H + h) * dv;
@@ -726,7 +849,7 @@ head_norm_gate_kernel(const float* __restrict__ o_raw, GemmOut<T> proj, int cols
     float ss = 0.f;
     for (int c = lane; c < dv; c += 32) { const float v = o[c]; ss = fmaf(v, v, ss); }
     ss = warp_sum(ss);
-    const float rstd = rsqrtf(ss / (float)dv + eps);
+    const float rstd = inv * rsqrtf(ss * inv * inv / (float)dv + eps);
     for (int c = lane; c < dv; c += 32) {
         const float g = proj.load((long long)t * cols + gate_off + h * dv + c);
         const float a = sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g);
@@ -842,6 +965,24 @@ CRANE_API int crane_decay_gate_prep(int dtype, const void* proj, const float* pr
     });
 }
 
+CRANE_API int crane_exp_gate_prep(int dtype, const void* proj, const float* proj_parts, int n_parts,
+                                  long long part_stride, int cols, const int* tok_entry, const int* cu_q,
+                                  const int* kv_len, const int* slots, int n_slots, float* state,
+                                  long long slot_stride, long long m_off, const float* bias_i, const float* bias_f,
+                                  float cap, float q_scale, float* aux, int aux_cols, int n_tokens, int n_entries,
+                                  int H, int d, int dv, int i_off, int f_off, int w_off, int* err, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
+    const int gate_blocks = (n_entries * H + 7) / 8;
+    int by = (2 * H * d + H * dv + 511) / 512;               // with few tokens a token's columns spread over more CTAs
+    while (by > 1 && (long long)n_tokens * by > 4 * 148) by = (by + 1) / 2;
+    DISPATCH_T(dtype, {
+        GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
+        return crane_launch(exp_gate_prep_kernel<T>, dim3(gate_blocks + n_tokens * by), dim3(256), 0, st, p, cols,
+                            tok_entry, cu_q, kv_len, slots, n_slots, state, slot_stride, m_off, bias_i, bias_f, cap,
+                            q_scale, aux, aux_cols, n_entries, H, d, dv, i_off, f_off, w_off, gate_blocks, by, err);
+    });
+}
+
 CRANE_API int crane_token_shift_mix(int dtype, const void* h, const float* mu, int mixes, const int* tok_entry,
                                     const int* cu_q, const int* kv_len, const int* slots, int n_slots,
                                     float* state, long long slot_stride, long long row_off, void* out,
@@ -942,19 +1083,19 @@ CRANE_API int crane_matrix_state_plan(int dk, int* rows, int* lanes) {
 CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off, int k_off, int v_off, int w_off,
                                       int beta_off, int w_vec, int mode, int qk_rep, const int* cu_q,
                                       const int* kv_len, const int* slots, int n_slots, float* state,
-                                      long long slot_stride, float* o_raw, int n_entries, int H, int dk, int dv,
-                                      int* err, cudaStream_t st) {
+                                      long long slot_stride, float* o_raw, float* den, int n_entries, int H, int dk,
+                                      int dv, int* err, cudaStream_t st) {
     if (n_entries <= 0) return 0;
     int rows, lanes;
-    if (crane_matrix_state_plan(dk, &rows, &lanes) || dv <= 0 || qk_rep <= 0 || mode < 0 || mode > 2 ||
-        (mode == SCAN_BONUS && !w_vec))
+    if (crane_matrix_state_plan(dk, &rows, &lanes) || dv <= 0 || qk_rep <= 0 || mode < 0 || mode > 3 ||
+        (mode == SCAN_BONUS && !w_vec) || (mode == SCAN_GATED && (w_vec || den == nullptr)))
         return (int)cudaErrorInvalidValue;
     int cpb = 256 / lanes;
     if (cpb > dv) cpb = dv;
     // few entries and heads: narrower blocks of columns, so that more SMs walk (a column's result does not
     // depend on the block it is in)
     while ((long long)n_entries * H * ((dv + cpb - 1) / cpb) < 148 && cpb > 8) cpb /= 2;
-    const int blocks = (dv + cpb - 1) / cpb;
+    const int blocks = (dv + (mode == SCAN_GATED ? 1 : 0) + cpb - 1) / cpb;
     const int walkers = ((cpb * lanes + 31) / 32) * 32;        // and a warp that copies
     const size_t per_token = (size_t)((3 * dk + cpb + 2 + 3) & ~3) * sizeof(float);
     const int vec4 = (dk % 4 == 0 && dv % 4 == 0 && cpb % 4 == 0 && aux_cols % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
@@ -970,6 +1111,8 @@ CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off,
         constexpr int R = decltype(rows_c)::value, L = decltype(lanes_c)::value;
         if (mode == SCAN_BONUS)
             return full ? matrix_state_scan_kernel<R, true, SCAN_BONUS, true, L> : matrix_state_scan_kernel<R, false, SCAN_BONUS, true, 0>;
+        if (mode == SCAN_GATED)
+            return full ? matrix_state_scan_kernel<R, true, SCAN_GATED, false, L> : matrix_state_scan_kernel<R, false, SCAN_GATED, false, 0>;
         if (full) return delta ? (w_vec ? matrix_state_scan_kernel<R, true, SCAN_DELTA, true, L> : matrix_state_scan_kernel<R, true, SCAN_DELTA, false, L>)
                                : (w_vec ? matrix_state_scan_kernel<R, true, SCAN_PLAIN, true, L> : matrix_state_scan_kernel<R, true, SCAN_PLAIN, false, L>);
         return delta ? (w_vec ? matrix_state_scan_kernel<R, false, SCAN_DELTA, true, 0> : matrix_state_scan_kernel<R, false, SCAN_DELTA, false, 0>)
@@ -984,19 +1127,21 @@ CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off,
     else kern = pick(integral_constant<int, 8>{}, integral_constant<int, 0>{});
     return crane_launch(kern, dim3(n_entries, H, blocks), dim3(walkers + 32), smem, st, aux, aux_cols, q_off, k_off,
                         v_off, w_off, beta_off, qk_rep, cu_q, kv_len, slots, n_slots, state, slot_stride,
-                        o_raw, H, dk, dv, lanes, cpb, tile_tokens, vec4, walkers, err);
+                        o_raw, H, dk, dv, lanes, cpb, tile_tokens, vec4, walkers, den, err);
 }
 
 CRANE_API int crane_head_norm_gate(int dtype, const float* o_raw, const void* proj, const float* proj_parts,
                                    int n_parts, long long part_stride, int cols, int gate_off,
                                    const int* tok_entry, const float* norm_w, int norm_step, int sigmoid_gate,
-                                   float eps, void* out, int n_tokens, int H, int dv, cudaStream_t st) {
+                                   float eps, const float* den, const float* floor_at, int floor_ld, float den_eps,
+                                   void* out, int n_tokens, int H, int dv, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     const long long warps = (long long)n_tokens * H;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
         return crane_launch(head_norm_gate_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, st, o_raw, p,
-                            cols, gate_off, tok_entry, norm_w, norm_step, sigmoid_gate, eps, (T*)out, n_tokens, H, dv);
+                            cols, gate_off, tok_entry, norm_w, norm_step, sigmoid_gate, eps, den, floor_at, floor_ld, den_eps,
+                            (T*)out, n_tokens, H, dv);
     });
 }
 

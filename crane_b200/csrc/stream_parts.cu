@@ -66,6 +66,35 @@ stream_enter_kernel(float* __restrict__ x, const float* __restrict__ kept, const
     }
 }
 
+// ------------------------------------------------------ the stream beside the embedding output
+// out[t] = [x[t] + delta[t] | kept[t]] in T: what a product that begins a pass reads.
+template <typename T>
+__global__ void __launch_bounds__(256)
+stream_beside_kernel(const float* __restrict__ x, GemmOut<T> delta, int has_delta, const float* __restrict__ kept,
+                     T* __restrict__ out, long long n, int hidden) {
+    pdl_launch_dependents();
+    pdl_wait();
+    if ((hidden & 1) == 0) {
+        for (long long i = 2 * ((long long)blockIdx.x * blockDim.x + threadIdx.x); i < n; i += 2 * (long long)gridDim.x * blockDim.x) {
+            float2 v = ld2(x + i);
+            if (has_delta) {
+                const float2 d = delta.load2(i);
+                v.x += d.x, v.y += d.y;
+            }
+            const float2 k = ld2(kept + i);
+            T* o = out + i / hidden * 2 * hidden + i % hidden;
+            st2(o, v.x, v.y);
+            st2(o + hidden, k.x, k.y);
+        }
+        return;
+    }
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        T* o = out + i / hidden * 2 * hidden + i % hidden;
+        o[0] = from_f32<T>(x[i] + (has_delta ? delta.load(i) : 0.f));
+        o[hidden] = from_f32<T>(kept[i]);
+    }
+}
+
 // ------------------------------------------------------ x += norm(delta); out = norm(x)
 // y = delta / sqrt(mean(delta^2) + eps) * wd;  x += y;  out = x / sqrt(mean(x^2) + eps) * wo (if out);
 // raw = x in T (if raw).  The weights are what the norms multiply by (an offset is folded in by the host).
@@ -243,10 +272,14 @@ ffn_activation_vec_kernel(const __nv_bfloat16* __restrict__ up, __nv_bfloat16* _
     const int c0 = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
     if (c0 >= cols) return;
     const long long row = blockIdx.y;
-    const uint4 raw = *(const uint4*)(up + row * cols + c0);
-    const __nv_bfloat162* in2 = (const __nv_bfloat162*)&raw;
     float w = 1.f;
     if (route != nullptr && c0 < routed_cols) w = route[row * experts + c0 / per_expert];
+    if (w == 0.f) {                                   // (an expert that was not chosen is not even read)
+        *(uint4*)(out + row * cols + c0) = make_uint4(0u, 0u, 0u, 0u);
+        return;
+    }
+    const uint4 raw = *(const uint4*)(up + row * cols + c0);
+    const __nv_bfloat162* in2 = (const __nv_bfloat162*)&raw;
     uint4 res;
     __nv_bfloat162* out2 = (__nv_bfloat162*)&res;
 #pragma unroll
@@ -264,11 +297,24 @@ ffn_activation_vec_kernel(const __nv_bfloat16* __restrict__ up, __nv_bfloat16* _
             } else {
                 a[k] = gelu_tanh_f(v);
             }
-            a[k] = w == 0.f ? 0.f : a[k] * w;
+            a[k] = a[k] * w;
         }
         out2[i] = __floats2bfloat162_rn(a[0], a[1]);
     }
     *(uint4*)(out + row * cols + c0) = res;
+}
+
+// ------------------------------------------------------ output gate
+// o[t][c] *= sigmoid(gate[t][gate_off + c])
+template <typename T>
+__global__ void __launch_bounds__(256)
+gate_mul_kernel(T* __restrict__ o, GemmOut<T> gate, int gate_ld, int gate_off, long long n, int cols) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const float z = gate.load(i / cols * gate_ld + gate_off + i % cols);
+        o[i] = from_f32<T>(to_f32(o[i]) / (1.f + expf(-z)));
+    }
 }
 
 // ------------------------------------------------------ router
@@ -336,6 +382,19 @@ CRANE_API int crane_stream_enter(float* x, const float* kept, const float* vec, 
     return crane_launch(stream_enter_kernel, dim3(blocks), dim3(256), 0, st, x, kept, vec, n, hidden);
 }
 
+CRANE_API int crane_stream_beside(int dtype, const float* x, const void* delta, const float* delta_parts, int n_parts,
+                                  long long part_stride, const float* kept, void* out, int n_rows, int hidden,
+                                  cudaStream_t st) {
+    if (n_rows <= 0) return 0;
+    const long long n = (long long)n_rows * hidden;
+    const int blocks = (int)((n + 511) / 512 < 4096 ? (n + 511) / 512 : 4096);
+    const int has = (delta != nullptr || delta_parts != nullptr) ? 1 : 0;
+    DISPATCH_T(dtype, {
+        GemmOut<T> d{(const T*)delta, delta_parts, n_parts, part_stride};
+        return crane_launch(stream_beside_kernel<T>, dim3(blocks), dim3(256), 0, st, x, d, has, kept, (T*)out, n, hidden);
+    });
+}
+
 CRANE_API int crane_add_normed_norm(int dtype, float* x, const void* delta, const float* delta_parts,
                                     int n_parts, long long part_stride, const float* wd, const float* wo,
                                     void* out, void* raw, int n_rows, int hidden, float eps_d, float eps_o,
@@ -383,6 +442,17 @@ CRANE_API int crane_ffn_activation(int dtype, const void* up, const float* up_pa
         GemmOut<T> u{(const T*)up, up_parts, n_parts, part_stride};
         return crane_launch(ffn_activation_kernel<T>, dim3(blocks), dim3(256), 0, st, u, (T*)out, n, cols, kind,
                             route, experts, per_expert, routed_cols);
+    });
+}
+
+CRANE_API int crane_gate_mul(int dtype, void* o, const void* gate, const float* gate_parts, int n_parts,
+                             long long part_stride, int gate_ld, int gate_off, int n_rows, int cols, cudaStream_t st) {
+    if (n_rows <= 0 || cols <= 0) return 0;
+    const long long n = (long long)n_rows * cols;
+    const int blocks = (int)((n + 255) / 256 < 8192 ? (n + 255) / 256 : 8192);
+    DISPATCH_T(dtype, {
+        GemmOut<T> g{(const T*)gate, gate_parts, n_parts, part_stride};
+        return crane_launch(gate_mul_kernel<T>, dim3(blocks), dim3(256), 0, st, (T*)o, g, gate_ld, gate_off, n, cols);
     });
 }
 

@@ -19,7 +19,7 @@ from .csrc import build
 P, I, L, F = c_void_p, c_int, c_longlong, c_float
 
 _SIGNATURES = {
-    "crane_embed_gather": [I, P, P, P, P, I, I, I, P, I, P, P],
+    "crane_embed_gather": [I, P, P, P, P, F, P, I, I, I, P, I, P, P],
     "crane_add_rmsnorm": [I, P, P, P, I, L, P, P, P, I, I, F, P],
     "crane_rope_norm_cache": [I, P, P, I, L, I, P, P, P, I, P, P, I, P, P, F, P, P, P, I, I, I, I,
                               I, I, I, I, I, I, I, F, P, P],
@@ -31,11 +31,11 @@ _SIGNATURES = {
     "crane_gemm_bf16_pair": [P, P, P, P, I, I, I, L, L, L, I, I, I, I, I, P, P],
     "crane_paged_attention_simt": [I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P, P],
     "crane_paged_decode_attention_supports": [I, I, I],
-    "crane_paged_decode_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, P],
+    "crane_paged_decode_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, L, I, I, I, P, P],
     "crane_paged_prefill_attention_supports": [I, I, I],
-    "crane_paged_prefill_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P],
+    "crane_paged_prefill_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P, P, I, L, I, I, P, P, P],
     "crane_paged_decode_attention_fused": [P, P, I, L, I, I, I, P, P, I, P, P, F, P, P, P, P, P, P, P, P,
-                                           I, I, I, I, I, I, I, I, F, I, I, I, I, F, P, P],
+                                           I, I, I, I, I, I, I, I, F, I, I, I, I, F, P, I, P, P],
     "crane_prefill_attention_tc_supports": [I, I, I, I],
     "crane_prefill_attention_tc": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
     "crane_embed_bigram": [I, P, P, P, P, I, I, I, I, L, L, P, P, P, P, P, I, P, I, P, P],
@@ -47,14 +47,16 @@ _SIGNATURES = {
     "crane_latent_attention_mma": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P],
     "crane_embed_sinusoid": [I, P, P, P, P, P, P, I, I, I, P, I, P, P],
     "crane_stream_enter": [P, P, P, I, I, P],
+    "crane_stream_beside": [I, P, P, P, I, L, P, P, I, I, P],
     "crane_add_normed_norm": [I, P, P, P, I, L, P, P, P, P, I, I, F, F, P],
     "crane_token_gate": [I, P, P, I, L, P, P, I, I, I, P, I, I, P, I, P, P],
     "crane_ffn_activation": [I, P, P, I, L, P, I, I, I, P, I, I, I, P],
+    "crane_gate_mul": [I, P, P, P, I, L, I, I, I, I, P],
     "crane_route_topk": [P, P, P, P, I, I, I, P],
     "crane_projection_norm_cache": [I, P, P, I, L, I, P, P, P, I, I, I, P, P, F, P, P, P, I, I, I, I, I, I, I,
                                     P, P, I, I, P, P, P],
     "crane_streams_norm": [I, P, L, I, P, P, P, I, L, P, P, P, P, P, P, I, I, F, P],
-    "crane_route_grouped": [P, P, I, L, I, P, P, I, I, I, I, I, I, I, P],
+    "crane_route_grouped": [P, P, I, L, I, P, P, I, I, I, I, I, I, I, I, F, P],
     "crane_gated_activation": [I, P, P, I, L, P, I, I, P, I, I, I, I, I, P],
     "crane_conv_delta_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, I, P, P],
     "crane_token_shift_mix": [I, P, P, I, P, P, P, P, I, P, L, L, P, L, I, I, P, P],
@@ -63,8 +65,12 @@ _SIGNATURES = {
                               P, P, I, I, I, I, I, I, P],
     "crane_decay_gate_prep": [I, P, P, I, L, I, P, P, P, I, F, F, P, I, I, I, I, I, P],
     "crane_matrix_state_plan": [I, P, P],
-    "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, I, I, I, I, P, P],
-    "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, I, I, F, P, I, I, I, P],
+    "crane_exp_gate_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, P, F, F, P, I, I, I, I, I, I, I, I, I, P, P],
+    "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, P, I, I, I, I, P, P],
+    "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, I, I, F, P, P, I, F, P, I, I, I, P],
+    "crane_gate_scan_mma_most": [],
+    "crane_gate_scan_prep": [I, P, P, I, L, I, I, I, P, P, P, P, I, P, L, L, L, P, P, I, P, I, P, P, P, P, P, I, I, I, I, P, P],
+    "crane_channel_scan": [I, P, P, P, I, L, I, I, I, P, P, P, I, P, L, L, L, I, P, I, I, P, P],
     "crane_head_talk_mix": [I, P, P, P, P, I, I, I, I, I, P],
     "crane_pair_norm_mean": [I, P, P, I, L, P, P, I, L, P, P, F, P, I, I, P],
     "crane_delta_rule_prep": [I, P, P, I, L, I, P, P, P, P, P, I, I, I, I, F, F, P],
@@ -177,12 +183,12 @@ class Kernels:
             raise KernelError(f"{what}: CUDA error {code}")
 
     # ---- elementwise ---------------------------------------------------
-    def embed_gather(self, tokens, table, x, err, deferred=None, raw=None) -> None:
-        """``deferred`` int32 [R]: a token id <= -2 is read from its row -id - 2.  ``raw``: the rows once more,
-        in the table's type."""
+    def embed_gather(self, tokens, table, x, err, deferred=None, raw=None, scale: float = 1.0, keep=None) -> None:
+        """x[t] = table[token] * scale.  ``deferred`` int32 [R]: a token id <= -2 is read from its row -id - 2.
+        ``raw``: the rows once more, in the table's type; ``keep``: once more in float."""
         n, hidden = x.shape
         self._check(self.lib.crane_embed_gather(_dt(table.dtype), tokens.data_ptr(), table.data_ptr(),
-                                                x.data_ptr(), _ptr(raw), n, hidden, table.shape[0],
+                                                x.data_ptr(), _ptr(raw), float(scale), _ptr(keep), n, hidden, table.shape[0],
                                                 deferred.data_ptr() if deferred is not None else None,
                                                 deferred.numel() if deferred is not None else 0,
                                                 err.data_ptr(), self._stream(x)), "embed_gather")
@@ -334,6 +340,13 @@ class Kernels:
         self._check(self.lib.crane_stream_enter(x.data_ptr(), _ptr(kept), vec.data_ptr(), x.shape[0], x.shape[1],
                                                 self._stream(x)), "stream_enter")
 
+    def stream_beside(self, x, delta: Optional[Act], kept, out) -> None:
+        """out[t] = [x[t] + delta[t] | kept[t]] in the model dtype; ``x`` and ``kept`` float, ``delta`` may be None."""
+        whole, parts, n_parts, stride = (None, None, 0, 0) if delta is None else _split(delta)
+        self._check(self.lib.crane_stream_beside(_dt(out.dtype), x.data_ptr(), whole, parts, n_parts, stride,
+                                                 kept.data_ptr(), out.data_ptr(), x.shape[0], x.shape[1],
+                                                 self._stream(x)), "stream_beside")
+
     def add_normed_norm(self, x, delta: Act, w_delta, eps_delta: float, w_out=None, eps_out: float = 0.0,
                         out=None, raw=None) -> None:
         """x += delta / rms(delta) * w_delta; then, if given, out = x / rms(x) * w_out and
@@ -365,6 +378,12 @@ class Kernels:
             _dt(out.dtype), whole, parts, n_parts, stride, out.data_ptr(), out.shape[0], out.shape[1],
             self.ACTIVATIONS[kind], _ptr(route), route.shape[1] if route is not None else 0, int(per_expert),
             int(routed_cols), self._stream(out)), "ffn_activation")
+
+    def gate_mul(self, o, gate: Act, cols: int, off: int) -> None:
+        """o *= sigmoid(columns off .. of ``gate``'s rows of ``cols``), ``o`` [rows, width] in place."""
+        whole, parts, n_parts, stride = _split(gate)
+        self._check(self.lib.crane_gate_mul(_dt(o.dtype), o.data_ptr(), whole, parts, n_parts, stride, int(cols),
+                                            int(off), o.shape[0], o.shape[1], self._stream(o)), "gate_mul")
 
     def route_topk(self, logits, route, idx, wt) -> None:
         """Per row of float ``logits`` [n, experts]: the ``top`` (= idx.shape[1]) largest, softmax over
@@ -436,18 +455,19 @@ class Kernels:
             out.shape[0], streams.shape[2], float(eps), self._stream(out)), "streams_norm")
 
     def route_grouped(self, z, correction, route, experts: int, top: int, groups: int, keep: int,
-                      shared_gate: bool, sigmoid: bool = False) -> None:
+                      shared_gate: bool, sigmoid: bool = False, renorm: bool = False, scale: float = 1.0) -> None:
         """Per row of float ``z`` [n, >= experts (+ 1)] (whole or as partial sums): scores = softmax over the experts (``sigmoid``: the
         sigmoid of each); the ``top`` largest
         of score + correction among the experts of the ``keep`` best of ``groups`` groups are chosen;
-        ``route`` [n, experts (+ 1)] gets their scores (zero elsewhere) and, ``shared_gate``, the
-        sigmoid of column ``experts`` behind them."""
+        ``route`` [n, experts (+ 1)] gets their scores (``renorm``: over the sum of the chosen ones + 1e-20) times
+        ``scale`` (zero elsewhere) and, ``shared_gate``, the sigmoid of column ``experts`` behind them."""
         whole, parts, n_parts, stride = _split(z)
         rows = z.parts[0] if isinstance(z, Partials) else z
         assert rows.dtype == torch.float32 and rows.stride(1) == 1 and route.is_contiguous()
         self._check(self.lib.crane_route_grouped(
             whole, parts, n_parts, stride, rows.stride(0), _ptr(correction), route.data_ptr(), rows.shape[0], int(experts), int(top),
-            int(groups), int(keep), 1 if shared_gate else 0, 1 if sigmoid else 0, self._stream(route)), "route_grouped")
+            int(groups), int(keep), 1 if shared_gate else 0, 1 if sigmoid else 0, 1 if renorm else 0, float(scale),
+            self._stream(route)), "route_grouped")
 
     def gated_activation(self, gu: Act, out, route=None, experts: int = 0, per_expert: int = 0,
                          routed_cols: int = 0, shared_gate: bool = False, on_input: bool = False) -> None:
@@ -582,30 +602,102 @@ class Kernels:
                          bonus.dv]),
             int(n), self._stream(a.out)), "low_rank_expand")
 
-    SCAN_MODES = {"plain": 0, "delta": 1, "bonus": 2}
+    SCAN_MODES = {"plain": 0, "delta": 1, "bonus": 2, "gated": 3}
+
+    def exp_gate_prep(self, proj: Act, cols, ctx, state, m_off, bias_i, bias_f, cap, q_scale, aux, H, d, dv, i_off,
+                      f_off, w_off, err, dtype) -> None:
+        """Rows [q | k | v | ...] of a merged projection, with the gates' columns at ``i_off`` and ``f_off``, ->
+        ``aux`` rows [q * q_scale | k | v | ...] in 32-bit with the kept share, the new token's share and the
+        floor of the normaliser (H each, one behind the other) at ``w_off``: i = cap tanh((z_i + bias_i) / cap),
+        f = log sigmoid(cap tanh((z_f + bias_f) / cap)), M' = max(f + M, i), exp(f + M - M'), exp(i - M'), exp(-M').
+        M lives in ``state`` [slots, floats] at ``m_off`` (H floats)."""
+        whole, parts, n_parts, stride = _split(proj)
+        self._check(self.lib.crane_exp_gate_prep(
+            _dt(dtype), whole, parts, n_parts, stride, int(cols), ctx.tok_entry.data_ptr(), ctx.cu_q.data_ptr(),
+            ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0), int(m_off),
+            bias_i.data_ptr(), bias_f.data_ptr(), float(cap), float(q_scale), aux.data_ptr(), aux.shape[1],
+            aux.shape[0], ctx.kv_len.shape[0], H, d, dv, int(i_off), int(f_off), int(w_off), err.data_ptr(),
+            self._stream(aux)), "exp_gate_prep")
+
+    # ---- recurrences with a number per channel ---------------------------
+    @dataclass
+    class GateScan:
+        """The fixed arguments of ``gate_scan_prep`` and ``channel_scan``: where y and x lie in a projection's rows,
+        where the state and the convolution's ring lie in a slot, the convolution ([taps, C], [C]), both gates'
+        matrices (``pack_gates``) with biases [C], softplus(lam) [C], the equal parts of the channels."""
+        y_off: int
+        x_off: int
+        s_off: int
+        ring_off: int
+        conv_w: torch.Tensor
+        conv_b: torch.Tensor
+        gates: torch.Tensor
+        mma: bool
+        rb: torch.Tensor
+        ib: torch.Tensor
+        sp: torch.Tensor
+        parts: int
+
+    def pack_gates(self, ra, ri, exact: bool):
+        """Two stacks of square matrices [parts, c, c] ([out, in]) as the kernel reads them, and whether the
+        tensor-core kernel takes them: rows padded with zeros to a multiple of 16, or turned over."""
+        parts, c, _ = ra.shape
+        padded = -(-c // 16) * 16
+        both = torch.stack([ra, ri])
+        if exact or ra.dtype != torch.bfloat16 or padded > self.lib.crane_gate_scan_mma_most():
+            return both.transpose(2, 3).contiguous(), False
+        out = torch.zeros((2, parts * c, padded), dtype=ra.dtype, device=ra.device)
+        out[:, :, :c] = both.reshape(2, parts * c, c)
+        return out, True
+
+    def gate_scan_prep(self, proj: Act, cols, ctx, state, g: "Kernels.GateScan", aux, out, err, dtype) -> None:
+        """u = conv(x) + bias, r and i = sigmoid(matrix u + bias) in parts, a = exp(-8 r softplus(lam)): ``aux`` float
+        [n, 2 C] = [a | sqrt(1 - a^2) i u] for ``channel_scan``.  In a step of single tokens (``ctx``): the token's
+        S <- a S + sqrt(1 - a^2) i u as well, ``out`` [n, C] = S gelu_tanh(y), and nothing is left to do."""
+        whole, parts, n_parts, stride = _split(proj)
+        self._check(self.lib.crane_gate_scan_prep(
+            _dt(dtype), whole, parts, n_parts, stride, int(cols), g.y_off, g.x_off, ctx.tok_entry.data_ptr(),
+            ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
+            state.stride(0), g.s_off, g.ring_off, g.conv_w.data_ptr(), g.conv_b.data_ptr(), g.conv_w.shape[0],
+            g.gates.data_ptr(), 1 if g.mma else 0, g.rb.data_ptr(), g.ib.data_ptr(), g.sp.data_ptr(), aux.data_ptr(),
+            out.data_ptr(), out.shape[0], out.shape[1], g.parts, 1 if step_of_single_tokens(ctx) else 0, err.data_ptr(),
+            self._stream(out)), "gate_scan_prep")
+
+    def channel_scan(self, aux, proj: Act, cols, ctx, state, g: "Kernels.GateScan", out, err) -> None:
+        """S <- a S + b per channel over every entry's tokens, (a, b) from ``aux`` [n, 2 C], from and to the slots;
+        ``out`` [n, C] = S gelu_tanh(y).  Moves the convolution's ring on."""
+        whole, parts, n_parts, stride = _split(proj)
+        self._check(self.lib.crane_channel_scan(
+            _dt(out.dtype), aux.data_ptr(), whole, parts, n_parts, stride, int(cols), g.y_off, g.x_off,
+            ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
+            state.stride(0), g.s_off, g.ring_off, g.conv_w.shape[0], out.data_ptr(), ctx.kv_len.shape[0], out.shape[1],
+            err.data_ptr(), self._stream(out)), "channel_scan")
 
     def matrix_state_scan(self, aux, offs, w_vec: bool, mode, qk_rep: int, ctx, state, o_raw, H, dk, dv,
-                          err) -> None:
+                          err, den=None) -> None:
         """The recurrence S <- diag(w) S; u = beta (v - S^T k) (``mode`` "delta" or True) or v ("plain" or
-        False); S <- S + k u^T; o = S^T q; or (``mode`` "bonus") o = S^T q + beta v; S <- diag(w) S + k v^T,
+        False); S <- S + k u^T; o = S^T q; or (``mode`` "bonus") o = S^T q + beta v; S <- diag(w) S + k v^T; or (``mode`` "gated")
+        S <- w S + beta k v^T, N <- w N + beta k, o = S^T q, ``den`` float [n, H] = N . q (N is column dv of S),
         over every entry's tokens, from and to ``state`` [slots, floats] (its leading H * rows * lanes * dv
         floats).  ``offs``: columns of q, k, v, w, beta in ``aux``; ``o_raw`` float [n, H dv]."""
         self._check(self.lib.crane_matrix_state_scan(
             aux.data_ptr(), aux.shape[1], *[int(o) for o in offs], 1 if w_vec else 0,
             self.SCAN_MODES[mode] if isinstance(mode, str) else int(bool(mode)), int(qk_rep),
             ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
-            state.stride(0), o_raw.data_ptr(), ctx.kv_len.shape[0], H, dk, dv, err.data_ptr(),
+            state.stride(0), o_raw.data_ptr(), _ptr(den), ctx.kv_len.shape[0], H, dk, dv, err.data_ptr(),
             self._stream(o_raw)), "matrix_state_scan")
 
     def head_norm_gate(self, o_raw, proj: Act, cols, gate_off, tok_entry, norm_w, eps, out, H, dv,
-                       sigmoid: bool = False) -> None:
+                       sigmoid: bool = False, den=None, floor=None, den_eps: float = 0.0) -> None:
         """out = o_raw / rms(o_raw per head) * norm_w * silu(gate columns of ``proj``), or ``sigmoid`` of them.
-        ``norm_w`` [dv] (shared by the heads) or [H dv]."""
+        ``norm_w`` [dv] (shared by the heads) or [H dv].  ``den`` float [n, H]: o_raw is first divided by
+        max(|den|, floor) + den_eps, ``floor`` float [n, H] (rows may be strided)."""
         norm_step = 0 if norm_w.numel() == dv else dv
         whole, parts, n_parts, stride = _split(proj)
         self._check(self.lib.crane_head_norm_gate(
             _dt(out.dtype), o_raw.data_ptr(), whole, parts, n_parts, stride, int(cols), int(gate_off),
-            tok_entry.data_ptr(), norm_w.data_ptr(), norm_step, 1 if sigmoid else 0, float(eps), out.data_ptr(),
+            tok_entry.data_ptr(), norm_w.data_ptr(), norm_step, 1 if sigmoid else 0, float(eps), _ptr(den), _ptr(floor),
+            floor.stride(0) if floor is not None else 0, float(den_eps), out.data_ptr(),
             out.shape[0], H, dv, self._stream(out)), "head_norm_gate")
 
     def head_talk_mix(self, cross, talk, tok_entry, out, H, G, dv, out_head) -> None:
@@ -985,15 +1077,24 @@ class Kernels:
         self.require_head_size(d)
         return bool(self.lib.crane_paged_decode_attention_supports(d, nq, nkv))
 
+    @staticmethod
+    def _gate(gate):
+        if gate is None:
+            return [None, None, 0, 0, 0, 0]
+        return [*_split(gate[0]), int(gate[1]), int(gate[2])]
+
     def paged_decode_attention(self, q, out, k_pool, v_pool, cu_q, kv_len, block_table, page_size,
                                nq, nkv, d, window, scale, n_splits, part_o, part_ml, err, sink: bool = False,
-                               cross: bool = False) -> None:
+                               cross: bool = False, sinks=None, gate=None) -> None:
         """The entries of exactly one token (bfloat16); entries with more or no
         rows are skipped.  ``part_o`` [entries * nq * n_splits * d] and ``part_ml``
         [entries * nq * n_splits * 2] floats are scratch for n_splits > 1.  ``sink``: the
         softmax has one more candidate of score 0 that has no value.  ``cross``: ``out`` is float
         [n, nq, nkv, d], every query head's weights applied to the values of EVERY key/value head
-        (for heads that exchange their weights); the scratch is always used and nkv times as large."""
+        (for heads that exchange their weights); the scratch is always used and nkv times as large.
+        ``sinks`` float [nq]: a candidate of that score without a value joins every softmax of its head.
+        ``gate`` (product, its row length, column): the result is multiplied by the sigmoid of the product's columns
+        column + h d .. of the token's row."""
         assert not cross or (out.dtype == torch.float32 and part_o is not None)
         n_entries = kv_len.shape[0]
         self.require_head_size(d)
@@ -1001,7 +1102,8 @@ class Kernels:
             q.data_ptr(), out.data_ptr(), _ptr(part_o), _ptr(part_ml), k_pool.data_ptr(),
             v_pool.data_ptr(), cu_q.data_ptr(), kv_len.data_ptr(), block_table.data_ptr(),
             block_table.shape[1], k_pool.shape[0], page_size, n_entries, nq, nkv, d, int(window),
-            float(scale), int(n_splits), 1 if sink else 0, 1 if cross else 0, err.data_ptr(), self._stream(q)),
+            float(scale), int(n_splits), 1 if sink else 0, _ptr(sinks), *self._gate(gate), 1 if cross else 0,
+            err.data_ptr(), self._stream(q)),
             "paged_decode_attention")
 
     def prefill_attention_supports(self, d: int, nq: int, nkv: int) -> bool:
@@ -1010,18 +1112,19 @@ class Kernels:
 
     def paged_prefill_attention(self, q, out, k_pool, v_pool, cu_q, kv_len, block_table, page_size,
                                 total_q_tiles, nq, nkv, d, window, scale, err, skip_single=False,
-                                sink: bool = False, cross: bool = False) -> None:
+                                sink: bool = False, cross: bool = False, sinks=None, gate=None) -> None:
         """Any mix of portions and single tokens (bfloat16).  ``total_q_tiles``:
         the sum over the entries of ceil(tokens / 64), or more.  ``skip_single``:
-        entries of exactly one token are left to the decode kernel.  ``sink`` and ``cross`` as in
-        ``paged_decode_attention``."""
+        entries of exactly one token are left to the decode kernel.  ``sink``, ``cross``, ``sinks`` and
+        ``gate`` as in ``paged_decode_attention``."""
         assert not cross or out.dtype == torch.float32
         self.require_head_size(d)
         self._check(self.lib.crane_paged_prefill_attention(
             q.data_ptr(), out.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), cu_q.data_ptr(),
             kv_len.data_ptr(), block_table.data_ptr(), block_table.shape[1], k_pool.shape[0],
             page_size, kv_len.shape[0], int(total_q_tiles), nq, nkv, d, int(window), float(scale),
-            1 if skip_single else 0, 1 if sink else 0, out.data_ptr() if cross else None, err.data_ptr(),
+            1 if skip_single else 0, 1 if sink else 0, _ptr(sinks), *self._gate(gate), out.data_ptr() if cross else None,
+            err.data_ptr(),
             self._stream(q)), "paged_prefill_attention")
 
     def prefill_attention_tc_supports(self, d: int, nq: int, nkv: int, page_size: int) -> bool:
@@ -1041,10 +1144,11 @@ class Kernels:
     def paged_decode_attention_fused(self, qkv: Act, qkv_cols, has_kv, cos, sin, q_norm_w, k_norm_w,
                                      eps, out, k_pool, v_pool, cu_q, kv_len, block_table, page_size,
                                      nq, nkv, d, window, scale, n_splits, part_o, part_ml, err,
-                                     rope=None) -> None:
+                                     rope=None, sinks=None, gate_off: int = -1) -> None:
         """One token per entry, straight from the q/k/v product: rotary encoding,
         per-head norm, cache write and attention in one kernel, then the merge of
-        the key slices.  ``rope`` as in ``rope_norm_cache``."""
+        the key slices.  ``rope`` as in ``rope_norm_cache``; ``sinks`` as in ``paged_decode_attention``;
+        ``gate_off`` >= 0: the result is multiplied by the sigmoid of the product's columns gate_off + h d .. ."""
         rd, inter, first, off = rope or (d, False, False, 0.0)
         whole, parts, n_parts, stride = _split(qkv)
         n_entries = kv_len.shape[0]
@@ -1056,7 +1160,7 @@ class Kernels:
             k_pool.data_ptr(), v_pool.data_ptr(), cu_q.data_ptr(), kv_len.data_ptr(),
             block_table.data_ptr(), block_table.shape[1], k_pool.shape[0], page_size, n_entries, nq,
             nkv, d, int(window), float(scale), int(n_splits), int(rd), 1 if inter else 0,
-            1 if first else 0, float(off), err.data_ptr(), self._stream(out)),
+            1 if first else 0, float(off), _ptr(sinks), int(gate_off), err.data_ptr(), self._stream(out)),
             "paged_decode_attention_fused")
 
     # ---- sampling -------------------------------------------------------

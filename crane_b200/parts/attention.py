@@ -31,54 +31,100 @@ class GqaAttention(Part):
     are rotated; default all), ``rope_pairing`` ("half": element i with
     i + rotary_dim/2, or "interleaved": 2i with 2i + 1), ``qk_norm_order``
     ("after_rope" or "before_rope"), ``qk_norm_offset`` (the norms multiply by
-    offset + w: 0, or 1 for weights stored as w - 1).
+    offset + w: 0, or 1 for weights stored as w - 1).  Beyond the reference:
+    ``sink`` (the softmax's sum also holds exp(sink_h), a learnt number per head without a key
+    or a value), ``gate`` (the heads' results times sigmoid(W_g h) before the output
+    projection), ``key_dim`` / ``value_dim`` (how wide a head's keys and values are where that
+    is less than ``head_dim``, the size they are stored at: the matrices, biases and norm
+    weights get zero rows, or columns, so that every kernel sees heads of ``head_dim``), ``names``.
     Tensors: ``<prefix>{q,k,v,o}_proj.weight`` (+ ``.bias``),
-    ``<prefix>query_layernorm.weight`` / ``key_layernorm.weight`` [head_dim]."""
+    ``<prefix>query_layernorm.weight`` / ``key_layernorm.weight`` [key_dim], gate [heads value_dim, hidden],
+    sink [heads] (float)."""
     kind = "mixer"
+    NAMES = dict({f"{n}": f"{n}_proj.weight" for n in "qkvo"}, **{f"{n}_bias": f"{n}_proj.bias" for n in "qkvo"},
+                 q_norm="query_layernorm.weight", k_norm="key_layernorm.weight", gate="g_proj.weight", sink="sinks")
+
+    @classmethod
+    def _dims(cls, a):
+        """(query heads, key/value heads, stored head size, a key's width, a value's width)"""
+        d = int(a["head_dim"])
+        return int(a["num_heads"]), int(a["num_kv_heads"]), d, int(a.get("key_dim") or d), int(a.get("value_dim") or d)
 
     @classmethod
     def manifest(cls, spec):
-        a = spec.params
-        h, nq, nkv, d = a["hidden_size"], a["num_heads"], a["num_kv_heads"], a["head_dim"]
-        p = spec.prefix
+        a, p = spec.params, spec.prefix
+        h = a["hidden_size"]
+        nq, nkv, _, d, dv = cls._dims(a)
+        nm = dict(cls.NAMES, **(a.get("names") or {}))
         own = a.get("own_kv", True)
-        m = {p + "q_proj.weight": TensorSpec((nq * d, h)), p + "o_proj.weight": TensorSpec((h, nq * d))}
+        m = {p + nm["q"]: TensorSpec((nq * d, h)), p + nm["o"]: TensorSpec((h, nq * dv))}
         if own:
-            m[p + "k_proj.weight"] = TensorSpec((nkv * d, h))
-            m[p + "v_proj.weight"] = TensorSpec((nkv * d, h))
+            m[p + nm["k"]] = TensorSpec((nkv * d, h))
+            m[p + nm["v"]] = TensorSpec((nkv * dv, h))
         if a.get("bias"):
-            m[p + "q_proj.bias"] = TensorSpec((nq * d,), "float32")
-            m[p + "o_proj.bias"] = TensorSpec((h,), "float32")
+            m[p + nm["q_bias"]] = TensorSpec((nq * d,), "float32")
+            m[p + nm["o_bias"]] = TensorSpec((h,), "float32")
             if own:
-                m[p + "k_proj.bias"] = TensorSpec((nkv * d,), "float32")
-                m[p + "v_proj.bias"] = TensorSpec((nkv * d,), "float32")
+                m[p + nm["k_bias"]] = TensorSpec((nkv * d,), "float32")
+                m[p + nm["v_bias"]] = TensorSpec((nkv * dv,), "float32")
         if a.get("qk_norm"):
-            m[p + "query_layernorm.weight"] = TensorSpec((d,), "float32")
+            norm = "scale" if a.get("names") else ""          # (what random weights are, where the name does not say)
+            m[p + nm["q_norm"]] = TensorSpec((d,), "float32", norm)
             if own:
-                m[p + "key_layernorm.weight"] = TensorSpec((d,), "float32")
+                m[p + nm["k_norm"]] = TensorSpec((d,), "float32", norm)
+        if a.get("gate"):
+            m[p + nm["gate"]] = TensorSpec((nq * dv, h))
+        if a.get("sink"):
+            m[p + nm["sink"]] = TensorSpec((nq,), "float32", "unit")
         return m
 
     def load(self, weights, rt):
         a, p = self.params, self.prefix
-        self.nq, self.nkv, self.d = int(a["num_heads"]), int(a["num_kv_heads"]), int(a["head_dim"])
+        self.nq, self.nkv, self.d, dk, dv = self._dims(a)
+        nm = dict(self.NAMES, **(a.get("names") or {}))
         self.own_kv = bool(a.get("own_kv", True))
         self.window = int(a.get("window") or 0)
-        self.scale = float(a.get("scale") or 1.0 / math.sqrt(self.d))
+        self.scale = float(a.get("scale") or 1.0 / math.sqrt(dk))
         self.eps = float(a.get("qk_norm_eps") or 0.0)
         if self.nq % self.nkv:
             raise ValueError(f"{p}: {self.nq} query heads are not a multiple of {self.nkv} kv heads")
-        if self.d % 2 or self.d > 256:
-            raise ValueError(f"{p}: head_dim {self.d} is not supported by the attention kernels "
-                             "(even sizes up to 256)")
-        names = ["q_proj"] + (["k_proj", "v_proj"] if self.own_kv else [])
-        ws = [weights.pop(p + n + ".weight") for n in names]
+        if self.d % 2 or self.d > 512 or max(dk, dv) > self.d:
+            raise ValueError(f"{p}: head_dim {self.d} (keys of {dk}, values of {dv}) is not supported by the attention "
+                             "kernels (even sizes up to 512)")
+        def stored(t, heads, width):
+            """Rows (of a matrix or a bias) of ``heads`` heads of ``width``, with zeros up to the stored size."""
+            if width == self.d:
+                return t
+            out = torch.zeros((heads, self.d) + tuple(t.shape[1:]), dtype=t.dtype, device=t.device)
+            out[:, :width] = t.view((heads, width) + tuple(t.shape[1:]))
+            return out.view((heads * self.d,) + tuple(t.shape[1:]))
+
+        blocks = [("q", self.nq, dk)] + ([("k", self.nkv, dk), ("v", self.nkv, dv)] if self.own_kv else [])
+        ws = [stored(weights.pop(p + nm[n]), heads, width) for n, heads, width in blocks]
+        biases = [stored(weights.pop(p + nm[n + "_bias"]), heads, width) for n, heads, width in blocks] if a.get("bias") else None
+        self.gate_off = -1
+        if a.get("gate"):                            # the gate's columns lie behind q, k and v in the same product
+            self.gate_off = sum(w.shape[0] for w in ws)
+            ws.append(stored(weights.pop(p + nm["gate"]), self.nq, dv))
+            if biases is not None:
+                biases.append(torch.zeros(ws[-1].shape[0], dtype=torch.float32, device=rt.device))
         self.qkv_w = torch.cat(ws, dim=0).contiguous() if len(ws) > 1 else ws[0]
-        self.qkv_b = (torch.cat([weights.pop(p + n + ".bias") for n in names]).contiguous()
-                      if a.get("bias") else None)
-        self.o_w = weights[p + "o_proj.weight"]
-        self.o_b = weights.get(p + "o_proj.bias") if a.get("bias") else None
-        self.q_norm = weights.get(p + "query_layernorm.weight") if a.get("qk_norm") else None
-        self.k_norm = weights.get(p + "key_layernorm.weight") if a.get("qk_norm") and self.own_kv else None
+        self.qkv_b = torch.cat(biases).contiguous() if biases is not None else None
+        self.o_w = weights[p + nm["o"]]
+        if dv != self.d:
+            self.o_w = stored(self.o_w.t().contiguous(), self.nq, dv).t().contiguous()
+        self.o_b = weights.get(p + nm["o_bias"]) if a.get("bias") else None
+        self.sinks = weights[p + nm["sink"]] if a.get("sink") else None
+        self.q_norm = weights.get(p + nm["q_norm"]) if a.get("qk_norm") else None
+        self.k_norm = weights.get(p + nm["k_norm"]) if a.get("qk_norm") and self.own_kv else None
+        offset = float(a.get("qk_norm_offset") or 0.0)
+        if dk != self.d and self.q_norm is not None:
+            # the kernels divide a head's sum of squares by the stored size D: with eps dk / D in the place of
+            # eps the root is sqrt(dk / D) times the one over dk elements, which the weights make up for
+            shrink = math.sqrt(dk / self.d)
+            self.q_norm = stored((self.q_norm + offset) * shrink, 1, dk).contiguous()
+            self.k_norm = stored((self.k_norm + offset) * shrink, 1, dk).contiguous() if self.k_norm is not None else None
+            self.eps, offset = self.eps * dk / self.d, 0.0
         self.position = build_part(a["position"]) if a.get("position") is not None else None
         if self.position is not None:
             self.position.load(weights, rt)          # a position encoding may have tensors of its own
@@ -91,8 +137,7 @@ class GqaAttention(Part):
             raise ValueError(f"{p}: rope_pairing is 'half' or 'interleaved', qk_norm_order 'after_rope' or "
                              f"'before_rope'; got {pairing!r}, {order!r}")
         # (rotated width, interleaved pairs, norm before the rotation, offset added to the norm weights)
-        self.rope = (rotary_dim, pairing == "interleaved", order == "before_rope",
-                     float(a.get("qk_norm_offset") or 0.0))
+        self.rope = (rotary_dim, pairing == "interleaved", order == "before_rope", offset)
         self.max_splits = int(os.environ.get("CRANE_DECODE_SPLITS", "64"))
 
     def cache_need(self) -> CacheNeed:
@@ -100,7 +145,7 @@ class GqaAttention(Part):
             return CacheNeed("none")
         return CacheNeed("kv", kv_heads=self.nkv, head_dim=self.d, window=self.window)
 
-    def forward(self, h, ctx, cache, rt):
+    def forward(self, h, ctx, cache, rt, hold: bool = False):
         n = h.shape[0]
         k = rt.kernels
         # (keys and values of more than a few MB stream through L2 between this product and the output
@@ -131,21 +176,22 @@ class GqaAttention(Part):
                                            self.k_norm, self.eps, o, cache.k, cache.v, ctx.cu_q,
                                            ctx.kv_len, table, cache.page_size, self.nq, self.nkv,
                                            self.d, self.window, self.scale, splits, part_o, part_ml,
-                                           rt.err, rope=self.rope)
+                                           rt.err, rope=self.rope, sinks=self.sinks, gate_off=self.gate_off)
             rt.launches += 1 if splits <= 8 else 2     # the merge is a launch of its own above 8 slices
-            return rt.linear(o, self.o_w, self.o_b, "attn_out")
+            return rt.linear(o, self.o_w, self.o_b, "attn_out", hold=hold)
         q = rt.ws.get("attn_q", n, self.nq * self.d, rt.dtype)
         k.rope_norm_cache(qkv, self.qkv_cols, rt.dtype, ctx.positions, ctx.tok_entry, table, cos,
                           sin, self.q_norm, self.k_norm, self.eps, q, cache.k, cache.v,
                           cache.page_size, self.nq, self.nkv, self.d, self.own_kv,
                           self.position is not None, rt.err, rope=self.rope)
+        gate = None if self.gate_off < 0 else (qkv, self.qkv_cols, self.gate_off)
         use_mma = not rt.exact and k.prefill_attention_supports(self.d, self.nq, self.nkv)
         # Whole prompts of at most 64 tokens take the warp-level kernel (64-row tiles, several CTAs per
         # SM) also at head size 128.  Measured at 16 / 4 heads, tcgen05 against warp-level: 256 prompts of
         # 8 tokens 244 / 144 us, 64 of 32: 44 / 28 us, 32 of 64: 22 / 19 us; 21 of 96: 22 / 23 us, 16 of 128:
         # 16 / 21 us; 16 portions of 32 behind 2,000 cached keys 50 / 94 us.
         short = bool(getattr(ctx, "short_prompts", False)) and use_mma
-        use_tc = (not rt.exact and rt.use_tc_attention and not short
+        use_tc = (not rt.exact and rt.use_tc_attention and not short and self.sinks is None and gate is None
                   and k.prefill_attention_tc_supports(self.d, self.nq, self.nkv, cache.page_size))
         # Decoded tokens beside prompt portions: the entries of one token go to the split-KV decode
         # kernel (which skips the others), the prompt portions to the prefill kernel (which skips them).
@@ -165,10 +211,10 @@ class GqaAttention(Part):
                 part_ml = rt.ws.get("attn_part_ml", rows, 2, torch.float32, cap=rows)
             k.paged_decode_attention(q, o, cache.k, cache.v, ctx.cu_q, ctx.kv_len, table,
                                      cache.page_size, self.nq, self.nkv, self.d, self.window,
-                                     self.scale, splits, part_o, part_ml, rt.err)
+                                     self.scale, splits, part_o, part_ml, rt.err, sinks=self.sinks, gate=gate)
             rt.launches += 3 if splits > 1 else 2
             if decode:
-                return rt.linear(o, self.o_w, self.o_b, "attn_out")
+                return rt.linear(o, self.o_w, self.o_b, "attn_out", hold=hold)
             rt.launches -= 1                      # the rotary kernel is counted once, below
         if use_tc:
             tiles = query_tiles(ctx, 128, skip_single=bool(singles))
@@ -180,14 +226,17 @@ class GqaAttention(Part):
             tiles = query_tiles(ctx, 64, skip_single=bool(singles))
             k.paged_prefill_attention(q, o, cache.k, cache.v, ctx.cu_q, ctx.kv_len, table,
                                       cache.page_size, tiles, self.nq, self.nkv, self.d, self.window,
-                                      self.scale, rt.err, skip_single=bool(singles))
+                                      self.scale, rt.err, skip_single=bool(singles), sinks=self.sinks, gate=gate)
             rt.launches += 2
         else:
             k.paged_attention_simt(q, o, cache.k, cache.v, ctx.positions, ctx.tok_entry, table,
                                    cache.page_size, self.nq, self.nkv, self.d, self.window,
-                                   self.scale, rt.err)
+                                   self.scale, rt.err, sinks=self.sinks)
             rt.launches += 2
-        return rt.linear(o, self.o_w, self.o_b, "attn_out")
+            if gate is not None:
+                k.gate_mul(o, qkv, self.qkv_cols, self.gate_off)
+                rt.launches += 1
+        return rt.linear(o, self.o_w, self.o_b, "attn_out", hold=hold)
 
 
 @register_part("mixer", "sink_attention")

@@ -5,6 +5,8 @@
 fused into the norm that follows it, so a block hands its last output on
 unadded ("pending") and receives the one of the block before it.
 
+Its ``ffn`` (and ``norm2``) may be absent.
+
 ``sandwich_residual``: every sublayer's result is normed before it is added,
 x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))); then an optional per-layer
 token input joins the stream.
@@ -36,20 +38,22 @@ from .norm import BranchSum, StreamUpdate, add_normed, combine_and_norm
 
 @register_block("prenorm_residual")
 class PreNormResidualBlock:
-    """parts: ``norm1``, ``mixer``, ``norm2``, ``ffn``."""
+    """parts: ``norm1``, ``mixer`` and, unless the layer has no feed-forward, ``norm2``, ``ffn``."""
 
     def __init__(self, layer_spec):
-        self.norm1 = build_part(layer_spec.parts["norm1"])
-        self.mixer = build_part(layer_spec.parts["mixer"])
-        self.norm2 = build_part(layer_spec.parts["norm2"])
-        self.ffn = build_part(layer_spec.parts["ffn"])
+        p = layer_spec.parts
+        self.norm1, self.mixer = build_part(p["norm1"]), build_part(p["mixer"])
+        self.ffn = build_part(p["ffn"]) if "ffn" in p else None
+        self.norm2 = build_part(p["norm2"]) if self.ffn is not None else None
 
     def parts(self):
-        return [self.norm1, self.mixer, self.norm2, self.ffn]
+        return [q for q in (self.norm1, self.mixer, self.norm2, self.ffn) if q is not None]
 
     def forward(self, x, pending, ctx, cache, rt):
         h = self.norm1.forward(x, pending, rt)
         a = self.mixer.forward(h, ctx, cache, rt)
+        if self.ffn is None:
+            return a
         h = self.norm2.forward(x, a, rt)
         return self.ffn.forward(h, ctx, rt)
 
@@ -152,6 +156,32 @@ class PassEntry(Part):
         kept = rt.ws.get("embedding_output", x.shape[0], self.size, torch.float32) if add_embedding else None
         rt.kernels.stream_enter(x, kept, self.rows[row])
         rt.launches += 1
+        return None
+
+
+@register_part("entry", "pass_projection")
+class PassProjection(Part):
+    """Where a pass over repeated layers begins, the stream x becomes W [x; x0], x0 the embedding output that the
+    embedding part kept (workspace buffer "embedding_output").  What the block before left pending joins x on the
+    way.  params: ``size``, ``tensor`` (name).  Tensor W [size, 2 size], the stream's columns first.  The product's
+    result is the stream, so it stays float."""
+    kind = "entry"
+
+    @classmethod
+    def manifest(cls, spec):
+        a = spec.params
+        return {spec.prefix + a["tensor"]: TensorSpec((int(a["size"]), 2 * int(a["size"])))}
+
+    def load(self, weights, rt):
+        self.w, self.size = weights[self.prefix + self.params["tensor"]], int(self.params["size"])
+
+    def forward(self, x, pending, ctx, rt):
+        n = x.shape[0]
+        kept = rt.ws.get("embedding_output", n, self.size, torch.float32)
+        both = rt.ws.get("pass_input", n, 2 * self.size, rt.dtype)
+        rt.kernels.stream_beside(x, pending, kept, both)
+        rt.launches += 1
+        rt.linear(both, self.w, None, "pass_input_product", out=x)
         return None
 
 

@@ -16,9 +16,12 @@ from .base import Part, register_part
 @register_part("embed", "token_embedding")
 class TokenEmbedding(Part):
     """params: ``vocab_size``, ``hidden_size``, ``table`` (tensor name behind the prefix; default
-    "weight"), ``model_copy`` (a workspace buffer that also gets the rows, in the model type: for blocks whose
-    sublayers read the stream itself).  Tensor [V,H]."""
+    "weight"), ``scale`` (a constant that multiplies the rows), ``model_copy`` (a workspace buffer that also gets
+    the rows, in the model type: for blocks whose sublayers read the stream itself), ``keep_copy`` (the rows are also
+    written to the workspace buffer "embedding_output", in float, for a model that reads the embedding output again
+    later).  Tensor [V,H]."""
     kind = "embed"
+    KEPT = "embedding_output"
 
     @classmethod
     def manifest(cls, spec):
@@ -27,6 +30,8 @@ class TokenEmbedding(Part):
 
     def load(self, weights, rt):
         self.table = weights[self.prefix + (self.params.get("table") or "weight")]
+        scale = self.params.get("scale")
+        self.scale = 1.0 if scale is None else float(scale)
 
     def forward(self, tokens, x, rt, deferred=None):
         """Writes the float residual rows ``x`` [N,H] for int32 ``tokens`` [N].
@@ -34,7 +39,8 @@ class TokenEmbedding(Part):
         device): a token sampled by an earlier launch that the host has not read."""
         copy = self.params.get("model_copy")
         raw = rt.ws.get(copy, x.shape[0], x.shape[1], rt.dtype) if copy else None
-        rt.kernels.embed_gather(tokens, self.table, x, rt.err, deferred, raw)
+        keep = rt.ws.get(self.KEPT, x.shape[0], x.shape[1], torch.float32) if self.params.get("keep_copy") else None
+        rt.kernels.embed_gather(tokens, self.table, x, rt.err, deferred, raw, self.scale, keep)
         rt.launches += 1
 
 

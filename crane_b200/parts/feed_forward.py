@@ -147,11 +147,14 @@ class ActMlp(Part):
 class RoutedExperts(Part):
     """A mixture of small feed-forwards down_e(act(up_e(h))): the router's logits z = W_r h are
     formed in 32-bit, the ``top`` largest choose a token's experts (ties to the lower index), and
-    their weights are the softmax over the chosen logits alone.  An optional shared expert of the
+    their weights are the softmax over the chosen logits alone.  With ``scores`` "sigmoid" the
+    choice goes by s = sigmoid(z), plus a learnt correction if there is one, and the weights are the
+    chosen experts' s over their sum (+ 1e-20), times ``route_scale``.  An optional shared expert of the
     same form runs for every token and is added.
     params: ``hidden_size``, ``experts``, ``top``, ``expert_size``, ``shared_size`` (0: none), ``act``,
-    ``names`` (router, expert: a pattern with {e}, shared, up, down).
-    Tensors: router [E,H]; per expert up [F,H], down [H,F]; shared up [Fs,H], down [H,Fs].
+    ``scores`` ("softmax", the default, or "sigmoid"), ``correction`` (tensor name or None), ``route_scale``
+    (default 1), ``names`` (router, expert: a pattern with {e}, shared, up, down).
+    Tensors: router [E,H]; correction [E] (float); per expert up [F,H], down [H,F]; shared up [Fs,H], down [H,Fs].
 
     All experts' up matrices (and the shared one's) are one matrix, and so are the down matrices:
     a step is two products with the activation between them, which multiplies every expert's
@@ -166,6 +169,8 @@ class RoutedExperts(Part):
         nm = dict(cls.NAMES, **(a.get("names") or {}))
         h, E, F, Fs = int(a["hidden_size"]), int(a["experts"]), int(a["expert_size"]), int(a.get("shared_size") or 0)
         m = {p + nm["router"]: TensorSpec((E, h))}
+        if a.get("correction"):
+            m[p + a["correction"]] = TensorSpec((E,), "float32", "offset")
         for e in range(E):
             q = p + nm["expert"].format(e=e)
             m[q + nm["up"]] = TensorSpec((F, h))
@@ -184,6 +189,12 @@ class RoutedExperts(Part):
             raise ValueError(f"{p}: {self.top} of {self.E} experts cannot be chosen")
         if self.act not in rt.kernels.ACTIVATIONS:
             raise ValueError(f"{p}: no activation '{self.act}'; there are: {', '.join(rt.kernels.ACTIVATIONS)}")
+        scores = str(a.get("scores") or "softmax")
+        self.sigmoid = scores == "sigmoid"
+        self.route_scale = 1.0 if a.get("route_scale") is None else float(a["route_scale"])
+        self.correction = weights[p + a["correction"]] if a.get("correction") else None
+        if scores not in ("softmax", "sigmoid") or not self.sigmoid and (self.correction is not None or self.route_scale != 1.0):
+            raise ValueError(f"{p}: scores are 'softmax', or 'sigmoid' with or without a correction and a scale")
         self.router = weights[p + nm["router"]]
         ups = [weights.pop(p + nm["expert"].format(e=e) + nm["up"]) for e in range(self.E)]
         downs = [weights.pop(p + nm["expert"].format(e=e) + nm["down"]) for e in range(self.E)]
@@ -197,11 +208,15 @@ class RoutedExperts(Part):
     def forward(self, h, ctx, rt):
         n = h.shape[0]
         k = rt.kernels
-        logits = rt.linear(h, self.router, None, "router_logits", out_dtype=torch.float32)
+        logits = rt.linear(h, self.router, None, "router_logits", out_dtype=torch.float32, keep_parts=self.sigmoid)
         route = rt.ws.get("route_weights", n, self.E, torch.float32)
-        idx = rt.ws.get("route_idx", n, self.top, torch.int32)
-        wt = rt.ws.get("route_wt", n, self.top, torch.float32)
-        k.route_topk(logits, route, idx, wt)
+        if self.sigmoid:
+            k.route_grouped(logits, self.correction, route, self.E, self.top, 1, 1, False, sigmoid=True, renorm=True,
+                            scale=self.route_scale)
+        else:
+            idx = rt.ws.get("route_idx", n, self.top, torch.int32)
+            wt = rt.ws.get("route_wt", n, self.top, torch.float32)
+            k.route_topk(logits, route, idx, wt)
         up = rt.linear(h, self.up, None, "experts_up")
         act = rt.ws.get("experts_act", n, self.inter, rt.dtype)
         k.ffn_activation(up, act, self.act, route, self.F, self.E * self.F)

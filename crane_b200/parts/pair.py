@@ -36,6 +36,11 @@ class ParallelPair(Part):
         keeps = [m for m in (self.left, self.right) if any(f.kind == "state" for f in m.cache_need().flat())]
         return all(getattr(m, "state_graph_safe", False) for m in keeps)
 
+    @property
+    def decode_bucket_safe(self):
+        keeps = [m for m in (self.left, self.right) if any(f.kind == "state" for f in m.cache_need().flat())]
+        return all(getattr(m, "decode_bucket_safe", False) for m in keeps)
+
     def load(self, weights, rt):
         a, p = self.params, self.prefix
         self.left.load(weights, rt)

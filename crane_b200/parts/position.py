@@ -98,3 +98,39 @@ class YarnRope(Part):
                 cos, sin = np.ones((n, 1), np.float32), np.zeros((n, 1), np.float32)
             _TABLES[key] = (torch.from_numpy(cos).to(rt.device), torch.from_numpy(sin).to(rt.device))
         return _TABLES[key]
+
+
+@register_part("position", "wavelength_rope")
+class WavelengthRope(Part):
+    """Rotary angles a = p * f_i over ``dims`` rotated elements, f_i = base^(-2i/dims), scaled by wavelength
+    l = 2 pi / f_i as Llama 3.1 does (``scaling``: factor, low, high, original; or None): f_i stays where
+    l < original / high, becomes f_i / factor where l > original / low, and in between
+    (1 - s) f_i / factor + s f_i with s = (original / l - low) / (high - low).
+    params: ``dims``, ``base``, ``scaling``, ``max_positions``.  No tensors.  ``tables(rt, limit)`` gives (cos, sin)
+    [positions < limit, dims / 2] in float; the angles are formed in 64-bit on the host and rounded once."""
+    kind = "position"
+
+    def width(self) -> int:
+        return int(self.params["dims"])
+
+    def frequencies(self):
+        dims, base = self.width(), float(self.params["base"])
+        f = base ** (-2.0 * np.arange(dims // 2, dtype=np.float64) / dims)
+        sc = self.params.get("scaling")
+        if not sc:
+            return f
+        factor, low, high, original = (float(sc[k]) for k in ("factor", "low", "high", "original"))
+        wavelength = 2.0 * np.pi / f
+        s = (original / wavelength - low) / (high - low) if high != low else np.zeros_like(f)
+        between = (1.0 - s) * f / factor + s * f
+        return np.where(wavelength < original / high, f, np.where(wavelength > original / low, f / factor, between))
+
+    def tables(self, rt, limit: int):
+        n = min(int(self.params["max_positions"]), int(limit))
+        sc = self.params.get("scaling") or {}
+        key = ("wavelength", self.width(), float(self.params["base"]),
+               tuple(sorted((k, float(v)) for k, v in sc.items())), n, str(rt.device))
+        if key not in _TABLES:
+            angles = np.arange(n, dtype=np.float64)[:, None] * self.frequencies()[None, :]
+            _TABLES[key] = tuple(torch.from_numpy(t.astype(np.float32)).to(rt.device) for t in (np.cos(angles), np.sin(angles)))
+        return _TABLES[key]

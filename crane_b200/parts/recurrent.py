@@ -21,6 +21,12 @@ token itself, its write scaled per key channel by u:
 
     o_t = (S + diag(u) k_t v_t^T)^T r_t;   S <- diag(w_t) S + k_t v_t^T
 
+``exponential_gates`` (the matrix memory of xLSTM): no correction, gates i and exp(f) per head whose
+logarithms are capped, f = log sigmoid(.), kept in range by a running maximum M, which starts at 0:
+
+    M' = max(f + M, i);  S <- exp(f + M - M') S + exp(i - M') k v^T;  N likewise with k alone
+    o = S^T q / (max(|N . q|, exp(-M')) + eps)
+
 State and everything between the projections and the output projection are 32-bit.  One kernel walks
 the recurrence for all of them (``matrix_state_scan``), prompts, portions and single tokens alike, so a
 state does not depend on how the tokens were cut.
@@ -37,6 +43,7 @@ from .base import CacheNeed, Part, register_part
 
 
 def _state_floats(rt, heads: int, dim: int, vdim: int, where: str) -> int:
+    """Floats of a slot's states of ``heads`` heads with ``vdim`` columns each."""
     rows, lanes = rt.kernels.matrix_state_plan(dim)
     if rows == 0:
         raise ValueError(f"{where}: keys of {dim} elements are wider than the recurrence kernel takes")
@@ -323,3 +330,67 @@ class WkvTimeMix(Part):
         k.head_norm_gate(o_raw, proj, self.cols, 3 * hd, ctx.tok_entry, self.norm_w, self.eps, o, H, d)
         rt.launches += 4
         return rt.linear(o, self.o_w, None, "time_mix_out")
+
+
+@register_part("mixer", "exponential_gates")
+class ExponentialGates(Part):
+    """params: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``gate_cap``, ``norm_eps`` (of the head norm), ``den_eps``
+    (what is added to the normaliser), ``names``.  Tensors: q, k [H dim, hidden], v, g [H vdim, hidden],
+    o [hidden, H vdim], i, f [H, hidden], and in 32-bit i_bias, f_bias [H], norm [H vdim].  The read-out is normed
+    per head, times ``norm``, times sigmoid(g).  The request's slot holds per head the state with the normaliser
+    as one more column, and behind the states the running maxima."""
+    kind = "mixer"
+    state_graph_safe = True
+    decode_bucket_safe = True
+    NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "i": "i", "f": "f", "i_bias": "i.b", "f_bias": "f.b",
+             "norm": "norm"}
+
+    @classmethod
+    def manifest(cls, spec):
+        a, p = spec.params, spec.prefix
+        w, H, d, m = (int(a[k]) for k in ("hidden_size", "heads", "dim", "vdim"))
+        nm = dict(cls.NAMES, **(a.get("names") or {}))
+        out = {p + nm["q"]: TensorSpec((H * d, w)), p + nm["k"]: TensorSpec((H * d, w)),
+               p + nm["v"]: TensorSpec((H * m, w)), p + nm["g"]: TensorSpec((H * m, w)),
+               p + nm["o"]: TensorSpec((w, H * m)), p + nm["norm"]: TensorSpec((H * m,), "float32", "scale")}
+        for gate in ("i", "f"):
+            out[p + nm[gate]] = TensorSpec((H, w))
+            out[p + nm[gate + "_bias"]] = TensorSpec((H,), "float32", "unit")
+        return out
+
+    def load(self, weights, rt):
+        a, p = self.params, self.prefix
+        self.H, self.d, self.m = (int(a[k]) for k in ("heads", "dim", "vdim"))
+        nm = dict(self.NAMES, **(a.get("names") or {}))
+        self.cap, self.eps, self.den_eps = float(a["gate_cap"]), float(a["norm_eps"]), float(a["den_eps"])
+        # one product for everything that reads the block's input: [q | k | v | g | i | f]
+        self.w_in = torch.cat([weights.pop(p + nm[n]) for n in ("q", "k", "v", "g", "i", "f")], dim=0).contiguous()
+        self.cols = self.w_in.shape[0]
+        self.bias_i, self.bias_f = weights[p + nm["i_bias"]], weights[p + nm["f_bias"]]
+        self.norm_w, self.o_w = weights[p + nm["norm"]], weights[p + nm["o"]]
+        # rows of the recurrence's inputs: [q | k | v | kept share | new share | floor]
+        self.w_at = 2 * self.H * self.d + self.H * self.m
+        self.aux_cols = -(-(self.w_at + 3 * self.H) // 4) * 4
+        self.max_off = _state_floats(rt, self.H, self.d, self.m + 1, p)
+        self.floats = self.max_off + self.H
+
+    def cache_need(self) -> CacheNeed:
+        return CacheNeed("state", state_shape=(self.floats,), state_dtype=torch.float32)
+
+    def forward(self, h, ctx, cache, rt, hold: bool = False):
+        n, k, H, d, m = h.shape[0], rt.kernels, self.H, self.d, self.m
+        hd, hv = H * d, H * m
+        proj = rt.linear(h, self.w_in, None, "exp_gates_proj")
+        aux = rt.ws.get("exp_gates_aux", n, self.aux_cols, torch.float32)
+        gates = 2 * hd + 2 * hv
+        k.exp_gate_prep(proj, self.cols, ctx, cache.state, self.max_off, self.bias_i, self.bias_f, self.cap, d ** -0.5,
+                        aux, H, d, m, gates, gates + H, self.w_at, rt.err, rt.dtype)
+        o_raw = rt.ws.get("exp_gates_o_raw", n, hv, torch.float32)
+        den = rt.ws.get("exp_gates_den", n, H, torch.float32)
+        k.matrix_state_scan(aux, (0, hd, 2 * hd, self.w_at, self.w_at + H), False, "gated", 1, ctx, cache.state, o_raw, H, d,
+                            m, rt.err, den=den)
+        o = rt.ws.get("exp_gates_o", n, hv, rt.dtype)
+        k.head_norm_gate(o_raw, proj, self.cols, 2 * hd + hv, ctx.tok_entry, self.norm_w, self.eps, o, H, m, sigmoid=True,
+                         den=den, floor=aux[:, self.w_at + 2 * H:], den_eps=self.den_eps)
+        rt.launches += 3
+        return rt.linear(o, self.o_w, None, "exp_gates_out", hold=hold)

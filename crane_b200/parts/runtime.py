@@ -97,7 +97,8 @@ class Runtime:
     # ---- matrix product -------------------------------------------------
     def linear(self, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], name: str,
                out_dtype: Optional[torch.dtype] = None, cap: Optional[int] = None,
-               hint_next: bool = True, hold: bool = False, keep_parts: bool = False) -> Act:
+               hint_next: bool = True, hold: bool = False, keep_parts: bool = False,
+               out: Optional[torch.Tensor] = None) -> Act:
         """x[M,K] @ w[N,K]^T (+ bias[N], float) -> [M,N] in ``out_dtype`` (the
         model dtype unless stated).  ``hint_next`` False: this product does not
         ask for the next product's weights (its caller streams so much between
@@ -105,11 +106,12 @@ class Runtime:
         only after other products have run (a branch of a parallel block): if it
         is left as partial sums, they get a buffer of this product's own name
         instead of the one that all products of its width share.  ``keep_parts``: a float
-        result may stay partial sums too (its reader adds them up)."""
+        result may stay partial sums too (its reader adds them up).  ``out``: a float tensor that gets the
+        result, instead of a buffer called ``name``."""
         M, K = x.shape
         N = w.shape[0]
-        out_dtype = out_dtype or self.dtype
-        out = self.ws.get(name, M, N, out_dtype, cap)
+        if out is None:
+            out = self.ws.get(name, M, N, out_dtype or self.dtype, cap)
         if self.exact:
             self.kernels.gemm_simt(x, w, bias, out)
             self.launches += 1

@@ -38,6 +38,7 @@ def model_folders(tmp_path_factory):
     import tiny_vodelix
     import tiny_zudarax
     import tiny_pogarax
+    import tiny_mufalix
     from crane_b200.weights.random_init import write_model_folder
     made = {}
 
@@ -46,7 +47,7 @@ def model_folders(tmp_path_factory):
         if key not in made:
             d = tmp_path_factory.mktemp(f"{name}_{dtype}")
             spec = next(t.TINY[name] for t in (tiny_configs, tiny_radorax, tiny_vodelix, tiny_mufevik, tiny_zudarax,
-                                                          tiny_pogarax) if name in t.TINY)
+                                                          tiny_pogarax, tiny_mufalix) if name in t.TINY)
             write_model_folder(str(d), spec["config"], spec["seed"], dtype, std=spec["std"],
                                norm_std=spec["norm_std"])
             made[key] = str(d)

@@ -260,7 +260,7 @@ def forward(cfg: dict, w: Dict[str, np.ndarray], tokens, state: Optional[list] =
     None: the start).  Returns (logits [n, V], the stream after every run [runs, n, W], state)."""
     eps = float(cfg["norm"]["eps"])
     runs = layer_runs(cfg)
-    x = w["embed"][np.asarray(tokens)] * float(cfg["embedding"]["scale"])
+    x = w["embed"][np.asarray(tokens)] * float((cfg.get("embedding") or {}).get("scale", 1.0))
     x0 = x.copy()
     state = [None] * len(runs) if state is None else list(state)
     streams = []

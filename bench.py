@@ -1460,6 +1460,234 @@ def pogarax_workload(args, pk):
     return out
 
 
+def mufalix_config(like, layers):
+    """A Mufalix model with the width, layer count and vocabulary of the Hunyuan configuration `like`: of every three
+    layers two are pairs (attention with the other's head counts, heads of 128, half of each rotated, a window of 1,024;
+    a gated linear recurrence over 5/4 of the width in 16 parts behind four taps) and one is a matrix memory (heads of
+    keys of 128 and values of 256 across the width); every layer has eight experts of a quarter of the other's inner
+    size of which two are chosen; layers 1 and 2 run twice."""
+    h, heads, kv = like["hidden_size"], like["num_attention_heads"], like["num_key_value_heads"]
+    left = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+            "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    right = {"width": h * 5 // 4, "blocks": 16, "conv": 4}
+    mlstm = {"heads": max(1, h // 256), "dim": 128, "vdim": 256, "gate_cap": 15.0}
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2, "scale": 1.5}, "expert": {"ff": like["intermediate_size"] // 4}}
+    ls = [{"type": "mlstm", "mixer": mlstm, "mlp": moe} if i % 3 == 1 else
+          {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe} for i in range(layers)]
+    cfg = {"architecture": "Mufalix", "vocab": like["vocab_size"], "width": h, "norm": {"eps": 1e-5},
+           "embedding": {"scale": 3.0}, "layers": ls}
+    if layers >= 3:
+        cfg["loop"] = {"start": 1, "stop": 3, "times": 2}
+    return cfg
+
+
+def mufalix_kernel_table(fcfg, pk, tokens, batch, context):
+    """Every kernel or option that only Mufalix runs beside the kernel of the engine's other models that does
+    the like job, each alone on synthetic operands of these layer sizes (L2 flushed between repetitions),
+    with the fraction of its roofline: algorithmic bytes over the measured copy rate, or FLOPs over the
+    measured bf16 rate, whichever takes longer."""
+    from types import SimpleNamespace
+    import numpy as np
+    import torch
+    from crane_b200.parts import Runtime
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    rt = Runtime(dev, bf, max(tokens, 256), head_sizes=(128,))
+    K = rt.kernels
+    flush = torch.zeros(128 << 20, dtype=f32, device=dev)
+    err = rt.err
+    W = fcfg["width"]
+    par = next(l["mixer"] for l in fcfg["layers"] if l["type"] == "parallel")
+    ml = next(l["mixer"] for l in fcfg["layers"] if l["type"] == "mlstm")
+    la, rr, moe = par["left"], par["right"], fcfg["layers"][0]["mlp"]
+    hbm, peak = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    rows = []
+
+    def add(name, like, ms, nbytes, flops, like_ms=0, like_bytes=0, like_flops=0):
+        def frac(ms_, b, f):
+            return round(max(b / hbm, f / peak) / (ms_ * 1e-3), 4)
+        rows.append({"kernel": name, "ms": round(ms, 4), "frac": frac(ms, nbytes, flops), "like": like,
+                     "like_ms": round(like_ms, 4) if like_ms else None,
+                     "like_frac": frac(like_ms, like_bytes, like_flops) if like_ms else None})
+
+    rnd = lambda *shape, dt=bf: torch.randn(*shape, device=dev, dtype=f32).to(dt)
+    t_of = lambda fn: _median_ms(fn, flush=flush)
+    ps = 64
+    E, top, F = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"]
+    for kind, n_req, q_len, kv in (("prefill", 1, tokens, tokens), ("decode", batch, 1, context)):
+        blocks = -(-kv // ps)
+        table = torch.arange(n_req * blocks, dtype=torch.int32, device=dev).view(n_req, blocks)
+        cu_d = torch.arange(n_req + 1, dtype=torch.int32, device=dev) * q_len
+        kv_d = torch.full((n_req,), kv, dtype=torch.int32, device=dev)
+        n = n_req * q_len
+        pos = torch.from_numpy(np.concatenate([np.arange(kv - q_len, kv, dtype=np.int32)] * n_req)).to(dev)
+        ent = torch.from_numpy(np.repeat(np.arange(n_req, dtype=np.int32), q_len)).to(dev)
+        slots = torch.arange(n_req, dtype=torch.int32, device=dev)
+        ctx = SimpleNamespace(tok_entry=ent, cu_q=cu_d, kv_len=kv_d, slots=slots, all_single=q_len == 1)
+        one = kind == "decode"
+        # ---- where a pass begins
+        x, y, x0, both = rnd(n, W, dt=f32), rnd(n, W), rnd(n, W, dt=f32), torch.empty(n, 2 * W, device=dev, dtype=bf)
+        vec, wp = rnd(W, dt=f32), rnd(W, 2 * W)
+        add(f"stream_beside ({kind})", "stream_enter (Vodelix)", t_of(lambda: K.stream_beside(x, y, x0, both)), n * W * 14, 0,
+            t_of(lambda: K.stream_enter(x, x0, vec)), n * W * 12, 0)
+        fl = 4 * n * W * W
+        add(f"pass product, float result ({kind})", "the same product, bfloat16 result",
+            t_of(lambda: rt.linear(both, wp, None, "b0", out=x)), 4 * W * W + n * W * 8, fl,
+            t_of(lambda: rt.linear(both, wp, None, "b1")), 4 * W * W + n * W * 6, fl)
+        # ---- router and activation
+        z, corr, route = rnd(n, E, dt=f32), rnd(E, dt=f32), torch.empty(n, E, device=dev)
+        t_p = t_of(lambda: K.route_grouped(z, corr, route, E, top, 1, 1, False, sigmoid=True, renorm=True, scale=1.5))
+        t_l = t_of(lambda: K.route_grouped(z, corr, route, E, top, 1, 1, False))
+        add(f"route_grouped, corrected sigmoid over the chosen sum ({kind})", "route_grouped, softmax (Mufevik)", t_p, n * E * 8, 0, t_l,
+            n * E * 8, 0)
+        up, act, gu = rnd(n, E * F), torch.empty(n, E * F, device=dev, dtype=bf), rnd(n, 2 * E * F)
+        K.route_grouped(z, corr, route, E, top, 1, 1, False, sigmoid=True, renorm=True, scale=1.5)
+        add(f"ffn_activation, squared relu of routed experts ({kind})", "gated_activation (Mufevik)",
+            t_of(lambda: K.ffn_activation(up, act, "relu2", route, F, E * F)), n * F * (top * 2 + E * 2), 0,
+            t_of(lambda: K.gated_activation(gu, act, route, E, F, E * F)), n * F * (top * 4 + E * 2), 0)
+        del up, act, gu, both, wp
+        # ---- attention
+        H, G, d, win, rd = la["heads"], la["kv_heads"], la["dim"], la["mask"]["size"], la["rot"]["dims"]
+        k_pool, v_pool = rnd(n_req * blocks, G, ps, d), rnd(n_req * blocks, G, ps, d)
+        qkv_cols = (H + 2 * G) * d
+        cols = qkv_cols + H * d
+        proj, plain = rnd(n, cols), rnd(n, qkv_cols)
+        q, o = torch.empty(n, H * d, device=dev, dtype=bf), torch.empty(n, H * d, device=dev, dtype=bf)
+        cos, cosf = torch.rand(kv, rd // 2, device=dev), torch.rand(kv, d // 2, device=dev)
+        qw, sinks = rnd(d, dt=f32), rnd(H, dt=f32)
+        rope = (rd, False, True, 0.0)
+        prep = lambda src, c, tab, r: K.rope_norm_cache(src, c, bf, pos, ent, table, tab, tab, qw, qw, 1e-5, q, k_pool, v_pool, ps, H, G, d,
+                                                        True, True, err, rope=r)
+        by = n * qkv_cols * 4
+        add(f"rope_norm_cache, norm before a partial rotation ({kind})", "rope_norm_cache (Hunyuan)", t_of(lambda: prep(proj, cols, cos, rope)),
+            by, 0, t_of(lambda: prep(plain, qkv_cols, cosf, None)), by, 0)
+        seen = lambda w_: sum(min(p + 1, w_ or p + 1) for p in range(kv - q_len, kv)) * n_req
+        read = lambda w_: n_req * min(kv, (w_ + q_len - 1) if w_ else kv) * G * d * 4 + n * H * d * 4
+        fl = lambda w_: 4 * seen(w_) * H * d
+        gb = n * H * d * 2
+        if not one:
+            tiles = -(-q_len // 64)
+            at = lambda w_, **kw: K.paged_prefill_attention(q, o, k_pool, v_pool, cu_d, kv_d, table, ps, tiles, H, G, d, w_, d ** -0.5, err, **kw)
+            own = dict(sinks=sinks, gate=(proj, cols, qkv_cols))
+            t_l = t_of(lambda: at(0, sink=True))
+            add(f"attention, window of {win}, sinks, gate ({kind})", "attention with a sink (Vodelix)", t_of(lambda: at(win, **own)), read(win) + gb,
+                fl(win), t_l, read(0), fl(0))
+            add(f"attention, sinks, gate, no window ({kind})", "attention with a sink (Vodelix)", t_of(lambda: at(0, **own)), read(0) + gb,
+                fl(0), t_l, read(0), fl(0))
+        else:
+            splits = K.decode_splits(n_req, G, rt.num_sms)
+            po, pml = torch.empty(n_req * H * splits * d, device=dev), torch.empty(n_req * H * splits * 2, device=dev)
+            at = lambda src, c, tab, w_, **kw: K.paged_decode_attention_fused(
+                src, c, True, tab, tab, qw, qw, 1e-5, o, k_pool, v_pool, cu_d, kv_d, table, ps, H, G, d, w_, d ** -0.5, splits, po, pml, err, **kw)
+            own = dict(rope=rope, sinks=sinks, gate_off=qkv_cols)
+            t_l = t_of(lambda: at(plain, qkv_cols, cosf, 0))
+            t_w = t_of(lambda: at(plain, qkv_cols, cosf, win))
+            add(f"fused attention, window of {win}, sinks, gate ({kind})", "fused attention with the same window (Hunyuan)",
+                t_of(lambda: at(proj, cols, cos, win, **own)), read(win) + gb, fl(win), t_w, read(win), fl(win))
+            add(f"fused attention, sinks, gate, no window ({kind})", "fused attention (Hunyuan)", t_of(lambda: at(proj, cols, cos, 0, **own)),
+                read(0) + gb, fl(0), t_l, read(0), fl(0))
+        del k_pool, v_pool, proj, plain, q, o
+        # ---- the linear recurrence
+        C, parts, taps = rr["width"], rr["blocks"], rr["conv"]
+        c = C // parts
+        state = torch.zeros(n_req, C * (1 + taps), device=dev)
+        proj, aux, out = rnd(n, 2 * C), torch.rand(n, 2 * C, device=dev), torch.empty(n, C, device=dev, dtype=bf)
+        gates, mma = K.pack_gates(rnd(parts, c, c), rnd(parts, c, c), False)
+        v = lambda: rnd(C, dt=f32)
+        scan = K.GateScan(y_off=0, x_off=C, s_off=0, ring_off=C, conv_w=rnd(taps, C, dt=f32), conv_b=v(), gates=gates, mma=mma, rb=v(), ib=v(),
+                          sp=v().abs(), parts=parts)
+        st = n_req * C * 8 * (2 if one else 0)
+        by, fl_g = n * C * (2 + (4 if one else 8)) + 4 * C * c + st, 4 * n * C * c
+        rank = 64
+        low, lw = rnd(n, rank), K.pack_low_rank(rnd(C, rank), False)[0]
+        lr = K.LowRank(lw, rank, 0, C, out=aux[:, :C], kind="exp_decay", bias=v(), mma=True)
+        t_l = t_of(lambda: K.low_rank_expand(low, rank, ent, n, bf, lr))
+        aux.uniform_(0.9, 1.0)
+        add(f"gate_scan_prep{', with the walk' if one else ''} ({kind})", "low_rank_expand, decay (Pogarax)",
+            t_of(lambda: K.gate_scan_prep(proj, 2 * C, ctx, state, scan, aux, out, err, bf)), by, fl_g, t_l,
+            n * rank * 2 + n * C * 4 + C * rank * 2, 2 * n * C * rank)
+        aux.uniform_(0.9, 1.0)
+        Hs, ds = W // 64, 64
+        rws, lanes = K.matrix_state_plan(ds)
+        st2 = torch.zeros(n_req, Hs * rws * lanes * ds, device=dev)
+        a2, o2 = torch.rand(n, 4 * Hs * ds, device=dev), torch.empty(n, Hs * ds, device=dev)
+        t_s = t_of(lambda: K.matrix_state_scan(a2, (0, Hs * ds, 2 * Hs * ds, 3 * Hs * ds, 0), True, "plain", 1, ctx, st2, o2, Hs, ds, ds, err))
+        b_s = n * 5 * Hs * ds * 4 + n_req * Hs * ds * ds * 8
+        if not one:
+            add(f"channel_scan ({kind})", "matrix_state_scan, decay per channel (Mufevik)",
+                t_of(lambda: K.channel_scan(aux, proj, 2 * C, ctx, state, scan, out, err)), n * C * (8 + 2 + 2), 0, t_s, b_s, 0)
+        del proj, aux, out, state, st2, a2, o2
+        # ---- the matrix memory
+        H, d, m = ml["heads"], ml["dim"], ml["vdim"]
+        hd, hv = H * d, H * m
+        cols, w_at = 2 * hd + 2 * hv + 2 * H, 2 * hd + hv
+        rws, lanes = K.matrix_state_plan(d)
+        m_off = H * rws * lanes * (m + 1)
+        state = torch.zeros(n_req, m_off + H, device=dev)
+        proj, aux = rnd(n, cols), torch.empty(n, -(-(w_at + 3 * H) // 4) * 4, device=dev)
+        bi = rnd(H, dt=f32)
+        t_p = t_of(lambda: K.exp_gate_prep(proj, cols, ctx, state, m_off, bi, bi, 15.0, d ** -0.5, aux, H, d, m, cols - 2 * H, cols - H, w_at,
+                                           err, bf))
+        ub, ba = rnd(H, d, dt=f32), torch.empty(n, w_at + 3 * H, device=dev)
+        t_l = t_of(lambda: K.bonus_prep(proj, cols, ent, ub, ba, w_at, H, d, m, bf))
+        add(f"exp_gate_prep ({kind})", "bonus_prep (Pogarax)", t_p, n * w_at * 6, 0, t_l, n * w_at * 6, 0)
+        o_raw, den = torch.empty(n, hv, device=dev), torch.empty(n, H, device=dev)
+        t_p = t_of(lambda: K.matrix_state_scan(aux, (0, hd, 2 * hd, w_at, w_at + H), False, "gated", 1, ctx, state, o_raw, H, d, m, err, den=den))
+        t_same = t_of(lambda: K.matrix_state_scan(aux, (0, hd, 2 * hd, w_at, w_at + H), False, "delta", 1, ctx, state, o_raw, H, d, m, err))
+        b_g = n * (w_at + hv) * 4 + n_req * H * d * m * 8
+        add(f"matrix_state_scan, gated with a normaliser ({kind})", "matrix_state_scan, delta rule (Mufevik's, at these sizes)", t_p, b_g, 0,
+            t_same, b_g, 0)
+        add(f"matrix_state_scan, gated with a normaliser ({kind})", "matrix_state_scan, decay per channel (Mufevik, heads of 64)", t_p, b_g, 0,
+            t_s, b_s, 0)
+        nw, o = rnd(hv, dt=f32), torch.empty(n, hv, device=dev, dtype=bf)
+        fin = lambda **kw: K.head_norm_gate(o_raw, proj, cols, 2 * hd + hv, ent, nw, 1e-5, o, H, m, sigmoid=True, **kw)
+        add(f"head_norm_gate behind a normaliser ({kind})", "head_norm_gate (Pogarax)",
+            t_of(lambda: fin(den=den, floor=aux[:, w_at + 2 * H:], den_eps=1e-6)), n * hv * 8, 0, t_of(fin), n * hv * 8, 0)
+        del proj, aux, state, o_raw
+    torch.cuda.synchronize()
+    assert int(err.item()) == 0
+    return rows
+
+
+def mufalix_workload(args, pk):
+    """Prefill and decode throughput of Mufalix at the layer sizes of --sizes beside Mufevik (the engine's closest
+    model: attention beside a linear recurrence, experts) with as many layers as Mufalix runs, at the same
+    width and vocabulary, random weights, and its kernels beside their likes."""
+    import gc
+    import torch
+    hcfg = dict(MODEL)
+    hcfg.update(OTHER_SIZES.get(args.sizes, {}))
+    layers = args.layers or 12
+    fcfg = mufalix_config(hcfg, layers)
+    loop = fcfg.get("loop")
+    runs = layers + ((loop["stop"] - loop["start"]) * (loop["times"] - 1) if loop else 0)
+    hcfg["num_hidden_layers"] = runs
+    page, pt = 64, args.prefill_tokens
+    out = {"workload": "mufalix", "sizes": args.sizes, "layers": layers, "layer_runs": runs, "batch": args.batch,
+           "context": args.context, "prefill_tokens": pt, "dtype": "bf16", "data": "synthetic", "models": {}}
+    for name, cfg in (("mufalix", fcfg), ("mufevik", mufevik_config(hcfg, runs))):
+        opts = dict(page_size=page, num_pages=(args.batch * (args.context + args.steps + args.warmup + 64) + pt) // page + 64,
+                    max_concurrent=max(64, args.batch), max_seq_len=max(args.context, pt) + 1024,
+                    max_batched_tokens=max(2048, pt), chunk_size=max(2048, pt))
+        model = build_model(cfg, opts)
+        pms = time_prefill(model, pt, cfg["vocab"], reps=3)
+        ids = fill_cache(model, args.batch, args.context)
+        with ClockSampler() as clk:
+            dms, launches = time_decode(model, ids, args.steps, args.warmup, cfg["vocab"])
+        weights = sum(t.numel() * t.element_size() for t in _model_tensors(model))
+        out["models"][name] = {"prefill_ms": round(pms, 3), "prefill_tokens_per_s": round(pt * 1000.0 / pms, 1),
+                               "decode_ms_per_step": round(dms, 4),
+                               "decode_tokens_per_s": round(args.batch * 1000.0 / dms, 1),
+                               "launches_per_decode_step": launches, "weight_bytes": weights,
+                               "layer_runs": len(model.runner.spec.schedule), "clocks": clk.summary()}
+        del model
+        gc.collect()
+        torch.cuda.empty_cache()
+    if not args.no_points:
+        out["kernels"] = mufalix_kernel_table(fcfg, pk, pt, args.batch, args.context)
+    out["peaks"] = pk
+    return out
+
+
 def _model_tensors(model):
     seen, out = set(), []
     parts = [model.runner.model.embed, model.runner.model.final_norm, model.runner.model.head]
@@ -1499,7 +1727,7 @@ def main():
                     help="layer sizes: Hunyuan 1.8B (the default, the headline configuration), 4B or 7B")
     ap.add_argument("--prefill-chunk", type=int, default=0,
                     help="with --only-prefill: also time the prompt in portions of this many tokens, a step each")
-    ap.add_argument("--workload", default="", choices=["", "serve", "mixed-step", "radorax", "vodelix", "mufevik", "zudarax", "pogarax"],
+    ap.add_argument("--workload", default="", choices=["", "serve", "mixed-step", "radorax", "vodelix", "mufevik", "zudarax", "pogarax", "mufalix"],
                     help="serve: a mix of requests through the scheduler; mixed-step: decoded tokens beside "
                          "one prompt portion in one step; radorax: prefill and decode of Radorax beside Hunyuan "
                          "Dense at equal layer sizes, and their kernels side by side; vodelix: the same for Vodelix; "
@@ -1523,6 +1751,9 @@ def main():
         return 2
     args.warmup = max(args.warmup, 3)
 
+    if args.workload == "mufalix":
+        print(json.dumps(mufalix_workload(args, peaks())))
+        return 0
     if args.workload == "pogarax":
         print(json.dumps(pogarax_workload(args, peaks())))
         return 0

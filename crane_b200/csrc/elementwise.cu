@@ -444,6 +444,92 @@ __global__ void rope_norm_cache_kernel(GemmOut<T> qkv, int qkv_stride,
     }
 }
 
+// Whole bf16 rows with the norm before a rotation of contiguous halves (or without a norm or a rotation): a lane per 8
+// neighbours of a head, so 16-byte loads and stores, LANES lanes a head (d <= 8 LANES).  What a rotated element is
+// paired with lies rotary_dim / 2 further on or before, in another lane's 8 (rotary_dim a multiple of 16), and comes by
+// shuffle.
+template <int LANES>
+__global__ void __launch_bounds__(256)
+norm_rope_cache_vec_kernel(const __nv_bfloat16* __restrict__ qkv, int qkv_stride, const int* __restrict__ positions,
+                           const int* __restrict__ tok_entry, const int* __restrict__ block_table, int max_blocks,
+                           const float* __restrict__ cos_tab, const float* __restrict__ sin_tab, int table_len,
+                           const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float eps,
+                           __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_pool,
+                           __nv_bfloat16* __restrict__ v_pool, int num_pages, int page_size, int n_tokens, int nq, int nkv,
+                           int d, int has_kv, int rotary, int rotary_dim, float norm_offset, int* err) {
+    pdl_launch_dependents();
+    const int heads = nq + (has_kv ? 2 * nkv : 0);
+    const int unit = (blockIdx.x * blockDim.x + threadIdx.x) / LANES, sub = threadIdx.x % LANES;
+    const bool in = unit < n_tokens * heads;
+    const int t = in ? unit / heads : 0, h = in ? unit % heads : 0;
+    const int pos = positions[t];
+    __nv_bfloat16* dst = in ? q_out + ((long long)t * nq + h) * d : nullptr;
+    const float* nw = q_norm_w;
+    bool turn = rotary != 0;
+    if (in && h >= nq) {
+        const int e = tok_entry[t];
+        const int page = e >= 0 ? block_table[(long long)e * max_blocks + pos / page_size] : -1;
+        const bool is_v = h >= nq + nkv;
+        const int g = is_v ? h - nq - nkv : h - nq;
+        dst = nullptr;
+        if (e >= 0 && (page < 0 || page >= num_pages)) { if (sub == 0) atomicOr(err, CRANE_ERR_PAGE_RANGE); }
+        else if (e >= 0) dst = (is_v ? v_pool : k_pool) + (((long long)page * nkv + g) * page_size + pos % page_size) * d;
+        nw = is_v ? nullptr : k_norm_w;
+        turn = turn && !is_v;
+    }
+    if (turn && (pos < 0 || pos >= table_len)) {
+        if (sub == 0) atomicOr(err, CRANE_ERR_POSITION_RANGE);
+        turn = false;
+    }
+    const bool have = in && 8 * sub < d;
+    const int half = rotary_dim >> 1, hl = half >> 3;           // half the rotated width, in elements and in lanes
+    const bool low = sub < hl, turned = turn && have && sub < 2 * hl;
+    float wv[8], c[8], sn[8];
+    if (have && nw != nullptr) {
+        const float4 w0 = *(const float4*)(nw + 8 * sub), w1 = *(const float4*)(nw + 8 * sub + 4);
+        wv[0] = w0.x, wv[1] = w0.y, wv[2] = w0.z, wv[3] = w0.w, wv[4] = w1.x, wv[5] = w1.y, wv[6] = w1.z, wv[7] = w1.w;
+    }
+    if (turned) {
+        const long long at = (long long)pos * half + 8 * (low ? sub : sub - hl);
+        const float4 c0 = *(const float4*)(cos_tab + at), c1 = *(const float4*)(cos_tab + at + 4);
+        const float4 s0 = *(const float4*)(sin_tab + at), s1 = *(const float4*)(sin_tab + at + 4);
+        c[0] = c0.x, c[1] = c0.y, c[2] = c0.z, c[3] = c0.w, c[4] = c1.x, c[5] = c1.y, c[6] = c1.z, c[7] = c1.w;
+        sn[0] = s0.x, sn[1] = s0.y, sn[2] = s0.z, sn[3] = s0.w, sn[4] = s1.x, sn[5] = s1.y, sn[6] = s1.z, sn[7] = s1.w;
+    }
+    pdl_wait();
+    float v[8];
+    uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+    if (have) raw = *(const uint4*)(qkv + (long long)t * qkv_stride + (long long)h * d + 8 * sub);
+    const __nv_bfloat162* r2 = (const __nv_bfloat162*)&raw;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(r2[i]);
+        v[2 * i] = f.x, v[2 * i + 1] = f.y;
+        ss += f.x * f.x + f.y * f.y;
+    }
+#pragma unroll
+    for (int o = LANES >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (nw != nullptr && have) {
+        const float rstd = rsqrtf(ss / (float)d + eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] *= rstd * (norm_offset + wv[i]);
+    }
+    const int lane = threadIdx.x & 31, from = rotary == 0 || sub >= 2 * hl ? lane : low ? lane + hl : lane - hl;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {                                // every lane takes part, whatever its head is
+        const float o = __shfl_sync(0xffffffffu, v[i], from);
+        if (turned) v[i] = low ? v[i] * c[i] - o * sn[i] : v[i] * c[i] + o * sn[i];
+    }
+    if (have && dst != nullptr) {
+        uint4 res;
+        __nv_bfloat162* o2 = (__nv_bfloat162*)&res;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o2[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        *(uint4*)(dst + 8 * sub) = res;
+    }
+}
+
 // The same for whole bf16 rows of head size 128, eight lanes per (token, head): a
 // lane owns eight neighbours of the first half and their partners in the second
 // half (16-byte loads and stores), four heads per warp.
@@ -757,6 +843,18 @@ CRANE_API int crane_rope_norm_cache(int dtype, const void* qkv, const float* qkv
                             max_blocks, cos_tab, sin_tab, table_len, q_norm_w, k_norm_w, eps,
                             (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, num_pages,
                             page_size, n_tokens, nq, nkv, has_kv, rotary, err);
+    }
+    if (general && dtype == 1 && qkv != nullptr && !rp.interleaved && (norm_first || (q_norm_w == nullptr && k_norm_w == nullptr)) &&
+        d % 8 == 0 && d <= 256 && (!rotary || rotary_dim % 16 == 0) && qkv_stride % 8 == 0 && n_tokens >= 32 &&
+        ((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)cos_tab | (uintptr_t)sin_tab |
+         (uintptr_t)q_norm_w | (uintptr_t)k_norm_w) % 16 == 0) {
+        const int lanes = d <= 64 ? 8 : d <= 128 ? 16 : 32;
+        const auto kern = d <= 64 ? norm_rope_cache_vec_kernel<8> : d <= 128 ? norm_rope_cache_vec_kernel<16>
+                                                                             : norm_rope_cache_vec_kernel<32>;
+        return crane_launch(kern, dim3((unsigned)((warps * lanes + 255) / 256)), dim3(256), 0, st, (const __nv_bfloat16*)qkv,
+                            qkv_stride, positions, tok_entry, block_table, max_blocks, cos_tab, sin_tab, table_len, q_norm_w,
+                            k_norm_w, eps, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, num_pages,
+                            page_size, n_tokens, nq, nkv, d, has_kv, rotary, rotary_dim, norm_offset, err);
     }
     DISPATCH_T(dtype, {
         GemmOut<T> src{(const T*)qkv, qkv_parts, n_parts, part_stride};

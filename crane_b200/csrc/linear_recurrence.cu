@@ -81,13 +81,20 @@ __device__ __forceinline__ float conv_at(const GateScanArgs<T>& g, const TileTok
     return acc;
 }
 
-// Token t, channel c: from the two products' sums to what the walk needs, or, SINGLE, through the walk.
+// Channel c: from the two products' sums to the decay and the addend.
+template <typename T>
+__device__ __forceinline__ void gate_scan_terms(const GateScanArgs<T>& g, int c, float zr, float zi, float u, float& a, float& add) {
+    const float r = lin_sigmoid(zr + g.rb[c]), i = lin_sigmoid(zi + g.ib[c]);
+    const float log_a = -LIN_RATE * r * g.sp[c];
+    a = expf(log_a);
+    add = sqrtf(-expm1f(2.f * log_a)) * i * u;
+}
+// Token t, channel c: to what the walk needs, or, SINGLE, through the walk.
 template <typename T, bool SINGLE>
 __device__ __forceinline__ void gate_scan_finish(const GateScanArgs<T>& g, const TileToken& k, int t, int c, float zr,
                                                  float zi, float u) {
-    const float r = lin_sigmoid(zr + g.rb[c]), i = lin_sigmoid(zi + g.ib[c]);
-    const float log_a = -LIN_RATE * r * g.sp[c];
-    const float a = expf(log_a), add = sqrtf(-expm1f(2.f * log_a)) * i * u;
+    float a, add;
+    gate_scan_terms(g, c, zr, zi, u, a, add);
     if (!SINGLE) {
         float* o = g.aux + (long long)t * 2 * g.C;
         o[c] = a;
@@ -154,203 +161,335 @@ __device__ __forceinline__ void lin_mma(float (&acc)[4], const uint32_t (&a)[4],
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// TOKENS x COLS of one part by TOKENS / 16 x (COLS / 16 / KSPLIT...) warps: WM x WN x WK warps, a warp 16 tokens and
-// COLS / WN columns (of both products) over every WK-th step of 16 along the inner dimension; with WK = 2 the second
-// half's sums go through shared memory.  Grid (token tiles, parts, column blocks of a part).
-// Shared memory: u's two parts [2][TOKENS][ld + 8], both matrices' rows [2][COLS][ld + 8], bfloat16.
-template <int TOKENS, int COLS, int WN, int WK, bool SINGLE>
-__global__ void __launch_bounds__(TOKENS / 16 * WN * WK * 32)
-gate_scan_prep_mma_kernel(const GateScanArgs<__nv_bfloat16> g) {
-    constexpr int WM = TOKENS / 16, NT = WM * WN * WK * 32;
-    constexpr int NB = COLS / WN / 8;                       // blocks of 8 columns a warp takes
-    static_assert(NB == 1 || NB % 2 == 0, "one block of 8 columns, or pairs of them");
-    extern __shared__ __align__(16) unsigned char lin_smem[];
-    __shared__ TileToken tok[TOKENS];
-    const int ldm = g.ld + 8;
-    __nv_bfloat16* u_hi = reinterpret_cast<__nv_bfloat16*>(lin_smem);
-    __nv_bfloat16* u_lo = u_hi + TOKENS * ldm;
-    __nv_bfloat16* w_s = u_lo + TOKENS * ldm;
-    const int t0 = blockIdx.x * TOKENS, part = blockIdx.y, c0 = blockIdx.z * COLS;
-    const int width = g.width, base_c = part * width;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = lane >> 2, t4 = lane & 3;
-    pdl_launch_dependents();
-    // the weights depend on no earlier kernel
-    const int pieces = g.ld >> 3;
-    for (int x = threadIdx.x; x < 2 * COLS * pieces; x += NT) {
-        const int r = x / pieces, q = x % pieces, m = r / COLS, c = c0 + r % COLS;
+// u of two neighbouring channels c, c + 1 at token t, everything it reads in flight at once (rows of even length; up to 4
+// taps, else one channel after the other).
+__device__ __forceinline__ float2 conv_at2(const GateScanArgs<__nv_bfloat16>& g, const TileToken& k, int t, int c) {
+    if (g.taps > 4) return make_float2(conv_at(g, k, t, c), conv_at(g, k, t, c + 1));
+    float2 x[4], w[4];
+    const float2 bias = ld2(g.conv_b + c);
+    const float* ring = g.state + (long long)k.slot * g.slot_stride + g.ring_off + c;
+#pragma unroll
+    for (int back = 0; back < 4; ++back) {
+        x[back] = w[back] = make_float2(0.f, 0.f);
+        if (back >= g.taps) continue;
+        w[back] = ld2(g.conv_w + (long long)(g.taps - 1 - back) * g.C + c);
+        const int p = k.start + k.place - back;
+        if (k.place >= back) x[back] = g.proj.load2((long long)(t - back) * g.cols + g.x_off + c);
+        else if (p >= 0) x[back] = ld2(ring + (long long)(p % g.taps) * g.C);
+    }
+    float2 u = bias;
+#pragma unroll
+    for (int back = 3; back >= 0; --back) {
+        u.x = fmaf(w[back].x, x[back].x, u.x);
+        u.y = fmaf(w[back].y, x[back].y, u.y);
+    }
+    return u;
+}
+// u as its rounding and what that leaves.
+__device__ __forceinline__ void split_store(__nv_bfloat16* hi, __nv_bfloat16* lo, float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    const float2 f = __bfloat1622float2(h);
+    *(__nv_bfloat162*)hi = h;
+    *(__nv_bfloat162*)lo = __floats2bfloat162_rn(a - f.x, b - f.y);
+}
+// The weights of `cols` columns from c0 on of both matrices: w_s [2][cols][ld + 8].
+__device__ __forceinline__ void load_gates(const GateScanArgs<__nv_bfloat16>& g, __nv_bfloat16* w_s, int cols, int base_c, int c0) {
+    const int pieces = g.ld >> 3, ldm = g.ld + 8;
+    for (int x = threadIdx.x; x < 2 * cols * pieces; x += blockDim.x) {
+        const int r = x / pieces, q = x % pieces, m = r / cols, c = c0 + r % cols;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (c < width) v = *reinterpret_cast<const uint4*>(g.gates + ((long long)m * g.C + base_c + c) * g.ld + q * 8);
+        if (c < g.width) v = *reinterpret_cast<const uint4*>(g.gates + ((long long)m * g.C + base_c + c) * g.ld + q * 8);
         *reinterpret_cast<uint4*>(w_s + r * ldm + q * 8) = v;
     }
+}
+// One step of 16 along the inner dimension: 16 tokens (rows from u_hi / u_lo on) by 16 columns of both matrices.
+__device__ __forceinline__ void gate_mma_step(float (&zr)[2][4], float (&zi)[2][4], const __nv_bfloat16* u_hi,
+                                              const __nv_bfloat16* u_lo, const __nv_bfloat16* wr, const __nv_bfloat16* wi, int ldm,
+                                              int ks, int lane) {
+    uint32_t ah[4], al[4], b0, b1, b2, b3;
+    const int at = (lane & 15) * ldm + ks * 16 + (lane >> 4) * 8;
+    const int bt = ((lane & 7) + (lane >> 4) * 8) * ldm + ks * 16 + ((lane >> 3) & 1) * 8;
+    lin_ldsm_x4(ah[0], ah[1], ah[2], ah[3], u_hi + at);
+    lin_ldsm_x4(al[0], al[1], al[2], al[3], u_lo + at);
+    lin_ldsm_x4(b0, b1, b2, b3, wr + bt);
+    lin_mma(zr[0], ah, b0, b1);
+    lin_mma(zr[1], ah, b2, b3);
+    lin_mma(zr[0], al, b0, b1);
+    lin_mma(zr[1], al, b2, b3);
+    lin_ldsm_x4(b0, b1, b2, b3, wi + bt);
+    lin_mma(zi[0], ah, b0, b1);
+    lin_mma(zi[1], ah, b2, b3);
+    lin_mma(zi[0], al, b0, b1);
+    lin_mma(zi[1], al, b2, b3);
+}
+
+// Few tokens: a CTA takes 16 tokens and 32 columns of one part, the inner dimension dealt out to FEW_SPLIT pairs of warps
+// (16 columns each); the sums meet in shared memory and every thread finishes its share of the tile.  Grid (token tiles,
+// parts, column blocks).  Shared memory: u [2][16][ld + 8], both matrices' rows [2][32][ld + 8].
+constexpr int FEW_SPLIT = 4, FEW_COLS = 32;
+template <bool SINGLE>
+__global__ void __launch_bounds__(2 * FEW_SPLIT * 32)
+gate_scan_prep_few_kernel(const GateScanArgs<__nv_bfloat16> g, int pairs) {
+    extern __shared__ __align__(16) unsigned char lin_smem[];
+    __shared__ TileToken tok[16];
+    __shared__ float sums[FEW_SPLIT][2][16][FEW_COLS + 1];
+    const int ldm = g.ld + 8;
+    __nv_bfloat16* u_hi = reinterpret_cast<__nv_bfloat16*>(lin_smem);
+    __nv_bfloat16* u_lo = u_hi + 16 * ldm;
+    __nv_bfloat16* w_s = u_lo + 16 * ldm;
+    const int t0 = blockIdx.x * 16, c0 = blockIdx.z * FEW_COLS, base_c = blockIdx.y * g.width;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_launch_dependents();
+    load_gates(g, w_s, FEW_COLS, base_c, c0);               // the weights depend on no earlier kernel
     pdl_wait();
-    if (threadIdx.x < TOKENS) tok[threadIdx.x] = tile_token(g, t0 + threadIdx.x);
+    if (threadIdx.x < 16) tok[threadIdx.x] = tile_token(g, t0 + threadIdx.x);
     __syncthreads();
-    // u of the part: a thread walks a run of tokens of one channel with the inputs sliding through registers
-    // (up to 4 taps), so that each is fetched once
-    constexpr int RUN = TOKENS >= 64 ? 16 : TOKENS >= 32 ? 8 : 1;
-    for (int x = threadIdx.x; x < g.ld * (TOKENS / RUN); x += NT) {
-        const int c = x % g.ld, first = x / g.ld * RUN;
-        if (c >= width || (RUN == 1 && tok[first].entry < 0)) {
-#pragma unroll
-            for (int tt = 0; tt < RUN; ++tt)
-                u_hi[(first + tt) * ldm + c] = u_lo[(first + tt) * ldm + c] = __float2bfloat16_rn(0.f);
-            continue;
-        }
-        const int cc = base_c + c;
-        float wv[4], win[4];
-        const bool slide = RUN > 1 && g.taps <= 4;
-        if (slide) {
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {                   // aligned to the last of 4 taps
-                wv[j] = j >= 4 - g.taps ? g.conv_w[(long long)(j - (4 - g.taps)) * g.C + cc] : 0.f;
-                win[j] = 0.f;
+    const int half = g.ld >> 1;
+#pragma unroll 2
+    for (int x = threadIdx.x; x < 16 * half; x += blockDim.x) {
+        const int tt = x / half, c = 2 * (x % half);
+        const TileToken k = tok[tt];
+        float2 u = make_float2(0.f, 0.f);
+        if (k.entry >= 0) {
+            if (pairs && c + 1 < g.width) u = conv_at2(g, k, t0 + tt, base_c + c);
+            else {
+                if (c < g.width) u.x = conv_at(g, k, t0 + tt, base_c + c);
+                if (c + 1 < g.width) u.y = conv_at(g, k, t0 + tt, base_c + c + 1);
             }
         }
-        const float bias = g.conv_b[cc];
+        split_store(u_hi + tt * ldm + c, u_lo + tt * ldm + c, u.x, u.y);
+    }
+    __syncthreads();
+    {
+        const int wn = warp & 1, wk = warp >> 1;
+        float zr[2][4] = {}, zi[2][4] = {};
+        for (int ks = wk; ks < (g.ld >> 4); ks += FEW_SPLIT)
+            gate_mma_step(zr, zi, u_hi, u_lo, w_s + wn * 16 * ldm, w_s + (FEW_COLS + wn * 16) * ldm, ldm, ks, lane);
 #pragma unroll
-        for (int tt = 0; tt < RUN; ++tt) {
-            const TileToken k = tok[first + tt];
-            float u = 0.f;
-            if (k.entry >= 0) {
-                if (slide) {
-                    const int t = t0 + first + tt;
-                    if (tt == 0 || k.place == 0) {          // a run's or a portion's beginning: the inputs before it
+        for (int b = 0; b < 2; ++b)
 #pragma unroll
-                        for (int j = 0; j < 3; ++j) win[j] = 3 - j < g.taps ? conv_input(g, k, t, cc, 3 - j) : 0.f;
-                    }
-                    win[3] = g.proj.load((long long)t * g.cols + g.x_off + cc);
-                    u = bias;
+            for (int j = 0; j < 4; ++j) {
+                const int tt = (lane >> 2) + (j >> 1) * 8, c = wn * 16 + b * 8 + 2 * (lane & 3) + (j & 1);
+                sums[wk][0][tt][c] = zr[b][j];
+                sums[wk][1][tt][c] = zi[b][j];
+            }
+    }
+    __syncthreads();
+    for (int x = threadIdx.x; x < 16 * FEW_COLS; x += blockDim.x) {
+        const int tt = x / FEW_COLS, cc = x % FEW_COLS, c = c0 + cc;
+        if (c >= g.width || tok[tt].entry < 0) continue;
+        float zr = 0.f, zi = 0.f;
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) u = fmaf(wv[j], win[j], u);
-#pragma unroll
-                    for (int j = 0; j < 3; ++j) win[j] = win[j + 1];
-                } else {
-                    u = conv_at(g, k, t0 + first + tt, cc);
+        for (int w = 0; w < FEW_SPLIT; ++w) zr += sums[w][0][tt][cc], zi += sums[w][1][tt][cc];
+        const float u = __bfloat162float(u_hi[tt * ldm + c]) + __bfloat162float(u_lo[tt * ldm + c]);
+        gate_scan_finish<__nv_bfloat16, SINGLE>(g, tok[tt], t0 + tt, base_c + c, zr, zi, u);
+    }
+}
+
+// Many tokens: a CTA takes 64 tokens and wn * 16 columns of one part, 4 x wn warps of 16 tokens and 16 columns.  The
+// inputs of the tile's tokens and of the three before it come into shared memory first; a thread then walks a run of
+// tokens of two channels with the inputs sliding through registers.  A portion's first tokens, which read the ring, and
+// convolutions of more taps go one by one.  Grid (token tiles, parts, column blocks).  Shared memory: inputs
+// [67][ld], u [2][64][ld + 8], both matrices' rows [2][wn * 16][ld + 8].
+constexpr int MANY_TOKENS = 64, MANY_RUN = 8, MANY_MAX_WN = 5;
+__global__ void __launch_bounds__(4 * MANY_MAX_WN * 32)
+gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, int pairs, int vec) {
+    extern __shared__ __align__(16) unsigned char lin_smem[];
+    __shared__ TileToken tok[MANY_TOKENS];
+    const int ldm = g.ld + 8, width = g.width, cols = wn_warps * 16;
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(lin_smem);
+    __nv_bfloat16* u_hi = xs + (MANY_TOKENS + 3) * g.ld;
+    __nv_bfloat16* u_lo = u_hi + MANY_TOKENS * ldm;
+    __nv_bfloat16* w_s = u_lo + MANY_TOKENS * ldm;
+    const int t0 = blockIdx.x * MANY_TOKENS, c0 = blockIdx.z * cols, base_c = blockIdx.y * width;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_launch_dependents();
+    load_gates(g, w_s, cols, base_c, c0);
+    pdl_wait();
+    if (threadIdx.x < MANY_TOKENS) tok[threadIdx.x] = tile_token(g, t0 + threadIdx.x);
+    if (vec) {                                              // rows of 16-byte pieces
+        const int pieces = g.ld >> 3;
+        for (int x = threadIdx.x; x < (MANY_TOKENS + 3) * pieces; x += blockDim.x) {
+            const int r = x / pieces, c = x % pieces * 8, t = t0 - 3 + r;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (t >= 0 && t < g.n && c < width) v = *reinterpret_cast<const uint4*>(g.proj.whole + (long long)t * g.cols + g.x_off + base_c + c);
+            *reinterpret_cast<uint4*>(xs + r * g.ld + c) = v;
+        }
+    } else {
+        const int half = g.ld >> 1;
+        for (int x = threadIdx.x; x < (MANY_TOKENS + 3) * half; x += blockDim.x) {
+            const int r = x / half, c = x % half * 2, t = t0 - 3 + r;
+            float2 v = make_float2(0.f, 0.f);
+            if (t >= 0 && t < g.n) {
+                const long long at = (long long)t * g.cols + g.x_off + base_c + c;
+                if (pairs && c + 1 < width) v = g.proj.load2(at);
+                else {
+                    if (c < width) v.x = g.proj.load(at);
+                    if (c + 1 < width) v.y = g.proj.load(at + 1);
                 }
             }
-            const __nv_bfloat16 hi = __float2bfloat16_rn(u);
-            u_hi[(first + tt) * ldm + c] = hi;
-            u_lo[(first + tt) * ldm + c] = __float2bfloat16_rn(u - __bfloat162float(hi));
+            st2(xs + r * g.ld + c, v.x, v.y);
         }
     }
     __syncthreads();
-    const int wm = warp % WM, wn = warp / WM % WN, wk = warp / (WM * WN);
-    float zr[NB][4], zi[NB][4];
+    {
+        const int half = g.ld >> 1;
+        for (int x = threadIdx.x; x < half * (MANY_TOKENS / MANY_RUN); x += blockDim.x) {
+            const int c = 2 * (x % half), first = x / half * MANY_RUN;
+            const bool in0 = c < width, in1 = c + 1 < width;
+            float2 w[4], win[4];
 #pragma unroll
-    for (int b = 0; b < NB; ++b) zr[b][0] = zr[b][1] = zr[b][2] = zr[b][3] = zi[b][0] = zi[b][1] = zi[b][2] = zi[b][3] = 0.f;
-    const int wcol = wn * NB * 8;
-    for (int ks = wk; ks < (g.ld >> 4); ks += WK) {
-        uint32_t ah[4], al[4];
-        const int at = (wm * 16 + (lane & 15)) * ldm + ks * 16 + (lane >> 4) * 8;
-        lin_ldsm_x4(ah[0], ah[1], ah[2], ah[3], u_hi + at);
-        lin_ldsm_x4(al[0], al[1], al[2], al[3], u_lo + at);
-        if (NB == 1) {
-            // one load brings the 8 columns of both matrices: lanes 0..15 R's two halves of 8, lanes 16..31 I's
-            uint32_t b0, b1, b2, b3;
-            lin_ldsm_x4(b0, b1, b2, b3, w_s + ((lane >> 4) * COLS + wcol + (lane & 7)) * ldm + ks * 16 + ((lane >> 3) & 1) * 8);
-            lin_mma(zr[0], ah, b0, b1);
-            lin_mma(zi[0], ah, b2, b3);
-            lin_mma(zr[0], al, b0, b1);
-            lin_mma(zi[0], al, b2, b3);
-        } else {
+            for (int j = 0; j < 4; ++j) {                   // aligned to the last of 4 taps
+                const int tap = j - (4 - g.taps);
+                const float* cw = g.conv_w + (long long)tap * g.C + base_c + c;
+                w[j] = make_float2(tap >= 0 && in0 ? cw[0] : 0.f, tap >= 0 && in1 ? cw[1] : 0.f);
+            }
+            const float2 bias = make_float2(in0 ? g.conv_b[base_c + c] : 0.f, in1 ? g.conv_b[base_c + c + 1] : 0.f);
 #pragma unroll
-            for (int b = 0; b + 1 < NB; b += 2) {
-                const int row = wcol + b * 8 + (lane & 7) + (lane >> 4) * 8, col = ks * 16 + ((lane >> 3) & 1) * 8;
-                uint32_t b0, b1, b2, b3;
-                lin_ldsm_x4(b0, b1, b2, b3, w_s + row * ldm + col);
-                lin_mma(zr[b], ah, b0, b1);
-                lin_mma(zr[b + 1], ah, b2, b3);
-                lin_mma(zr[b], al, b0, b1);
-                lin_mma(zr[b + 1], al, b2, b3);
-                lin_ldsm_x4(b0, b1, b2, b3, w_s + (COLS + row) * ldm + col);
-                lin_mma(zi[b], ah, b0, b1);
-                lin_mma(zi[b + 1], ah, b2, b3);
-                lin_mma(zi[b], al, b0, b1);
-                lin_mma(zi[b + 1], al, b2, b3);
+            for (int j = 0; j < 3; ++j) win[j] = ld2(xs + (first + j) * g.ld + c);
+#pragma unroll
+            for (int tt = 0; tt < MANY_RUN; ++tt) {
+                const TileToken k = tok[first + tt];
+                win[3] = ld2(xs + (first + tt + 3) * g.ld + c);
+                float2 u = bias;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) u.x = fmaf(w[j].x, win[j].x, u.x), u.y = fmaf(w[j].y, win[j].y, u.y);
+                if (k.entry < 0) u = make_float2(0.f, 0.f);
+                else if (k.place < g.taps - 1 || g.taps > 4)
+                    u = make_float2(in0 ? conv_at(g, k, t0 + first + tt, base_c + c) : 0.f,
+                                    in1 ? conv_at(g, k, t0 + first + tt, base_c + c + 1) : 0.f);
+                split_store(u_hi + (first + tt) * ldm + c, u_lo + (first + tt) * ldm + c, u.x, u.y);
+#pragma unroll
+                for (int j = 0; j < 3; ++j) win[j] = win[j + 1];
             }
         }
     }
-    if (WK == 2) {
-        __shared__ float half[WK == 2 ? WM * WN * 32 : 1][NB * 8 + 1];
-        float* mine = half[(wn * WM + wm) * 32 + lane];
-        if (wk == 1) {
+    __syncthreads();
+    const int wm = warp & 3, wn = warp >> 2;
+    float zr[2][4] = {}, zi[2][4] = {};
+    for (int ks = 0; ks < (g.ld >> 4); ++ks)
+        gate_mma_step(zr, zi, u_hi + wm * 16 * ldm, u_lo + wm * 16 * ldm, w_s + wn * 16 * ldm, w_s + (cols + wn * 16) * ldm, ldm, ks, lane);
 #pragma unroll
-            for (int b = 0; b < NB; ++b)
+    for (int b = 0; b < 2; ++b) {
+        const int c = c0 + wn * 16 + b * 8 + 2 * (lane & 3);
 #pragma unroll
-                for (int j = 0; j < 4; ++j) mine[b * 8 + j] = zr[b][j], mine[b * 8 + 4 + j] = zi[b][j];
-        }
-        __syncthreads();
-        if (wk == 1) return;
-#pragma unroll
-        for (int b = 0; b < NB; ++b)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) zr[b][j] += mine[b * 8 + j], zi[b][j] += mine[b * 8 + 4 + j];
-    }
-#pragma unroll
-    for (int b = 0; b < NB; ++b)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int tt = wm * 16 + quad + (j >> 1) * 8, c = c0 + wcol + b * 8 + 2 * t4 + (j & 1);
+        for (int h = 0; h < 2; ++h) {
+            const int tt = wm * 16 + (lane >> 2) + h * 8;
             if (c >= width || tok[tt].entry < 0) continue;
-            const float u = __bfloat162float(u_hi[tt * ldm + c]) + __bfloat162float(u_lo[tt * ldm + c]);
-            gate_scan_finish<__nv_bfloat16, SINGLE>(g, tok[tt], t0 + tt, base_c + c, zr[b][j], zi[b][j], u);
+            const float2 uh = ld2(u_hi + tt * ldm + c), ul = ld2(u_lo + tt * ldm + c);
+            float a0, b0, a1, b1;
+            gate_scan_terms(g, base_c + c, zr[b][2 * h], zi[b][2 * h], uh.x + ul.x, a0, b0);
+            float* o = g.aux + (long long)(t0 + tt) * 2 * g.C + base_c + c;
+            if (c + 1 < width) {
+                gate_scan_terms(g, base_c + c + 1, zr[b][2 * h + 1], zi[b][2 * h + 1], uh.y + ul.y, a1, b1);
+                if (pairs) { st2(o, a0, a1); st2(o + g.C, b0, b1); }
+                else { o[0] = a0; o[1] = a1; o[g.C] = b0; o[g.C + 1] = b1; }
+            } else {
+                o[0] = a0;
+                o[g.C] = b0;
+            }
         }
+    }
 }
 
 // ------------------------------------------------------ the walk
-// Grid (blocks of 32 channels, entries); a lane per channel, a warp per run of RUN tokens of a round of WARPS * RUN.
-// A run is first composed to (product of the a's, its sum from zero); from the runs' pairs every warp works out the
-// state before its run, and walks it.  The last warp's state begins the next round.
-constexpr int SCAN_WARPS = 16, SCAN_RUN = 8;
-template <typename T>
+// Grid (share of the entry's tokens, blocks of 32 channels, entries); a lane per channel.  The CTAs of an entry's shares
+// are one cluster.  A warp takes a run of RUN tokens of a round of WARPS * RUN: a run is first composed to (product of
+// the a's, its sum from zero); from the runs' pairs every warp works out the state before its run, and walks it.  With
+// more than one share, every CTA first composes its whole share and reads the pairs of the shares before it from their
+// CTAs' shared memory.
+constexpr int SCAN_WARPS = 8, SCAN_RUN = 8, SCAN_MAX_SHARES = 8;
+template <typename T, bool CLUSTER>
 __global__ void __launch_bounds__(SCAN_WARPS * 32)
 channel_scan_kernel(const float* __restrict__ aux, GemmOut<T> proj, int cols, int y_off, int x_off,
                     const int* __restrict__ cu_q, const int* __restrict__ kv_len, const int* __restrict__ slots,
                     int n_slots, float* __restrict__ state, long long slot_stride, long long s_off, long long ring_off,
                     int taps, T* __restrict__ out, int C, int* err) {
     __shared__ float2 pair[2][SCAN_WARPS][32];
+    __shared__ float2 whole[32];
     pdl_launch_dependents();
     pdl_wait();
-    const int e = blockIdx.y;
+    const int e = blockIdx.z;
     const int first = cu_q[e], q_len = cu_q[e + 1] - first;
     if (q_len <= 0) return;                                 // an entry that pads the step: no slot is touched
     const int slot = slots[e];
-    if (slot < 0 || slot >= n_slots) {
+    if (slot < 0 || slot >= n_slots) {                      // (all CTAs of the cluster leave)
         if (threadIdx.x == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
         return;
     }
+    constexpr int ROUND = SCAN_WARPS * SCAN_RUN;
+    const int shares = CLUSTER ? (int)gridDim.x : 1, share = CLUSTER ? (int)blockIdx.x : 0;
+    // shares of whole rounds: tokens begin .. end - 1 are this CTA's
+    const int per = ((q_len + shares - 1) / shares + ROUND - 1) / ROUND * ROUND;
+    const int begin = min(q_len, share * per), end = min(q_len, begin + per);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c = blockIdx.x * 32 + lane;
+    const int c = blockIdx.y * 32 + lane;
     const bool live = c < C;
     const int start = kv_len[e] - q_len;
     float* mine = state + (long long)slot * slot_stride;
     float s0 = live && start > 0 ? mine[s_off + c] : 0.f;    // the state before the round
-    constexpr int ROUND = SCAN_WARPS * SCAN_RUN;
-    float a[SCAN_RUN], b[SCAN_RUN], an[SCAN_RUN], bn[SCAN_RUN];
-    auto fetch = [&](int t, float (&pa)[SCAN_RUN], float (&pb)[SCAN_RUN]) {       // tokens past the end change nothing
+    float a[SCAN_RUN], b[SCAN_RUN];
+    auto fetch = [&](int t) {                                // tokens past the end change nothing
 #pragma unroll
         for (int j = 0; j < SCAN_RUN; ++j) {
-            const bool in = live && t + j < q_len;
+            const bool in = live && t + j < end;
             const float* row = aux + (long long)(first + t + j) * 2 * C + c;
-            pa[j] = in ? row[0] : 1.f;
-            pb[j] = in ? row[C] : 0.f;
+            a[j] = in ? row[0] : 1.f;
+            b[j] = in ? row[C] : 0.f;
         }
     };
-    fetch(warp * SCAN_RUN, a, b);
-    for (int t0 = 0, it = 0; t0 < q_len; t0 += ROUND, ++it) {
-        const int t = t0 + warp * SCAN_RUN;
-        if (t0 + ROUND < q_len) fetch(t + ROUND, an, bn);
-        float y[SCAN_RUN];
-#pragma unroll
-        for (int j = 0; j < SCAN_RUN; ++j)
-            y[j] = live && t + j < q_len ? proj.load((long long)(first + t + j) * cols + y_off + c) : 0.f;
+    auto compose = [&]() {
         float A = 1.f, B = 0.f;
 #pragma unroll
         for (int j = 0; j < SCAN_RUN; ++j) {
             B = fmaf(a[j], B, b[j]);
             A *= a[j];
         }
-        pair[it & 1][warp][lane] = make_float2(A, B);
+        return make_float2(A, B);
+    };
+    if (CLUSTER) {
+        float2 total = make_float2(1.f, 0.f);                // of the rounds so far, of this warp's runs alone ...
+        for (int t0 = begin; t0 < end; t0 += ROUND) {
+            fetch(t0 + warp * SCAN_RUN);
+            pair[0][warp][lane] = compose();
+            __syncthreads();
+            if (warp == 0) {                                 // ... warp 0 puts the round's runs together
+#pragma unroll
+                for (int w = 0; w < SCAN_WARPS; ++w) {
+                    const float2 p = pair[0][w][lane];
+                    total = make_float2(total.x * p.x, fmaf(p.x, total.y, p.y));
+                }
+            }
+            __syncthreads();
+        }
+        if (warp == 0) whole[lane] = total;
+        asm volatile("barrier.cluster.arrive.release.aligned;\n"
+                     "barrier.cluster.wait.acquire.aligned;" ::: "memory");
+        const uint32_t at = (uint32_t)__cvta_generic_to_shared(&whole[lane]);
+        float2 p[SCAN_MAX_SHARES];
+#pragma unroll
+        for (int r = 0; r < SCAN_MAX_SHARES; ++r) {
+            p[r] = make_float2(1.f, 0.f);
+            if (r < share) {
+                uint32_t ra;
+                asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(at), "r"(r));
+                asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(p[r].x), "=f"(p[r].y) : "r"(ra) : "memory");
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < SCAN_MAX_SHARES; ++r) s0 = fmaf(p[r].x, s0, p[r].y);
+        // nobody leaves, or writes the slot, while a CTA of the cluster may still read
+        asm volatile("barrier.cluster.arrive.release.aligned;\n"
+                     "barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    }
+    for (int t0 = begin, it = 0; t0 < end; t0 += ROUND, ++it) {
+        const int t = t0 + warp * SCAN_RUN;
+        fetch(t);
+        float y[SCAN_RUN];
+#pragma unroll
+        for (int j = 0; j < SCAN_RUN; ++j)
+            y[j] = live && t + j < end ? proj.load((long long)(first + t + j) * cols + y_off + c) : 0.f;
+        pair[it & 1][warp][lane] = compose();
         __syncthreads();
         float s = s0, mine_s = s0;
 #pragma unroll
@@ -363,13 +502,11 @@ channel_scan_kernel(const float* __restrict__ aux, GemmOut<T> proj, int cols, in
 #pragma unroll
         for (int j = 0; j < SCAN_RUN; ++j) {
             mine_s = fmaf(a[j], mine_s, b[j]);
-            if (live && t + j < q_len)
+            if (live && t + j < end)
                 out[(long long)(first + t + j) * C + c] = from_f32<T>(mine_s * lin_gelu_tanh(y[j]));
-            a[j] = an[j];
-            b[j] = bn[j];
         }
     }
-    if (!live) return;
+    if (!live || end != q_len || begin == end) return;       // the CTA with the last token moves the slot on
     if (warp == 0) mine[s_off + c] = s0;
     // the last inputs of the convolution: those of this step (older ones stay where they are)
     for (int back = warp; back < taps && back < q_len; back += SCAN_WARPS) {
@@ -387,24 +524,38 @@ int launch_simt(const GateScanArgs<T>& g, int parts, cudaStream_t st) {
     return crane_launch(kern, dim3((g.n + SIMT_TOKENS - 1) / SIMT_TOKENS, parts, (g.width + 127) / 128), dim3(128), smem, st, g);
 }
 
-template <int TOKENS, int COLS, int WN, int WK, bool SINGLE>
-int launch_mma(const GateScanArgs<__nv_bfloat16>& g, int parts, cudaStream_t st) {
-    const size_t smem = (size_t)2 * (TOKENS + COLS) * (g.ld + 8) * sizeof(__nv_bfloat16);
-    const auto kern = gate_scan_prep_mma_kernel<TOKENS, COLS, WN, WK, SINGLE>;
+constexpr int LIN_SMEM = 208 * 1024;
+int launch_tensor(const GateScanArgs<__nv_bfloat16>& g, int parts, int all_single, cudaStream_t st) {
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024) != cudaSuccess)
-            return (int)cudaGetLastError();
+        const void* kerns[] = {(const void*)gate_scan_prep_few_kernel<true>, (const void*)gate_scan_prep_few_kernel<false>,
+                               (const void*)gate_scan_prep_many_kernel};
+        for (const void* k : kerns)
+            if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, LIN_SMEM) != cudaSuccess)
+                return (int)cudaGetLastError();
         configured = true;
     }
-    if (smem > 208 * 1024) return (int)cudaErrorInvalidValue;
-    return crane_launch(kern, dim3((g.n + TOKENS - 1) / TOKENS, parts, (g.width + COLS - 1) / COLS),
-                        dim3(TOKENS / 16 * WN * WK * 32), smem, st, g);
-}
-
-int launch_tensor(const GateScanArgs<__nv_bfloat16>& g, int parts, int all_single, cudaStream_t st) {
-    if (all_single) return g.n <= 16 ? launch_mma<16, 16, 2, 2, true>(g, parts, st) : launch_mma<32, 32, 2, 1, true>(g, parts, st);
-    return g.n <= 16 ? launch_mma<16, 16, 2, 2, false>(g, parts, st) : launch_mma<64, 64, 2, 1, false>(g, parts, st);
+    const int ldm = g.ld + 8;
+    // two neighbours a load and a store where every row and every place in it is even
+    const int pairs = ((g.C | g.width | g.cols | g.x_off | g.y_off) & 1) == 0 && ((g.slot_stride | g.ring_off | g.proj.part_stride) & 1) == 0 &&
+                      (((uintptr_t)g.state | (uintptr_t)g.conv_w | (uintptr_t)g.conv_b) & 7) == 0;
+    if (all_single || g.n <= 16) {
+        const size_t smem = (size_t)2 * (16 + FEW_COLS) * ldm * sizeof(__nv_bfloat16);
+        const auto kern = all_single ? gate_scan_prep_few_kernel<true> : gate_scan_prep_few_kernel<false>;
+        return crane_launch(kern, dim3((g.n + 15) / 16, parts, (g.width + FEW_COLS - 1) / FEW_COLS), dim3(2 * FEW_SPLIT * 32), smem,
+                            st, g, pairs);
+    }
+    const int vec = g.proj.parts == nullptr && ((g.width | g.cols | g.x_off) & 7) == 0 && ((uintptr_t)g.proj.whole & 15) == 0;
+    const size_t base = (size_t)((MANY_TOKENS + 3) * g.ld + 2 * MANY_TOKENS * ldm) * sizeof(__nv_bfloat16);
+    const size_t per_wn = (size_t)2 * 16 * ldm * sizeof(__nv_bfloat16);
+    const int groups = (g.width + 15) / 16;
+    int wn = groups < MANY_MAX_WN ? groups : MANY_MAX_WN;
+    while (wn > 1 && base + wn * per_wn > LIN_SMEM) --wn;
+    if (base + per_wn > LIN_SMEM) return (int)cudaErrorInvalidValue;
+    const int blocks = (groups + wn - 1) / wn;
+    wn = (groups + blocks - 1) / blocks;                    // (as even as it gets)
+    return crane_launch(gate_scan_prep_many_kernel, dim3((g.n + MANY_TOKENS - 1) / MANY_TOKENS, parts, blocks), dim3(4 * wn * 32),
+                        base + wn * per_wn, st, g, wn, pairs, vec);
 }
 int launch_tensor(const GateScanArgs<float>&, int, int, cudaStream_t) { return (int)cudaErrorInvalidValue; }
 
@@ -439,14 +590,20 @@ CRANE_API int crane_gate_scan_prep(int dtype, const void* proj, const float* pro
 CRANE_API int crane_channel_scan(int dtype, const float* aux, const void* proj, const float* proj_parts, int n_parts,
                                  long long part_stride, int cols, int y_off, int x_off, const int* cu_q,
                                  const int* kv_len, const int* slots, int n_slots, float* state, long long slot_stride,
-                                 long long s_off, long long ring_off, int taps, void* out, int n_entries, int C,
-                                 int* err, cudaStream_t st) {
+                                 long long s_off, long long ring_off, int taps, void* out, int n_entries, int n_tokens,
+                                 int C, int* err, cudaStream_t st) {
     if (n_entries <= 0) return 0;
     if (taps < 1 || taps > LIN_MAX_TAPS || C <= 0) return (int)cudaErrorInvalidValue;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
-        return crane_launch(channel_scan_kernel<T>, dim3((C + 31) / 32, n_entries), dim3(SCAN_WARPS * 32), 0, st, aux, p,
-                            cols, y_off, x_off, cu_q, kv_len, slots, n_slots, state, slot_stride, s_off, ring_off, taps,
-                            (T*)out, C, err);
+        // shares of about four rounds: enough CTAs for a long prompt, no more than a cluster holds
+        int shares = 1;
+        while (shares < SCAN_MAX_SHARES && n_tokens / n_entries >= shares * 4 * SCAN_WARPS * SCAN_RUN) shares *= 2;
+        const dim3 grid(shares, (C + 31) / 32, n_entries), block(SCAN_WARPS * 32);
+        if (shares == 1)
+            return crane_launch(channel_scan_kernel<T, false>, grid, block, 0, st, aux, p, cols, y_off, x_off, cu_q, kv_len, slots,
+                                n_slots, state, slot_stride, s_off, ring_off, taps, (T*)out, C, err);
+        return crane_launch_cluster(channel_scan_kernel<T, true>, grid, block, 0, dim3(shares, 1, 1), st, aux, p, cols, y_off, x_off,
+                                    cu_q, kv_len, slots, n_slots, state, slot_stride, s_off, ring_off, taps, (T*)out, C, err);
     });
 }

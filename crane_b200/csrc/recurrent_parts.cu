@@ -200,11 +200,11 @@ decay_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
 //     i = cap tanh((z_i + bias_i) / cap),  f = log sigmoid(cap tanh((z_f + bias_f) / cap))
 //     M' = max(f + M, i);  w = exp(f + M - M'),  b = exp(i - M'),  floor = exp(-M')
 // M (0 before a request's first token) lies in the slot, [H] at `m_off`.  The first `gate_blocks` CTAs work out the
-// gates, a warp per (entry, head); the others copy q, k and v, `by` CTAs a token.  M -> max(M + A, B) composes to
-// maps of the same form, so a warp takes 128 tokens at a time, four a lane, and finds the M before every lane's four by
-// a scan over the lanes; within a lane it goes token by token, and a token's w is taken from the very M that the token
-// before it left.
-template <typename T>
+// gates, a CTA per (entry, head), or (SINGLE: every entry of the step has one token) a thread; the others copy q, k and
+// v, `by` CTAs a token.  M -> max(M + A, B) composes to maps of the same form, so a CTA takes 1,024 tokens at a time,
+// four a thread, and finds the M before every thread's four by a scan over lanes and warps; a thread goes token by
+// token, and a token's w is taken from the very M that the token before it left.
+template <typename T, bool SINGLE>
 __global__ void __launch_bounds__(256)
 exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, const int* __restrict__ cu_q,
                      const int* __restrict__ kv_len, const int* __restrict__ slots, int n_slots,
@@ -233,44 +233,66 @@ exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entr
         }
         return;
     }
-    const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    // li = -inf and lf = 0 (past a portion's end) leave M as it is
+    auto gates = [&](float zi, float zf, float bi, float bf, float& li, float& lf) {
+        const float x = cap * tanhf((zf + bf) / cap);
+        li = cap * tanhf((zi + bi) / cap);
+        lf = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
+    };
+    auto write = [&](long long t, int h, float li, float lf, float before, float m) {
+        float* out = aux + t * aux_cols + w_off + h;
+        out[0] = expf(lf + before - m);
+        out[H] = expf(li - m);
+        out[2 * H] = expf(-m);
+    };
+    const int wid = SINGLE ? (int)(blockIdx.x * blockDim.x + threadIdx.x) : (int)blockIdx.x;
     if (wid >= n_entries * H) return;
     const int e = wid / H, h = wid % H;
     const int first = cu_q[e], q_len = cu_q[e + 1] - first;
     if (q_len <= 0) return;
     const int slot = slots[e];
     if (slot < 0 || slot >= n_slots) {
-        if (lane == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
+        if (SINGLE || threadIdx.x == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
         return;
     }
     float* kept = state + (long long)slot * slot_stride + m_off + h;
     float m0 = kv_len[e] > q_len ? *kept : 0.f;
     const float bi = bias_i[h], bf = bias_f[h];
-    constexpr int PER = 4;
+    if (SINGLE) {
+        float li, lf;
+        const long long row = (long long)first * cols + h;
+        gates(proj.load(row + i_off), proj.load(row + f_off), bi, bf, li, lf);
+        const float m = fmaxf(lf + m0, li);
+        write(first, h, li, lf, m0, m);
+        *kept = m;
+        return;
+    }
+    constexpr int PER = 4, WARPS = 8;
+    __shared__ float part_a[WARPS], part_b[WARPS], last[WARPS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float zi[PER], zf[PER];
     auto fetch = [&](int t0) {
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
-            const int t = t0 + lane * PER + j;
+            const int t = t0 + (int)threadIdx.x * PER + j;
             const long long row = (long long)(first + (t < q_len ? t : q_len - 1)) * cols + h;
             zi[j] = proj.load(row + i_off);
             zf[j] = proj.load(row + f_off);
         }
     };
     fetch(0);
-    for (int t0 = 0; t0 < q_len; t0 += 32 * PER) {
+    for (int t0 = 0; t0 < q_len; t0 += WARPS * 32 * PER) {
+        const int t = t0 + (int)threadIdx.x * PER;
         float li[PER], lf[PER], m[PER];
         float A = 0.f, B = -INFINITY;
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
-            const bool in = t0 + lane * PER + j < q_len;
-            const float x = cap * tanhf((zf[j] + bf) / cap);
-            li[j] = in ? cap * tanhf((zi[j] + bi) / cap) : -INFINITY;          // (past the end: M stays)
-            lf[j] = in ? fminf(x, 0.f) - log1pf(expf(-fabsf(x))) : 0.f;
+            gates(zi[j], zf[j], bi, bf, li[j], lf[j]);
+            if (t + j >= q_len) li[j] = -INFINITY, lf[j] = 0.f;
             B = fmaxf(B + lf[j], li[j]);
             A += lf[j];
         }
-        if (t0 + 32 * PER < q_len) fetch(t0 + 32 * PER);
+        if (t0 + WARPS * 32 * PER < q_len) fetch(t0 + WARPS * 32 * PER);
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float pa = __shfl_up_sync(0xffffffffu, A, o), pb = __shfl_up_sync(0xffffffffu, B, o);
@@ -279,26 +301,26 @@ exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entr
                 A += pa;
             }
         }
+        if (lane == 31) part_a[warp] = A, part_b[warp] = B;
         const float pa = __shfl_up_sync(0xffffffffu, A, 1), pb = __shfl_up_sync(0xffffffffu, B, 1);
-        float run = lane == 0 ? m0 : fmaxf(m0 + pa, pb);
+        __syncthreads();
+        float run = m0;                                     // M before the warp's tokens, then before the thread's
+        for (int w = 0; w < warp; ++w) run = fmaxf(run + part_a[w], part_b[w]);
+        if (lane > 0) run = fmaxf(run + pa, pb);
 #pragma unroll
         for (int j = 0; j < PER; ++j) m[j] = run = fmaxf(lf[j] + run, li[j]);
-        const float left = __shfl_up_sync(0xffffffffu, m[PER - 1], 1);
-        float before = lane == 0 ? m0 : left;
+        if (lane == 31) last[warp] = m[PER - 1];
+        float before = __shfl_up_sync(0xffffffffu, m[PER - 1], 1);
+        __syncthreads();
+        if (lane == 0) before = warp == 0 ? m0 : last[warp - 1];
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
-            const int t = t0 + lane * PER + j;
-            if (t < q_len) {
-                float* out = aux + (long long)(first + t) * aux_cols + w_off + h;
-                out[0] = expf(lf[j] + before - m[j]);
-                out[H] = expf(li[j] - m[j]);
-                out[2 * H] = expf(-m[j]);
-            }
+            if (t + j < q_len) write(first + t + j, h, li[j], lf[j], before, m[j]);
             before = m[j];
         }
-        m0 = __shfl_sync(0xffffffffu, m[PER - 1], 31);
+        m0 = last[WARPS - 1];                               // (a round later `part_a` and `last` are written behind two barriers)
     }
-    if (lane == 0) *kept = m0;
+    if (threadIdx.x == 0) *kept = m0;
 }
 
 // ------------------------------------------------------ what the bonus recurrence's projections read
@@ -879,16 +901,53 @@ head_talk_mix_kernel(const float* __restrict__ cross, const float* __restrict__ 
 
 // ------------------------------------------------------ two mixers side by side
 // out = (a / rms(a) * wa + b / rms(b) * wb) / 2 over the width; a CTA per row.
+// Four neighbours of a product (aligned), all slices' loads in flight eight at a time, added in slice order.
 template <typename T>
-__global__ void __launch_bounds__(256)
+__device__ __forceinline__ float4 load4(const GemmOut<T>& g, long long idx) {
+    if (g.parts == nullptr) {
+        const float2 a = ld2(g.whole + idx), b = ld2(g.whole + idx + 2);
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+    float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < g.n_parts; i += 8) {
+        float4 q[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            q[j] = i + j < g.n_parts ? *(const float4*)(g.parts + (long long)(i + j) * g.part_stride + idx)
+                                     : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) d.x += q[j].x, d.y += q[j].y, d.z += q[j].z, d.w += q[j].w;
+    }
+    return make_float4(to_f32(from_f32<T>(d.x)), to_f32(from_f32<T>(d.y)), to_f32(from_f32<T>(d.z)), to_f32(from_f32<T>(d.w)));
+}
+template <typename T>
+__global__ void __launch_bounds__(1024)
 pair_norm_mean_kernel(GemmOut<T> a, GemmOut<T> b, const float* __restrict__ wa, const float* __restrict__ wb,
-                      float eps, T* __restrict__ out, int hidden) {
+                      float eps, T* __restrict__ out, int hidden, int quad) {
     extern __shared__ float row2[];                   // [2 hidden]
     __shared__ float scratch[32];
     pdl_launch_dependents();
-    pdl_wait();
     const long long base = (long long)blockIdx.x * hidden;
     float sa = 0.f, sb = 0.f;
+    // Rows of four columns a thread: everything a thread reads is in flight at once, the weights before the wait for
+    // the kernel before, and stays in its registers.
+    if (quad) {
+        const int c = threadIdx.x * 4;
+        const bool in = c < hidden;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 va = in ? *(const float4*)(wa + c) : zero, vb = in ? *(const float4*)(wb + c) : zero;
+        pdl_wait();
+        const float4 x = in ? load4(a, base + c) : zero, y = in ? load4(b, base + c) : zero;
+        sa = block_sum((x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w), scratch);
+        sb = block_sum((y.x * y.x + y.y * y.y) + (y.z * y.z + y.w * y.w), scratch);
+        const float ra = rsqrtf(sa / (float)hidden + eps), rb = rsqrtf(sb / (float)hidden + eps);
+        if (in) {
+            st2(out + base + c, 0.5f * (x.x * ra * va.x + y.x * rb * vb.x), 0.5f * (x.y * ra * va.y + y.y * rb * vb.y));
+            st2(out + base + c + 2, 0.5f * (x.z * ra * va.z + y.z * rb * vb.z), 0.5f * (x.w * ra * va.w + y.w * rb * vb.w));
+        }
+        return;
+    }
+    pdl_wait();
     const bool pairs = (hidden & 1) == 0;             // rows of even length: two neighbours a load and a store
     if (pairs) {
         for (int c = 2 * threadIdx.x; c < hidden; c += 2 * blockDim.x) {
@@ -970,14 +1029,16 @@ CRANE_API int crane_exp_gate_prep(int dtype, const void* proj, const float* proj
                                   const int* kv_len, const int* slots, int n_slots, float* state,
                                   long long slot_stride, long long m_off, const float* bias_i, const float* bias_f,
                                   float cap, float q_scale, float* aux, int aux_cols, int n_tokens, int n_entries,
-                                  int H, int d, int dv, int i_off, int f_off, int w_off, int* err, cudaStream_t st) {
+                                  int H, int d, int dv, int i_off, int f_off, int w_off, int all_single, int* err,
+                                  cudaStream_t st) {
     if (n_tokens <= 0) return 0;
-    const int gate_blocks = (n_entries * H + 7) / 8;
+    const int gate_blocks = all_single ? (n_entries * H + 255) / 256 : n_entries * H;
     int by = (2 * H * d + H * dv + 511) / 512;               // with few tokens a token's columns spread over more CTAs
     while (by > 1 && (long long)n_tokens * by > 4 * 148) by = (by + 1) / 2;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
-        return crane_launch(exp_gate_prep_kernel<T>, dim3(gate_blocks + n_tokens * by), dim3(256), 0, st, p, cols,
+        const auto kern = all_single ? exp_gate_prep_kernel<T, true> : exp_gate_prep_kernel<T, false>;
+        return crane_launch(kern, dim3(gate_blocks + n_tokens * by), dim3(256), 0, st, p, cols,
                             tok_entry, cu_q, kv_len, slots, n_slots, state, slot_stride, m_off, bias_i, bias_f, cap,
                             q_scale, aux, aux_cols, n_entries, H, d, dv, i_off, f_off, w_off, gate_blocks, by, err);
     });
@@ -1164,7 +1225,11 @@ CRANE_API int crane_pair_norm_mean(int dtype, const void* a, const float* a_part
         GemmOut<T> gb{(const T*)b, b_parts, bn, bstr};
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(pair_norm_mean_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        return crane_launch(pair_norm_mean_kernel<T>, dim3(n_rows), dim3(256), smem, st, ga, gb, wa, wb, eps, (T*)out,
-                            hidden);
+        const int quad = hidden % 4 == 0 && hidden <= 4096 && ((astr | bstr) & 3) == 0 &&
+                         (((uintptr_t)wa | (uintptr_t)wb | (uintptr_t)a_parts | (uintptr_t)b_parts) & 15) == 0 &&
+                         (((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & 7) == 0;
+        const int threads = quad ? (hidden / 4 + 31) / 32 * 32 : 256;
+        return crane_launch(pair_norm_mean_kernel<T>, dim3(n_rows), dim3(threads), quad ? 0 : smem, st, ga, gb, wa, wb, eps,
+                            (T*)out, hidden, quad);
     });
 }

@@ -65,12 +65,12 @@ _SIGNATURES = {
                               P, P, I, I, I, I, I, I, P],
     "crane_decay_gate_prep": [I, P, P, I, L, I, P, P, P, I, F, F, P, I, I, I, I, I, P],
     "crane_matrix_state_plan": [I, P, P],
-    "crane_exp_gate_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, P, F, F, P, I, I, I, I, I, I, I, I, I, P, P],
+    "crane_exp_gate_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, P, F, F, P, I, I, I, I, I, I, I, I, I, I, P, P],
     "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, P, I, I, I, I, P, P],
     "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, I, I, F, P, P, I, F, P, I, I, I, P],
     "crane_gate_scan_mma_most": [],
     "crane_gate_scan_prep": [I, P, P, I, L, I, I, I, P, P, P, P, I, P, L, L, L, P, P, I, P, I, P, P, P, P, P, I, I, I, I, P, P],
-    "crane_channel_scan": [I, P, P, P, I, L, I, I, I, P, P, P, I, P, L, L, L, I, P, I, I, P, P],
+    "crane_channel_scan": [I, P, P, P, I, L, I, I, I, P, P, P, I, P, L, L, L, I, P, I, I, I, P, P],
     "crane_head_talk_mix": [I, P, P, P, P, I, I, I, I, I, P],
     "crane_pair_norm_mean": [I, P, P, I, L, P, P, I, L, P, P, F, P, I, I, P],
     "crane_delta_rule_prep": [I, P, P, I, L, I, P, P, P, P, P, I, I, I, I, F, F, P],
@@ -616,8 +616,8 @@ class Kernels:
             _dt(dtype), whole, parts, n_parts, stride, int(cols), ctx.tok_entry.data_ptr(), ctx.cu_q.data_ptr(),
             ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0), int(m_off),
             bias_i.data_ptr(), bias_f.data_ptr(), float(cap), float(q_scale), aux.data_ptr(), aux.shape[1],
-            aux.shape[0], ctx.kv_len.shape[0], H, d, dv, int(i_off), int(f_off), int(w_off), err.data_ptr(),
-            self._stream(aux)), "exp_gate_prep")
+            aux.shape[0], ctx.kv_len.shape[0], H, d, dv, int(i_off), int(f_off), int(w_off),
+            1 if step_of_single_tokens(ctx) else 0, err.data_ptr(), self._stream(aux)), "exp_gate_prep")
 
     # ---- recurrences with a number per channel ---------------------------
     @dataclass
@@ -670,8 +670,8 @@ class Kernels:
         self._check(self.lib.crane_channel_scan(
             _dt(out.dtype), aux.data_ptr(), whole, parts, n_parts, stride, int(cols), g.y_off, g.x_off,
             ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
-            state.stride(0), g.s_off, g.ring_off, g.conv_w.shape[0], out.data_ptr(), ctx.kv_len.shape[0], out.shape[1],
-            err.data_ptr(), self._stream(out)), "channel_scan")
+            state.stride(0), g.s_off, g.ring_off, g.conv_w.shape[0], out.data_ptr(), ctx.kv_len.shape[0], out.shape[0],
+            out.shape[1], err.data_ptr(), self._stream(out)), "channel_scan")
 
     def matrix_state_scan(self, aux, offs, w_vec: bool, mode, qk_rep: int, ctx, state, o_raw, H, dk, dv,
                           err, den=None) -> None:

@@ -518,6 +518,48 @@ def test_attention_part(dtype, H, G, d, m, rot, window):
     rt.check_errors()
 
 
+@pytest.mark.parametrize("d, rot, norm", [(128, 64, True), (96, 32, True), (64, 64, True), (200, 48, True), (256, 256, True), (128, 0, True),
+                                          (24, 16, True), (128, 32, False), (8, 0, True)])
+def test_norm_before_a_partial_rotation(K, d, rot, norm):
+    """Whole bfloat16 rows of many tokens (16-byte loads, the partner by shuffle) against NumPy, with rows of no entry,
+    a missing page and pages in no order."""
+    rng = np.random.default_rng(d + rot)
+    n, H, G, ps, eps, off = 70, 3, 1, 8, 1e-3, 0.5
+    cols = (H + 2 * G) * d + 16
+    x = _dev(rng.standard_normal((n, cols)) * 0.05, torch.bfloat16)
+    pos = rng.permutation(80)[:n]
+    table = np.array([rng.permutation(12)[:10]], dtype=np.int32)
+    table[0, 9] = -1
+    ent = np.zeros(n, dtype=np.int32)
+    ent[5] = -1
+    f = pm.rotary_frequencies(rot, 300.0)
+    ang = np.arange(80)[:, None] * f[None]
+    cos, sin = (_dev(np.cos(ang)), _dev(np.sin(ang))) if rot else (None, None)
+    qw, kw = (rng.standard_normal(d), rng.standard_normal(d)) if norm else (None, None)
+    q = torch.full((n, H * d), 5.0, dtype=torch.bfloat16, device=DEV)
+    kp, vp = (torch.full((12, G, ps, d), 5.0, dtype=torch.bfloat16, device=DEV) for _ in range(2))
+    err = _err()
+    K.rope_norm_cache(x, cols, torch.bfloat16, _i32(pos), _i32(ent), _i32(table), cos, sin, None if qw is None else _dev(qw),
+                      None if kw is None else _dev(kw), eps, q, kp, vp, ps, H, G, d, True, rot > 0, err, rope=(rot or d, False, True, off))
+    xn = _np(x)
+
+    def heads(a, w):
+        y = a.reshape(n, -1, d)
+        return pm.rotate_half(pm.over_rms(y, eps) * (off + w) if w is not None else y, pos, f)
+    want_q, want_k = heads(xn[:, :H * d], qw), heads(xn[:, H * d:(H + G) * d], kw)
+    assert np.abs(_np(q).reshape(n, H, d) - want_q).max() < 1e-2 * max(1.0, np.abs(want_q).max())
+    for t in range(n):
+        page = table[0, pos[t] // ps]
+        if ent[t] < 0 or page < 0:
+            continue
+        k, v = _np(kp)[page, :, pos[t] % ps], _np(vp)[page, :, pos[t] % ps]
+        assert np.abs(k - want_k[t]).max() < 1e-2 * max(1.0, np.abs(want_k).max()), t
+        assert np.abs(v - xn[t, (H + G) * d:(H + 2 * G) * d].reshape(G, d)).max() == 0
+    used = {int(p) for p in table[0] if p >= 0}
+    assert all((kp[p] == 5.0).all() for p in range(12) if p not in used)
+    assert int(err.item()) == (2 if (pos // ps == 9).any() else 0)
+
+
 @pytest.mark.parametrize("experts, top, scale", [(3, 3, 1.0), (12, 1, 2.5), (6, 2, 0.7), (64, 6, 1.0), (40, 8, 1.6)])
 def test_route_by_corrected_scores(K, experts, top, scale):
     """The correction chooses and the score weighs; the weights are over the chosen scores' sum."""

@@ -1619,7 +1619,7 @@ def mufalix_kernel_table(fcfg, pk, tokens, batch, context):
         # ---- the matrix memory
         H, d, m = ml["heads"], ml["dim"], ml["vdim"]
         hd, hv = H * d, H * m
-        cols, w_at = 2 * hd + 2 * hv + 2 * H, 2 * hd + hv
+        cols, w_at = -(-(2 * hd + 2 * hv + 2 * H) // 8) * 8, 2 * hd + hv
         rws, lanes = K.matrix_state_plan(d)
         m_off = H * rws * lanes * (m + 1)
         state = torch.zeros(n_req, m_off + H, device=dev)
@@ -1638,6 +1638,16 @@ def mufalix_kernel_table(fcfg, pk, tokens, batch, context):
             t_same, b_g, 0)
         add(f"matrix_state_scan, gated with a normaliser ({kind})", "matrix_state_scan, decay per channel (Mufevik, heads of 64)", t_p, b_g, 0,
             t_s, b_s, 0)
+        if not one and K.memory_chunks_takes(proj, cols, d, m):
+            logs = torch.empty(n, 2 * H, device=dev)
+            least = 24
+            t_p = t_of(lambda: K.exp_gate_prep(proj, cols, ctx, state, m_off, bi, bi, 15.0, d ** -0.5, aux, H, d, m, cols - 2 * H, cols - H,
+                                               w_at, err, bf, logs=logs, logs_min=least))
+            add(f"exp_gate_prep for chunks ({kind})", "bonus_prep (Pogarax)", t_p, n * H * 16, 0, t_l, n * w_at * 6, 0)
+            t_p = t_of(lambda: K.memory_chunks(proj, cols, (0, hd, 2 * hd), logs, ctx, state, o_raw, den, H, d, m, d ** -0.5, least, err))
+            fl = 2 * n * H * (32 * (d + m) + 2 * d * m)          # (half of a chunk's scores, on average)
+            add(f"memory_chunks ({kind})", "matrix_state_scan, decay per channel (Mufevik, heads of 64)", t_p, n * (w_at * 2 + hv * 4), fl, t_s,
+                b_s, 0)
         nw, o = rnd(hv, dt=f32), torch.empty(n, hv, device=dev, dtype=bf)
         fin = lambda **kw: K.head_norm_gate(o_raw, proj, cols, 2 * hd + hv, ent, nw, 1e-5, o, H, m, sigmoid=True, **kw)
         add(f"head_norm_gate behind a normaliser ({kind})", "head_norm_gate (Pogarax)",

@@ -26,6 +26,13 @@ __device__ __forceinline__ float lin_gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+// 1 - exp(x) for x <= 0, exp(x) given: near 0 from the series of the exponential, -x (1 + x/2 (1 + x/3 (...))), which
+// loses nothing to the subtraction.
+__device__ __forceinline__ float one_minus_exp(float x, float exp_x) {
+    const float series = -x * fmaf(x * 0.5f, fmaf(x * (1.f / 3.f), fmaf(x * 0.25f, fmaf(x * 0.2f, fmaf(x * (1.f / 6.f), 1.f, 1.f), 1.f), 1.f), 1.f), 1.f);
+    return x > -0.25f ? series : 1.f - exp_x;
+}
+
 template <typename T>
 struct GateScanArgs {
     GemmOut<T> proj;
@@ -87,7 +94,7 @@ __device__ __forceinline__ void gate_scan_terms(const GateScanArgs<T>& g, int c,
     const float r = lin_sigmoid(zr + g.rb[c]), i = lin_sigmoid(zi + g.ib[c]);
     const float log_a = -LIN_RATE * r * g.sp[c];
     a = expf(log_a);
-    add = sqrtf(-expm1f(2.f * log_a)) * i * u;
+    add = sqrtf(one_minus_exp(2.f * log_a, a * a)) * i * u;
 }
 // Token t, channel c: to what the walk needs, or, SINGLE, through the walk.
 template <typename T, bool SINGLE>
@@ -286,13 +293,13 @@ gate_scan_prep_few_kernel(const GateScanArgs<__nv_bfloat16> g, int pairs) {
     }
 }
 
-// Many tokens: a CTA takes 64 tokens and wn * 16 columns of one part, 4 x wn warps of 16 tokens and 16 columns.  The
+// Many tokens: a CTA takes 48 tokens and wn * 16 columns of one part, 3 x wn warps of 16 tokens and 16 columns.  The
 // inputs of the tile's tokens and of the three before it come into shared memory first; a thread then walks a run of
 // tokens of two channels with the inputs sliding through registers.  A portion's first tokens, which read the ring, and
 // convolutions of more taps go one by one.  Grid (token tiles, parts, column blocks).  Shared memory: inputs
-// [67][ld], u [2][64][ld + 8], both matrices' rows [2][wn * 16][ld + 8].
-constexpr int MANY_TOKENS = 64, MANY_RUN = 8, MANY_MAX_WN = 5;
-__global__ void __launch_bounds__(4 * MANY_MAX_WN * 32)
+// [51][ld], u [2][48][ld + 8], both matrices' rows [2][wn * 16][ld + 8].
+constexpr int MANY_TOKENS = 48, MANY_RUN = 8, MANY_MAX_WN = 5;
+__global__ void __launch_bounds__(MANY_TOKENS / 16 * MANY_MAX_WN * 32)
 gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, int pairs, int vec) {
     extern __shared__ __align__(16) unsigned char lin_smem[];
     __shared__ TileToken tok[MANY_TOKENS];
@@ -365,7 +372,7 @@ gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, in
         }
     }
     __syncthreads();
-    const int wm = warp & 3, wn = warp >> 2;
+    const int wm = warp % (MANY_TOKENS / 16), wn = warp / (MANY_TOKENS / 16);
     float zr[2][4] = {}, zi[2][4] = {};
     for (int ks = 0; ks < (g.ld >> 4); ++ks)
         gate_mma_step(zr, zi, u_hi + wm * 16 * ldm, u_lo + wm * 16 * ldm, w_s + wn * 16 * ldm, w_s + (cols + wn * 16) * ldm, ldm, ks, lane);
@@ -397,8 +404,8 @@ gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, in
 // are one cluster.  A warp takes a run of RUN tokens of a round of WARPS * RUN: a run is first composed to (product of
 // the a's, its sum from zero); from the runs' pairs every warp works out the state before its run, and walks it.  With
 // more than one share, every CTA first composes its whole share and reads the pairs of the shares before it from their
-// CTAs' shared memory.
-constexpr int SCAN_WARPS = 8, SCAN_RUN = 8, SCAN_MAX_SHARES = 8;
+// CTAs' shared memory; a share of one round keeps its terms in registers meanwhile.
+constexpr int SCAN_WARPS = 16, SCAN_RUN = 16, SCAN_MAX_SHARES = 8;
 template <typename T, bool CLUSTER>
 __global__ void __launch_bounds__(SCAN_WARPS * 32)
 channel_scan_kernel(const float* __restrict__ aux, GemmOut<T> proj, int cols, int y_off, int x_off,
@@ -484,7 +491,7 @@ channel_scan_kernel(const float* __restrict__ aux, GemmOut<T> proj, int cols, in
     }
     for (int t0 = begin, it = 0; t0 < end; t0 += ROUND, ++it) {
         const int t = t0 + warp * SCAN_RUN;
-        fetch(t);
+        if (!CLUSTER || end - begin > ROUND) fetch(t);
         float y[SCAN_RUN];
 #pragma unroll
         for (int j = 0; j < SCAN_RUN; ++j)
@@ -554,7 +561,7 @@ int launch_tensor(const GateScanArgs<__nv_bfloat16>& g, int parts, int all_singl
     if (base + per_wn > LIN_SMEM) return (int)cudaErrorInvalidValue;
     const int blocks = (groups + wn - 1) / wn;
     wn = (groups + blocks - 1) / blocks;                    // (as even as it gets)
-    return crane_launch(gate_scan_prep_many_kernel, dim3((g.n + MANY_TOKENS - 1) / MANY_TOKENS, parts, blocks), dim3(4 * wn * 32),
+    return crane_launch(gate_scan_prep_many_kernel, dim3((g.n + MANY_TOKENS - 1) / MANY_TOKENS, parts, blocks), dim3(MANY_TOKENS / 16 * wn * 32),
                         base + wn * per_wn, st, g, wn, pairs, vec);
 }
 int launch_tensor(const GateScanArgs<float>&, int, int, cudaStream_t) { return (int)cudaErrorInvalidValue; }
@@ -596,9 +603,9 @@ CRANE_API int crane_channel_scan(int dtype, const float* aux, const void* proj, 
     if (taps < 1 || taps > LIN_MAX_TAPS || C <= 0) return (int)cudaErrorInvalidValue;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
-        // shares of about four rounds: enough CTAs for a long prompt, no more than a cluster holds
+        // shares of a round: enough CTAs for a long prompt, no more than a cluster holds
         int shares = 1;
-        while (shares < SCAN_MAX_SHARES && n_tokens / n_entries >= shares * 4 * SCAN_WARPS * SCAN_RUN) shares *= 2;
+        while (shares < SCAN_MAX_SHARES && n_tokens / n_entries > shares * SCAN_WARPS * SCAN_RUN) shares *= 2;
         const dim3 grid(shares, (C + 31) / 32, n_entries), block(SCAN_WARPS * 32);
         if (shares == 1)
             return crane_launch(channel_scan_kernel<T, false>, grid, block, 0, st, aux, p, cols, y_off, x_off, cu_q, kv_len, slots,

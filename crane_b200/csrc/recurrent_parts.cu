@@ -204,6 +204,8 @@ decay_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_en
 // v, `by` CTAs a token.  M -> max(M + A, B) composes to maps of the same form, so a CTA takes 1,024 tokens at a time,
 // four a thread, and finds the M before every thread's four by a scan over lanes and warps; a thread goes token by
 // token, and a token's w is taken from the very M that the token before it left.
+// `logs` (or null): for entries of at least `logs_min` tokens, which walk in chunks, log w and log b go to
+// [n][2 H] there instead of w and b to aux, and nothing is copied.
 template <typename T, bool SINGLE>
 __global__ void __launch_bounds__(256)
 exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entry, const int* __restrict__ cu_q,
@@ -211,13 +213,14 @@ exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entr
                      float* __restrict__ state, long long slot_stride, long long m_off,
                      const float* __restrict__ bias_i, const float* __restrict__ bias_f, float cap, float q_scale,
                      float* __restrict__ aux, int aux_cols, int n_entries, int H, int d, int dv, int i_off, int f_off,
-                     int w_off, int gate_blocks, int by, int* err) {
+                     int w_off, int gate_blocks, int by, float* __restrict__ logs, int logs_min, int* err) {
     pdl_launch_dependents();
     pdl_wait();
     const int hd = H * d, hv = H * dv;
     if ((int)blockIdx.x >= gate_blocks) {
         const int t = ((int)blockIdx.x - gate_blocks) / by, part = ((int)blockIdx.x - gate_blocks) % by;
-        if (tok_entry[t] < 0) return;
+        const int te = tok_entry[t];
+        if (te < 0 || (logs != nullptr && cu_q[te + 1] - cu_q[te] >= logs_min)) return;
         const long long row = (long long)t * cols;
         float* out = aux + (long long)t * aux_cols;
         const int n = 2 * hd + hv;
@@ -239,11 +242,17 @@ exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entr
         li = cap * tanhf((zi + bi) / cap);
         lf = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
     };
+    bool as_logs = false;
     auto write = [&](long long t, int h, float li, float lf, float before, float m) {
         float* out = aux + t * aux_cols + w_off + h;
+        out[2 * H] = expf(-m);
+        if (as_logs) {
+            logs[t * 2 * H + h] = lf + before - m;
+            logs[t * 2 * H + H + h] = li - m;
+            return;
+        }
         out[0] = expf(lf + before - m);
         out[H] = expf(li - m);
-        out[2 * H] = expf(-m);
     };
     const int wid = SINGLE ? (int)(blockIdx.x * blockDim.x + threadIdx.x) : (int)blockIdx.x;
     if (wid >= n_entries * H) return;
@@ -258,6 +267,7 @@ exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entr
     float* kept = state + (long long)slot * slot_stride + m_off + h;
     float m0 = kv_len[e] > q_len ? *kept : 0.f;
     const float bi = bias_i[h], bf = bias_f[h];
+    as_logs = logs != nullptr && q_len >= logs_min;
     if (SINGLE) {
         float li, lf;
         const long long row = (long long)first * cols + h;
@@ -650,7 +660,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
                          const int* __restrict__ kv_len, const int* __restrict__ slots, int n_slots,
                          float* __restrict__ state, long long slot_stride, float* __restrict__ o_raw,
                          int H, int dk, int dv, int lanes_rt, int cols_per_block, int tile_tokens, int vec4,
-                         int walkers, float* __restrict__ den, int* err) {
+                         int walkers, float* __restrict__ den, int max_len, int* err) {
     constexpr bool DELTA = MODE == SCAN_DELTA, BONUS = MODE == SCAN_BONUS, GATED = MODE == SCAN_GATED;
     const int dvt = dv + (GATED ? 1 : 0);             // columns of the state
     extern __shared__ __align__(16) float tile[];     // two tiles of [tile_tokens][3 dk + cols + 2, to a multiple of 4]
@@ -658,7 +668,7 @@ matrix_state_scan_kernel(const float* __restrict__ aux, int aux_cols, int q_off,
     pdl_wait();
     const int e = blockIdx.x, h = blockIdx.y;
     const int first = cu_q[e], q_len = cu_q[e + 1] - first;
-    if (q_len <= 0) return;
+    if (q_len <= 0 || (max_len > 0 && q_len >= max_len)) return;      // (long entries may be another kernel's)
     const int slot = slots[e];
     if (slot < 0 || slot >= n_slots) {
         if (threadIdx.x == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
@@ -1029,8 +1039,8 @@ CRANE_API int crane_exp_gate_prep(int dtype, const void* proj, const float* proj
                                   const int* kv_len, const int* slots, int n_slots, float* state,
                                   long long slot_stride, long long m_off, const float* bias_i, const float* bias_f,
                                   float cap, float q_scale, float* aux, int aux_cols, int n_tokens, int n_entries,
-                                  int H, int d, int dv, int i_off, int f_off, int w_off, int all_single, int* err,
-                                  cudaStream_t st) {
+                                  int H, int d, int dv, int i_off, int f_off, int w_off, int all_single, float* logs,
+                                  int logs_min, int* err, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     const int gate_blocks = all_single ? (n_entries * H + 255) / 256 : n_entries * H;
     int by = (2 * H * d + H * dv + 511) / 512;               // with few tokens a token's columns spread over more CTAs
@@ -1038,9 +1048,11 @@ CRANE_API int crane_exp_gate_prep(int dtype, const void* proj, const float* proj
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
         const auto kern = all_single ? exp_gate_prep_kernel<T, true> : exp_gate_prep_kernel<T, false>;
-        return crane_launch(kern, dim3(gate_blocks + n_tokens * by), dim3(256), 0, st, p, cols,
+        // (one entry that walks in chunks, whatever padding of less than 64 rows the step has: nothing to copy)
+        const int copies = logs != nullptr && n_entries == 1 && n_tokens >= logs_min + 64 ? 0 : n_tokens * by;
+        return crane_launch(kern, dim3(gate_blocks + copies), dim3(256), 0, st, p, cols,
                             tok_entry, cu_q, kv_len, slots, n_slots, state, slot_stride, m_off, bias_i, bias_f, cap,
-                            q_scale, aux, aux_cols, n_entries, H, d, dv, i_off, f_off, w_off, gate_blocks, by, err);
+                            q_scale, aux, aux_cols, n_entries, H, d, dv, i_off, f_off, w_off, gate_blocks, by, logs, logs_min, err);
     });
 }
 
@@ -1145,7 +1157,7 @@ CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off,
                                       int beta_off, int w_vec, int mode, int qk_rep, const int* cu_q,
                                       const int* kv_len, const int* slots, int n_slots, float* state,
                                       long long slot_stride, float* o_raw, float* den, int n_entries, int H, int dk,
-                                      int dv, int* err, cudaStream_t st) {
+                                      int dv, int max_len, int* err, cudaStream_t st) {
     if (n_entries <= 0) return 0;
     int rows, lanes;
     if (crane_matrix_state_plan(dk, &rows, &lanes) || dv <= 0 || qk_rep <= 0 || mode < 0 || mode > 3 ||
@@ -1188,7 +1200,7 @@ CRANE_API int crane_matrix_state_scan(const float* aux, int aux_cols, int q_off,
     else kern = pick(integral_constant<int, 8>{}, integral_constant<int, 0>{});
     return crane_launch(kern, dim3(n_entries, H, blocks), dim3(walkers + 32), smem, st, aux, aux_cols, q_off, k_off,
                         v_off, w_off, beta_off, qk_rep, cu_q, kv_len, slots, n_slots, state, slot_stride,
-                        o_raw, H, dk, dv, lanes, cpb, tile_tokens, vec4, walkers, den, err);
+                        o_raw, H, dk, dv, lanes, cpb, tile_tokens, vec4, walkers, den, max_len, err);
 }
 
 CRANE_API int crane_head_norm_gate(int dtype, const float* o_raw, const void* proj, const float* proj_parts,

@@ -65,8 +65,10 @@ _SIGNATURES = {
                               P, P, I, I, I, I, I, I, P],
     "crane_decay_gate_prep": [I, P, P, I, L, I, P, P, P, I, F, F, P, I, I, I, I, I, P],
     "crane_matrix_state_plan": [I, P, P],
-    "crane_exp_gate_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, P, F, F, P, I, I, I, I, I, I, I, I, I, I, P, P],
-    "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, P, I, I, I, I, P, P],
+    "crane_exp_gate_prep": [I, P, P, I, L, I, P, P, P, P, I, P, L, L, P, P, F, F, P, I, I, I, I, I, I, I, I, I, I, P, I, P, P],
+    "crane_memory_chunks_supports": [I, I],
+    "crane_memory_chunks": [P, I, I, I, I, P, I, P, P, P, I, P, L, P, P, I, I, I, I, I, I, F, I, P, P],
+    "crane_matrix_state_scan": [P, I, I, I, I, I, I, I, I, I, P, P, P, I, P, L, P, P, I, I, I, I, I, P, P],
     "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, I, I, F, P, P, I, F, P, I, I, I, P],
     "crane_gate_scan_mma_most": [],
     "crane_gate_scan_prep": [I, P, P, I, L, I, I, I, P, P, P, P, I, P, L, L, L, P, P, I, P, I, P, P, P, P, P, I, I, I, I, P, P],
@@ -605,19 +607,38 @@ class Kernels:
     SCAN_MODES = {"plain": 0, "delta": 1, "bonus": 2, "gated": 3}
 
     def exp_gate_prep(self, proj: Act, cols, ctx, state, m_off, bias_i, bias_f, cap, q_scale, aux, H, d, dv, i_off,
-                      f_off, w_off, err, dtype) -> None:
+                      f_off, w_off, err, dtype, logs=None, logs_min: int = 0) -> None:
         """Rows [q | k | v | ...] of a merged projection, with the gates' columns at ``i_off`` and ``f_off``, ->
         ``aux`` rows [q * q_scale | k | v | ...] in 32-bit with the kept share, the new token's share and the
         floor of the normaliser (H each, one behind the other) at ``w_off``: i = cap tanh((z_i + bias_i) / cap),
         f = log sigmoid(cap tanh((z_f + bias_f) / cap)), M' = max(f + M, i), exp(f + M - M'), exp(i - M'), exp(-M').
-        M lives in ``state`` [slots, floats] at ``m_off`` (H floats)."""
+        M lives in ``state`` [slots, floats] at ``m_off`` (H floats).  ``logs`` float [n, 2 H]: for entries of at least
+        ``logs_min`` tokens, which ``memory_chunks`` walks, the logarithms of both shares go there and of ``aux`` only
+        the floors are written."""
         whole, parts, n_parts, stride = _split(proj)
         self._check(self.lib.crane_exp_gate_prep(
             _dt(dtype), whole, parts, n_parts, stride, int(cols), ctx.tok_entry.data_ptr(), ctx.cu_q.data_ptr(),
             ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0), int(m_off),
             bias_i.data_ptr(), bias_f.data_ptr(), float(cap), float(q_scale), aux.data_ptr(), aux.shape[1],
             aux.shape[0], ctx.kv_len.shape[0], H, d, dv, int(i_off), int(f_off), int(w_off),
-            1 if step_of_single_tokens(ctx) else 0, err.data_ptr(), self._stream(aux)), "exp_gate_prep")
+            1 if step_of_single_tokens(ctx) else 0, _ptr(logs), int(logs_min), err.data_ptr(), self._stream(aux)),
+            "exp_gate_prep")
+
+    def memory_chunks_takes(self, proj: Act, cols: int, dk: int, dv: int) -> bool:
+        """Whether ``memory_chunks`` takes heads of these sizes from this product."""
+        return (not isinstance(proj, Partials) and proj.dtype == torch.bfloat16 and cols % 8 == 0
+                and proj.data_ptr() % 16 == 0 and bool(self.lib.crane_memory_chunks_supports(int(dk), int(dv))))
+
+    def memory_chunks(self, proj, cols, offs, logs, ctx, state, o_raw, den, H, dk, dv, q_scale, min_len, err) -> None:
+        """``matrix_state_scan`` mode "gated" for the entries of at least ``min_len`` tokens, in chunks of 64 tokens on the
+        tensor cores, straight from the projection's rows (bfloat16; ``offs``: the columns of q, k, v) and the
+        logarithms of ``exp_gate_prep``."""
+        rows, lanes = self.matrix_state_plan(dk)
+        self._check(self.lib.crane_memory_chunks(
+            proj.data_ptr(), int(cols), *[int(o) for o in offs], logs.data_ptr(), logs.shape[1], ctx.cu_q.data_ptr(),
+            ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(), state.stride(0), o_raw.data_ptr(),
+            den.data_ptr(), ctx.kv_len.shape[0], H, dk, dv, rows, lanes, float(q_scale), int(min_len), err.data_ptr(),
+            self._stream(o_raw)), "memory_chunks")
 
     # ---- recurrences with a number per channel ---------------------------
     @dataclass
@@ -674,18 +695,18 @@ class Kernels:
             out.shape[1], err.data_ptr(), self._stream(out)), "channel_scan")
 
     def matrix_state_scan(self, aux, offs, w_vec: bool, mode, qk_rep: int, ctx, state, o_raw, H, dk, dv,
-                          err, den=None) -> None:
+                          err, den=None, max_len: int = 0) -> None:
         """The recurrence S <- diag(w) S; u = beta (v - S^T k) (``mode`` "delta" or True) or v ("plain" or
         False); S <- S + k u^T; o = S^T q; or (``mode`` "bonus") o = S^T q + beta v; S <- diag(w) S + k v^T; or (``mode`` "gated")
         S <- w S + beta k v^T, N <- w N + beta k, o = S^T q, ``den`` float [n, H] = N . q (N is column dv of S),
         over every entry's tokens, from and to ``state`` [slots, floats] (its leading H * rows * lanes * dv
-        floats).  ``offs``: columns of q, k, v, w, beta in ``aux``; ``o_raw`` float [n, H dv]."""
+        floats).  ``offs``: columns of q, k, v, w, beta in ``aux``; ``o_raw`` float [n, H dv].  ``max_len`` > 0: entries of that many tokens or more are left to another kernel."""
         self._check(self.lib.crane_matrix_state_scan(
             aux.data_ptr(), aux.shape[1], *[int(o) for o in offs], 1 if w_vec else 0,
             self.SCAN_MODES[mode] if isinstance(mode, str) else int(bool(mode)), int(qk_rep),
             ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
-            state.stride(0), o_raw.data_ptr(), _ptr(den), ctx.kv_len.shape[0], H, dk, dv, err.data_ptr(),
-            self._stream(o_raw)), "matrix_state_scan")
+            state.stride(0), o_raw.data_ptr(), _ptr(den), ctx.kv_len.shape[0], H, dk, dv, int(max_len),
+            err.data_ptr(), self._stream(o_raw)), "matrix_state_scan")
 
     def head_norm_gate(self, o_raw, proj: Act, cols, gate_off, tok_entry, norm_w, eps, out, H, dv,
                        sigmoid: bool = False, den=None, floor=None, den_eps: float = 0.0) -> None:

@@ -29,7 +29,9 @@ logarithms are capped, f = log sigmoid(.), kept in range by a running maximum M,
 
 State and everything between the projections and the output projection are 32-bit.  One kernel walks
 the recurrence for all of them (``matrix_state_scan``), prompts, portions and single tokens alike, so a
-state does not depend on how the tokens were cut.
+state does not depend on how the tokens were cut.  (``exponential_gates`` has a second one, for portions of a
+few tokens or more of large bfloat16 steps: ``memory_chunks``, 64 tokens at a time on the tensor cores, equal to
+the walk but for 32-bit rounding.)
 """
 from __future__ import annotations
 
@@ -342,6 +344,7 @@ class ExponentialGates(Part):
     kind = "mixer"
     state_graph_safe = True
     decode_bucket_safe = True
+    CHUNK_MIN = 24               # from this many tokens on an entry walks in chunks
     NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "i": "i", "f": "f", "i_bias": "i.b", "f_bias": "f.b",
              "norm": "norm"}
 
@@ -365,6 +368,8 @@ class ExponentialGates(Part):
         self.cap, self.eps, self.den_eps = float(a["gate_cap"]), float(a["norm_eps"]), float(a["den_eps"])
         # one product for everything that reads the block's input: [q | k | v | g | i | f]
         self.w_in = torch.cat([weights.pop(p + nm[n]) for n in ("q", "k", "v", "g", "i", "f")], dim=0).contiguous()
+        if self.w_in.shape[0] % 8:                    # rows of whole 16-byte pieces
+            self.w_in = torch.cat([self.w_in, self.w_in.new_zeros(-self.w_in.shape[0] % 8, self.w_in.shape[1])])
         self.cols = self.w_in.shape[0]
         self.bias_i, self.bias_f = weights[p + nm["i_bias"]], weights[p + nm["f_bias"]]
         self.norm_w, self.o_w = weights[p + nm["norm"]], weights[p + nm["o"]]
@@ -383,14 +388,23 @@ class ExponentialGates(Part):
         proj = rt.linear(h, self.w_in, None, "exp_gates_proj")
         aux = rt.ws.get("exp_gates_aux", n, self.aux_cols, torch.float32)
         gates = 2 * hd + 2 * hv
+        chunked = not rt.exact and not step_of_single_tokens(ctx) and k.memory_chunks_takes(proj, self.cols, d, m)
+        logs = rt.ws.get("exp_gates_logs", n, 2 * H, torch.float32) if chunked else None
         k.exp_gate_prep(proj, self.cols, ctx, cache.state, self.max_off, self.bias_i, self.bias_f, self.cap, d ** -0.5,
-                        aux, H, d, m, gates, gates + H, self.w_at, rt.err, rt.dtype)
+                        aux, H, d, m, gates, gates + H, self.w_at, rt.err, rt.dtype, logs=logs, logs_min=self.CHUNK_MIN)
         o_raw = rt.ws.get("exp_gates_o_raw", n, hv, torch.float32)
         den = rt.ws.get("exp_gates_den", n, H, torch.float32)
-        k.matrix_state_scan(aux, (0, hd, 2 * hd, self.w_at, self.w_at + H), False, "gated", 1, ctx, cache.state, o_raw, H, d,
-                            m, rt.err, den=den)
+        if chunked:
+            k.memory_chunks(proj, self.cols, (0, hd, 2 * hd), logs, ctx, cache.state, o_raw, den, H, d, m, d ** -0.5,
+                            self.CHUNK_MIN, rt.err)
+            rt.launches += 1
+        # (one entry of a step that is padded by less than 64 rows walks in chunks whole)
+        if not chunked or ctx.kv_len.shape[0] > 1 or n < self.CHUNK_MIN + 64:
+            k.matrix_state_scan(aux, (0, hd, 2 * hd, self.w_at, self.w_at + H), False, "gated", 1, ctx, cache.state, o_raw,
+                                H, d, m, rt.err, den=den, max_len=self.CHUNK_MIN if chunked else 0)
+            rt.launches += 1
         o = rt.ws.get("exp_gates_o", n, hv, rt.dtype)
         k.head_norm_gate(o_raw, proj, self.cols, 2 * hd + hv, ctx.tok_entry, self.norm_w, self.eps, o, H, m, sigmoid=True,
                          den=den, floor=aux[:, self.w_at + 2 * H:], den_eps=self.den_eps)
-        rt.launches += 3
+        rt.launches += 2
         return rt.linear(o, self.o_w, None, "exp_gates_out", hold=hold)

@@ -256,6 +256,61 @@ def test_exponential_gates_over_steps(K, dtype, H, d, dv, cap, plan, lens):
     assert int(err.item()) == 0
 
 
+@pytest.mark.parametrize("H, d, dv, lens", [(2, 16, 8, [64]), (3, 32, 24, [63, 1, 65, 23, 24, 200]), (1, 64, 64, [300]), (2, 128, 40, [130, 64]),
+                                            (1, 256, 16, [97]), (1, 144, 48, [200, 30]), (4, 48, 136, [3, 70])])
+@pytest.mark.parametrize("spread", [1.0, 6.0])
+def test_chunks_of_the_matrix_memory_equal_the_walk(K, H, d, dv, lens, spread):
+    """Portions in chunks of 64 tokens against the walk token by token, read-outs and normalisers in 32-bit and the
+    states they leave, for fresh and continued requests; entries below the limit are left to the walk.  ``spread``
+    1: forget gates near 1, so the first token shows in the last; 6: gates from one end to the other."""
+    rng = np.random.default_rng(d + dv)
+    hd, hv = H * d, H * dv
+    cols = -(-(2 * hd + 2 * hv + 2 * H) // 8) * 8
+    g_off = 2 * hd + 2 * hv
+    n, w_at = sum(lens), 2 * hd + hv
+    x = rng.standard_normal((n, cols))
+    x[:, g_off:g_off + H] *= spread
+    x[:, g_off + H:g_off + 2 * H] = x[:, g_off + H:g_off + 2 * H] * spread * 1.5 + (7.0 if spread == 1.0 else 2.0)
+    cu = np.concatenate([[0], np.cumsum(lens)])
+    x[cu[:-1], 2 * hd:2 * hd + hv] *= 8.0
+    x = _dev(x, torch.bfloat16)
+    start = [0 if i % 2 == 0 else 77 for i in range(len(lens))]
+    ctx = SimpleNamespace(cu_q=_i32(cu), kv_len=_i32(np.asarray(lens) + start), slots=_i32(rng.permutation(len(lens))),
+                          tok_entry=_i32(np.repeat(np.arange(len(lens)), lens)))
+    rows_, lanes = K.matrix_state_plan(d)
+    m_off = H * rows_ * lanes * (dv + 1)
+    seed = torch.randn(len(lens), m_off + H + 1, device=DEV)
+    if rows_ * lanes > d:                                    # rows past the keys are zeros and stay so
+        st = seed[:, :m_off].view(len(lens), H, rows_, dv + 1, lanes)
+        r = torch.arange(lanes, device=DEV)[None] * rows_ + torch.arange(rows_, device=DEV)[:, None]
+        st *= (r < d)[None, None, :, None, :]
+    err, bias = _err(), _dev(np.zeros(H))
+    least = 24
+    got = {}
+    for way in ("walk", "chunks"):
+        state = seed.clone()
+        aux = torch.full((n, -(-(w_at + 3 * H) // 4) * 4), 5.0, device=DEV)
+        o_raw, den = torch.full((n, hv), 5.0, device=DEV), torch.full((n, H), 5.0, device=DEV)
+        logs = torch.full((n, 2 * H), 5.0, device=DEV) if way == "chunks" else None
+        K.exp_gate_prep(x, cols, ctx, state, m_off, bias, bias, 15.0, d ** -0.5, aux, H, d, dv, g_off, g_off + H, w_at, err, torch.bfloat16,
+                        logs=logs, logs_min=least)
+        if logs is not None:
+            assert K.memory_chunks_takes(x, cols, d, dv)
+            K.memory_chunks(x, cols, (0, hd, 2 * hd), logs, ctx, state, o_raw, den, H, d, dv, d ** -0.5, least, err)
+            short = np.repeat(np.asarray(lens) < least, lens)
+            assert (o_raw[torch.from_numpy(short).to(DEV)] == 5.0).all()
+        if logs is None or min(lens) < least:
+            K.matrix_state_scan(aux, (0, hd, 2 * hd, w_at, w_at + H), False, "gated", 1, ctx, state, o_raw, H, d, dv, err, den=den,
+                                max_len=least if logs is not None else 0)
+        got[way] = (_np(o_raw), _np(den), _np(state), _np(aux)[:, w_at + 2 * H:w_at + 3 * H])
+    for a, b, what in zip(got["walk"], got["chunks"], ("read-outs", "normalisers", "states", "floors")):
+        assert np.abs(a - b).max() < 1e-4 * np.abs(a).max(), what
+    o, den = got["walk"][:2]
+    rms = lambda a: np.sqrt((a.reshape(n, H, -1) ** 2).mean(axis=(1, 2)))          # and token by token
+    assert (rms(o - got["chunks"][0]) < 2e-3 * rms(o) + 1e-5 * rms(o).max()).all()
+    assert int(err.item()) == 0
+
+
 @pytest.mark.parametrize("n", [1, 3, 31, 128, 129, 700])
 def test_exponential_gates_alone(K, n):
     """The three numbers per token against the walk in NumPy, from a maximum the request brings along, whole and

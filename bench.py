@@ -1573,6 +1573,13 @@ def mufalix_kernel_table(fcfg, pk, tokens, batch, context):
                 fl(win), t_l, read(0), fl(0))
             add(f"attention, sinks, gate, no window ({kind})", "attention with a sink (Vodelix)", t_of(lambda: at(0, **own)), read(0) + gb,
                 fl(0), t_l, read(0), fl(0))
+            tc = lambda w_, **kw: K.prefill_attention_tc(q, o, k_pool, v_pool, cu_d, kv_d, table, ps, -(-q_len // 128), H, G, d, w_, d ** -0.5, err,
+                                                         **kw)
+            t_l = t_of(lambda: tc(0))
+            add(f"tcgen05 attention, window of {win}, sinks, gate ({kind})", "tcgen05 attention (Hunyuan)", t_of(lambda: tc(win, **own)),
+                read(win) + gb, fl(win), t_l, read(0), fl(0))
+            add(f"tcgen05 attention, sinks, gate, no window ({kind})", "tcgen05 attention (Hunyuan)", t_of(lambda: tc(0, **own)), read(0) + gb,
+                fl(0), t_l, read(0), fl(0))
         else:
             splits = K.decode_splits(n_req, G, rt.num_sms)
             po, pml = torch.empty(n_req * H * splits * d, device=dev), torch.empty(n_req * H * splits * 2, device=dev)

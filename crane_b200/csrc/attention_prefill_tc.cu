@@ -189,9 +189,30 @@ struct Params {
     int max_blocks, num_pages, page_size, n_entries, nq, nkv, window;
     int skip_single;             // entries of one token have no tile here (the decode kernel takes them)
     float scale_log2;
+    const float* sinks;          // [nq] or null: a candidate of that score without a value joins every softmax of its head
+    GemmOut<__nv_bfloat16> gate; // gate_ld > 0: the result times the sigmoid of columns gate_off + h D .. of the row
+    int gate_ld, gate_off;
     int* err;
 };
 
+// The sink's part of a row's sum (scores relative to m_ref, in units of log2 e).
+__device__ __forceinline__ float sink_term(const Params& p, int h, float m_ref) {
+    return p.sinks != nullptr ? exp2f(p.sinks[h] * 1.4426950408889634f - m_ref) : 0.f;
+}
+// 32 neighbouring results of a row times their gates.
+__device__ __forceinline__ void gate_row(const Params& p, long long row, int h, int c0, uint32_t (&v)[32]) {
+    if (p.gate_ld <= 0) return;
+    const long long at = row * p.gate_ld + p.gate_off + h * D + c0;
+#pragma unroll
+    for (int i = 0; i < 32; i += 2) {
+        const float2 z = p.gate.load2(at + i);
+        v[i] = __float_as_uint(__fdividef(__uint_as_float(v[i]), 1.f + __expf(-z.x)));
+        v[i + 1] = __float_as_uint(__fdividef(__uint_as_float(v[i + 1]), 1.f + __expf(-z.y)));
+    }
+}
+
+// MODS: the instantiation that knows sinks and gates (code that the serving kernel never runs would cost it registers).
+template <bool MODS>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const Params p) {
@@ -486,6 +507,10 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
             for (int o = 0; o < SPLIT; ++o) l += xch[o * BQ + r];            // the same order for every thread
         }
+        if (MODS) {
+            pdl_wait();                                     // (the gate is an earlier kernel's)
+            l += sink_term(p, h, m_ref);
+        }
         const float inv = l > 0.f ? 1.f / l : 0.f;
         const bool store = r_begin + r < r_end;
         __nv_bfloat16* orow = p.out + ((long long)(row0 + r_begin + r) * p.nq + h) * D;
@@ -495,6 +520,7 @@ prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             tmem_ld32(tmem_o + lane_addr + c0, v);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (store) {
+                if (MODS) gate_row(p, row0 + r_begin + r, h, c0, v);
 #pragma unroll
                 for (int i = 0; i < 32; i += 8) {
                     uint4 w;
@@ -545,6 +571,7 @@ done:
 // two softmax warpgroups take registers over from the first one (setmaxnreg).
 constexpr int PAIR_THREADS = 384;
 
+template <bool MODS>
 __global__ void __launch_bounds__(PAIR_THREADS, 1)
 prefill_attn_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const Params p) {
@@ -794,6 +821,10 @@ prefill_attn_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // ---- epilogue: O / l ----
             if (!mbar_wait(smem_u32(o_done), 0, abort_flag)) goto done;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (MODS) {
+                pdl_wait();                                 // (the gate is an earlier kernel's)
+                l += sink_term(p, h_a + x, m_ref);
+            }
             const float inv = l > 0.f ? 1.f / l : 0.f;
             const bool store = r_begin + r < r_end;
             __nv_bfloat16* orow = p.out + ((long long)(row0 + r_begin + r) * p.nq + h_a + x) * D;
@@ -803,6 +834,7 @@ prefill_attn_tc_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 tmem_ld32(tmem_ox + c0, o);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 if (store) {
+                    if (MODS) gate_row(p, row0 + r_begin + r, h_a + x, c0, o);
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
                         uint4 w;
@@ -878,14 +910,19 @@ CRANE_API int crane_prefill_attention_tc_supports(int d, int nq, int nkv, int pa
 }
 
 // total_q_tiles: sum over the entries of ceil(q_len / 128) (or more).  q is [n_tokens, nq * 128].
-// skip_single != 0: entries of exactly one token are left out and count no tile.
+// skip_single != 0: entries of exactly one token are left out and count no tile.  sinks and the gate as in
+// crane_paged_prefill_attention.
 CRANE_API int crane_prefill_attention_tc(const void* q, void* out, const void* k_pool, const void* v_pool,
                                          const int* cu_q, const int* kv_len, const int* block_table,
                                          int max_blocks, int num_pages, int page_size, int n_entries,
                                          int n_tokens, int total_q_tiles, int nq, int nkv, int d, int window,
-                                         float scale, int skip_single, int* err, cudaStream_t st) {
+                                         float scale, int skip_single, const float* sinks, const void* gate,
+                                         const float* gate_parts, int gate_n_parts, long long gate_stride,
+                                         int gate_ld, int gate_off, int* err, cudaStream_t st) {
     if (n_entries <= 0 || total_q_tiles <= 0) return 0;
-    if (!crane_prefill_attention_tc_supports(d, nq, nkv, page_size)) return (int)cudaErrorInvalidValue;
+    if (!crane_prefill_attention_tc_supports(d, nq, nkv, page_size) ||
+        (gate_ld > 0 && (((gate_ld | gate_off) & 1) || (gate_stride & 1))))
+        return (int)cudaErrorInvalidValue;
     CUtensorMap mq, mk, mv;
     const long long pool_rows = (long long)num_pages * nkv * page_size;
     if (!make_map(&mq, q, n_tokens, (long long)nq * D, BQ) || !make_map(&mk, k_pool, pool_rows, D, page_size < BKV ? page_size : BKV) ||
@@ -895,12 +932,15 @@ CRANE_API int crane_prefill_attention_tc(const void* q, void* out, const void* k
     p.out = (__nv_bfloat16*)out; p.cu_q = cu_q; p.kv_len = kv_len; p.block_table = block_table;
     p.max_blocks = max_blocks; p.num_pages = num_pages; p.page_size = page_size; p.n_entries = n_entries;
     p.nq = nq; p.nkv = nkv; p.window = window; p.skip_single = skip_single; p.scale_log2 = scale * 1.4426950408889634f; p.err = err;
+    p.sinks = sinks; p.gate_ld = gate_ld; p.gate_off = gate_off;
+    p.gate = GemmOut<__nv_bfloat16>{(const __nv_bfloat16*)gate, gate_parts, gate_n_parts, gate_stride};
     // Two heads of a kv head per CTA (every K and V tile serves both, the heads take turns on the
     // tensor cores) where there are CTAs enough to keep every SM busy to the end even so.  Measured
     // at 16 / 4 heads, one head against two per CTA: a whole prompt of 4,096 tokens 88 against 78 us, of
     // 8,192 the same (265 us, 0.63 of the bf16 peak), 2,048 rows behind 30,000 cached keys 562 against
     // 519 us; below that the coarser grain loses (2,048 tokens 29 against 44 us; 512 rows behind 8,192
     // keys, 64 CTAs against 32, 81 against 143 us).
+    const bool mods = sinks != nullptr || gate_ld > 0;
     int sms = 0, dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -909,22 +949,26 @@ CRANE_API int crane_prefill_attention_tc(const void* q, void* out, const void* k
         constexpr size_t pair_smem = 6 * TILE_BYTES + 14 * 8 + 16 + 1024;
         static bool pair_configured = false;
         if (!pair_configured) {
-            if (cudaFuncSetAttribute(prefill_attn_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+            if (cudaFuncSetAttribute(prefill_attn_tc_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                     (int)pair_smem) != cudaSuccess ||
+                cudaFuncSetAttribute(prefill_attn_tc_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                      (int)pair_smem) != cudaSuccess)
                 return (int)cudaGetLastError();
             pair_configured = true;
         }
-        return crane_launch(prefill_attn_tc_pair_kernel, dim3(nq / 2, total_q_tiles), dim3(PAIR_THREADS), pair_smem,
+        return crane_launch(mods ? prefill_attn_tc_pair_kernel<true> : prefill_attn_tc_pair_kernel<false>, dim3(nq / 2, total_q_tiles), dim3(PAIR_THREADS), pair_smem,
                             st, mq, mk, mv, p);
     }
     constexpr size_t smem = 5 * TILE_BYTES + 18 * 8 + 2 * SPLIT * BQ * 4 + 16 + 1024;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(prefill_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        if (cudaFuncSetAttribute(prefill_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                 (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(prefill_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)smem) != cudaSuccess)
             return (int)cudaGetLastError();
         configured = true;
     }
-    return crane_launch(prefill_attn_tc_kernel, dim3(nq, total_q_tiles), dim3(NUM_THREADS), smem, st, mq, mk,
+    return crane_launch(mods ? prefill_attn_tc_kernel<true> : prefill_attn_tc_kernel<false>, dim3(nq, total_q_tiles), dim3(NUM_THREADS), smem, st, mq, mk,
                         mv, p);
 }

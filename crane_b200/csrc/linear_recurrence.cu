@@ -6,8 +6,10 @@
 //     log a = -8 r softplus(lam);   S <- a S + sqrt(1 - a^2) i u;   out = S gelu_tanh(y)
 //
 // x and y are columns of one merged projection.  `gate_scan_prep` forms, of every token and channel, a and
-// sqrt(1 - a^2) i u in 32-bit; `channel_scan` walks each request's tokens.  In a step of single tokens the first
-// kernel does the walk's one token as well and there is no second one.
+// b = sqrt(1 - a^2) i u in 32-bit, and of a tile of tokens what its walk comes to: A_t and B_t with S_t = A_t S + B_t for
+// the state S before the tile, A_t = 0 from a portion's first token on (the slot's state is in its B_t).  `channel_scan`
+// works out the states before the tiles from the tiles' last rows, and the read-outs.  In a step of single tokens the
+// first kernel does the walk's one token as well and there is no second one.
 // The products with the square matrices: on the bfloat16 path warp-level MMA, u as the sum of two bfloat16 numbers
 // (its rounding and what that leaves), so that the gates see u with 16 bits of mantissa; on the 32-bit path, and
 // for parts wider than the tensor-core kernel takes, FP32 cores, inner dimension in order.
@@ -46,7 +48,7 @@ struct GateScanArgs {
     const T* gates;                            // MMA: [2][C][ld] (R's rows, then I's; ld = part width, zero-filled to 16);
                                                // FP32 cores: [2][B][width][width], columns (outputs) side by side
     const float *rb, *ib, *sp;                 // [C]; sp = softplus(lam)
-    float* aux;                                // [n][2 C]: a, then the addend
+    float* aux;                                // [n][2 C]: A, then B
     T* out;                                    // [n][C] (single tokens)
     int n, C, width, ld;
     int* err;
@@ -96,23 +98,25 @@ __device__ __forceinline__ void gate_scan_terms(const GateScanArgs<T>& g, int c,
     a = expf(log_a);
     add = sqrtf(one_minus_exp(2.f * log_a, a * a)) * i * u;
 }
-// Token t, channel c: to what the walk needs, or, SINGLE, through the walk.
-template <typename T, bool SINGLE>
-__device__ __forceinline__ void gate_scan_finish(const GateScanArgs<T>& g, const TileToken& k, int t, int c, float zr,
-                                                 float zi, float u) {
+// A portion's first token: the slot's state joins the addend, and what came before counts no more.
+template <typename T>
+__device__ __forceinline__ void gate_scan_open(const GateScanArgs<T>& g, const TileToken& k, int c, float& a, float& add) {
+    if (k.place != 0) return;
+    if (k.start > 0) add = fmaf(g.state[(long long)k.slot * g.slot_stride + g.s_off + c], a, add);
+    a = 0.f;
+}
+// A single token, channel c: the walk, the read-out, the slot.
+template <typename T>
+__device__ __forceinline__ void gate_scan_single(const GateScanArgs<T>& g, const TileToken& k, int t, int c, float zr, float zi,
+                                                 float u) {
+    const float x = g.proj.load((long long)t * g.cols + g.x_off + c), y = g.proj.load((long long)t * g.cols + g.y_off + c);
+    float* slot = g.state + (long long)k.slot * g.slot_stride;
     float a, add;
     gate_scan_terms(g, c, zr, zi, u, a, add);
-    if (!SINGLE) {
-        float* o = g.aux + (long long)t * 2 * g.C;
-        o[c] = a;
-        o[g.C + c] = add;
-        return;
-    }
-    float* slot = g.state + (long long)k.slot * g.slot_stride;
     const float s = fmaf(k.start > 0 ? slot[g.s_off + c] : 0.f, a, add);
     slot[g.s_off + c] = s;
-    slot[g.ring_off + (long long)(k.start % g.taps) * g.C + c] = g.proj.load((long long)t * g.cols + g.x_off + c);
-    g.out[(long long)t * g.C + c] = from_f32<T>(s * lin_gelu_tanh(g.proj.load((long long)t * g.cols + g.y_off + c)));
+    slot[g.ring_off + (long long)(k.start % g.taps) * g.C + c] = x;
+    g.out[(long long)t * g.C + c] = from_f32<T>(s * lin_gelu_tanh(y));
 }
 
 // ------------------------------------------------------ FP32 cores
@@ -150,10 +154,24 @@ gate_scan_prep_simt_kernel(const GateScanArgs<T> g) {
             zi[tt] = fmaf(b, u, zi[tt]);
         }
     }
+    const int cc = part * g.width + c;
+    float A = 1.f, B = 0.f;
 #pragma unroll
-    for (int tt = 0; tt < SIMT_TOKENS; ++tt)
-        if (tok[tt].entry >= 0)
-            gate_scan_finish<T, SINGLE>(g, tok[tt], t0 + tt, part * g.width + c, zr[tt], zi[tt], lin_us[tt * g.width + c]);
+    for (int tt = 0; tt < SIMT_TOKENS; ++tt) {
+        if (tok[tt].entry < 0) continue;
+        if (SINGLE) {
+            gate_scan_single(g, tok[tt], t0 + tt, cc, zr[tt], zi[tt], lin_us[tt * g.width + c]);
+            continue;
+        }
+        float a, b;
+        gate_scan_terms(g, cc, zr[tt], zi[tt], lin_us[tt * g.width + c], a, b);
+        gate_scan_open(g, tok[tt], cc, a, b);
+        A *= a;
+        B = fmaf(a, B, b);
+        float* o = g.aux + (long long)(t0 + tt) * 2 * g.C + cc;
+        o[0] = A;
+        o[g.C] = B;
+    }
 }
 
 // ------------------------------------------------------ tensor cores
@@ -247,10 +265,11 @@ gate_scan_prep_few_kernel(const GateScanArgs<__nv_bfloat16> g, int pairs) {
     const int t0 = blockIdx.x * 16, c0 = blockIdx.z * FEW_COLS, base_c = blockIdx.y * g.width;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_launch_dependents();
-    load_gates(g, w_s, FEW_COLS, base_c, c0);               // the weights depend on no earlier kernel
-    pdl_wait();
+    // (the weights depend on no earlier kernel, and what the step's entries are was written before the step began)
     if (threadIdx.x < 16) tok[threadIdx.x] = tile_token(g, t0 + threadIdx.x);
+    load_gates(g, w_s, FEW_COLS, base_c, c0);
     __syncthreads();
+    pdl_wait();
     const int half = g.ld >> 1;
 #pragma unroll 2
     for (int x = threadIdx.x; x < 16 * half; x += blockDim.x) {
@@ -289,7 +308,28 @@ gate_scan_prep_few_kernel(const GateScanArgs<__nv_bfloat16> g, int pairs) {
 #pragma unroll
         for (int w = 0; w < FEW_SPLIT; ++w) zr += sums[w][0][tt][cc], zi += sums[w][1][tt][cc];
         const float u = __bfloat162float(u_hi[tt * ldm + c]) + __bfloat162float(u_lo[tt * ldm + c]);
-        gate_scan_finish<__nv_bfloat16, SINGLE>(g, tok[tt], t0 + tt, base_c + c, zr, zi, u);
+        if (SINGLE) {
+            gate_scan_single(g, tok[tt], t0 + tt, base_c + c, zr, zi, u);
+            continue;
+        }
+        float a, b;
+        gate_scan_terms(g, base_c + c, zr, zi, u, a, b);
+        gate_scan_open(g, tok[tt], base_c + c, a, b);
+        sums[0][0][tt][cc] = a;                             // (read by this thread alone)
+        sums[0][1][tt][cc] = b;
+    }
+    if (SINGLE) return;
+    __syncthreads();
+    if (threadIdx.x < FEW_COLS && c0 + threadIdx.x < g.width) {
+        float A = 1.f, B = 0.f;
+        for (int tt = 0; tt < 16 && tok[tt].entry >= 0; ++tt) {
+            const float a = sums[0][0][tt][threadIdx.x];
+            A *= a;
+            B = fmaf(a, B, sums[0][1][tt][threadIdx.x]);
+            float* o = g.aux + (long long)(t0 + tt) * 2 * g.C + base_c + c0 + threadIdx.x;
+            o[0] = A;
+            o[g.C] = B;
+        }
     }
 }
 
@@ -299,7 +339,12 @@ gate_scan_prep_few_kernel(const GateScanArgs<__nv_bfloat16> g, int pairs) {
 // convolutions of more taps go one by one.  Grid (token tiles, parts, column blocks).  Shared memory: inputs
 // [51][ld], u [2][48][ld + 8], both matrices' rows [2][wn * 16][ld + 8].
 constexpr int MANY_TOKENS = 48, MANY_RUN = 8, MANY_MAX_WN = 5;
-__global__ void __launch_bounds__(MANY_TOKENS / 16 * MANY_MAX_WN * 32)
+// Bytes before the weights: the inputs and u, later the tile's terms in their place.
+__host__ __device__ constexpr int many_front(int ld, int cols) {
+    const int u = ((MANY_TOKENS + 3) * ld + 2 * MANY_TOKENS * (ld + 8)) * 2, terms = 2 * MANY_TOKENS * (cols + 1) * 4;
+    return ((u > terms ? u : terms) + 15) / 16 * 16;
+}
+__global__ void __launch_bounds__(MANY_TOKENS / 16 * MANY_MAX_WN * 32, 2)
 gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, int pairs, int vec) {
     extern __shared__ __align__(16) unsigned char lin_smem[];
     __shared__ TileToken tok[MANY_TOKENS];
@@ -307,13 +352,13 @@ gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, in
     __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(lin_smem);
     __nv_bfloat16* u_hi = xs + (MANY_TOKENS + 3) * g.ld;
     __nv_bfloat16* u_lo = u_hi + MANY_TOKENS * ldm;
-    __nv_bfloat16* w_s = u_lo + MANY_TOKENS * ldm;
+    __nv_bfloat16* w_s = reinterpret_cast<__nv_bfloat16*>(lin_smem + many_front(g.ld, cols));
     const int t0 = blockIdx.x * MANY_TOKENS, c0 = blockIdx.z * cols, base_c = blockIdx.y * width;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_launch_dependents();
+    if (threadIdx.x < MANY_TOKENS) tok[threadIdx.x] = tile_token(g, t0 + threadIdx.x);
     load_gates(g, w_s, cols, base_c, c0);
     pdl_wait();
-    if (threadIdx.x < MANY_TOKENS) tok[threadIdx.x] = tile_token(g, t0 + threadIdx.x);
     if (vec) {                                              // rows of 16-byte pieces
         const int pieces = g.ld >> 3;
         for (int x = threadIdx.x; x < (MANY_TOKENS + 3) * pieces; x += blockDim.x) {
@@ -376,149 +421,153 @@ gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, in
     float zr[2][4] = {}, zi[2][4] = {};
     for (int ks = 0; ks < (g.ld >> 4); ++ks)
         gate_mma_step(zr, zi, u_hi + wm * 16 * ldm, u_lo + wm * 16 * ldm, w_s + wn * 16 * ldm, w_s + (cols + wn * 16) * ldm, ldm, ks, lane);
+    // the terms of the tile, [48][cols + 1] each, in the place of the inputs and of u
+    const int ldt = cols + 1;
+    float* ta = reinterpret_cast<float*>(lin_smem);
+    float* tb = ta + MANY_TOKENS * ldt;
 #pragma unroll
-    for (int b = 0; b < 2; ++b) {
-        const int c = c0 + wn * 16 + b * 8 + 2 * (lane & 3);
+    for (int b = 0; b < 2; ++b)
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            const int tt = wm * 16 + (lane >> 2) + h * 8;
-            if (c >= width || tok[tt].entry < 0) continue;
-            const float2 uh = ld2(u_hi + tt * ldm + c), ul = ld2(u_lo + tt * ldm + c);
-            float a0, b0, a1, b1;
-            gate_scan_terms(g, base_c + c, zr[b][2 * h], zi[b][2 * h], uh.x + ul.x, a0, b0);
-            float* o = g.aux + (long long)(t0 + tt) * 2 * g.C + base_c + c;
-            if (c + 1 < width) {
-                gate_scan_terms(g, base_c + c + 1, zr[b][2 * h + 1], zi[b][2 * h + 1], uh.y + ul.y, a1, b1);
-                if (pairs) { st2(o, a0, a1); st2(o + g.C, b0, b1); }
-                else { o[0] = a0; o[1] = a1; o[g.C] = b0; o[g.C + 1] = b1; }
-            } else {
-                o[0] = a0;
-                o[g.C] = b0;
+        for (int h = 0; h < 4; ++h) {
+            const int tt = wm * 16 + (lane >> 2) + (h >> 1) * 8, c = c0 + wn * 16 + b * 8 + 2 * (lane & 3) + (h & 1);
+            float a = 1.f, add = 0.f;                       // (rows of no entry and columns behind the part)
+            if (c < width && tok[tt].entry >= 0) {
+                const float u = __bfloat162float(u_hi[tt * ldm + c]) + __bfloat162float(u_lo[tt * ldm + c]);
+                gate_scan_terms(g, base_c + c, zr[b][h], zi[b][h], u, a, add);
+                gate_scan_open(g, tok[tt], base_c + c, a, add);
+            }
+            zr[b][h] = a;
+            zi[b][h] = add;
+        }
+    __syncthreads();
+#pragma unroll
+    for (int b = 0; b < 2; ++b)
+#pragma unroll
+        for (int h = 0; h < 4; ++h) {
+            const int tt = wm * 16 + (lane >> 2) + (h >> 1) * 8, cc = wn * 16 + b * 8 + 2 * (lane & 3) + (h & 1);
+            ta[tt * ldt + cc] = zr[b][h];
+            tb[tt * ldt + cc] = zi[b][h];
+        }
+    __syncthreads();
+    // a thread walks a run of 8 tokens of one column (there are as many runs as threads), the runs meet in shared memory
+    {
+        const int cc = threadIdx.x % cols, run = threadIdx.x / cols, first = run * MANY_RUN;
+        float A = 1.f, B = 0.f;
+#pragma unroll
+        for (int j = 0; j < MANY_RUN; ++j) {
+            const float a = ta[(first + j) * ldt + cc];
+            A *= a;
+            B = fmaf(a, B, tb[(first + j) * ldt + cc]);
+        }
+        float2* ends = reinterpret_cast<float2*>(w_s);      // [runs][cols]; the weights have been read
+        ends[run * cols + cc] = make_float2(A, B);
+        __syncthreads();
+        A = 1.f, B = 0.f;
+        for (int r = 0; r < run; ++r) {
+            const float2 p = ends[r * cols + cc];
+            A *= p.x;
+            B = fmaf(p.x, B, p.y);
+        }
+        const int c = c0 + cc;
+        float* o = g.aux + (long long)(t0 + first) * 2 * g.C + base_c + c;
+#pragma unroll
+        for (int j = 0; j < MANY_RUN; ++j, o += 2 * g.C) {
+            const float a = ta[(first + j) * ldt + cc];
+            A *= a;
+            B = fmaf(a, B, tb[(first + j) * ldt + cc]);
+            if (c < width && tok[first + j].entry >= 0) {
+                o[0] = A;
+                o[g.C] = B;
             }
         }
     }
 }
 
 // ------------------------------------------------------ the walk
-// Grid (share of the entry's tokens, blocks of 32 channels, entries); a lane per channel.  The CTAs of an entry's shares
-// are one cluster.  A warp takes a run of RUN tokens of a round of WARPS * RUN: a run is first composed to (product of
-// the a's, its sum from zero); from the runs' pairs every warp works out the state before its run, and walks it.  With
-// more than one share, every CTA first composes its whole share and reads the pairs of the shares before it from their
-// CTAs' shared memory; a share of one round keeps its terms in registers meanwhile.
-constexpr int SCAN_WARPS = 16, SCAN_RUN = 16, SCAN_MAX_SHARES = 8;
-template <typename T, bool CLUSTER>
-__global__ void __launch_bounds__(SCAN_WARPS * 32)
+// Grid (tiles of `tile` tokens, the preparation's; blocks of 64 channels); 2 channels a lane, APPLY_ROWS warps that take a
+// token each in turn.  The state before the tile is what the tiles before it come to, from the one in which the request
+// of the tile's first token began: their last rows, a share of them per warp, put together in shared memory.
+constexpr int APPLY_ROWS = 8;
+template <typename T>
+__global__ void __launch_bounds__(APPLY_ROWS * 32)
 channel_scan_kernel(const float* __restrict__ aux, GemmOut<T> proj, int cols, int y_off, int x_off,
-                    const int* __restrict__ cu_q, const int* __restrict__ kv_len, const int* __restrict__ slots,
-                    int n_slots, float* __restrict__ state, long long slot_stride, long long s_off, long long ring_off,
-                    int taps, T* __restrict__ out, int C, int* err) {
-    __shared__ float2 pair[2][SCAN_WARPS][32];
-    __shared__ float2 whole[32];
+                    const int* __restrict__ tok_entry, const int* __restrict__ cu_q, const int* __restrict__ kv_len,
+                    const int* __restrict__ slots, int n_slots, float* __restrict__ state, long long slot_stride,
+                    long long s_off, long long ring_off, int taps, T* __restrict__ out, int n, int C, int tile, int pairs,
+                    int* err) {
+    __shared__ float4 part[APPLY_ROWS][32];
     pdl_launch_dependents();
+    const int tile_id = blockIdx.x, t0 = tile_id * tile;
+    const int e0 = tok_entry[t0];
+    if (e0 < 0) return;                                     // nothing but padding from here on
+    const int row = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int c = blockIdx.y * 64 + 2 * lane;
+    const bool in0 = c < C, in1 = c + 1 < C;
+    const int first_tile = cu_q[e0] / tile;
     pdl_wait();
-    const int e = blockIdx.z;
-    const int first = cu_q[e], q_len = cu_q[e + 1] - first;
-    if (q_len <= 0) return;                                 // an entry that pads the step: no slot is touched
-    const int slot = slots[e];
-    if (slot < 0 || slot >= n_slots) {                      // (all CTAs of the cluster leave)
-        if (threadIdx.x == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
-        return;
-    }
-    constexpr int ROUND = SCAN_WARPS * SCAN_RUN;
-    const int shares = CLUSTER ? (int)gridDim.x : 1, share = CLUSTER ? (int)blockIdx.x : 0;
-    // shares of whole rounds: tokens begin .. end - 1 are this CTA's
-    const int per = ((q_len + shares - 1) / shares + ROUND - 1) / ROUND * ROUND;
-    const int begin = min(q_len, share * per), end = min(q_len, begin + per);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c = blockIdx.y * 32 + lane;
-    const bool live = c < C;
-    const int start = kv_len[e] - q_len;
-    float* mine = state + (long long)slot * slot_stride;
-    float s0 = live && start > 0 ? mine[s_off + c] : 0.f;    // the state before the round
-    float a[SCAN_RUN], b[SCAN_RUN];
-    auto fetch = [&](int t) {                                // tokens past the end change nothing
-#pragma unroll
-        for (int j = 0; j < SCAN_RUN; ++j) {
-            const bool in = live && t + j < end;
-            const float* row = aux + (long long)(first + t + j) * 2 * C + c;
-            a[j] = in ? row[0] : 1.f;
-            b[j] = in ? row[C] : 0.f;
-        }
+    auto load = [&](const float* p) {
+        if (pairs) return in0 ? ld2(p) : make_float2(0.f, 0.f);
+        return make_float2(in0 ? p[0] : 0.f, in1 ? p[1] : 0.f);
     };
-    auto compose = [&]() {
-        float A = 1.f, B = 0.f;
-#pragma unroll
-        for (int j = 0; j < SCAN_RUN; ++j) {
-            B = fmaf(a[j], B, b[j]);
-            A *= a[j];
+    float2 carry = make_float2(0.f, 0.f);
+    const int before = tile_id - first_tile;
+    if (before > 0) {
+        const int per = (before + APPLY_ROWS - 1) / APPLY_ROWS;
+        const int lo = first_tile + min(before, row * per), hi = first_tile + min(before, (row + 1) * per);
+        float4 s = make_float4(1.f, 1.f, 0.f, 0.f);         // (A, A', B, B')
+#pragma unroll 4
+        for (int j = lo; j < hi; ++j) {
+            const float* p = aux + (long long)((j + 1) * tile - 1) * 2 * C + c;
+            const float2 a = load(p), b = load(p + C);
+            s = make_float4(s.x * a.x, s.y * a.y, fmaf(a.x, s.z, b.x), fmaf(a.y, s.w, b.y));
         }
-        return make_float2(A, B);
-    };
-    if (CLUSTER) {
-        float2 total = make_float2(1.f, 0.f);                // of the rounds so far, of this warp's runs alone ...
-        for (int t0 = begin; t0 < end; t0 += ROUND) {
-            fetch(t0 + warp * SCAN_RUN);
-            pair[0][warp][lane] = compose();
-            __syncthreads();
-            if (warp == 0) {                                 // ... warp 0 puts the round's runs together
-#pragma unroll
-                for (int w = 0; w < SCAN_WARPS; ++w) {
-                    const float2 p = pair[0][w][lane];
-                    total = make_float2(total.x * p.x, fmaf(p.x, total.y, p.y));
-                }
-            }
-            __syncthreads();
-        }
-        if (warp == 0) whole[lane] = total;
-        asm volatile("barrier.cluster.arrive.release.aligned;\n"
-                     "barrier.cluster.wait.acquire.aligned;" ::: "memory");
-        const uint32_t at = (uint32_t)__cvta_generic_to_shared(&whole[lane]);
-        float2 p[SCAN_MAX_SHARES];
-#pragma unroll
-        for (int r = 0; r < SCAN_MAX_SHARES; ++r) {
-            p[r] = make_float2(1.f, 0.f);
-            if (r < share) {
-                uint32_t ra;
-                asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(at), "r"(r));
-                asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(p[r].x), "=f"(p[r].y) : "r"(ra) : "memory");
-            }
-        }
-#pragma unroll
-        for (int r = 0; r < SCAN_MAX_SHARES; ++r) s0 = fmaf(p[r].x, s0, p[r].y);
-        // nobody leaves, or writes the slot, while a CTA of the cluster may still read
-        asm volatile("barrier.cluster.arrive.release.aligned;\n"
-                     "barrier.cluster.wait.acquire.aligned;" ::: "memory");
-    }
-    for (int t0 = begin, it = 0; t0 < end; t0 += ROUND, ++it) {
-        const int t = t0 + warp * SCAN_RUN;
-        if (!CLUSTER || end - begin > ROUND) fetch(t);
-        float y[SCAN_RUN];
-#pragma unroll
-        for (int j = 0; j < SCAN_RUN; ++j)
-            y[j] = live && t + j < end ? proj.load((long long)(first + t + j) * cols + y_off + c) : 0.f;
-        pair[it & 1][warp][lane] = compose();
+        part[row][lane] = s;
         __syncthreads();
-        float s = s0, mine_s = s0;
 #pragma unroll
-        for (int w = 0; w < SCAN_WARPS; ++w) {
-            if (w == warp) mine_s = s;
-            const float2 p = pair[it & 1][w][lane];
-            s = fmaf(p.x, s, p.y);
-        }
-        s0 = s;
-#pragma unroll
-        for (int j = 0; j < SCAN_RUN; ++j) {
-            mine_s = fmaf(a[j], mine_s, b[j]);
-            if (live && t + j < end)
-                out[(long long)(first + t + j) * C + c] = from_f32<T>(mine_s * lin_gelu_tanh(y[j]));
+        for (int r = 0; r < APPLY_ROWS; ++r) {
+            const float4 p = part[r][lane];
+            carry = make_float2(fmaf(p.x, carry.x, p.z), fmaf(p.y, carry.y, p.w));
         }
     }
-    if (!live || end != q_len || begin == end) return;       // the CTA with the last token moves the slot on
-    if (warp == 0) mine[s_off + c] = s0;
-    // the last inputs of the convolution: those of this step (older ones stay where they are)
-    for (int back = warp; back < taps && back < q_len; back += SCAN_WARPS) {
-        const int p = kv_len[e] - 1 - back;
-        mine[ring_off + (long long)(p % taps) * C + c] = proj.load((long long)(first + q_len - 1 - back) * cols + x_off + c);
+    const int end = min(n, t0 + tile);
+#pragma unroll 2
+    for (int t = t0 + row; t < end; t += APPLY_ROWS) {
+        const int e = tok_entry[t];
+        if (e < 0) break;
+        const int slot = slots[e];
+        if (slot < 0 || slot >= n_slots) {
+            if (lane == 0) atomicOr(err, CRANE_ERR_SLOT_RANGE);
+            continue;
+        }
+        const float* p = aux + (long long)t * 2 * C + c;
+        const float2 a = load(p), b = load(p + C);
+        const long long at = (long long)t * cols + c;
+        float2 y = make_float2(0.f, 0.f);
+        if (pairs) { if (in0) y = proj.load2(at + y_off); }
+        else {
+            if (in0) y.x = proj.load(at + y_off);
+            if (in1) y.y = proj.load(at + y_off + 1);
+        }
+        const float2 s = make_float2(fmaf(a.x, carry.x, b.x), fmaf(a.y, carry.y, b.y));
+        T* o = out + (long long)t * C + c;
+        const float ox = s.x * lin_gelu_tanh(y.x), oy = s.y * lin_gelu_tanh(y.y);
+        if (pairs) { if (in0) st2(o, ox, oy); }
+        else {
+            if (in0) o[0] = from_f32<T>(ox);
+            if (in1) o[1] = from_f32<T>(oy);
+        }
+        // a portion's last tokens: the state, and the convolution's last inputs (older ones stay where they are)
+        const int back = cu_q[e + 1] - 1 - t;
+        if (back < taps) {
+            float* mine = state + (long long)slot * slot_stride + c;
+            float* ring = mine + ring_off + (long long)((kv_len[e] - 1 - back) % taps) * C;
+            if (in0) ring[0] = proj.load(at + x_off);
+            if (in1) ring[1] = proj.load(at + x_off + 1);
+            if (back == 0) {
+                if (in0) mine[s_off] = s.x;
+                if (in1) mine[s_off + 1] = s.y;
+            }
+        }
     }
 }
 
@@ -553,16 +602,15 @@ int launch_tensor(const GateScanArgs<__nv_bfloat16>& g, int parts, int all_singl
                             st, g, pairs);
     }
     const int vec = g.proj.parts == nullptr && ((g.width | g.cols | g.x_off) & 7) == 0 && ((uintptr_t)g.proj.whole & 15) == 0;
-    const size_t base = (size_t)((MANY_TOKENS + 3) * g.ld + 2 * MANY_TOKENS * ldm) * sizeof(__nv_bfloat16);
-    const size_t per_wn = (size_t)2 * 16 * ldm * sizeof(__nv_bfloat16);
+    const auto smem_for = [&](int w) { return (size_t)many_front(g.ld, w * 16) + (size_t)w * 2 * 16 * ldm * sizeof(__nv_bfloat16); };
     const int groups = (g.width + 15) / 16;
     int wn = groups < MANY_MAX_WN ? groups : MANY_MAX_WN;
-    while (wn > 1 && base + wn * per_wn > LIN_SMEM) --wn;
-    if (base + per_wn > LIN_SMEM) return (int)cudaErrorInvalidValue;
+    while (wn > 1 && smem_for(wn) > LIN_SMEM) --wn;
+    if (smem_for(wn) > LIN_SMEM) return (int)cudaErrorInvalidValue;
     const int blocks = (groups + wn - 1) / wn;
     wn = (groups + blocks - 1) / blocks;                    // (as even as it gets)
     return crane_launch(gate_scan_prep_many_kernel, dim3((g.n + MANY_TOKENS - 1) / MANY_TOKENS, parts, blocks), dim3(MANY_TOKENS / 16 * wn * 32),
-                        base + wn * per_wn, st, g, wn, pairs, vec);
+                        smem_for(wn), st, g, wn, pairs, vec);
 }
 int launch_tensor(const GateScanArgs<float>&, int, int, cudaStream_t) { return (int)cudaErrorInvalidValue; }
 
@@ -594,23 +642,22 @@ CRANE_API int crane_gate_scan_prep(int dtype, const void* proj, const float* pro
     });
 }
 
+// The tokens of a tile of `crane_gate_scan_prep` for these arguments (not in a step of single tokens).
+CRANE_API int crane_gate_scan_tile(int mma, int n_tokens) { return !mma || n_tokens <= 16 ? 16 : MANY_TOKENS; }
+
 CRANE_API int crane_channel_scan(int dtype, const float* aux, const void* proj, const float* proj_parts, int n_parts,
-                                 long long part_stride, int cols, int y_off, int x_off, const int* cu_q,
-                                 const int* kv_len, const int* slots, int n_slots, float* state, long long slot_stride,
-                                 long long s_off, long long ring_off, int taps, void* out, int n_entries, int n_tokens,
-                                 int C, int* err, cudaStream_t st) {
-    if (n_entries <= 0) return 0;
+                                 long long part_stride, int cols, int y_off, int x_off, const int* tok_entry,
+                                 const int* cu_q, const int* kv_len, const int* slots, int n_slots, float* state,
+                                 long long slot_stride, long long s_off, long long ring_off, int taps, void* out,
+                                 int n_tokens, int C, int mma, int* err, cudaStream_t st) {
+    if (n_tokens <= 0) return 0;
     if (taps < 1 || taps > LIN_MAX_TAPS || C <= 0) return (int)cudaErrorInvalidValue;
+    const int tile = crane_gate_scan_tile(mma, n_tokens);
+    const int pairs = ((C | cols | y_off) & 1) == 0 && (part_stride & 1) == 0 && ((uintptr_t)aux & 7) == 0;
     DISPATCH_T(dtype, {
         GemmOut<T> p{(const T*)proj, proj_parts, n_parts, part_stride};
-        // shares of a round: enough CTAs for a long prompt, no more than a cluster holds
-        int shares = 1;
-        while (shares < SCAN_MAX_SHARES && n_tokens / n_entries > shares * SCAN_WARPS * SCAN_RUN) shares *= 2;
-        const dim3 grid(shares, (C + 31) / 32, n_entries), block(SCAN_WARPS * 32);
-        if (shares == 1)
-            return crane_launch(channel_scan_kernel<T, false>, grid, block, 0, st, aux, p, cols, y_off, x_off, cu_q, kv_len, slots,
-                                n_slots, state, slot_stride, s_off, ring_off, taps, (T*)out, C, err);
-        return crane_launch_cluster(channel_scan_kernel<T, true>, grid, block, 0, dim3(shares, 1, 1), st, aux, p, cols, y_off, x_off,
-                                    cu_q, kv_len, slots, n_slots, state, slot_stride, s_off, ring_off, taps, (T*)out, C, err);
+        return crane_launch(channel_scan_kernel<T>, dim3((n_tokens + tile - 1) / tile, (C + 63) / 64), dim3(APPLY_ROWS * 32), 0, st,
+                            aux, p, cols, y_off, x_off, tok_entry, cu_q, kv_len, slots, n_slots, state, slot_stride, s_off,
+                            ring_off, taps, (T*)out, n_tokens, C, tile, pairs, err);
     });
 }

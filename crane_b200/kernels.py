@@ -37,7 +37,7 @@ _SIGNATURES = {
     "crane_paged_decode_attention_fused": [P, P, I, L, I, I, I, P, P, I, P, P, F, P, P, P, P, P, P, P, P,
                                            I, I, I, I, I, I, I, I, F, I, I, I, I, F, P, I, P, P],
     "crane_prefill_attention_tc_supports": [I, I, I, I],
-    "crane_prefill_attention_tc": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
+    "crane_prefill_attention_tc": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P, I, L, I, I, P, P],
     "crane_embed_bigram": [I, P, P, P, P, I, I, I, I, L, L, P, P, P, P, P, I, P, I, P, P],
     "crane_combine_layernorm": [I, P, P, L, I, P, P, I, L, P, P, I, L, P, P, P, P, P, P, P, P, I, I, F, P],
     "crane_xielu": [I, P, P, I, L, P, L, P, P],
@@ -72,7 +72,7 @@ _SIGNATURES = {
     "crane_head_norm_gate": [I, P, P, P, I, L, I, I, P, P, I, I, F, P, P, I, F, P, I, I, I, P],
     "crane_gate_scan_mma_most": [],
     "crane_gate_scan_prep": [I, P, P, I, L, I, I, I, P, P, P, P, I, P, L, L, L, P, P, I, P, I, P, P, P, P, P, I, I, I, I, P, P],
-    "crane_channel_scan": [I, P, P, P, I, L, I, I, I, P, P, P, I, P, L, L, L, I, P, I, I, I, P, P],
+    "crane_channel_scan": [I, P, P, P, I, L, I, I, I, P, P, P, P, I, P, L, L, L, I, P, I, I, I, P, P],
     "crane_head_talk_mix": [I, P, P, P, P, I, I, I, I, I, P],
     "crane_pair_norm_mean": [I, P, P, I, L, P, P, I, L, P, P, F, P, I, I, P],
     "crane_delta_rule_prep": [I, P, P, I, L, I, P, P, P, P, P, I, I, I, I, F, F, P],
@@ -672,9 +672,10 @@ class Kernels:
         return out, True
 
     def gate_scan_prep(self, proj: Act, cols, ctx, state, g: "Kernels.GateScan", aux, out, err, dtype) -> None:
-        """u = conv(x) + bias, r and i = sigmoid(matrix u + bias) in parts, a = exp(-8 r softplus(lam)): ``aux`` float
-        [n, 2 C] = [a | sqrt(1 - a^2) i u] for ``channel_scan``.  In a step of single tokens (``ctx``): the token's
-        S <- a S + sqrt(1 - a^2) i u as well, ``out`` [n, C] = S gelu_tanh(y), and nothing is left to do."""
+        """u = conv(x) + bias, r and i = sigmoid(matrix u + bias) in parts, a = exp(-8 r softplus(lam)), b = sqrt(1 - a^2) i u:
+        ``aux`` float [n, 2 C] = what the walk S <- a S + b from each tile of tokens comes to, for ``channel_scan``.  In a
+        step of single tokens (``ctx``): the token's walk as well, ``out`` [n, C] = S gelu_tanh(y), and nothing is left
+        to do."""
         whole, parts, n_parts, stride = _split(proj)
         self._check(self.lib.crane_gate_scan_prep(
             _dt(dtype), whole, parts, n_parts, stride, int(cols), g.y_off, g.x_off, ctx.tok_entry.data_ptr(),
@@ -685,14 +686,14 @@ class Kernels:
             self._stream(out)), "gate_scan_prep")
 
     def channel_scan(self, aux, proj: Act, cols, ctx, state, g: "Kernels.GateScan", out, err) -> None:
-        """S <- a S + b per channel over every entry's tokens, (a, b) from ``aux`` [n, 2 C], from and to the slots;
-        ``out`` [n, C] = S gelu_tanh(y).  Moves the convolution's ring on."""
+        """The states S of every entry's tokens from ``gate_scan_prep``'s ``aux``, to the slots; ``out`` [n, C] =
+        S gelu_tanh(y).  Moves the convolution's ring on."""
         whole, parts, n_parts, stride = _split(proj)
         self._check(self.lib.crane_channel_scan(
             _dt(out.dtype), aux.data_ptr(), whole, parts, n_parts, stride, int(cols), g.y_off, g.x_off,
-            ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0], state.data_ptr(),
-            state.stride(0), g.s_off, g.ring_off, g.conv_w.shape[0], out.data_ptr(), ctx.kv_len.shape[0], out.shape[0],
-            out.shape[1], err.data_ptr(), self._stream(out)), "channel_scan")
+            ctx.tok_entry.data_ptr(), ctx.cu_q.data_ptr(), ctx.kv_len.data_ptr(), ctx.slots.data_ptr(), state.shape[0],
+            state.data_ptr(), state.stride(0), g.s_off, g.ring_off, g.conv_w.shape[0], out.data_ptr(), out.shape[0],
+            out.shape[1], 1 if g.mma else 0, err.data_ptr(), self._stream(out)), "channel_scan")
 
     def matrix_state_scan(self, aux, offs, w_vec: bool, mode, qk_rep: int, ctx, state, o_raw, H, dk, dv,
                           err, den=None, max_len: int = 0) -> None:
@@ -1152,15 +1153,17 @@ class Kernels:
         return bool(self.lib.crane_prefill_attention_tc_supports(d, nq, nkv, page_size))
 
     def prefill_attention_tc(self, q, out, k_pool, v_pool, cu_q, kv_len, block_table, page_size,
-                             total_q_tiles, nq, nkv, d, window, scale, err, skip_single=False) -> None:
+                             total_q_tiles, nq, nkv, d, window, scale, err, skip_single=False, sinks=None,
+                             gate=None) -> None:
         """Flash attention on tcgen05 (head size 128).  ``total_q_tiles``: the sum
         over the entries of ceil(tokens / 128), or more.  ``skip_single`` as in
-        ``paged_prefill_attention``."""
+        ``paged_prefill_attention``, ``sinks`` and ``gate`` as in ``paged_decode_attention``."""
         self._check(self.lib.crane_prefill_attention_tc(
             q.data_ptr(), out.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), cu_q.data_ptr(),
             kv_len.data_ptr(), block_table.data_ptr(), block_table.shape[1], k_pool.shape[0],
             page_size, kv_len.shape[0], q.shape[0], int(total_q_tiles), nq, nkv, d, int(window),
-            float(scale), 1 if skip_single else 0, err.data_ptr(), self._stream(q)), "prefill_attention_tc")
+            float(scale), 1 if skip_single else 0, _ptr(sinks), *self._gate(gate), err.data_ptr(), self._stream(q)),
+            "prefill_attention_tc")
 
     def paged_decode_attention_fused(self, qkv: Act, qkv_cols, has_kv, cos, sin, q_norm_w, k_norm_w,
                                      eps, out, k_pool, v_pool, cu_q, kv_len, block_table, page_size,

@@ -191,7 +191,7 @@ class GqaAttention(Part):
         # 8 tokens 244 / 144 us, 64 of 32: 44 / 28 us, 32 of 64: 22 / 19 us; 21 of 96: 22 / 23 us, 16 of 128:
         # 16 / 21 us; 16 portions of 32 behind 2,000 cached keys 50 / 94 us.
         short = bool(getattr(ctx, "short_prompts", False)) and use_mma
-        use_tc = (not rt.exact and rt.use_tc_attention and not short and self.sinks is None and gate is None
+        use_tc = (not rt.exact and rt.use_tc_attention and not short
                   and k.prefill_attention_tc_supports(self.d, self.nq, self.nkv, cache.page_size))
         # Decoded tokens beside prompt portions: the entries of one token go to the split-KV decode
         # kernel (which skips the others), the prompt portions to the prefill kernel (which skips them).
@@ -220,7 +220,7 @@ class GqaAttention(Part):
             tiles = query_tiles(ctx, 128, skip_single=bool(singles))
             k.prefill_attention_tc(q, o, cache.k, cache.v, ctx.cu_q, ctx.kv_len, table, cache.page_size,
                                    tiles, self.nq, self.nkv, self.d, self.window, self.scale, rt.err,
-                                   skip_single=bool(singles))
+                                   skip_single=bool(singles), sinks=self.sinks, gate=gate)
             rt.launches += 2
         elif use_mma:
             tiles = query_tiles(ctx, 64, skip_single=bool(singles))

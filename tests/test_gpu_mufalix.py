@@ -508,9 +508,34 @@ def test_attention_with_gate_window_and_sinks(K, dtype, window, d, nq, nkv, ps, 
             K.paged_prefill_attention(q_all, both, k_pool, v_pool, _i32(cu), _i32(lens), table, ps, tiles + 3, nq, nkv, d, window, scale, err,
                                       sinks=sk, gate=(g, gate_cols, gate_off))
             assert np.abs(_np(both) - want).max() < tol * max(1.0, np.abs(want).max()), form
+            if K.prefill_attention_tc_supports(d, nq, nkv, ps):          # the same on tcgen05, every entry and portions alone
+                for skip in (False, True):
+                    both.fill_(5.0)
+                    K.prefill_attention_tc(q_all, both, k_pool, v_pool, _i32(cu), _i32(lens), table, ps, len(lens) + 1, nq, nkv, d, window,
+                                           scale, err, skip_single=skip, sinks=sk, gate=(g, gate_cols, gate_off))
+                    rows = [i for i in range(N) if not skip or i not in single]
+                    assert np.abs(_np(both)[rows] - want[rows]).max() < tol * max(1.0, np.abs(want).max()), (form, skip)
+                    assert not skip or (both[single] == 5.0).all()
         bad = np.abs(_np(out) - want).max(axis=1) >= tol * max(1.0, np.abs(want).max())
         assert not bad.any(), (form, np.nonzero(bad)[0][:5])
     assert int(err.item()) == 0
+
+
+@pytest.mark.parametrize("window", [0, 200])
+def test_long_prompts_two_heads_a_block(K, window):
+    """As many tiles as make the tcgen05 kernel take two heads at a time: sinks, gate and window against the kernel of
+    64-row tiles."""
+    torch.manual_seed(window)
+    T, nq, nkv, d, ps = 4096, 16, 4, 128, 64
+    q, gate = torch.randn(T, nq * d, device=DEV).bfloat16(), torch.randn(T, nq * d + 8, device=DEV).bfloat16()
+    kp, vp = (torch.randn(T // ps, nkv, ps, d, device=DEV).bfloat16() for _ in range(2))
+    table, cu, kvl, err = _i32([torch.randperm(T // ps).tolist()]), _i32([0, T]), _i32([T]), _err()
+    sinks = torch.linspace(-2, 9, nq, device=DEV)
+    a, b = torch.empty_like(q), torch.empty_like(q)
+    g = (gate, nq * d + 8, 8)
+    K.prefill_attention_tc(q, a, kp, vp, cu, kvl, table, ps, T // 128, nq, nkv, d, window, d ** -0.5, err, sinks=sinks, gate=g)
+    K.paged_prefill_attention(q, b, kp, vp, cu, kvl, table, ps, T // 64, nq, nkv, d, window, d ** -0.5, err, sinks=sinks, gate=g)
+    assert float((a.float() - b.float()).abs().max()) < 2e-2 * float(b.float().abs().max()) and int(err.item()) == 0
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -203,6 +203,20 @@ __device__ __forceinline__ float sink_term(const Params& p, int h, float m_ref) 
 __device__ __forceinline__ void gate_row(const Params& p, long long row, int h, int c0, uint32_t (&v)[32]) {
     if (p.gate_ld <= 0) return;
     const long long at = row * p.gate_ld + p.gate_off + h * D + c0;
+    if (p.gate.parts == nullptr && ((p.gate_ld | p.gate_off) & 7) == 0 && ((uintptr_t)p.gate.whole & 15) == 0) {
+#pragma unroll
+        for (int i = 0; i < 32; i += 8) {
+            const uint4 raw = *(const uint4*)(p.gate.whole + at + i);
+            const __nv_bfloat162* z2 = (const __nv_bfloat162*)&raw;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float2 z = __bfloat1622float2(z2[j]);
+                v[i + 2 * j] = __float_as_uint(__fdividef(__uint_as_float(v[i + 2 * j]), 1.f + __expf(-z.x)));
+                v[i + 2 * j + 1] = __float_as_uint(__fdividef(__uint_as_float(v[i + 2 * j + 1]), 1.f + __expf(-z.y)));
+            }
+        }
+        return;
+    }
 #pragma unroll
     for (int i = 0; i < 32; i += 2) {
         const float2 z = p.gate.load2(at + i);

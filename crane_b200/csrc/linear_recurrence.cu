@@ -24,6 +24,13 @@ constexpr int LIN_MAX_TAPS = 16;
 constexpr float LIN_RATE = 8.f;                // log a = -LIN_RATE r softplus(lam)
 
 __device__ __forceinline__ float lin_sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
+// On the bfloat16 path: the device's fast forms, errors of a few units in the last place of 32-bit.
+__device__ __forceinline__ float lin_sigmoid_fast(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+__device__ __forceinline__ float lin_sqrt_fast(float v) {
+    float r;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
 __device__ __forceinline__ float lin_gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
@@ -93,10 +100,14 @@ __device__ __forceinline__ float conv_at(const GateScanArgs<T>& g, const TileTok
 // Channel c: from the two products' sums to the decay and the addend.
 template <typename T>
 __device__ __forceinline__ void gate_scan_terms(const GateScanArgs<T>& g, int c, float zr, float zi, float u, float& a, float& add) {
-    const float r = lin_sigmoid(zr + g.rb[c]), i = lin_sigmoid(zi + g.ib[c]);
+    constexpr bool FAST = sizeof(T) == 2;
+    zr += g.rb[c];
+    zi += g.ib[c];
+    const float r = FAST ? lin_sigmoid_fast(zr) : lin_sigmoid(zr), i = FAST ? lin_sigmoid_fast(zi) : lin_sigmoid(zi);
     const float log_a = -LIN_RATE * r * g.sp[c];
     a = expf(log_a);
-    add = sqrtf(one_minus_exp(2.f * log_a, a * a)) * i * u;
+    const float rest = one_minus_exp(2.f * log_a, a * a);
+    add = (FAST ? lin_sqrt_fast(rest) : sqrtf(rest)) * i * u;
 }
 // A portion's first token: the slot's state joins the addend, and what came before counts no more.
 template <typename T>
@@ -219,12 +230,15 @@ __device__ __forceinline__ void split_store(__nv_bfloat16* hi, __nv_bfloat16* lo
 }
 // The weights of `cols` columns from c0 on of both matrices: w_s [2][cols][ld + 8].
 __device__ __forceinline__ void load_gates(const GateScanArgs<__nv_bfloat16>& g, __nv_bfloat16* w_s, int cols, int base_c, int c0) {
-    const int pieces = g.ld >> 3, ldm = g.ld + 8;
-    for (int x = threadIdx.x; x < 2 * cols * pieces; x += blockDim.x) {
-        const int r = x / pieces, q = x % pieces, m = r / cols, c = c0 + r % cols;
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (c < g.width) v = *reinterpret_cast<const uint4*>(g.gates + ((long long)m * g.C + base_c + c) * g.ld + q * 8);
-        *reinterpret_cast<uint4*>(w_s + r * ldm + q * 8) = v;
+    const int pieces = g.ld >> 3, ldm = g.ld + 8;            // (8 threads a row: a piece each, then the next 8)
+    for (int r = threadIdx.x >> 3; r < 2 * cols; r += blockDim.x >> 3) {
+        const int m = r >= cols, c = c0 + r - m * cols;
+        const __nv_bfloat16* src = g.gates + ((long long)m * g.C + base_c + c) * g.ld;
+        for (int q = threadIdx.x & 7; q < pieces; q += 8) {
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (c < g.width) v = *reinterpret_cast<const uint4*>(src + q * 8);
+            *reinterpret_cast<uint4*>(w_s + r * ldm + q * 8) = v;
+        }
     }
 }
 // One step of 16 along the inner dimension: 16 tokens (rows from u_hi / u_lo on) by 16 columns of both matrices.
@@ -361,11 +375,14 @@ gate_scan_prep_many_kernel(const GateScanArgs<__nv_bfloat16> g, int wn_warps, in
     pdl_wait();
     if (vec) {                                              // rows of 16-byte pieces
         const int pieces = g.ld >> 3;
-        for (int x = threadIdx.x; x < (MANY_TOKENS + 3) * pieces; x += blockDim.x) {
-            const int r = x / pieces, c = x % pieces * 8, t = t0 - 3 + r;
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (t >= 0 && t < g.n && c < width) v = *reinterpret_cast<const uint4*>(g.proj.whole + (long long)t * g.cols + g.x_off + base_c + c);
-            *reinterpret_cast<uint4*>(xs + r * g.ld + c) = v;
+        for (int r = threadIdx.x >> 3; r < MANY_TOKENS + 3; r += blockDim.x >> 3) {
+            const int t = t0 - 3 + r;
+            const __nv_bfloat16* src = g.proj.whole + (long long)t * g.cols + g.x_off + base_c;
+            for (int c = (threadIdx.x & 7) * 8; c < pieces * 8; c += 64) {
+                uint4 v = make_uint4(0u, 0u, 0u, 0u);
+                if (t >= 0 && t < g.n && c < width) v = *reinterpret_cast<const uint4*>(src + c);
+                *reinterpret_cast<uint4*>(xs + r * g.ld + c) = v;
+            }
         }
     } else {
         const int half = g.ld >> 1;

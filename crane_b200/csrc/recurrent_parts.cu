@@ -328,7 +328,7 @@ exp_gate_prep_kernel(GemmOut<T> proj, int cols, const int* __restrict__ tok_entr
             if (t + j < q_len) write(first + t + j, h, li[j], lf[j], before, m[j]);
             before = m[j];
         }
-        m0 = last[WARPS - 1];                               // (a round later `part_a` and `last` are written behind two barriers)
+        m0 = last[WARPS - 1];                               // (`part_a` and `last` are written again behind a barrier that all readers have reached)
     }
     if (threadIdx.x == 0) *kept = m0;
 }

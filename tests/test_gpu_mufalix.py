@@ -753,6 +753,31 @@ def test_greedy_batch_bfloat16_through_the_scheduler(name, model_folders):
     assert m.runner.graph_replays > 0 and m.runner._pad_with_copies       # (the batch-size buckets)
 
 
+def test_decode_batches_of_changing_size_without_the_decode_kernel(model_folders):
+    """Heads that the decode kernel does not take: single tokens go through the kernel for portions, also in the
+    batch-size buckets' graphs, which are recorded with fewer requests than later steps have."""
+    from crane_b200.config import EngineConfig
+    from crane_b200.engine import ModelRunner, StepEntry
+    folder = model_folders("FG", "bfloat16")
+    cfg, w = pm.load_folder(folder)
+    runner = ModelRunner(folder, EngineConfig(dtype="bfloat16", page_size=16, num_pages=24, max_concurrent=4, max_batched_tokens=64,
+                                              max_seq_len=128))
+    rng = np.random.default_rng(2)
+    toks = [rng.integers(0, cfg["vocab"], 40).tolist() for _ in range(4)]
+    want = [pm.logits_all(cfg, w, t) for t in toks]
+    done = [9, 14, 3, 6]
+    for r in range(4):
+        runner.step([StepEntry(r, toks[r][:done[r]], [])])
+    for live in [(0, 1, 2)] * 3 + [(0, 1, 2, 3)] * 4 + [(1, 2, 3)] * 2 + [(2,)] * 2 + [(0, 1, 2, 3)] * 3:
+        got = runner.step([StepEntry(r, [toks[r][done[r]]], [0]) for r in live]).cpu().numpy()
+        for i, r in enumerate(live):
+            row = want[r][done[r]]
+            assert np.sqrt(((got[i] - row) ** 2).mean()) < 6e-2 * np.sqrt((row ** 2).mean()), (live, r)
+            done[r] += 1
+    runner.rt.check_errors()
+    assert runner.graph_replays > 0 and runner._pad_with_copies
+
+
 def test_command_line(model_folders):
     """bin/crane picks the model class from config.json."""
     import os

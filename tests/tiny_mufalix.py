@@ -103,6 +103,17 @@ FL = {
 }
 
 
+# more query heads per key/value head than the decode kernel's tile has rows
+FG = {
+    "architecture": "Mufalix", "vocab": 120, "width": 64, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.5},
+    "layers": [
+        _none(_parallel(_attention(20, 1, 16, 16, 0.3, 12, (8, 100.0, None)), 32, 2, 3)),
+        _moe(_mlstm(2, 16, 16, 6.0), 3, 3, 1.2, 16),
+        _none(_parallel(_attention(34, 2, 32, 24, 0.2, 0, None), 48, 1, 4)),
+    ],
+}
+
+
 def all_chosen(config):
     """The same with every expert of every layer chosen: no choice that rounding could flip, so whole-model logits
     can be compared closely in bfloat16."""
@@ -119,6 +130,7 @@ TINY = {
     "FC": {"config": FC, "seed": 63, "std": 0.14, "norm_std": 0.05, "page_size": 16},
     "FD": {"config": FD, "seed": 64, "std": 0.15, "norm_std": 0.05, "page_size": 32},
     "FL": {"config": FL, "seed": 65, "std": 0.045, "norm_std": 0.05, "page_size": 64},
+    "FG": {"config": FG, "seed": 66, "std": 0.12, "norm_std": 0.05, "page_size": 16},
 }
 for _name in list(TINY):
     TINY[_name + "-all"] = dict(TINY[_name], config=all_chosen(TINY[_name]["config"]), seed=TINY[_name]["seed"] + 10)
